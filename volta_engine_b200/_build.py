@@ -29,6 +29,8 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=default",
     "--expt-relaxed-constexpr", "-diag-suppress", "177,550",
 ]
+# sources whose results follow the 32-bit definitions of exp / tanh / division to rounding
+PRECISE = {"rowops.cu", "linattn.cu", "latent.cu", "gemv_rows.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-pthread", "-Wall", "-Wno-unused-function"]
 
 
@@ -64,15 +66,18 @@ def _build_lib(name: str, srcs: list[Path], headers: list[Path], compiler: list[
     objdir = OUT / f"obj_{name}"
     objdir.mkdir(exist_ok=True)
     jobs = []
+
+    def flags_of(s: Path) -> list[str]:
+        return [f for f in flags if f != "--use_fast_math"] if s.name in PRECISE else flags
     for s in srcs:
-        dig = _digest([s] + headers, " ".join(flags))
+        dig = _digest([s] + headers, " ".join(flags_of(s)))
         obj = objdir / (s.stem + ".o")
         tag = objdir / (s.stem + ".sha")
         if force or not obj.exists() or not tag.exists() or tag.read_text() != dig:
             jobs.append((s, obj, tag, dig))
     if jobs:
         with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
-            futs = [ex.submit(_run, compiler + flags + ["-I", str(CSRC), "-c", str(s), "-o", str(o)])
+            futs = [ex.submit(_run, compiler + flags_of(s) + ["-I", str(CSRC), "-c", str(s), "-o", str(o)])
                     for s, o, _, _ in jobs]
             for f in futs:
                 f.result()

@@ -116,7 +116,7 @@ gemm_kernel(const GemmParams p, const __grid_constant__ CUtensorMap amap, const 
     sf_tile = (size_t)tt.x * (p.n_per_expert / 128) + blockIdx.x;
     if (p.alpha_tab) alpha = p.alpha_tab[tt.x];
   }
-  const int nkt = p.K / KT;
+  const int nkt = MODE == 0 ? (p.K + KT - 1) / KT : p.K / KT;   // bf16 operands: the map's zero fill completes the last step
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) {
@@ -309,7 +309,7 @@ static int launch_gemm(const GemmParams& p, const CUtensorMap& amap, const CUten
   constexpr int SF = MODE == 1 ? 1024 : (MODE == 2 ? 2048 + 2048 * ((BN + 127) / 128) : 0);
   constexpr int smem = STAGES * (A_RAW + A_DEQ + B_BYTES + SF) + 1024;
   static_assert(smem <= 227 * 1024, "shared memory budget");
-  if (p.K % KT) return (int)cudaErrorInvalidValue;
+  if (MODE != 0 && p.K % KT) return (int)cudaErrorInvalidValue;
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(gemm_kernel<MODE, BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);

@@ -107,8 +107,8 @@ __global__ void mla_expand_out_kernel(const __nv_bfloat16* __restrict__ o_lat, c
 }
 
 struct MlaParams {
-  const __nv_bfloat16* q_abs;   // [rows, heads, 576]
-  float* o_part;                // [rows, heads, nsplit, 512]
+  const __nv_bfloat16* q_abs;   // [rows, heads, row]
+  float* o_part;                // [rows, heads, nsplit, latent columns]
   float* lse_part;              // [rows, heads, nsplit]
   const int* pos;
   const int* slot;
@@ -116,6 +116,7 @@ struct MlaParams {
   int max_pages, heads, nsplit;
   float scale_log2;
   int* status;
+  int row;                      // cache row width in elements (a multiple of 64) where it is not a template constant
 };
 
 VE_DEVINL void m_ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
@@ -130,18 +131,28 @@ VE_DEVINL void m_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-constexpr int kQPitch = kLatRow * 2 + 16;     // bytes per Q row in shared memory (padded against bank conflicts)
-constexpr int kMlaTile = kMlaPage * kLatRow * 2;   // 73728 bytes: 9 sub-tiles of 64 keys x 128 B
+// a page tile: row / 64 sub-tiles of 64 keys x 128 B; Q rows in shared memory are padded by 16 B against bank conflicts
+constexpr int mla_smem_bytes(int row) { return 2 * kMlaPage * row * 2 + 16 * (row * 2 + 16) + 16 * 68 * 4 + 1024; }
 constexpr int kSPitch = 68;                    // floats per row of the score exchange buffer
 
-// grid (tokens * slabs_per_token, nsplit), 128 threads.
+// grid (tokens * slabs_per_token, nsplit), 128 threads. NB: 16-column blocks of the latent part per warp (latent width up to
+// 64 * NB); ROW: cache row width, 0 = p.row; P2: the softmax weights enter P.V as two bf16 terms (value and remainder), so
+// they keep 32-bit quality.
+template <int NB, int ROW, bool P2>
 __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, const __grid_constant__ CUtensorMap kmap) {
+  constexpr int LATC = NB * 64;
+  const int roww = ROW ? ROW : p.row;
+  const int kMlaTile = kMlaPage * roww * 2, kQPitch = roww * 2 + 16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* ktile[2] = {smem, smem + kMlaTile};
   uint8_t* qs = smem + 2 * kMlaTile;                         // 16 x kQPitch
   float* ss = reinterpret_cast<float*>(qs + 16 * kQPitch);   // 16 x kSPitch
   __shared__ uint64_t full[2];
+  if (P2) {                     // (the launch is a programmatic dependent only in this form)
+    grid_dep_wait();
+    grid_dep_launch();
+  }
 
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int slabs = (p.heads + 15) / 16;
@@ -159,10 +170,10 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
     mbar_fence_init();
   }
   // Q rows of this slab into shared memory (zero rows beyond the head count)
-  for (int i = tid; i < 16 * (kLatRow / 8); i += 128) {
-    const int r = i / (kLatRow / 8), c = (i % (kLatRow / 8)) * 8;
+  for (int i = tid; i < 16 * (roww / 8); i += 128) {
+    const int r = i / (roww / 8), c = (i % (roww / 8)) * 8;
     bf16x8 v;
-    if (head0 + r < p.heads) v = *reinterpret_cast<const bf16x8*>(p.q_abs + ((long)tok * p.heads + head0 + r) * kLatRow + c);
+    if (head0 + r < p.heads) v = *reinterpret_cast<const bf16x8*>(p.q_abs + ((long)tok * p.heads + head0 + r) * roww + c);
     else v.v[0] = v.v[1] = v.v[2] = v.v[3] = __floats2bfloat162_rn(0.f, 0.f);
     *reinterpret_cast<bf16x8*>(qs + r * kQPitch + c * 2) = v;
   }
@@ -171,13 +182,13 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
     const int page = p.page_table[(long)s * p.max_pages + kt];
     mbar_expect_tx(&full[stage], kMlaTile);
 #pragma unroll
-    for (int c = 0; c < kLatRow / 64; ++c) tma_load_2d(ktile[stage] + c * 8192, &kmap, &full[stage], c * 64, page * kMlaPage);
+    for (int c = 0; c < roww / 64; ++c) tma_load_2d(ktile[stage] + c * 8192, &kmap, &full[stage], c * 64, page * kMlaPage);
   };
   if (tid == 0 && kt_begin < kt_end) issue(kt_begin, 0);
 
-  float o[16][4];
+  float o[2 * NB][4];
 #pragma unroll
-  for (int i = 0; i < 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int i = 0; i < 2 * NB; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f};
   const uint32_t q_base = smem_u32(qs);
   bool failed = false;
@@ -191,7 +202,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
     // ---- scores of this warp's 16 keys over the 576-wide row
     float sacc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll 4
-    for (int kk = 0; kk < kLatRow / 16; ++kk) {
+    for (int kk = 0; kk < roww / 16; ++kk) {
       uint32_t a[4];
       {
         const int mi = lane >> 3, rr = lane & 7;     // matrices: (rows 0-7,k lo) (rows 8-15,k lo) (rows 0-7,k hi) (rows 8-15,k hi)
@@ -238,7 +249,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
       m_run[h] = m_new;
       l_run[h] *= corr[h];
     }
-    uint32_t pf[4][4];
+    uint32_t pf[4][4], pl[P2 ? 4 : 1][4];
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) {
       float pv[4];
@@ -251,27 +262,37 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
       __nv_bfloat162 lo = __floats2bfloat162_rn(pv[0], pv[1]), hi = __floats2bfloat162_rn(pv[2], pv[3]);
       pf[nt >> 1][(nt & 1) * 2 + 0] = *reinterpret_cast<uint32_t*>(&lo);
       pf[nt >> 1][(nt & 1) * 2 + 1] = *reinterpret_cast<uint32_t*>(&hi);
+      if (P2) {
+        lo = __floats2bfloat162_rn(pv[0] - __low2float(lo), pv[1] - __high2float(lo));
+        hi = __floats2bfloat162_rn(pv[2] - __low2float(hi), pv[3] - __high2float(hi));
+        pl[P2 ? nt >> 1 : 0][(nt & 1) * 2 + 0] = *reinterpret_cast<uint32_t*>(&lo);
+        pl[P2 ? nt >> 1 : 0][(nt & 1) * 2 + 1] = *reinterpret_cast<uint32_t*>(&hi);
+      }
     }
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 2 * NB; ++i) {
       o[i][0] *= corr[0];
       o[i][1] *= corr[0];
       o[i][2] *= corr[1];
       o[i][3] *= corr[1];
     }
-    // ---- O[:, warp*128 .. +128) += P . C   (the latent part of the same tile is V)
+    // ---- O[:, warp*NB*16 .. +NB*16) += P . C   (the latent part of the same tile is V)
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks)
 #pragma unroll
-      for (int dp = 0; dp < 8; ++dp) {
+      for (int dp = 0; dp < NB; ++dp) {
         const int mi = lane >> 3, rr = lane & 7;
         const int key = ks * 16 + (mi & 1) * 8 + rr;
-        const int d = warp * 128 + dp * 16 + (mi >> 1) * 8;
+        const int d = warp * NB * 16 + dp * 16 + (mi >> 1) * 8;
         const int c = d / 64, ch = (d % 64) / 8;
         uint32_t b0, b1, b2, b3;
         m_ldsm_x4_t(kb + c * 8192 + key * 128 + ((ch ^ (key & 7)) << 4), b0, b1, b2, b3);
         m_mma(o[2 * dp], pf[ks], b0, b1);
         m_mma(o[2 * dp + 1], pf[ks], b2, b3);
+        if (P2) {
+          m_mma(o[2 * dp], pl[P2 ? ks : 0], b0, b1);
+          m_mma(o[2 * dp + 1], pl[P2 ? ks : 0], b2, b3);
+        }
       }
   }
   if (failed) {
@@ -289,9 +310,9 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
     if (head >= p.heads) continue;
     const float inv = l_run[h] > 0.f ? 1.f / l_run[h] : 0.f;
     const long base = ((long)tok * p.heads + head) * p.nsplit + z;
-    float* orow = p.o_part + base * kLat + warp * 128;
+    float* orow = p.o_part + base * LATC + warp * NB * 16;
 #pragma unroll
-    for (int nt = 0; nt < 16; ++nt)
+    for (int nt = 0; nt < 2 * NB; ++nt)
       *reinterpret_cast<float2*>(orow + nt * 8 + 2 * t) = make_float2(o[nt][2 * h] * inv, o[nt][2 * h + 1] * inv);
     if (warp == 0 && t == 0) p.lse_part[base] = l_run[h] > 0.f ? m_run[h] + log2f(l_run[h]) : -FLT_MAX;
   }
@@ -370,24 +391,72 @@ int ve_mla_decode(const void* q_abs, void* o_lat, void* o_part, void* lse_part, 
   p.nsplit = nsplit;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = (int*)status;
+  p.row = kLatRow;
   CUtensorMap kmap;
   int rc = make_tmap_2d(&kmap, pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)pool_pages * kMlaPage, kLatRow,
                         (uint64_t)kLatRow * 2, kMlaPage, 64, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
-  constexpr int smem = 2 * kMlaTile + 16 * kQPitch + 16 * kSPitch * 4 + 1024;
+  constexpr int smem = mla_smem_bytes(kLatRow);
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(mla_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(mla_decode_kernel<8, kLatRow, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
   const int slabs = (heads + 15) / 16;
   dim3 grid(rows * slabs, nsplit);
-  mla_decode_kernel<<<grid, 128, smem, st>>>(p, kmap);
+  mla_decode_kernel<8, kLatRow, false><<<grid, 128, smem, st>>>(p, kmap);
   rc = (int)cudaGetLastError();
   if (rc) return rc;
   mla_reduce_kernel<<<rows * heads, kLat, 0, st>>>((const float*)o_part, (const float*)lse_part, (__nv_bfloat16*)o_lat,
                                                    (const int*)slot, heads, nsplit);
+  VE_CHECK_LAUNCH();
+}
+
+// The decode kernel for other row layouts: q_abs [rows, heads, row] and pool rows of `pitch` elements, of which the first
+// `row` (a multiple of 64) are used; latent part in the first `lat` <= 512 columns. Leaves split partials o_part
+// [rows, heads, nsplit, lat rounded up to 64 * {1, 2, 4, 8}] and lse_part (log2 units); a split without keys leaves
+// lse = -FLT_MAX. The merge is part of latent_expand.
+int ve_latent_decode(const void* q_abs, void* o_part, void* lse_part, const void* pos, const void* slot, const void* page_table, int max_pages,
+                     void* pool, long pool_pages, int pitch, int row, int lat, int rows, int heads, int nsplit, float scale, void* status,
+                     cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const int nb = lat <= 64 ? 1 : lat <= 128 ? 2 : lat <= 256 ? 4 : 8;
+  if (row % 64 || row < nb * 64 || row > 704 || lat > 512 || pitch < row || pitch % 8 || nsplit < 1) return cudaErrorInvalidValue;
+  MlaParams p;
+  p.q_abs = (const __nv_bfloat16*)q_abs;
+  p.o_part = (float*)o_part;
+  p.lse_part = (float*)lse_part;
+  p.pos = (const int*)pos;
+  p.slot = (const int*)slot;
+  p.page_table = (const int*)page_table;
+  p.max_pages = max_pages;
+  p.heads = heads;
+  p.nsplit = nsplit;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.status = (int*)status;
+  p.row = row;
+  CUtensorMap kmap;
+  int rc = make_tmap_2d(&kmap, pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)pool_pages * kMlaPage, pitch, (uint64_t)pitch * 2, kMlaPage, 64,
+                        CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  const int smem = mla_smem_bytes(row);
+  const dim3 grid(rows * ((heads + 15) / 16), nsplit);
+#define VE_LD(NB)                                                                                                          \
+  do {                                                                                                                     \
+    static int attr = 0;                                                                                                   \
+    if (smem > attr) {                                                                                                     \
+      cudaError_t e = cudaFuncSetAttribute(mla_decode_kernel<NB, 0, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
+      if (e != cudaSuccess) return (int)e;                                                                                 \
+      attr = smem;                                                                                                         \
+    }                                                                                                                      \
+    launch_pdl(mla_decode_kernel<NB, 0, true>, grid, dim3(128), smem, st, p, kmap);                                        \
+  } while (0)
+  if (nb == 1) VE_LD(1);
+  else if (nb == 2) VE_LD(2);
+  else if (nb == 4) VE_LD(4);
+  else VE_LD(8);
+#undef VE_LD
   VE_CHECK_LAUNCH();
 }
 

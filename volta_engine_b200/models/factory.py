@@ -21,6 +21,8 @@ from .dense import DenseConfig, DenseLayer, DenseModel
 DENSE_TYPES = {"llama", "mistral", "qwen2", "qwen3", "gemma2", "gemma3_text", "glm4", "dense"}
 MOE_TYPES = {"qwen3_moe", "glm4_moe", "mixtral", "moe"}
 MLA_TYPES = {"deepseek_v2", "deepseek_v3", "kimi_k2", "mla"}
+# designs that config.json names under "architecture": module and loader (config dict, tensor source, device, comm, dtype=)
+ARCHITECTURES = {"Fofosun": ("fofosun", "load_fofosun")}
 
 
 def dense_config_from_hf(c: dict) -> DenseConfig:
@@ -224,8 +226,8 @@ def load_dense_weights(model: DenseModel, src: TensorSource, gemm_mode="w4a16", 
 
 
 def load_model(model_dir, device="cuda:0", comm=None, gemm_mode="w4a16", quantize=None, prefer=None, overlay: dict | None = None,
-               nvfp4_dense: str = ""):
-    """-> (model, hf_config dict). Raises for model types this build has no pipeline for. ``overlay``: keyword arguments of
+               nvfp4_dense: str = "", dtype: str = "bf16"):
+    """-> (model, hf_config dict). ``dtype``: bf16, or fp32 for the families that have an all-32-bit form. Raises for model types this build has no pipeline for. ``overlay``: keyword arguments of
     :func:`overlay_from_options` (parts of the model taken from other directories); ``nvfp4_dense``: comma list of dense
     groups quantised to NVFP4 at load beyond the default (``head``, or ``all``)."""
     d = Path(model_dir)
@@ -233,6 +235,15 @@ def load_model(model_dir, device="cuda:0", comm=None, gemm_mode="w4a16", quantiz
     if "text_config" in hf and "num_hidden_layers" not in hf:
         hf = dict(hf["text_config"], **{k: v for k, v in hf.items() if k != "text_config"})
     mt = hf.get("model_type", "")
+    arch = ARCHITECTURES.get(hf.get("architecture", ""))
+    if arch is not None:
+        import importlib
+        if quantize or overlay or nvfp4_dense:
+            raise NotImplementedError(f"{hf['architecture']}: the weights are not quantised at load and have no overlays")
+        loader = getattr(importlib.import_module("." + arch[0], __package__), arch[1])
+        return loader(hf, TensorSource(d, prefer), device, comm, dtype=dtype), hf
+    if dtype not in ("bf16", "bfloat16"):
+        raise NotImplementedError(f"dtype {dtype!r}: model_type {mt!r} runs in bf16 only")
     if mt == "deepseek_v41":
         return load_dsv41(hf, d, device, comm), hf
     if mt in ("glm5_next", "glm5-next"):

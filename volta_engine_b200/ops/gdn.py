@@ -112,18 +112,24 @@ class GDNJournal:
     def __init__(self, st: GDNState, shadow: tuple | None = None):
         """``shadow``: (conv [1, ...], rec [1, ...]) buffers shared by the journals of one layer (one per row count of the
         verify step: each CUDA graph keeps its own operands, and only the last step's shadow is ever needed)."""
-        self.shadow_conv, self.shadow_rec = shadow if shadow is not None else (torch.zeros_like(st.conv[:1]),
-                                                                               torch.zeros_like(st.rec[:1]))
+        self.shadow_conv, self.shadow_rec = shadow if shadow is not None else self.make_shadow(st)
         self.rows = None          # operands of the last journalled block
         self.fn = None            # callable(keep): applies rows [0, keep) to the state
 
+    @staticmethod
+    def make_shadow(st) -> tuple:
+        """States without a short convolution have ``conv`` None."""
+        return (torch.zeros_like(st.conv[:1]) if st.conv is not None else None, torch.zeros_like(st.rec[:1]))
+
     def begin(self, st: GDNState, slot: torch.Tensor):
         idx = slot[:1].clamp(min=0).long()
-        torch.index_select(st.conv, 0, idx, out=self.shadow_conv)
+        if st.conv is not None:
+            torch.index_select(st.conv, 0, idx, out=self.shadow_conv)
         torch.index_select(st.rec, 0, idx, out=self.shadow_rec)
 
     def replay(self, st: GDNState, slot: int, keep: int):
-        st.conv[slot].copy_(self.shadow_conv[0])
+        if st.conv is not None:
+            st.conv[slot].copy_(self.shadow_conv[0])
         st.rec[slot].copy_(self.shadow_rec[0])
         if keep > 0 and self.fn is not None:
             self.fn(keep)

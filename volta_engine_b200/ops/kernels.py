@@ -533,6 +533,14 @@ def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False):
     return out
 
 
+def gemm_f32(W, x):
+    """out[t, n] = sum_k W[n, k] x[t, k], true fp32."""
+    N, K = W.shape
+    out = torch.empty(x.shape[0], N, dtype=torch.float32, device=x.device)
+    call("gemm_f32", "plplpliii", ptr(W), W.stride(0), ptr(x), x.stride(0), ptr(out), N, x.shape[0], N, K)
+    return out
+
+
 GEMM_WIDE = os.environ.get("VOLTA_GEMM_WIDE", "1") != "0"
 
 

@@ -27,10 +27,14 @@ GEMV_KERNEL = os.environ.get("VOLTA_GEMV", "auto")
 
 class LinearBF16:
     def __init__(self, weight: torch.Tensor):
-        self.weight = weight.contiguous()  # [N, K]
         self.out_features, self.in_features = weight.shape
+        if self.in_features % 8:           # 16-byte rows for the loaders: zero columns behind the real ones
+            weight = torch.nn.functional.pad(weight, (0, -self.in_features % 8))
+        self.weight = weight.contiguous()  # [N, K]
 
     def forward(self, x, residual=None, out=None, out_f32=False):
+        if x.shape[1] != self.weight.shape[1]:
+            x = torch.nn.functional.pad(x, (0, self.weight.shape[1] - x.shape[1]))
         if not x.is_cuda:
             y = x.float() @ self.weight.float().t()
             if residual is not None:
@@ -47,6 +51,22 @@ class LinearBF16:
 
     def nbytes(self):
         return self.weight.numel() * self.weight.element_size()
+
+
+class LinearF32:
+    """fp32 weight and activations: the linears of a model's all-32-bit form."""
+
+    def __init__(self, weight: torch.Tensor):
+        self.weight = weight.float().contiguous()
+        self.out_features, self.in_features = weight.shape
+
+    def forward(self, x, out_f32=True):
+        if not x.is_cuda:
+            return x @ self.weight.t()
+        return K.gemm_f32(self.weight, x)
+
+    def nbytes(self):
+        return self.weight.numel() * 4
 
 
 class LinearNVFP4:

@@ -1,0 +1,121 @@
+"""Linear attention with a decayed outer-product state (csrc/cuda/linattn.cu): per slot and head an fp32 state S [dk, dv] with
+
+    S_t = diag(d_t) S_(t-1) + k_t v_t^T,     o_t = S_t^T q_t
+
+over projection rows [ q (heads dk) | x (heads dk) | v (heads dv) | ... ]; q = silu(q) and either
+
+  * ``decay`` given (lightning attention): d = decay[head], k = silu(x), v = silu(v), or
+  * ``lower`` / ``bias`` given (HGRN2): the forget gate f = lower + (1 - lower) sigmoid(x + bias) per channel is the decay and
+    its complement 1 - f the key; v as projected.
+
+A row at position 0 starts its slot from a zero state; rows of one slot inside a batch are consecutive positions in order.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from .._lib import call, ptr
+from .gdn import GDNJournal
+
+CHUNK_MIN = 16            # shortest portion that takes the chunked kernels
+
+
+@dataclass
+class LinAttnSpec:
+    heads: int
+    dk: int
+    dv: int
+    decay: torch.Tensor | None = None       # fp32 [heads]
+    lower: torch.Tensor | None = None       # fp32 [heads * dk]
+    bias: torch.Tensor | None = None        # fp32 [heads * dk]
+
+    @property
+    def mode(self) -> int:
+        return 0 if self.decay is not None else 1
+
+    @property
+    def cols(self) -> int:
+        return self.heads * (2 * self.dk + self.dv)
+
+
+class LinAttnState:
+    """rec [slots, heads, dk, dv] fp32 of one layer."""
+    conv = None
+
+    def __init__(self, spec: LinAttnSpec, max_slots: int, device):
+        self.rec = torch.zeros(max_slots, spec.heads, spec.dk, spec.dv, dtype=torch.float32, device=device)
+
+    def nbytes(self):
+        return self.rec.numel() * 4
+
+    def snapshot(self, slot: int) -> dict:
+        return {"rec": self.rec[slot].cpu().clone()}
+
+    def restore(self, slot: int, snap: dict):
+        self.rec[slot].copy_(snap["rec"])
+
+
+def gates(x, spec: LinAttnSpec):
+    """fp32 rows of the second projection block -> (decay, key), each [rows, heads, dk]."""
+    n = x.shape[0]
+    if spec.mode == 0:
+        k = torch.nn.functional.silu(x).reshape(n, spec.heads, spec.dk)
+        return spec.decay.reshape(1, spec.heads, 1).expand_as(k), k
+    z = x + spec.bias
+    f = spec.lower + (1.0 - spec.lower) * torch.sigmoid(z)
+    k = (1.0 - spec.lower) * torch.sigmoid(-z)
+    return f.reshape(n, spec.heads, spec.dk), k.reshape(n, spec.heads, spec.dk)
+
+
+def linattn_reference(proj, pos, slot, st: LinAttnState, spec: LinAttnSpec) -> torch.Tensor:
+    """CPU statement over the rows of a batch; updates ``st`` in place -> fp32 [rows, heads * dv]."""
+    n, H, dk, dv = proj.shape[0], spec.heads, spec.dk, spec.dv
+    pf = proj.float()
+    q = torch.nn.functional.silu(pf[:, : H * dk]).reshape(n, H, dk)
+    d, k = gates(pf[:, H * dk: 2 * H * dk], spec)
+    v = pf[:, 2 * H * dk: spec.cols].reshape(n, H, dv)
+    if spec.mode == 0:
+        v = torch.nn.functional.silu(v)
+    o = torch.zeros(n, H, dv)
+    for i in range(n):
+        s = int(slot[i])
+        if s < 0:
+            continue
+        S = st.rec[s]
+        if int(pos[i]) == 0:
+            S.zero_()
+        S.mul_(d[i][:, :, None]).add_(k[i][:, :, None] * v[i][:, None, :])
+        o[i] = torch.einsum("hkv,hk->hv", S, q[i])
+    return o.reshape(n, H * dv)
+
+
+def _step(proj, pos, slot, st, spec, o, rows, segs=None):
+    x32 = 1 if proj.dtype == torch.float32 else 0
+    first, count, n = segs if segs is not None else (None, None, 0)
+    call("linattn_step", "plipp" + "ppi" + "pppp" + "pliiiii", ptr(proj), proj.stride(0), x32, ptr(pos), ptr(slot), ptr(first), ptr(count), n,
+         ptr(st.rec), ptr(spec.bias), ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), rows, spec.heads, spec.dk, spec.dv, spec.mode)
+
+
+def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJournal | None = None, rows=None) -> torch.Tensor:
+    """Rows of batch ``b`` through the recurrence -> fp32 [rows, heads * dv]. ``rows`` = (pos, slot) that outlive the step
+    when ``journal`` keeps the block's operands for a replay."""
+    pos, slot = rows if rows is not None else (b.pos, b.slot)
+    if journal is not None:
+        journal.begin(st, slot)
+    if not proj.is_cuda:
+        if journal is not None:
+            journal.fn = lambda keep: linattn_reference(proj[:keep], pos[:keep], slot[:keep], st, spec)
+        return linattn_reference(proj, pos, slot, st, spec)
+    n = proj.shape[0]
+    o = torch.empty(n, spec.heads * spec.dv, dtype=torch.float32, device=proj.device)
+    if b.row_path:
+        _step(proj, pos, slot, st, spec, o, n)
+        if journal is not None:
+            o2 = torch.empty_like(o)
+            journal.fn = lambda keep: _step(proj, pos, slot, st, spec, o2, keep)
+        return o
+    t = b.segments()
+    _step(proj, pos, slot, st, spec, o, n, (t.first, t.count, t.n))
+    return o

@@ -1,0 +1,127 @@
+"""Row operators of decoders with an fp32 residual stream, and the linears of their decode steps that take the operator in
+front as a prologue (csrc/cuda/rowops.cu, gemv_rows.cu). CPU tensors run the same formulas in fp32 PyTorch.
+
+Activations are bf16, or fp32 for the all-32-bit form of a model; the residual is always fp32 and every operator computes
+in fp32.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from .._lib import call, ptr
+
+FUSED_ROWS = 8            # decode rows that take the prologue forms
+FUSED_SMEM = 200 << 10
+
+
+def _f32(t) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+@dataclass
+class DynamicTanh:
+    """y = tanh(alpha x) * w + b: an element-wise stand-in for a norm layer (no statistics)."""
+    w: torch.Tensor           # fp32
+    b: torch.Tensor           # fp32
+    alpha: float
+
+    @classmethod
+    def load(cls, src, name: str, device):
+        return cls(src.tensor(name, device, torch.float32).contiguous(), src.tensor(name + ".b", device, torch.float32).contiguous(),
+                   float(src.tensor(name + ".alpha").float()))
+
+    def rows(self, h, out_dtype, part=None, scale=None):
+        """h += scale * part (in place, optional), then the norm of h."""
+        rows, H = h.shape
+        if not h.is_cuda:
+            if part is not None:
+                h += part.float() * (scale if scale is not None else 1.0)
+            return (torch.tanh(self.alpha * h) * self.w + self.b).to(out_dtype)
+        out = torch.empty(rows, H, dtype=out_dtype, device=h.device)
+        call("dyt_rows", "pplpppfpliii", ptr(h), ptr(part), part.stride(0) if part is not None else 0, ptr(scale), ptr(self.w), ptr(self.b),
+             self.alpha, ptr(out), out.stride(0), rows, H, _f32(out))
+        return out
+
+    def prologue(self, h):
+        return {"pro": 1, "x": h, "w": self.w, "b": self.b, "alpha": self.alpha}
+
+
+@dataclass
+class GroupRMS:
+    """RMS norm over groups of ``group`` columns (0: the whole row) with a plain weight that repeats with its own length,
+    optionally times sigmoid(gate)."""
+    w: torch.Tensor           # fp32
+    eps: float
+    group: int = 0
+
+    def rows(self, x, out_dtype, gate=None):
+        rows, cols = x.shape
+        G = self.group or cols
+        if not x.is_cuda:
+            v = x.float().reshape(rows, cols // G, G)
+            v = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + self.eps)).reshape(rows, cols)
+            v = v * self.w.repeat(cols // self.w.numel())
+            if gate is not None:
+                v = v * torch.sigmoid(gate.float())
+            return v.to(out_dtype)
+        out = torch.empty(rows, cols, dtype=out_dtype, device=x.device)
+        assert gate is None or gate.dtype == x.dtype
+        call("group_rms", "plipipl" + "pliiifi", ptr(x), x.stride(0), _f32(x), ptr(self.w), self.w.numel(), ptr(gate),
+             gate.stride(0) if gate is not None else 0, ptr(out), out.stride(0), rows, cols, G, float(self.eps), _f32(out))
+        return out
+
+    def prologue(self, x, gate=None):
+        return {"pro": 2, "x": x, "w": self.w, "G": self.group or x.shape[1], "wlen": self.w.numel(), "gate": gate, "eps": self.eps}
+
+
+@dataclass
+class PolyNorm:
+    """c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 with N = division by the row's root mean square."""
+    coef: torch.Tensor        # fp32 [4]
+    eps: float
+
+    def rows(self, z, out_dtype):
+        rows, F = z.shape
+        if not z.is_cuda:
+            v = z.float()
+            n = [p / torch.sqrt(p.pow(2).mean(-1, keepdim=True) + self.eps) for p in (v, v * v, v * v * v)]
+            return (self.coef[0] * n[0] + self.coef[1] * n[1] + self.coef[2] * n[2] + self.coef[3]).to(out_dtype)
+        out = torch.empty(rows, F, dtype=out_dtype, device=z.device)
+        call("polynorm", "plipplii" + "fi", ptr(z), z.stride(0), _f32(z), ptr(self.coef), ptr(out), out.stride(0), rows, F, float(self.eps), _f32(out))
+        return out
+
+    def prologue(self, z):
+        return {"pro": 3, "x": z, "coef": self.coef, "eps": self.eps}
+
+
+def embed_rows(ids, table):
+    """-> fp32 [rows, H]."""
+    if not table.is_cuda:
+        return table[ids.long()].float()
+    V, H = table.shape
+    out = torch.empty(ids.numel(), H, dtype=torch.float32, device=table.device)
+    call("embed_rows", "pppiiii", ptr(ids), ptr(table), ptr(out), ids.numel(), H, V, _f32(table))
+    return out
+
+
+def fused_fits(lin, rows: int) -> bool:
+    """The prologue form of ``lin`` takes this many rows."""
+    return rows <= FUSED_ROWS and rows * (lin.weight.shape[1] + 64) * 2 <= FUSED_SMEM
+
+
+def gemv_rows(lin, M: int, *, x, pro=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, out_f32=False, residual=None):
+    """A bf16 linear on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
+    ``residual`` = (h fp32, scale | None): h += scale * y in place; otherwise the product is returned."""
+    W = lin.weight
+    N, K = W.shape
+    dev = W.device
+    out = None
+    if residual is None:
+        out = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=dev)
+    h, scale = residual if residual is not None else (None, None)
+    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp", ptr(W), W.stride(0), N, K, M, pro, x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
+         float(alpha), G, wlen, ptr(gate), gate.stride(0) if gate is not None else 0, ptr(coef), float(eps),
+         ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, N, ptr(h), h.stride(0) if h is not None else 0, ptr(scale))
+    return out

@@ -16,6 +16,66 @@ MAX_CHUNK_ROWS = 4096  # prefill chunk upper bound
 LOGITS_ALL = "all"
 LOGITS_LAST = "last"
 LOGITS_NONE = "none"
+LOGITS_ROWS = "rows"   # the rows listed in BatchRows.want
+
+LONG_SEGMENT = 16      # portions of at least this many rows take the prompt kernels, shorter ones the decode kernels
+
+
+@dataclass
+class SegmentTable:
+    """Runs of consecutive rows of one slot inside a batch that is known on the host. Device tables are int32."""
+    n: int                          # segments
+    first: torch.Tensor             # [n] first row
+    count: torch.Tensor             # [n] rows
+    host: list                      # [(slot, first row, rows, first position)]
+    short_rows: int                 # leading rows that belong to segments shorter than LONG_SEGMENT
+    ctx_slot: torch.Tensor | None   # per segment behind those rows: its slot and the first row of its context when the contexts
+    ctx_base: torch.Tensor | None   # (positions 0 .. last) of these segments are laid out one after the other
+    ctx_total: int
+    tile_first: torch.Tensor | None  # tiles of at most 64 rows of one of these segments; rows counted from short_rows
+    tile_count: torch.Tensor | None
+    tile_base: torch.Tensor | None   # the segment's ctx_base
+    chunk_seg: torch.Tensor | None   # chunks of at most 64 rows of these segments: segment (0 = the first behind short_rows),
+    chunk_first: torch.Tensor | None  # first row (in the batch) and rows
+    chunk_count: torch.Tensor | None
+    seg_chunk0: torch.Tensor | None   # [segments + 1] first chunk of every such segment
+
+    @classmethod
+    def build(cls, slots, pos, device):
+        host, i, n = [], 0, len(slots)
+        while i < n:
+            j = i
+            while j < n and slots[j] == slots[i] and pos[j] == pos[i] + (j - i):
+                j += 1
+            host.append((slots[i], i, j - i, pos[i]))
+            i = j
+
+        def dev(v):
+            return torch.tensor(v, dtype=torch.int32).to(device, non_blocking=True)
+        k = 0
+        while k < len(host) and host[k][2] < LONG_SEGMENT:
+            k += 1
+        rest = host[k:]
+        short = rest[0][1] if rest else n
+        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 7))
+        if rest:
+            base, total = [], 0
+            tf, tc, tb, cs, cf, cc, c0 = [], [], [], [], [], [], [0]
+            for g, (s, f, c, p0) in enumerate(rest):
+                base.append(total)
+                for o in range(0, c, 64):
+                    tf.append(f + o - short)
+                    tc.append(min(64, c - o))
+                    tb.append(total)
+                    cs.append(g)
+                    cf.append(f + o)
+                    cc.append(min(64, c - o))
+                c0.append(len(cs))
+                total += p0 + c
+            t.ctx_slot, t.ctx_base, t.ctx_total = dev([h[0] for h in rest]), dev(base), total
+            t.tile_first, t.tile_count, t.tile_base = dev(tf), dev(tc), dev(tb)
+            t.chunk_seg, t.chunk_first, t.chunk_count, t.seg_chunk0 = dev(cs), dev(cf), dev(cc), dev(c0)
+        return t
 
 
 @dataclass
@@ -34,6 +94,28 @@ class BatchRows:
     embeds: torch.Tensor | None = None      # [n, H] rows that replace the token embedding where embed_mask is set
     embed_mask: torch.Tensor | None = None  # [n] bool
     tree: tuple | None = None               # (base int32 [n], mask int64 [n]): rows of a verification tree (ops.kernels.attention)
+
+    want: torch.Tensor | None = None        # LOGITS_ROWS: int64 row indices
+    seg_table: SegmentTable | None = None
+
+    @property
+    def row_path(self) -> bool:
+        """Few rows: kernels that handle every row by itself (and find rows of one slot on the device)."""
+        return self.n <= MAX_GRAPH_ROWS
+
+    def segments(self) -> SegmentTable:
+        if self.seg_table is None:
+            assert len(self.host_slots) == self.n, "the batch's rows are not known on the host"
+            self.seg_table = SegmentTable.build(self.host_slots, self.host_pos, self.ids.device)
+        return self.seg_table
+
+    def select_logits(self, x):
+        """Rows of ``x`` whose logits are asked for (None: no rows)."""
+        if self.logits == LOGITS_NONE:
+            return None
+        if self.logits == LOGITS_LAST:
+            return x[self.n - 1: self.n]
+        return x.index_select(0, self.want) if self.logits == LOGITS_ROWS else x
 
     @classmethod
     def make(cls, ids, pos, slots, device, logits=LOGITS_ALL, G=1, prefill=False, nsplit=1):

@@ -16,7 +16,7 @@ from dataclasses import dataclass
 import torch
 
 from ..ops import kernels as K
-from .batch import BatchRows, LOGITS_ALL, LOGITS_LAST, LOGITS_NONE, MAX_GRAPH_ROWS
+from .batch import BatchRows, LOGITS_ALL, LOGITS_LAST, LOGITS_NONE, LOGITS_ROWS, MAX_GRAPH_ROWS
 from .kv_cache import PagedKVCache
 
 
@@ -72,6 +72,7 @@ class Engine:
         pin = self.cuda
         self.h_in = torch.zeros(3, R, dtype=torch.int32, pin_memory=pin)
         self.h_tok = torch.zeros(R, dtype=torch.int32, pin_memory=pin)
+        self._h_in_read = None
         from .sampling import NUM_CANDIDATES
         self.s_cand_ids = torch.zeros(R, NUM_CANDIDATES, dtype=torch.int32, device=dev)
         self.s_cand_vals = torch.zeros(R, NUM_CANDIDATES, dtype=torch.float32, device=dev)
@@ -163,7 +164,7 @@ class Engine:
             self.model.begin_journal(journal, rows)
         key = (rows, nsplit, self.feedback, topk, journal)
         if not self.use_graphs or rows > MAX_GRAPH_ROWS:
-            self._forward_static(rows, nsplit, topk)
+            self.row_logits = self._forward_static(rows, nsplit, topk)
             return
         g = self.graphs.get(key)
         if g is None:
@@ -171,25 +172,33 @@ class Engine:
         g.calls += 1
         if g.graph is not None:
             g.graph.replay()
+            self.row_logits = g.logits
         elif g.calls == 1:
-            self._forward_static(rows, nsplit, topk)
+            self.row_logits = self._forward_static(rows, nsplit, topk)
         else:
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(graph):
-                self._forward_static(rows, nsplit, topk)
+                g.logits = self._forward_static(rows, nsplit, topk)
             g.graph = graph
             graph.replay()
+            self.row_logits = g.logits
 
     def set_rows(self, ids: list[int], pos: list[int], slots: list[int]):
         """Upload one step's row descriptor from pinned host memory (async on the current stream)."""
         n = len(ids)
+        if self._h_in_read is not None:            # the copies of the step in front may still read the pinned rows
+            self._h_in_read.synchronize()
         self.h_in[0, :n] = torch.tensor(ids, dtype=torch.int32)
         self.h_in[1, :n] = torch.tensor(pos, dtype=torch.int32)
         self.h_in[2, :n] = torch.tensor(slots, dtype=torch.int32)
         self.s_ids[:n].copy_(self.h_in[0, :n], non_blocking=True)
         self.s_pos[:n].copy_(self.h_in[1, :n], non_blocking=True)
         self.s_slot[:n].copy_(self.h_in[2, :n], non_blocking=True)
+        if self.cuda:
+            if self._h_in_read is None:
+                self._h_in_read = torch.cuda.Event()
+            self._h_in_read.record()
 
     @property
     def supports_journal(self) -> bool:
@@ -255,13 +264,20 @@ class Engine:
     def step_candidates(self, ids: list[int], pos: list[int], slots: list[int], journal: bool = False):
         """Like :meth:`step` but returns, per row, the merged top-16 candidates (ids, logits, lse) for the
         host sampler instead of the greedy token."""
-        from .sampling import Candidates, merge_shards
         n = len(ids)
         for s, p in zip(slots, pos):
             self.kv.reserve(s, p + 2)
         self.set_rows(ids, pos, slots)
         self._run_rows(n, topk=True, journal=journal)
-        cid, cval, clse = self.s_cand_ids[:n], self.s_cand_vals[:n], self.s_cand_lse[:n]
+        return self._merge_candidates(self.s_cand_ids[:n], self.s_cand_vals[:n], self.s_cand_lse[:n])
+
+    def _candidates(self, logits):
+        from .sampling import NUM_CANDIDATES
+        return self._merge_candidates(*K.topk(logits.contiguous(), NUM_CANDIDATES, self.comm.rank * self.model.vocab_local))
+
+    def _merge_candidates(self, cid, cval, clse):
+        from .sampling import Candidates, merge_shards
+        n = cid.shape[0]
         if self.comm.size > 1:
             cid, cval, clse = (self.comm.all_gather_rows(t) for t in (cid, cval, clse))
         cid, cval, clse = cid.cpu(), cval.cpu(), clse.cpu()
@@ -308,8 +324,63 @@ class Engine:
         if not want_token:
             return -1
         rows = logits.shape[0]
+        self.row_logits = logits
         self._sample_greedy(logits, self.s_tok, self.s_val, rows)
         return int(self.s_tok[rows - 1].item())
+
+    def prefill_candidates(self):
+        """Candidates (as :meth:`step_candidates` returns them) of the last row of the last ``prefill_rows(want_token=True)``:
+        what a sampled request's first token comes from when its prompt row must not run twice (recurrent state)."""
+        return self._candidates(self.row_logits[-1:])[0]
+
+    # ------------------------------------------------------------------------------------------ mixed batches
+    @property
+    def supports_mixed(self) -> bool:
+        """Models that take prompt portions and decode rows of several sequences in one forward."""
+        return bool(getattr(self.model, "supports_mixed", False))
+
+    def forward_segments(self, segs) -> torch.Tensor | None:
+        """One forward over ``segs`` = [(slot, tokens, first position, [places among the tokens whose logits are wanted])]:
+        portions of prompts beside single decode rows. Every slot appears once. Returns the wanted fp32 logits in the order of
+        the arguments ([wanted, local vocabulary]; None when nothing is wanted). Valid until the next step."""
+        for slot, toks, p0, _ in segs:
+            self.kv.reserve(slot, p0 + len(toks))
+        total = sum(len(s[1]) for s in segs)
+        n_want = sum(len(s[3]) for s in segs)
+        if total <= MAX_GRAPH_ROWS and all(len(s[1]) == 1 for s in segs):
+            # decode rows only: the step's own path (graph replay)
+            self.set_rows([s[1][0] for s in segs], [s[2] for s in segs], [s[0] for s in segs])
+            self._run_rows(total)
+            idx = [r for r, s in enumerate(segs) for _ in s[3]]
+            if not idx:
+                return None
+            return self.row_logits[:total] if idx == list(range(total)) else self.row_logits[torch.tensor(idx, device=self.device)]
+        order = sorted(range(len(segs)), key=lambda i: len(segs[i][1]))         # short segments in front (decode kernels)
+        ids, pos, slots, at = [], [], [], {}
+        for i in order:
+            slot, toks, p0, _ = segs[i]
+            at[i] = len(ids)
+            ids += toks
+            pos += range(p0, p0 + len(toks))
+            slots += [slot] * len(toks)
+        if self.supports_journal:
+            self.model.begin_journal(False, total)
+        b = BatchRows.make(ids, pos, slots, self.device, LOGITS_ROWS if n_want else LOGITS_NONE, 1, prefill=False, nsplit=self._nsplit(total))
+        if n_want:
+            b.want = torch.tensor([at[i] + w for i, s in enumerate(segs) for w in s[3]], dtype=torch.int64).to(self.device, non_blocking=True)
+        return self.model.forward(b, self.kv)
+
+    def step_mixed(self, segs, candidates: bool = False) -> list:
+        """:meth:`forward_segments`, then the greedy token (or the candidates) of every wanted row."""
+        logits = self.forward_segments(segs)
+        if logits is None:
+            return []
+        if candidates:
+            return self._candidates(logits)
+        n = logits.shape[0]
+        tok, val = torch.empty(n, dtype=torch.int32, device=self.device), torch.empty(n, dtype=torch.float32, device=self.device)
+        self._sample_greedy(logits, tok, val, n)
+        return tok.tolist()
 
     def decode_chain(self, first_ids: list[int], pos: list[int], slots: list[int], steps: int) -> torch.Tensor:
         """``steps`` greedy steps for the given rows with the token fed back on the device (no host sync

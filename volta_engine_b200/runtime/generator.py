@@ -180,6 +180,10 @@ class Generator:
         self.prefill_cooldown = max(0, getattr(options, "prefill_cooldown", 0)) if options else 0
         self._since_prefill = 1 << 30
         self.cache_reply = getattr(options, "prefix_cache_reply", True) if options else True
+        # a sampled request's first token: models without per-slot recurrent state run the prompt's last row once more
+        self.rerun_last_row = not (self._state_snaps and self.speculator != "mtp")
+        # prompt portions beside decode rows in one forward (plain decoding only: speculative rounds keep their own steps)
+        self.mixed = bool(getattr(engine, "supports_mixed", False)) and self.speculator == "none"
         self.drafter = None                    # block drafter (speculator "dflash"): object with draft(slot, anchor, pos, depth)
         self.mtp = None
         if self.speculator == "mtp":
@@ -261,8 +265,13 @@ class Generator:
                     return
 
     def step(self):
-        """One scheduler iteration: admit, one prefill slice, one decode / speculative step."""
+        """One scheduler iteration: admit, one prefill slice, one decode / speculative step; models that take mixed batches
+        run the prompt portions and the decode rows of the iteration in one forward."""
         self._admit()
+        if self._mixed_ready():
+            prefilled, decoded = self._mixed_step()
+            self.metrics.tick(decoded, prefilled, sum(1 for s in self.slots if s.phase != "idle"))
+            return
         prefilled = self._prefill_slice()
         decoded = self._decode_step()
         active = sum(1 for s in self.slots if s.phase != "idle")
@@ -337,6 +346,78 @@ class Generator:
         self.metrics.prompt_tokens += len(req.prompt)
         self.metrics.cached_tokens += s.cached_tokens
 
+    # ------------------------------------------------------------------------------------------ mixed batches
+    def _mixed_ready(self) -> bool:
+        """Something to prefill beside something else to run. A prompt alone and decode rows alone keep their own steps."""
+        if not self.mixed or self.drafter is not None:
+            return False
+        pre = [s for s in self.slots if s.phase == "prefill" and not s.req.cancelled]
+        if not pre or any(s.req.mm is not None or s.req.steer_probe for s in pre) or getattr(self, "probe_files", None):
+            return False
+        dec = sum(1 for s in self.slots if s.phase == "decode")
+        if dec and self._since_prefill < self.prefill_cooldown:
+            return False
+        return dec > 0 or len(pre) > 1
+
+    def _mixed_step(self) -> tuple[int, int]:
+        """One forward over the next portion of every prompt in turn (as many rows as a chunk holds) and one row of every
+        decoding slot. Returns (prompt rows, decode rows)."""
+        for s in [s for s in self.slots if s.req is not None and s.req.cancelled]:
+            self._finish(s, "cancelled")
+        self._since_prefill = 0
+        t0 = time.time()
+        dec = [s for s in self.slots if s.phase == "decode"]
+        segs = [(s.idx, [s.next_tok], s.pos, [0]) for s in dec]
+        room = max(1, self.engine.prefill_chunk - len(dec))
+        pre = []
+        for s in sorted((s for s in self.slots if s.phase == "prefill"), key=lambda s: s.t_start):
+            if room <= 0:
+                break
+            end = min(len(s.req.prompt), s.cursor + room)
+            end = min([end] + [p for p in self._snapshot_points(s) if s.cursor < p])
+            last = end == len(s.req.prompt)
+            pre.append((s, end, last))
+            segs.append((s.idx, list(s.req.prompt[s.cursor:end]), s.cursor, [end - s.cursor - 1] if last else []))
+            room -= end - s.cursor
+        ask = dec + [s for s, _, last in pre if last]
+        sampled = any(not s.req.params.greedy or s.req.params.logprobs for s in ask)
+        res = self.engine.step_mixed(segs, candidates=sampled)
+        ms = (time.time() - t0) * 1e3
+        got = {}
+        for s, r in zip(ask, res):
+            if sampled:
+                c = penalize(r, s.req.params, s.counts.counts)
+                got[s.idx] = (sample_token(c, s.req.params, s.rng), r)
+            else:
+                got[s.idx] = (r, None)
+        rows = 0
+        for s, end, last in pre:
+            rows += end - s.cursor
+            s.cursor = s.pos = end
+            s.t_prefill_ms += ms
+            if self.cache is not None and s.req.cache_prefix and end in self._snapshot_points(s):
+                self._store_prefix(s, end)
+            if last:
+                s.next_tok, s.phase = got[s.idx][0], "decode"
+        self.metrics.tokens_prefilled += rows
+        for s in dec:
+            t, c = got[s.idx]
+            t = self._think_gate(s, t)
+            s.pos += 1
+            s.next_tok = t
+            self._emit(s, [t], self._logprobs(s, t, c))
+        for s, _, last in pre:
+            if last:
+                self._emit(s, [s.next_tok])
+        return rows, len(dec)
+
+    @staticmethod
+    def _logprobs(s: SlotState, t: int, c):
+        if c is None or not s.req.params.logprobs:
+            return None
+        return [{"token": t, "logprob": logprob_of(c, t),
+                 "top": [(i, l - c.lse) for i, l in list(zip(c.ids, c.logits))[: s.req.params.logprobs]]}]
+
     # ------------------------------------------------------------------------------------------ prefill
     def _snapshot_points(self, s: SlotState) -> list[int]:
         n = len(s.req.prompt)
@@ -387,10 +468,13 @@ class Generator:
                 s.phase = "decode"
                 s.t_prefill_ms += (time.time() - t0) * 1e3
                 if not s.req.params.greedy:
-                    # re-run the last row through the candidate path so the first token is sampled, not argmax
-                    s.pos -= 1
-                    cand = self.engine.step_candidates([prompt[-1]], [s.pos], [s.idx])[0]
-                    s.pos += 1
+                    if self.rerun_last_row:
+                        # re-run the last row through the candidate path so the first token is sampled, not argmax
+                        s.pos -= 1
+                        cand = self.engine.step_candidates([prompt[-1]], [s.pos], [s.idx])[0]
+                        s.pos += 1
+                    else:                     # the row already advanced the slot's recurrent state
+                        cand = self.engine.prefill_candidates()
                     cand = penalize(cand, s.req.params, s.counts.counts)
                     s.next_tok = sample_token(cand, s.req.params, s.rng)
                 self.metrics.tokens_prefilled += done_rows
@@ -486,11 +570,7 @@ class Generator:
             s.next_tok = t
             if s.ctrl is not None:
                 s.ctrl.record_plain(ms)
-            lp = None
-            if c is not None and s.req.params.logprobs:
-                lp = [{"token": t, "logprob": logprob_of(c, t),
-                       "top": [(i, l - c.lse) for i, l in list(zip(c.ids, c.logits))[: s.req.params.logprobs]]}]
-            self._emit(s, [t], lp)
+            self._emit(s, [t], self._logprobs(s, t, c))
         return len(act)
 
     def _think_gate(self, s: SlotState, t: int) -> int:

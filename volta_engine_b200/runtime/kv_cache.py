@@ -19,7 +19,8 @@ class OutOfPages(RuntimeError):
 
 # whole-cache element formats: bf16, E5M2 bytes, or the scaled forms "k8v4" (int8 keys + 4-bit Hadamard-rotated values, one
 # fp16 scale per 64 elements) and "nvfp4" (E2M1 with one E4M3 scale per 16). Attention expands pages to bf16 on chip.
-KV_FORMATS = {"bf16": torch.bfloat16, "fp16": torch.bfloat16, "fp8": torch.float8_e5m2, "k8v4": "k8v4", "nvfp4": "nvfp4"}
+KV_FORMATS = {"bf16": torch.bfloat16, "fp16": torch.bfloat16, "fp8": torch.float8_e5m2, "k8v4": "k8v4", "nvfp4": "nvfp4",
+              "fp32": torch.float32}   # fp32: caches of models that run in 32-bit throughout
 
 
 class PagedKVCache:

@@ -17,6 +17,7 @@ _TABLE = [
     ("max_slots", int, 8, "concurrent sequences"),
     ("kv_pool", int, 0, "KV pool size in tokens (0 = size from free memory)"),
     ("kv_format", str, "bf16", "KV cache element format: bf16 | fp8 | k8v4 | nvfp4"),
+    ("dtype", str, "bf16", "arithmetic of the model families that offer both: bf16 | fp32 (32-bit throughout; kv_format follows)"),
     ("vram_reserve_mib", int, 2048, "device memory left unallocated"),
     ("prefill_chunk", int, 2048, "rows per prefill forward"),
     ("spec_tree", int, 0, "suffix speculator: > 1 verifies up to this many different continuations of the current suffix "

@@ -110,7 +110,8 @@ class _SnapHandle:
         return (int, (self.hid,))
 
 
-_ENGINE_CALLS = ("prefill", "prefill_rows", "step", "step_candidates", "decode_chain", "set_rows")
+_ENGINE_CALLS = ("prefill", "prefill_rows", "step", "step_candidates", "decode_chain", "set_rows",
+                 "prefill_candidates", "forward_segments", "step_mixed")
 _KV_CALLS = ("reserve", "release")
 
 

@@ -168,7 +168,8 @@ def build_engine(cfg: LaunchConfig, device=None, comm=None, agree=None):
     device = device or ("cuda:0" if torch.cuda.is_available() else "cpu")
     overlay = {k: getattr(o, k) for k in ("nvfp4_experts", "nvfp4_expert_layers", "mtp_head_dir", "mtp_nvfp4", "nvfp4_dense_dir", "nvfp4_dense_src")
                if getattr(o, k)}
-    model, hf = load_model(cfg.model_dir, device, comm, gemm_mode=o.gemm_mode, overlay=overlay or None, nvfp4_dense=o.nvfp4_dense)
+    model, hf = load_model(cfg.model_dir, device, comm, gemm_mode=o.gemm_mode, overlay=overlay or None, nvfp4_dense=o.nvfp4_dense,
+                           dtype=o.dtype)
     mcfg = model.cfg
     model.side_streams = bool(o.side_streams)
     if o.trace_layers:
@@ -177,11 +178,13 @@ def build_engine(cfg: LaunchConfig, device=None, comm=None, agree=None):
     configure_expert_tier(model, o, getattr(comm, "rank", 0) if comm is not None else 0)
     configure_cpu_experts(model, o)
     from ..runtime.kv_cache import KV_FORMATS
-    if o.kv_format not in KV_FORMATS:
-        raise ValueError(f"kv_format '{o.kv_format}': this build has {sorted(KV_FORMATS)}")
+    kv_format = "fp32" if o.dtype in ("fp32", "float32") else o.kv_format
+    if kv_format not in KV_FORMATS:
+        raise ValueError(f"kv_format '{kv_format}': this build has {sorted(KV_FORMATS)}")
     # bytes per cached element, scales included: bf16 2, E5M2 1, k8v4 (1 + 1/32 + 1/2 + 1/32) / 2, nvfp4 1/2 + 1/16
-    kv_bytes = {"fp8": 1.0, "k8v4": 0.78125, "nvfp4": 0.5625}.get(o.kv_format, 2.0)
-    bpt = int(getattr(model, "kv_layers", mcfg.n_layers) * model.nkv * 2 * mcfg.head_dim * kv_bytes)
+    kv_bytes = {"fp8": 1.0, "k8v4": 0.78125, "nvfp4": 0.5625, "fp32": 4.0}.get(kv_format, 2.0)
+    v_dim = getattr(model, "kv_v_dim", mcfg.head_dim)             # models with one cached row per token need no value pool
+    bpt = max(1, int(getattr(model, "kv_layers", mcfg.n_layers) * model.nkv * (mcfg.head_dim + v_dim) * kv_bytes))
     on_gpu = torch.device(device).type == "cuda"
     scratch_bytes = max(0, o.scratch_mib) << 20
     budget = None
@@ -201,17 +204,17 @@ def build_engine(cfg: LaunchConfig, device=None, comm=None, agree=None):
     if agree is not None:
         pool_tokens = agree(pool_tokens)
     kv_layers = getattr(model, "kv_layers", mcfg.n_layers)       # hybrid models keep KV only for their attention layers
-    pages = max(2, pool_tokens // 64)
+    pages = max(2, pool_tokens // 64 + 1)                        # page 0 is the null page
     arena = scratch = None
     if on_gpu:
         from ..ops import kernels as K
         from ..runtime.arena import Arena, ScratchRegistry
-        arena = Arena(PagedKVCache.pool_bytes(kv_layers, model.nkv, mcfg.head_dim, pages, o.kv_format) + scratch_bytes
+        arena = Arena(PagedKVCache.pool_bytes(kv_layers, model.nkv, mcfg.head_dim, pages, kv_format, v_dim) + scratch_bytes
                       + (1 << 20), device)
         scratch = ScratchRegistry(arena, overflow=True)
         K.use_scratch(scratch, device)
     kv = PagedKVCache(kv_layers, model.nkv, mcfg.head_dim, pages, o.max_slots, o.max_seq, device,
-                      dtype=o.kv_format, arena=arena)
+                      dtype=kv_format, v_head_dim=v_dim, arena=arena)
     engine = Engine(model, kv, use_graphs=not o.no_graphs and torch.device(device).type == "cuda",
                     prefill_chunk=o.prefill_chunk)
     engine.arena, engine.scratch = arena, scratch
@@ -408,7 +411,7 @@ def build_server(cfg: LaunchConfig, device=None, comm=None, chan=None, agree=Non
         # compressor rings, indexer keys) run without the cache instead of resuming from a stale state
         from ..runtime.prefix_cache import model_fingerprint
         kvc = engine.kv
-        fp = model_fingerprint(cfg.model_dir, kv_format=o.kv_format, tp=cfg.tp_size, layers=kvc.n_layers, kv_heads=kvc.n_kv,
+        fp = model_fingerprint(cfg.model_dir, kv_format=o.kv_format if o.dtype == "bf16" else o.dtype, tp=cfg.tp_size, layers=kvc.n_layers, kv_heads=kvc.n_kv,
                                head_dim=kvc.head_dim, v_head_dim=kvc.v_head_dim, model_type=getattr(model.cfg, "model_type", ""))
         cache = PrefixCache(o.prefix_cache_mib << 20, o.prefix_cache_dir or None, fingerprint=fp,
                             disk_budget_bytes=max(0, o.prefix_cache_disk_gib) << 30)
@@ -471,7 +474,7 @@ def build_server(cfg: LaunchConfig, device=None, comm=None, chan=None, agree=Non
             if k in gc:
                 defaults[k] = gc[k]
     name = cfg.model_name or os.path.basename(os.path.normpath(cfg.model_dir))
-    srv = VoltaServer(gen, tok, template, model_name=name, model_type=hf.get("model_type", "dense"), host=cfg.host,
+    srv = VoltaServer(gen, tok, template, model_name=name, model_type=hf.get("model_type", "") or getattr(model.cfg, "model_type", "dense"), host=cfg.host,
                       port=cfg.port, api_key=cfg.api_key, defaults=defaults, max_context=o.max_seq,
                       default_max_tokens=cfg.default_max_tokens, request_timeout_s=cfg.request_timeout_s,
                       info={"tp": o.tp, "kv_tokens": pool_tokens, "options": dict(o.values)})
