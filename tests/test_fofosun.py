@@ -1,0 +1,227 @@
+"""The Fofosun decoder against its plain statement: whole prompts, portions, token-by-token decoding, mixed batches, slots and
+pages that are used again, long decoding; in fp32 and bf16, on the CPU statements and on the GPU kernels."""
+import io
+import json
+
+import pytest
+import torch
+
+from fofosun_util import CONFIGS, DEVICES, DTYPES, TOL, engine, make, off, one_thread, reference, tokens, write_model  # noqa: F401
+
+NAMES = list(CONFIGS)
+
+
+def run(eng, slot, toks, cuts, p0=0):
+    """Tokens of one sequence in portions of the given sizes -> logits of all of them."""
+    out, at = [], 0
+    for c in cuts:
+        part = toks[at:at + c]
+        out.append(eng.forward_segments([(slot, part, p0 + at, list(range(len(part))))]).float().clone())
+        at += c
+    assert at == len(toks)
+    return torch.cat(out)
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_whole_prompt(name, dtype, device):
+    cfg, _, model = make(name, device, dtype)
+    toks = tokens(150, cfg["vocab"])
+    got = run(engine(model), 2, toks, [150])
+    assert got.shape == (150, cfg["vocab"]) and off(got, reference(name, toks)) < TOL[dtype]
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_residual_after_every_layer(device):
+    import fofosun_plain as plain
+    cfg, w, model = make("eights", device, "fp32")
+    toks = tokens(40, cfg["vocab"], 5)
+    _, want = plain.forward(cfg, w, toks)
+    for cuts in ([40], [1] * 40):
+        model.layer_tap = tap = []
+        try:
+            run(engine(model, use_graphs=False), 0, toks, cuts)
+        finally:
+            model.layer_tap = None
+        n = len(cfg["layers"])
+        got = torch.cat([torch.stack(tap[i:i + n]) for i in range(0, len(tap), n)], 1).double().cpu()
+        assert (got - want).abs().max() < 2e-4 * want.abs().max()
+
+
+CUTS = {"one by one": [1] * 150, "twos": [2] * 75, "prompt then decode": [110] + [1] * 40, "around pages": [63, 1, 1, 63, 2, 20],
+        "short and long": [3, 17, 2, 64, 15, 16, 33], "halves": [75, 75]}
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["eights", "odd", "wide"])
+def test_portions_and_decoding(name, dtype, device):
+    cfg, _, model = make(name, device, dtype)
+    toks = tokens(150, cfg["vocab"])
+    want = reference(name, toks)
+    eng = engine(model)
+    for i, (what, cuts) in enumerate(CUTS.items()):
+        if device == "cpu" and dtype == "bf16" and i % 2:
+            continue
+        slot = i % 4
+        assert off(run(eng, slot, toks, cuts), want) < TOL[dtype], what
+        eng.kv.release(slot)                     # the next way of cutting gets used pages and a used state slot
+    assert eng.kv.free_pages() == eng.kv.num_pages - 1
+
+
+def schedule(lengths, seed):
+    """Random steps over several requests: portions of some beside single tokens of others; at most four live at once."""
+    g = torch.Generator().manual_seed(seed)
+    left, live, steps = list(range(len(lengths))), [], []
+    done = [0] * len(lengths)
+    while left or live:
+        while left and len(live) < 4:
+            live.append(left.pop(0))
+        step, ended = [], []
+        for r in list(live):
+            if len(live) > 1 and torch.rand((), generator=g) < 0.2:
+                continue                         # left out of this step
+            rest = lengths[r] - done[r]
+            n = [1, 1, 2, 3, 16, 29, 64, 90][int(torch.randint(0, 8, (), generator=g))] if rest > 12 else 1
+            n = min(n, rest)
+            step.append((r, done[r], n))
+            done[r] += n
+            if done[r] == lengths[r]:
+                ended.append(r)
+        live = [r for r in live if r not in ended]
+        if step:
+            steps.append((step, ended))
+    return steps
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["eights", "odd", "recurrent"])
+def test_mixed_batches_equal_each_alone(name, dtype, device):
+    cfg, _, model = make(name, device, dtype)
+    lengths = [150, 1, 23, 97, 64, 65, 130, 2]
+    seqs = [tokens(150, cfg["vocab"])[:n] if n != 97 else tokens(97, cfg["vocab"], 9) for n in lengths]
+    full = reference(name, seqs[0])
+    want = [full[:n] if n != 97 else reference(name, seqs[3]) for n in lengths]
+    pages = 1 + 3 * 3 + 2                        # what four live requests need at most: pages come round again
+    eng = engine(model, pages=pages if model.kv_layers else 12)
+    slots, free = {}, [3, 2, 1, 0]
+    worst = 0.0
+    for step, ended in schedule(lengths, 11):
+        segs = []
+        for r, at, n in step:
+            if r not in slots:
+                slots[r] = free.pop()
+            segs.append((slots[r], seqs[r][at:at + n], at, list(range(n))))
+        got = eng.forward_segments(segs)
+        exp = torch.cat([want[r][at:at + n] for r, at, n in step])
+        worst = max(worst, off(got, exp))
+        for r in ended:
+            eng.kv.release(slots[r])
+            free.append(slots.pop(r))
+    assert worst < TOL[dtype]
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_only_the_wanted_rows_come_back_in_order(device):
+    cfg, _, model = make("eights", device, "fp32")
+    a, b = tokens(40, cfg["vocab"], 1), tokens(9, cfg["vocab"], 2)
+    ra, rb = reference("eights", a), reference("eights", b)
+    eng = engine(model)
+    got = eng.forward_segments([(0, a[:30], 0, [29, 3]), (1, b[:5], 0, []), (2, b[:7], 0, [0, 6])])
+    assert off(got, torch.stack([ra[29], ra[3], rb[0], rb[6]])) < 1e-4
+    assert eng.forward_segments([(0, a[30:31], 30, []), (1, b[5:6], 5, [])]) is None
+    got = eng.forward_segments([(1, b[6:7], 6, [0]), (0, a[31:32], 31, []), (2, b[7:8], 7, [0])])
+    assert off(got, torch.stack([rb[6], rb[7]])) < 1e-4
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_decoding_keeps_the_state(dtype, device):
+    cfg, _, model = make("eights", device, dtype)
+    n = 400 if device == "cuda" else 230
+    toks = tokens(n, cfg["vocab"], 4)
+    eng = engine(model)
+    got = run(eng, 1, toks, [20] + [1] * (n - 20))
+    assert off(got, reference("eights", toks)) < TOL[dtype]
+
+
+@pytest.mark.gpu
+def test_steps_without_wanted_logits_do_not_overtake_each_other():
+    """Rows of a step are uploaded from pinned memory; a step whose result nobody reads must not be overwritten by the next."""
+    cfg, _, model = make("wide", "cuda", "fp32")
+    toks = tokens(120, cfg["vocab"], 6)
+    want = reference("wide", toks)
+    eng = engine(model)
+    for _ in range(2):
+        for i, t in enumerate(toks[:-1]):
+            eng.forward_segments([(0, [t], i, [])])
+        assert off(eng.forward_segments([(0, toks[-1:], 119, [0])]), want[-1:]) < 1e-4
+        eng.kv.release(0)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("rows", [1, 3, 8, 9, 16])
+def test_decode_row_counts_and_graph_replay(rows):
+    """Fused and separate forms of a decode step, eager and replayed."""
+    cfg, _, model = make("wide", "cuda", "bf16")
+    seqs = [tokens(24, cfg["vocab"], 20 + r) for r in range(rows)]
+    want = [reference("wide", s) for s in seqs]
+    for graphs in (False, True):
+        eng = engine(model, pages=2 * rows + 2, slots=rows, use_graphs=graphs)
+        for r, s in enumerate(seqs):
+            eng.forward_segments([(r, s[:18], 0, [])])
+        for i in range(18, 24):
+            got = eng.forward_segments([(r, [s[i]], i, [0]) for r, s in enumerate(seqs)])
+            assert off(got, torch.stack([w[i] for w in want])) < TOL["bf16"], (graphs, i)
+
+
+# ------------------------------------------------------------------------------------------ the framework's own entry points
+@pytest.mark.parametrize("device", DEVICES)
+def test_model_directory_through_the_launcher_and_trace_run(tmp_path, device, capsys):
+    from volta_engine_b200.tools import trace_run
+    write_model(tmp_path / "m", "eights")
+    toks = tokens(100, CONFIGS["eights"]["vocab"], 8)
+    want = reference("eights", toks)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:70], "want": [69, 0]}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": toks[70:71], "want": []}, {"id": "y", "tokens": toks[:2], "want": [1]}], "end": []},
+             {"step": 2, "entries": [{"id": "x", "tokens": toks[71:100], "want": [28]}], "end": ["x", "y"]},
+             {"step": 3, "entries": [{"id": "z", "tokens": toks[:1], "want": [0]}], "end": ["z"]}]
+    rows = {0: [69, 0], 1: [1], 2: [99], 3: [0]}
+    for dtype, tol in (("float32", 1e-4), ("bfloat16", TOL["bf16"])):
+        rc = trace_run.main(["--model", str(tmp_path / "m"), "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "192"],
+                            stdin=io.StringIO("\n".join(json.dumps(s) for s in steps) + "\n"), device=device)
+        assert rc == 0
+        assert [ln for ln in capsys.readouterr().out.splitlines() if ln.startswith("done")] == [f"done {i}" for i in range(4)]
+        for i, ps in rows.items():
+            raw = torch.frombuffer(bytearray((tmp_path / f"{i}.f32").read_bytes()), dtype=torch.float32)
+            assert off(raw.reshape(len(ps), -1), want[ps]) < tol
+
+
+def test_pool_of_exactly_the_asked_tokens_and_slots(tmp_path):
+    from volta_engine_b200.tools import trace_run
+    write_model(tmp_path, "eights")
+    eng = trace_run.build(str(tmp_path), "float32", 130, 2, "cpu")
+    assert eng.kv.free_pages() == 3 and eng.kv.max_slots == 2
+    run_ = trace_run.TraceRunner(eng)
+    t = tokens(128, CONFIGS["eights"]["vocab"])
+    for _ in range(3):                           # 64 + 128 tokens live at a time, again and again
+        run_.step([{"id": "a", "tokens": t[:64]}, {"id": "b", "tokens": t[:128]}], ["a", "b"])
+    run_.step([{"id": "a", "tokens": t[:1]}, {"id": "b", "tokens": t[:1]}], [])
+    with pytest.raises(RuntimeError):
+        run_.step([{"id": "c", "tokens": t[:1]}], [])
+
+
+def test_other_designs_are_refused(tmp_path):
+    from volta_engine_b200.models.factory import load_model
+    from volta_engine_b200.models.fofosun import FofosunConfig
+    bad = dict(CONFIGS["eights"], layers=[dict(CONFIGS["eights"]["layers"][0], type="mamba")])
+    with pytest.raises(NotImplementedError):
+        FofosunConfig.from_dict(bad)
+    bad = dict(CONFIGS["eights"], layers=[dict(CONFIGS["eights"]["layers"][0], mlp={"kind": "moe", "ff": 8})])
+    with pytest.raises(NotImplementedError):
+        FofosunConfig.from_dict(bad)
+    write_model(tmp_path, "eights")
+    with pytest.raises(NotImplementedError):
+        load_model(tmp_path, "cpu", quantize="nvfp4")

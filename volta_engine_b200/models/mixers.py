@@ -24,8 +24,6 @@ def make_linear(src, names, device, dtype):
 def apply_linear(lin, x, out_f32: bool = False):
     """``lin`` on rows of its activation type: the decode kernel up to 16 rows, the tensor-core GEMM above."""
     if x.is_cuda and isinstance(lin, LinearBF16) and x.shape[0] <= 16:
-        if x.shape[1] != lin.weight.shape[1]:
-            x = torch.nn.functional.pad(x, (0, lin.weight.shape[1] - x.shape[1]))
         return gemv_rows(lin, x.shape[0], x=x, out_f32=out_f32)
     return lin.forward(x, out_f32=out_f32)
 

@@ -117,6 +117,8 @@ def gemv_rows(lin, M: int, *, x, pro=0, w=None, b=None, alpha=0.0, G=0, wlen=0, 
     W = lin.weight
     N, K = W.shape
     dev = W.device
+    if pro == 0 and x.shape[1] != K:              # weight rows padded to 16 bytes
+        x = torch.nn.functional.pad(x, (0, K - x.shape[1]))
     out = None
     if residual is None:
         out = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=dev)
