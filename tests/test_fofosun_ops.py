@@ -165,10 +165,11 @@ LIN = [("hgrn2", 2, 32, 32), ("hgrn2", 3, 24, 40), ("hgrn2", 1, 128, 128), ("hgr
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("form", ["fp32", "bf16 rows", "chunked"])
 @pytest.mark.parametrize("mode,H,dk,dv", LIN)
-def test_recurrence_in_portions(mode, H, dk, dv, dtype, device):
+def test_recurrence_in_portions(mode, H, dk, dv, form, device):
     """One long sequence in portions of all kinds beside a second one, in slots that hold another sequence's state before."""
+    dtype = torch.bfloat16 if form == "bf16 rows" else torch.float32
     base = lin_case(mode, H, dk, dv)
     spec = on(base, device)
     st = LinAttnState(spec, 3, device)
@@ -176,6 +177,7 @@ def test_recurrence_in_portions(mode, H, dk, dv, dtype, device):
     cols = spec.cols + 5
     a, b = rnd(330, cols, seed=3, scale=1.5).to(dtype), rnd(90, cols, seed=4, scale=1.5).to(dtype)
     a[:, H * dk:2 * H * dk] *= 2
+    a[37, H * dk:2 * H * dk] = -60.0              # everything forgettable is forgotten at this row
     wa, Sa = lin_plain(base, a)
     wb, _ = lin_plain(base, b)
     got_a, got_b, at, bt = [], [], 0, 0
@@ -183,15 +185,15 @@ def test_recurrence_in_portions(mode, H, dk, dv, dtype, device):
         ids = list(range(at, at + na)) + list(range(bt, bt + nb))
         batch = BatchRows.make(ids, ids, [2] * na + [0] * nb, device)
         proj = torch.cat([a[at:at + na], b[bt:bt + nb]]).to(device)
-        o = linattn_rows(proj, batch, st, spec)
+        o = linattn_rows(proj, batch, st, spec, chunked=form == "chunked")
         got_a.append(o[:na].cpu())
         got_b.append(o[na:].cpu())
         at, bt = at + na, bt + nb
     for got, want in ((torch.cat(got_a), wa), (torch.cat(got_b), wb)):
         ref = want.pow(2).mean().sqrt()
-        tol = 3e-5 if dtype == torch.float32 else 6e-3      # (bf16 activations: v and q may be rounded once)
+        tol = 3e-3 if form == "chunked" else 3e-5            # the chunked form rounds the values to bf16
         assert (got.double() - want).abs().max() < tol * (want.abs().max() + ref)
-    assert (st.rec[2].double().cpu() - Sa).abs().max() < (3e-5 if dtype == torch.float32 else 6e-3) * Sa.abs().max()
+    assert (st.rec[2].double().cpu() - Sa).abs().max() < tol * Sa.abs().max()
     assert bool((st.rec[1] == 7.0).all())         # the slot nobody used
 
 
@@ -340,3 +342,39 @@ def test_rotation_is_exact_at_far_positions(device):
         qs.append(qo[:, 8:].cpu() @ r.kv.k[1, page, 0, off:off + 6, 16:24].cpu().t())
     assert (qs[0] - qs[1]).abs().max() < 1e-5
     assert near.shape == far.shape
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("mode,H,dk,dv", [("hgrn2", 2, 128, 128), ("lightning", 3, 64, 32), ("hgrn2", 5, 24, 40)])
+def test_chunked_recurrence_of_a_large_batch(mode, H, dk, dv):
+    """Several sequences, portions longer than many chunks, values that are exact in bf16: then everything else of the chunked
+    form keeps 32-bit quality."""
+    base = lin_case(mode, H, dk, dv, seed=5)
+    spec = on(base, "cuda")
+    if mode == "lightning":
+        base.decay = base.decay.clone()
+    st = LinAttnState(spec, 4, "cuda")
+    lens = [700, 16, 433, 17]
+    rows = []
+    for i, n in enumerate(lens):
+        r = rnd(n, spec.cols, seed=30 + i, scale=1.5)
+        v = r[:, 2 * H * dk:2 * H * dk + H * dv]
+        v.copy_(v.to(torch.bfloat16))
+        rows.append(r)
+    want = [lin_plain(base, r) for r in rows]
+    cut = [300, 0, 150, 0]
+    for part in (0, 1):
+        segs = [(i, 0 if part == 0 else cut[i], cut[i] if part == 0 else lens[i]) for i in range(4)]
+        segs = [s for s in segs if s[2] > s[1]]
+        pos = [p for i, a, b in segs for p in range(a, b)]
+        slot = [3 - i for i, a, b in segs for _ in range(a, b)]
+        batch = BatchRows.make(pos, pos, slot, "cuda")
+        o = linattn_rows(torch.cat([rows[i][a:b] for i, a, b in segs]).cuda(), batch, st, spec).double().cpu()
+        at = 0
+        for i, a, b in segs:
+            w = want[i][0]
+            assert (o[at:at + b - a] - w[a:b]).abs().max() < (3e-3 if mode == "lightning" else 6e-5) * w.abs().max()
+            at += b - a
+    for i in range(4):
+        S = want[i][1]
+        assert (st.rec[3 - i].double().cpu() - S).abs().max() < (3e-3 if mode == "lightning" else 6e-5) * S.abs().max()

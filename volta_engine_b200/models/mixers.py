@@ -62,7 +62,7 @@ class LinearRecurrence:
 
     def rows(self, x, b, kv, journal=(None, None)):
         proj = apply_linear(self.in_proj, x, out_f32=True)         # gates and keys enter the recurrence unrounded
-        o = linattn_rows(proj, b, self.bind(kv), self.spec, *journal)
+        o = linattn_rows(proj, b, self.bind(kv), self.spec, *journal, chunked=self.dtype != torch.float32)
         y = self.norm.rows(o, self.dtype, gate=self._gate(proj))
         return apply_linear(self.out, y)
 

@@ -19,9 +19,6 @@ import torch
 from .._lib import call, ptr
 from .gdn import GDNJournal
 
-CHUNK_MIN = 16            # shortest portion that takes the chunked kernels
-
-
 @dataclass
 class LinAttnSpec:
     heads: int
@@ -98,8 +95,10 @@ def _step(proj, pos, slot, st, spec, o, rows, segs=None):
          ptr(st.rec), ptr(spec.bias), ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), rows, spec.heads, spec.dk, spec.dv, spec.mode)
 
 
-def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJournal | None = None, rows=None) -> torch.Tensor:
-    """Rows of batch ``b`` through the recurrence -> fp32 [rows, heads * dv]. ``rows`` = (pos, slot) that outlive the step
+def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJournal | None = None, rows=None,
+                 chunked: bool = True) -> torch.Tensor:
+    """Rows of batch ``b`` through the recurrence -> fp32 [rows, heads * dv]. ``chunked``: long portions may take the
+    tensor-core form, which rounds the values v to bf16 (off in the all-32-bit form of a model). ``rows`` = (pos, slot) that outlive the step
     when ``journal`` keeps the block's operands for a replay."""
     pos, slot = rows if rows is not None else (b.pos, b.slot)
     if journal is not None:
@@ -117,5 +116,16 @@ def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJourn
             journal.fn = lambda keep: _step(proj, pos, slot, st, spec, o2, keep)
         return o
     t = b.segments()
-    _step(proj, pos, slot, st, spec, o, n, (t.first, t.count, t.n))
+    if not chunked or spec.dk > 128 or spec.dv > 128 or proj.dtype != torch.float32:
+        _step(proj, pos, slot, st, spec, o, n, (t.first, t.count, t.n))
+        return o
+    if t.n_short:
+        _step(proj, pos, slot, st, spec, o, n, (t.first, t.count, t.n_short))
+    if t.chunks:
+        multi = t.longest > 1
+        start = torch.empty((t.chunks, spec.heads, spec.dk, spec.dv) if multi else (1,), dtype=torch.float32, device=proj.device)
+        total = torch.empty((t.chunks, spec.heads, spec.dk) if multi else (1,), dtype=torch.float32, device=proj.device)
+        call("linattn_chunk", "plpppppp" + "iii" + "ppp" + "pppp" + "liiii", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
+             ptr(t.chunk_count), ptr(t.seg_chunk0), t.chunks, t.seg_chunk0.numel() - 1, t.longest, ptr(st.rec), ptr(start), ptr(total), ptr(spec.bias),
+             ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), spec.heads, spec.dk, spec.dv, spec.mode)
     return o

@@ -18,6 +18,7 @@ LOGITS_LAST = "last"
 LOGITS_NONE = "none"
 LOGITS_ROWS = "rows"   # the rows listed in BatchRows.want
 
+CHUNK_ROWS = 128       # rows of one chunk of the chunked recurrences (half of it in small batches, for more parallel work)
 LONG_SEGMENT = 16      # portions of at least this many rows take the prompt kernels, shorter ones the decode kernels
 
 
@@ -35,10 +36,13 @@ class SegmentTable:
     tile_first: torch.Tensor | None  # tiles of at most 64 rows of one of these segments; rows counted from short_rows
     tile_count: torch.Tensor | None
     tile_base: torch.Tensor | None   # the segment's ctx_base
-    chunk_seg: torch.Tensor | None   # chunks of at most 64 rows of these segments: segment (0 = the first behind short_rows),
+    chunk_seg: torch.Tensor | None   # chunks of at most CHUNK_ROWS rows of these segments: segment (0 = the first behind short_rows),
     chunk_first: torch.Tensor | None  # first row (in the batch) and rows
     chunk_count: torch.Tensor | None
     seg_chunk0: torch.Tensor | None   # [segments + 1] first chunk of every such segment
+    n_short: int = 0                  # leading segments that make up short_rows
+    chunks: int = 0
+    longest: int = 0                  # most chunks of any segment
 
     @classmethod
     def build(cls, slots, pos, device):
@@ -57,21 +61,24 @@ class SegmentTable:
             k += 1
         rest = host[k:]
         short = rest[0][1] if rest else n
-        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 7))
+        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 7), n_short=k)
         if rest:
             base, total = [], 0
             tf, tc, tb, cs, cf, cc, c0 = [], [], [], [], [], [], [0]
+            per = CHUNK_ROWS if n >= 1024 else CHUNK_ROWS // 2
             for g, (s, f, c, p0) in enumerate(rest):
                 base.append(total)
                 for o in range(0, c, 64):
                     tf.append(f + o - short)
                     tc.append(min(64, c - o))
                     tb.append(total)
+                for o in range(0, c, per):
                     cs.append(g)
                     cf.append(f + o)
-                    cc.append(min(64, c - o))
+                    cc.append(min(per, c - o))
                 c0.append(len(cs))
                 total += p0 + c
+            t.chunks, t.longest = len(cs), max(b - a for a, b in zip(c0, c0[1:]))
             t.ctx_slot, t.ctx_base, t.ctx_total = dev([h[0] for h in rest]), dev(base), total
             t.tile_first, t.tile_count, t.tile_base = dev(tf), dev(tc), dev(tb)
             t.chunk_seg, t.chunk_first, t.chunk_count, t.seg_chunk0 = dev(cs), dev(cf), dev(cc), dev(c0)

@@ -29,7 +29,7 @@ TABLE = {
     "mla_expand_out": ("MLALatent", P),
     "latent_rope_store": ("LatentAttention", P), "latent_absorb": ("LatentAttention", P), "latent_attn": ("LatentAttention", P),
     "latent_expand": ("LatentAttention", P), "latent_gather": ("LatentAttention", P), "latent_prefill": ("LatentAttention", P),
-    "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P),
+    "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P), "linattn_chunk": ("LinearAttention", P),
     "embed_rows": ("RowOps (fp32 residual)", P), "dyt_rows": ("RowOps (fp32 residual)", P), "group_rms": ("RowOps (fp32 residual)", P),
     "polynorm": ("RowOps (fp32 residual)", P), "gemv_rows": ("LinearBF16 decode", P), "gemm_f32": ("Gemm (fp32)", P),
     "dsa_prep": ("DSA", P), "dsa_pool_update": ("DSA", P), "dsa_score": ("DSA / QSA", P), "dsa_select": ("DSA / QSA", P),
