@@ -86,9 +86,23 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
     for (int m = 0; m < a.M; ++m) {
       float s1 = 0.f, s2 = 0.f, s3 = 0.f;
       for (int i = tid; i < a.kx; i += 256) poly_sums(src[m * a.ldx + i], s1, s2, s3);
-      s1 = block_sum(s1, red);
-      s2 = block_sum(s2, red);
-      s3 = block_sum(s3, red);
+      s1 = warp_sum(s1);
+      s2 = warp_sum(s2);
+      s3 = warp_sum(s3);
+      __syncthreads();                                     // (readers of the row in front)
+      if (lane == 0) {
+        red[warp] = s1;
+        red[33 + warp] = s2;
+        red[66 + warp] = s3;
+      }
+      __syncthreads();
+      s1 = s2 = s3 = 0.f;
+#pragma unroll
+      for (int y = 0; y < 8; ++y) {
+        s1 += red[y];
+        s2 += red[33 + y];
+        s3 += red[66 + y];
+      }
       const PolyScale ps = poly_scale(s1, s2, s3, a.kx, a.eps, a.coef);
       for (int i = tid; i < a.kx; i += 256) put(m, i, poly_of(src[m * a.ldx + i], ps));
     }
@@ -96,64 +110,117 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
   __syncthreads();
 }
 
-// 8 warps: R tiles of 8 weight rows x KS slices of k. Units of 32 k; slice s takes units s, s + KS, ...
-template <int KS, bool FUSED>
-__global__ void __launch_bounds__(256, 2) gemv_rows_kernel(const RowsArgs a) {
-  constexpr int R = 8 / KS, PF = 8;
+// 8 warps: R tiles of 8 weight rows x KS slices of k; units of 32 k, slice s takes units s, s + KS, ... CTAs are resident and walk
+// the groups of R tiles; the ring of requested weights (8 units per warp) runs on across groups. XM 0: all activations in shared
+// memory (made by the prologue, or copied), rows 8..15 only with HI. XM 1: they pass through shared memory in slabs of 8 units
+// per slice (many rows of a long k).
+template <int KS, int XM, bool HI>
+__global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
+  constexpr int R = 8 / KS, PF = 8, SLAB = KS * PF * 32, SP = SLAB * 2 + 64;
   extern __shared__ __align__(16) uint8_t xs[];
-  __shared__ float part[8][16][8], red[33];
+  __shared__ float part[2][8][HI ? 16 : 8][8], red[3][33];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-  const int ks = warp % KS, rt = warp / KS, n0 = (blockIdx.x * R + rt) * 8;
-  const int units = (a.K + 31) / 32, mine = units > ks ? (units - ks + KS - 1) / KS : 0;
-  const __nv_bfloat16* wr = a.W + (long)min(n0 + g, a.N - 1) * a.ldw + t * 8;
-  auto load_w = [&](int j) -> uint4 {
-    const int k = (ks + j * KS) * 32 + t * 8;
-    if (j < mine && k < a.K) return __ldcs(reinterpret_cast<const uint4*>(wr + (k - t * 8)));
+  const int ks = warp % KS, rt = warp / KS;
+  const int units = (a.K + 31) / 32, batches = ((units + KS - 1) / KS + PF - 1) / PF;
+  const int groups = ((a.N + 7) / 8 + R - 1) / R;
+  auto row_of = [&](int grp) { return a.W + (long)min((grp * R + rt) * 8 + g, a.N - 1) * a.ldw + t * 8; };
+  auto load_w = [&](const __nv_bfloat16* wr, int u, bool in) -> uint4 {
+    if (in && u * 32 + t * 8 < a.K) return __ldcs(reinterpret_cast<const uint4*>(wr + u * 32));
     return make_uint4(0, 0, 0, 0);
   };
-  uint4 cur[PF];
+  int grp = blockIdx.x;
+  uint4 buf[PF];
+  {
+    const __nv_bfloat16* wr = row_of(grp);
 #pragma unroll
-  for (int j = 0; j < PF; ++j) cur[j] = load_w(j);
+    for (int j = 0; j < PF; ++j) buf[j] = load_w(wr, ks + j * KS, true);
+  }
   grid_dep_wait();
   grid_dep_launch();
-  if (FUSED) rows_prologue(a, xs, red);
   const __nv_bfloat16* xg = reinterpret_cast<const __nv_bfloat16*>(a.x);
-  auto load_x = [&](int m, int k) -> uint4 {
-    if (m >= a.M || k >= a.K) return make_uint4(0, 0, 0, 0);
-    if (FUSED) return *reinterpret_cast<const uint4*>(xs + m * a.pitch + k * 2);
-    return *reinterpret_cast<const uint4*>(xg + m * a.ldx + k);
+  auto slab = [&](int b, int stage) {                     // activations of batch b -> xs[stage]
+    constexpr int C8 = SLAB / 8;
+    for (int i = tid; i < (HI ? 16 : 8) * C8; i += 256) {
+      const int m = i / C8, k = b * SLAB + (i % C8) * 8;
+      const bool in = m < a.M && k < a.K;
+      const int n = in ? 16 : 0;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(xs + (stage * (HI ? 16 : 8) + m) * SP + (i % C8) * 16)),
+                   "l"(xg + (in ? m * a.ldx + k : 0)), "r"(n) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float c[4] = {0.f, 0.f, 0.f, 0.f};
-  for (int j0 = 0; j0 < mine; j0 += PF) {
-    uint4 nxt[PF];
+  if (XM == 0) {
+    if (a.pro) {
+      rows_prologue(a, xs, &red[0][0]);
+    } else {
+      const int K32 = units * 32;
+      for (int i = tid; i < a.M * (K32 / 8); i += 256) {
+        const int m = i / (K32 / 8), k = (i % (K32 / 8)) * 8;
+        *reinterpret_cast<uint4*>(xs + m * a.pitch + k * 2) = k < a.K ? *reinterpret_cast<const uint4*>(xg + m * a.ldx + k) : make_uint4(0, 0, 0, 0);
+      }
+      __syncthreads();
+    }
+  } else {
+    slab(0, 0);
+  }
+  int pb = 0, stage = 0;
+  for (; grp < groups; grp += gridDim.x) {
+    float c[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int b = 0; b < batches; ++b) {
+      const bool last = b + 1 == batches;
+      const int ngrp = last ? grp + gridDim.x : grp, nu = last ? ks : ks + (b + 1) * PF * KS;
+      const __nv_bfloat16* wr = row_of(ngrp);
+      if (XM == 1) {
+        if (!last || ngrp < groups) {
+          slab(last ? 0 : b + 1, stage ^ 1);
+          asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+          asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+      }
 #pragma unroll
-    for (int j = 0; j < PF; ++j) nxt[j] = load_w(j0 + PF + j);
-#pragma unroll
-    for (int j = 0; j < PF; ++j) {
-      if (j0 + j < mine) {
-        const int k = (ks + (j0 + j) * KS) * 32 + t * 8;
-        const uint4 lo = load_x(g, k), hi = FUSED ? make_uint4(0, 0, 0, 0) : load_x(g + 8, k);     // fused rows: M <= 8
-        rows_mma(c, lo.x, hi.x, lo.y, hi.y, cur[j].x, cur[j].y);
-        rows_mma(c, lo.z, hi.z, lo.w, hi.w, cur[j].z, cur[j].w);
+      for (int j = 0; j < PF; ++j) {
+        const uint4 w = buf[j];
+        buf[j] = load_w(wr, nu + j * KS, ngrp < groups);
+        const int u = ks + (b * PF + j) * KS;
+        if (u < units) {
+          uint4 lo = make_uint4(0, 0, 0, 0), hi = make_uint4(0, 0, 0, 0);
+          if (XM == 0) {
+            if (g < a.M) lo = *reinterpret_cast<const uint4*>(xs + g * a.pitch + u * 64 + t * 16);
+            if (HI && g + 8 < a.M) hi = *reinterpret_cast<const uint4*>(xs + (g + 8) * a.pitch + u * 64 + t * 16);
+          } else {
+            const uint8_t* p = xs + (stage * (HI ? 16 : 8) + g) * SP + (j * KS + ks) * 64 + t * 16;
+            lo = *reinterpret_cast<const uint4*>(p);
+            if (HI) hi = *reinterpret_cast<const uint4*>(p + 8 * SP);
+          }
+          rows_mma(c, lo.x, hi.x, lo.y, hi.y, w.x, w.y);
+          rows_mma(c, lo.z, hi.z, lo.w, hi.w, w.z, w.w);
+        }
+      }
+      if (XM == 1) {
+        stage ^= 1;
+        __syncthreads();                                  // the slab behind may be overwritten now
       }
     }
+    part[pb][warp][g][2 * t] = c[0];
+    part[pb][warp][g][2 * t + 1] = c[1];
+    if (HI) {
+      part[pb][warp][(HI ? 8 : 0) + g][2 * t] = c[2];
+      part[pb][warp][(HI ? 8 : 0) + g][2 * t + 1] = c[3];
+    }
+    __syncthreads();
+    for (int i = tid; i < a.M * R * 8; i += 256) {
+      const int m = i / (R * 8), q = i % (R * 8), r = q / 8, e = q % 8, n = (grp * R + r) * 8 + e;
+      if (n >= a.N) continue;
+      float v = 0.f;
 #pragma unroll
-    for (int j = 0; j < PF; ++j) cur[j] = nxt[j];
-  }
-  part[warp][g][2 * t] = c[0];
-  part[warp][g][2 * t + 1] = c[1];
-  part[warp][g + 8][2 * t] = c[2];
-  part[warp][g + 8][2 * t + 1] = c[3];
-  __syncthreads();
-  for (int i = tid; i < a.M * R * 8; i += 256) {
-    const int m = i / (R * 8), q = i % (R * 8), r = q / 8, e = q % 8, n = (blockIdx.x * R + r) * 8 + e;
-    if (n >= a.N) continue;
-    float v = 0.f;
-#pragma unroll
-    for (int s = 0; s < KS; ++s) v += part[r * KS + s][m][e];
-    if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
-    else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
-    else a.out[m * a.ldo + n] = f2bf(v);
+      for (int s = 0; s < KS; ++s) v += part[pb][r * KS + s][m][e];
+      if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
+      else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
+      else a.out[m * a.ldo + n] = f2bf(v);
+    }
+    pb ^= 1;                                              // (the other buffer's readers are done: they passed the barrier above)
   }
 }
 
@@ -191,17 +258,19 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       if (t0 + tt + i < T && n0 + tn + j < N) out[(long)(t0 + tt + i) * ldo + n0 + tn + j] = acc[i][j];
 }
 
-template <int KS, bool FUSED>
+template <int KS, int XM, bool HI>
 static int launch_rows(const RowsArgs& a, cudaStream_t st) {
-  const int smem = FUSED ? a.M * a.pitch : 0;
+  constexpr int SP = KS * 8 * 32 * 2 + 64;
+  const int smem = XM ? 2 * (HI ? 16 : 8) * SP : a.M * a.pitch;
   static int attr = 0;
   if (smem > attr) {
-    cudaError_t e = cudaFuncSetAttribute(gemv_rows_kernel<KS, FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(gemv_rows_kernel<KS, XM, HI>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     attr = smem;
   }
-  const int tiles = (a.N + 7) / 8;
-  launch_pdl(gemv_rows_kernel<KS, FUSED>, dim3((tiles + 8 / KS - 1) / (8 / KS)), dim3(256), smem, st, a);
+  const int groups = ((a.N + 7) / 8 + 8 / KS - 1) / (8 / KS);
+  const int per = (smem + (HI ? 9 : 5) * 1024) * 3 <= 222 * 1024 ? 3 : (smem + (HI ? 9 : 5) * 1024) * 2 <= 222 * 1024 ? 2 : 1;
+  launch_pdl(gemv_rows_kernel<KS, XM, HI>, dim3(groups < 148 * per ? groups : 148 * per), dim3(256), smem, st, a);
   return (int)cudaGetLastError();
 }
 
@@ -220,25 +289,28 @@ int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, 
   if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 3) return cudaErrorInvalidValue;
   RowsArgs a{(const __nv_bfloat16*)W, ldw, N, K, M, pro, kx, x, ldx, (const float*)w, (const float*)b, alpha, G, wlen, (const float*)gate, ldg,
              (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale, 0};
+  const int K32 = (K + 31) / 32 * 32;
+  a.pitch = K32 * 2 + ((K32 * 2) % 128 == 0 ? 64 : 0);            // rows of a quad pair land in different halves of the banks
   if (pro) {
-    const int K32 = (K + 31) / 32 * 32;
-    a.pitch = K32 * 2 + ((K32 * 2) % 128 == 0 ? 64 : 0);          // rows of a quad pair land in different halves of the banks
-    if (M > 8 || (long)M * a.pitch > 200 * 1024) return cudaErrorInvalidValue;
+    if (M > 8 || (long)M * a.pitch > 100 * 1024) return cudaErrorInvalidValue;
     if ((pro == 1 && (!w || !b || h)) || (pro == 2 && (!w || G < 1 || kx % G || wlen < 1)) || (pro == 3 && !coef)) return cudaErrorInvalidValue;
   } else if (kx != K || ldx % 8 || ((uintptr_t)x & 15)) {
     return cudaErrorInvalidValue;
   }
-  const int tiles = (N + 7) / 8;
-  if (pro) {
-    if (tiles <= 148 * 2) return launch_rows<8, true>(a, st);
-    if (tiles <= 148 * 4) return launch_rows<4, true>(a, st);
-    if (tiles <= 148 * 16) return launch_rows<2, true>(a, st);
-    return launch_rows<1, true>(a, st);
+  const int tiles = (N + 7) / 8, units = (K + 31) / 32;
+  if ((long)M * a.pitch <= 100 * 1024) {
+    // at least eight units per warp where k is long enough; otherwise fewer slices of k and more rows per group
+#define VE_GR(KS) (M <= 8 ? launch_rows<KS, 0, false>(a, st) : launch_rows<KS, 0, true>(a, st))
+    if (units >= 48 || tiles < 148) return VE_GR(8);
+    if (units >= 24) return VE_GR(4);
+    return VE_GR(2);
+#undef VE_GR
   }
-  if (tiles <= 148 * 4) return launch_rows<8, false>(a, st);
-  if (tiles <= 148 * 8) return launch_rows<4, false>(a, st);
-  if (tiles <= 148 * 16) return launch_rows<2, false>(a, st);
-  return launch_rows<1, false>(a, st);
+#define VE_GR(KS) (M <= 8 ? launch_rows<KS, 1, false>(a, st) : launch_rows<KS, 1, true>(a, st))
+  if (tiles >= 4 * 120) return VE_GR(2);
+  if (tiles >= 2 * 120) return VE_GR(4);
+  return VE_GR(8);
+#undef VE_GR
 }
 
 int ve_gemm_f32(const void* W, long ldw, const void* x, long ldx, void* out, long ldo, int T, int N, int K, cudaStream_t st) {

@@ -232,43 +232,49 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims n, co
 }
 
 // out[row][h dv + v] = sum_c o[c] W_uv[h dv + v][c], o = merged split partials (o_part [rows][H][nsplit][ldp], lse in log2
-// units; lse null: one finished partial). grid (rows, H, nz), 128 threads, a warp per value row. Dynamic shared memory: kr floats.
+// units; lse null: one finished partial). grid (rows, H, nz), 512 threads: four groups share the splits (every partial's load is
+// in flight at once), then a warp per value row. Dynamic shared memory: 4 kr floats.
 template <int VEC, typename T>
-__global__ void __launch_bounds__(128) latent_expand_kernel(const LatentDims n, const float* __restrict__ o_part, const float* __restrict__ lse,
+__global__ void __launch_bounds__(512) latent_expand_kernel(const LatentDims n, const float* __restrict__ o_part, const float* __restrict__ lse,
                                                             int nsplit, int ldp, const T* __restrict__ w_uv, const int* __restrict__ slot,
                                                             T* __restrict__ out, long ldo, int vper) {
-  extern __shared__ float os[];
+  extern __shared__ float os[];                           // [4][kr]
+  __shared__ float sw[64], s_inv;
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
-  const int h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sg = tid >> 7;
   const int v0 = blockIdx.z * vper, v1 = min(n.dv, v0 + vper);
   if (slot[row] < 0) {
-    for (int v = v0 + threadIdx.x; v < v1; v += 128) out[row * ldo + (long)h * n.dv + v] = from_f<T>(0.f);
+    for (int v = v0 + tid; v < v1; v += 512) out[row * ldo + (long)h * n.dv + v] = from_f<T>(0.f);
     return;
   }
   const long base = (row * n.H + h) * nsplit;
-  float mx = -FLT_MAX;
-  if (lse)
-    for (int i = 0; i < nsplit; ++i) mx = fmaxf(mx, lse[base + i]);
-  for (int c = threadIdx.x; c < n.kr; c += 128) {
-    if (!lse) {
-      os[c] = o_part[base * ldp + c];
-      continue;
+  if (lse) {
+    if (warp == 0) {                                      // weights of at most 64 splits
+      const float l0 = lane < nsplit ? lse[base + lane] : -FLT_MAX, l1 = lane + 32 < nsplit ? lse[base + lane + 32] : -FLT_MAX;
+      const float mx = warp_max(fmaxf(l0, l1));
+      const float w0 = l0 == -FLT_MAX ? 0.f : exp2f(l0 - mx), w1 = l1 == -FLT_MAX ? 0.f : exp2f(l1 - mx);
+      sw[lane] = w0;
+      sw[lane + 32] = w1;
+      const float ws = warp_sum(w0 + w1);
+      if (lane == 0) s_inv = ws > 0.f ? 1.f / ws : 0.f;
     }
-    float acc = 0.f, ws = 0.f;
-#pragma unroll 4
-    for (int i = 0; i < nsplit; ++i) {
-      const float l = lse[base + i];
-      if (l == -FLT_MAX) continue;               // a split without keys wrote no partial
-      const float w = exp2f(l - mx);
-      ws += w;
-      acc = fmaf(w, o_part[(base + i) * ldp + c], acc);
+    __syncthreads();
+    for (int c = tid & 127; c < n.kr; c += 128) {
+      float acc = 0.f;
+#pragma unroll 16
+      for (int i = sg; i < nsplit; i += 4) acc = fmaf(sw[i], sw[i] != 0.f ? o_part[(base + i) * ldp + c] : 0.f, acc);   // (an empty split left nothing)
+      os[sg * n.kr + c] = acc;
     }
-    os[c] = ws > 0.f ? acc / ws : 0.f;
+    __syncthreads();
+    const float inv = s_inv;
+    for (int c = tid; c < n.kr; c += 512) os[c] = (os[c] + os[n.kr + c] + os[2 * n.kr + c] + os[3 * n.kr + c]) * inv;
+  } else {
+    for (int c = tid; c < n.kr; c += 512) os[c] = o_part[base * ldp + c];
   }
   __syncthreads();
-  for (int v = v0 + warp; v < v1; v += 4) {
+  for (int v = v0 + warp; v < v1; v += 16) {
     const T* w = w_uv + ((long)h * n.dv + v) * n.kr;
     float acc = 0.f;
 #pragma unroll 2
@@ -569,10 +575,10 @@ int ve_latent_expand(VE_LDIMS, const void* o_part, const void* lse, int nsplit, 
                      int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const LatentDims n = VE_LMAKE;
-  if (!ldims_ok(n) || nsplit < 1 || kr > 8192) return cudaErrorInvalidValue;
+  if (!ldims_ok(n) || nsplit < 1 || nsplit > 64 || kr > 3072) return cudaErrorInvalidValue;
   const bool al = !((uintptr_t)w_uv & 15);
-  const int vper = rows * H >= 148 ? dv : 16;
-#define VE_EX(V, T) launch_pdl(latent_expand_kernel<V, T>, dim3(rows, H, (dv + vper - 1) / vper), dim3(128), (size_t)kr * 4, st, n, (const float*)o_part, \
+  const int vper = rows * H >= 296 ? dv : rows * H >= 74 ? 32 : 16;
+#define VE_EX(V, T) launch_pdl(latent_expand_kernel<V, T>, dim3(rows, H, (dv + vper - 1) / vper), dim3(512), (size_t)kr * 16, st, n, (const float*)o_part, \
     (const float*)lse, nsplit, ldp, (const T*)w_uv, (const int*)slot, (T*)out, ldo, vper)
   if (f32) {
     if (al && kr % 4 == 0) VE_EX(4, float);

@@ -100,7 +100,7 @@ def latent_reference(spec: LatentSpec, q, kv, w_norm, w_uk, w_uv, b, cache, pool
     return out.reshape(n, H * dv).to(dt)
 
 
-def _absorbed(spec, q, kv, w_norm, w_uk, w_uv, pos, slot, cache, pool, nsplit):
+def _absorbed(spec, q, kv, w_norm, w_uk, w_uv, pos, slot, cache, pool):
     """Absorbed attention of the rows of ``q``; writes their cache rows first (rows of one sequence may follow each other: all
     cache rows are written before the attention launch)."""
     n, dev, dt = q.shape[0], q.device, pool.dtype
@@ -113,7 +113,7 @@ def _absorbed(spec, q, kv, w_norm, w_uk, w_uv, pos, slot, cache, pool, nsplit):
          ptr(spec.freq), ptr(pos), ptr(slot), ptr(table), table.shape[1], ptr(pool), ptr(q_abs), qw, n, float(spec.eps), f32)
     out = torch.empty(n, spec.heads * spec.vdim, dtype=dt, device=dev)
     if spec.tc_decode and not f32:
-        nsplit = max(1, min(nsplit, 64))
+        nsplit = max(1, min(64, 296 // (n * ((spec.heads + 15) // 16))))        # two CTAs per SM, whatever the position
         part = torch.empty(n, spec.heads, nsplit, spec.lat_cols, dtype=torch.float32, device=dev)
         lse = torch.empty(n, spec.heads, nsplit, dtype=torch.float32, device=dev)
         call("latent_decode", "ppppppiplii" + "iiiifp", ptr(q_abs), ptr(part), ptr(lse), ptr(pos), ptr(slot), ptr(table), table.shape[1], ptr(pool),
@@ -156,11 +156,11 @@ def latent_rows(spec: LatentSpec, q, kv, w_norm, w_uk, w_uv, ukv, b, cache, pool
         return latent_reference(spec, q, kv, w_norm, w_uk, w_uv, b, cache, pool)
     n = q.shape[0]
     if b.row_path or pool.dtype == torch.float32 or not spec.tc_prefill:
-        return _absorbed(spec, q, kv, w_norm, w_uk, w_uv, b.pos, b.slot, cache, pool, b.nsplit if b.row_path else 1)
+        return _absorbed(spec, q, kv, w_norm, w_uk, w_uv, b.pos, b.slot, cache, pool)
     t = b.segments()
     out = torch.empty(n, spec.heads * spec.vdim, dtype=pool.dtype, device=q.device)
     r0 = t.short_rows
     if r0:
-        out[:r0] = _absorbed(spec, q[:r0], kv[:r0], w_norm, w_uk, w_uv, b.pos[:r0], b.slot[:r0], cache, pool, max(1, min(32, 444 // r0)))
+        out[:r0] = _absorbed(spec, q[:r0], kv[:r0], w_norm, w_uk, w_uv, b.pos[:r0], b.slot[:r0], cache, pool)
     _expanded(spec, q, kv, w_norm, ukv, b, cache, pool, out, r0)
     return out

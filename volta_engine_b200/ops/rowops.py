@@ -13,7 +13,7 @@ import torch
 from .._lib import call, ptr
 
 FUSED_ROWS = 8            # decode rows that take the prologue forms
-FUSED_SMEM = 200 << 10
+FUSED_SMEM = 100 << 10
 
 
 def _f32(t) -> int:
