@@ -59,10 +59,11 @@ def _run(cmd: list[str]) -> None:
 
 
 def _build_lib(name: str, srcs: list[Path], headers: list[Path], compiler: list[str],
-               flags: list[str], link: list[str], force: bool) -> Path:
+               flags: list[str], link: list[str], force: bool, part: str = "") -> Path:
+    """``part``: link only these sources, as ``lib<name>_<part>.so`` (the objects are shared with the whole library)."""
     OUT.mkdir(exist_ok=True)
-    lib = OUT / f"lib{name}.so"
-    stamp = OUT / f"{name}.stamp"
+    lib = OUT / f"lib{name}{part and '_' + part}.so"
+    stamp = OUT / f"{name}{part and '_' + part}.stamp"
     objdir = OUT / f"obj_{name}"
     objdir.mkdir(exist_ok=True)
     jobs = []
@@ -91,17 +92,19 @@ def _build_lib(name: str, srcs: list[Path], headers: list[Path], compiler: list[
     return lib
 
 
-def build_kernels(force: bool = False) -> Path:
+def build_kernels(force: bool = False, sources=None, part: str = "") -> Path:
+    """The kernel library, or with ``sources`` (file names) a part of it: what one model needs, for tools that run a single
+    model out of a checkout in which nothing is built yet."""
     nvcc = _nvcc()
-    lib = OUT / "libvolta_kernels.so"
+    lib = OUT / f"libvolta_kernels{part and '_' + part}.so"
     if nvcc is None:
         if lib.exists():
             return lib
-        raise RuntimeError("nvcc not found and libvolta_kernels.so is not built")
-    srcs = sorted((CSRC / "cuda").glob("*.cu"))
+        raise RuntimeError(f"nvcc not found and {lib.name} is not built")
+    srcs = sorted(p for p in (CSRC / "cuda").glob("*.cu") if sources is None or p.name in sources)
     headers = sorted((CSRC / "cuda").glob("*.cuh")) + sorted((CSRC / "cuda").glob("*.h"))
     return _build_lib("volta_kernels", srcs, headers, [nvcc], NVCC_FLAGS,
-                      ["-Xcompiler", "-fPIC", "-lcudart"], force)
+                      ["-Xcompiler", "-fPIC", "-lcudart"], force, part)
 
 
 def build_host(force: bool = False) -> Path:

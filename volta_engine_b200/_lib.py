@@ -50,6 +50,18 @@ def kernels() -> ctypes.CDLL:
     return _kernels
 
 
+def kernels_of(part: str, sources) -> ctypes.CDLL:
+    """Make do with a part of the kernel library when the whole one is not built: the kernels of ``sources`` (see
+    ``_build.build_kernels``). Entry points of other sources are then missing (an error when one is called)."""
+    global _kernels
+    if _kernels is None and not (Path(__file__).resolve().parent / "_native" / "libvolta_kernels.so").exists():
+        from . import _build
+        with _lock:
+            if _kernels is None:
+                _kernels = ctypes.CDLL(str(_build.build_kernels(sources=sources, part=part)), mode=ctypes.RTLD_GLOBAL)
+    return kernels()
+
+
 def host() -> ctypes.CDLL:
     global _host
     if _host is None:

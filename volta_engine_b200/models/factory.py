@@ -44,6 +44,16 @@ def dense_config_from_hf(c: dict) -> DenseConfig:
         rope_theta_local=float(c.get("rope_local_base_freq") or 0.0), sandwich_norm=gemma, model_type=mt)
 
 
+def kernel_sources(model_dir):
+    """(part name, CUDA source names) of the kernels a model directory needs, for models that say so; None: the whole library."""
+    hf = json.loads((Path(model_dir) / "config.json").read_text())
+    arch = ARCHITECTURES.get(hf.get("architecture", ""))
+    if arch is None:
+        return None
+    import importlib
+    return arch[0], importlib.import_module("." + arch[0], __package__).KERNEL_SOURCES
+
+
 class TensorSource:
     """Checkpoint-name view over a safetensors repository or a GGUF file."""
 

@@ -38,7 +38,8 @@ class LinearRecurrence:
         f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
         self.gated = kind == "lightning"
         if kind == "lightning":
-            self.spec = LinAttnSpec(H, dk, dv, decay=torch.tensor([float(d) for d in m["decay"]], dtype=torch.float32, device=device))
+            decay = m["decay"] if isinstance(m["decay"], (list, tuple)) else [m["decay"]] * H
+            self.spec = LinAttnSpec(H, dk, dv, decay=torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device))
             if self.spec.decay.numel() != H:
                 raise ValueError(f"{p}: {self.spec.decay.numel()} decays for {H} heads")
         else:

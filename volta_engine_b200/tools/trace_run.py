@@ -54,7 +54,13 @@ class TraceRunner:
 
 
 def build(model_dir: str, dtype: str, max_tokens: int, slots: int, device=None):
+    import torch
+    from .. import _lib
+    from ..models.factory import kernel_sources
     from ..server.cli import build_engine, resolve_config
+    part = kernel_sources(model_dir)
+    if part is not None and torch.cuda.is_available() and device != "cpu":
+        _lib.kernels_of(*part)                             # in a fresh checkout: compile what this model needs
     n = (max_tokens + 63) // 64 * 64
     cfg, _ = resolve_config(["--model-dir", model_dir, "--set", f"dtype={'fp32' if dtype == 'float32' else 'bf16'}", "--set", f"kv_pool={n}",
                              "--set", f"max_seq={n}", "--set", f"max_slots={slots}", "--set", "scratch_mib=64"], env={})
