@@ -125,6 +125,26 @@ def test_linears_of_widths_that_are_not_multiples_of_the_tile():
         assert (got.double().cpu() - e).abs().max() < 1e-5 * e.abs().max()
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("T,N,K", [(130, 256, 64), (257, 300, 104), (520, 1000, 33), (129, 5, 712), (300, 513, 256)])
+def test_wide_gemm_at_the_edges_of_its_tiles(T, N, K):
+    from volta_engine_b200._lib import call, ptr
+    from volta_engine_b200.ops.kernels import status_word
+    Kp = -(-K // 8) * 8
+    W, x = torch.zeros(N, Kp, dtype=torch.bfloat16), torch.zeros(T, Kp, dtype=torch.bfloat16)
+    W[:, :K], x[:, :K] = rnd(N, K, seed=1).to(torch.bfloat16), rnd(T, K, seed=2).to(torch.bfloat16)
+    res = rnd(T, N, seed=3).to(torch.bfloat16)
+    e = x.double() @ W.double().t()
+    Wd, xd, rd = W.cuda(), x.cuda(), res.cuda()
+    for f32 in (True, False):
+        out = torch.full((T + 1, N), 9.0, dtype=torch.float32 if f32 else torch.bfloat16, device="cuda")
+        call("gemm_bf16_wide", "plplplppliiifp", ptr(Wd), Kp, ptr(xd), Kp, 0 if f32 else ptr(out), N, ptr(out) if f32 else 0, 0 if f32 else ptr(rd), N, T, N, Kp,
+             1.0, ptr(status_word(Wd.device)))
+        want = e if f32 else e + res.double()
+        assert (out[:T].double().cpu() - want).abs().max() < (1e-5 if f32 else 6e-3) * want.abs().max()
+        assert bool((out[T] == 9.0).all())
+
+
 # ------------------------------------------------------------------------------------------ recurrences
 def lin_case(mode, H, dk, dv, seed=0):
     if mode == "lightning":
@@ -285,6 +305,33 @@ def test_latent_attention_in_portions(H, d, rot, dv, kr, dtype, device):
             at += cnt
         got = torch.cat(got)[:at]
         assert (got.double() - want[:at]).abs().max() < tol * want.abs().max(), (n, cuts)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,d,rot,dv,kr", [c for c in LAT if c[1] % 8 == 0])
+def test_latent_attention_on_the_mma_kernel(H, d, rot, dv, kr, monkeypatch):
+    from volta_engine_b200.ops import latent as L
+    monkeypatch.setattr(L, "TC_PREFILL", False)
+    test_latent_attention_in_portions(H, d, rot, dv, kr, torch.bfloat16, "cuda")
+
+
+@pytest.mark.gpu
+def test_latent_prompt_of_many_key_tiles():
+    """Both streams, moving references and several query tiles: scores grow along the sequence, then fall."""
+    spec, w = latent_case(2, 64, 32, 96, 64, seed=3)
+    T = 600
+    kv = rnd(T, 96, seed=5).to(torch.bfloat16).float()
+    q = (rnd(T, 2 * 96, seed=6) * torch.linspace(0.2, 3, T)[:, None]).to(torch.bfloat16).float()
+    kv[:, 64:] *= torch.cat([torch.linspace(0.1, 2.5, T // 2), torch.linspace(2.5, 0.1, T - T // 2)])[:, None]
+    kv = kv.to(torch.bfloat16).float()
+    want, _ = latent_plain(spec, w, q, kv)
+    for cuts in ([T], [1, 399, 200], [129, 127, 344]):
+        r, at, got = LatentRun(spec, w, torch.bfloat16, "cuda"), 0, []
+        for cnt in cuts:
+            got.append(r.rows([(2, at, q[at:at + cnt], kv[at:at + cnt])]))
+            at += cnt
+        err = ((torch.cat(got).double() - want).abs().max() / want.abs().max()).item()
+        assert err < 0.03, err
 
 
 @pytest.mark.parametrize("device", DEVICES)

@@ -22,41 +22,9 @@
 
 namespace ve {
 
-VE_DEVINL void tmem_st32(uint32_t taddr, const uint32_t* r) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-      "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
-      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
-        "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]),
-        "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]),
-        "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-      : "memory");
-}
-VE_DEVINL void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
-// Descriptor of an MN-major operand stored with the 128-byte swizzle: 64 contiguous elements of the M / N extent per
-// 128 B row, 8 rows (8 steps of K) per 1024 B atom; `lbo` = bytes to the next 64 elements of M / N, `sbo` = bytes to
-// the next 8 steps of K.
-VE_DEVINL uint64_t make_desc_sw128_mn(uint32_t saddr, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= (uint64_t)((saddr & 0x3FFFF) >> 4);
-  d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(sbo >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
-
 constexpr int kTcRows = 128;        // query rows of a tile
 constexpr int kTcThreads = 320;
 constexpr float kTcLazyLog2 = 8.f;  // the reference maximum moves only when a page raises it by more than this
-
-VE_DEVINL float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 
 template <int HD, int NST>
 __global__ void __launch_bounds__(kTcThreads, 1) attn_prefill_tc_kernel(const AttnParams p, const __grid_constant__ CUtensorMap kmap,

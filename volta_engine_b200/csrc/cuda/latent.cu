@@ -8,10 +8,12 @@
 //   latent_expand   merges split partials and multiplies by W_uv
 //   latent_gather   a sequence's cache rows, contiguous
 //   latent_prefill  prompt rows against expanded keys / values: mma.sync flash attention, 64 rows x 64 keys; scores and
-//                   weights keep 32-bit quality (weights enter the second product as two bf16 terms)
+//                   weights keep 32-bit quality (weights enter the second product as two bf16 terms). On tcgen05 (latent_tc.cuh)
+//                   where plain + rotated width are at most three chunks of 64 columns and the values two, else on mma.sync
 // Angles are formed in double from a frequency table, so they are exact at any position. No fast-math in this file.
 // Neighbouring dimensions (2i, 2i + 1) form a rotation pair.
 #include "rowmath.cuh"
+#include "tmap.h"
 #include <float.h>
 
 namespace ve {
@@ -505,6 +507,7 @@ static int launch_latent_prefill(const LatentPrefill& p, int ntiles, cudaStream_
 }
 
 }  // namespace ve
+#include "latent_tc.cuh"
 
 using namespace ve;
 
@@ -624,6 +627,33 @@ int ve_latent_prefill(VE_LDIMS, const void* q, long ldq, const void* up, long ld
     return launch_latent_prefill<256, 128>(p, ntiles, st);
   }
   return launch_latent_prefill<256, 256>(p, ntiles, st);
+}
+
+// The same on tcgen05: tiles of at most 128 rows; d and rot in at most three chunks of 64 columns together, dv <= 128. up
+// [up_rows][...] and lat [up_rows][lat_w] are read through tensor maps.
+int ve_latent_prefill_tc(VE_LDIMS, const void* q, long ldq, const void* up, long ldu, const void* lat, int lat_w, long up_rows, const void* pos,
+                         const void* tile_first, const void* tile_count, const void* tile_base, int ntiles, void* out, long ldo, float scale, void* status,
+                         cudaStream_t st) {
+  if (ntiles <= 0) return 0;
+  const LatentDims n = VE_LMAKE;
+  const int uc = (d + 63) / 64, qc = uc + (rot + 63) / 64, vc = (dv + 63) / 64;
+  if (!ldims_ok(n) || d % 8 || rot % 8 || dv % 8 || rot0 % 8 || lat_w % 8 || ldq % 8 || ldu % 8 || ldo % 8 || qc > 3 || vc > 2 || scale <= 0.f ||
+      ((uintptr_t)q & 15) || ((uintptr_t)out & 15)) return cudaErrorInvalidValue;
+  CUtensorMap um, rm;
+  int rc = make_tmap_2d(&um, up, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, up_rows, (uint64_t)H * (d + dv), (uint64_t)ldu * 2, 64, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  rc = make_tmap_2d(&rm, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, up_rows, lat_w, (uint64_t)lat_w * 2, 64, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  LatentTc p{n, (const __nv_bfloat16*)q, ldq, (const int*)pos, (const int*)tile_first, (const int*)tile_count, (const int*)tile_base, (__nv_bfloat16*)out, ldo,
+             scale * 1.4426950408889634f, uc, (int*)status};
+  if (vc == 1) {
+    if (qc == 1) return launch_latent_tc<1, 1>(p, um, rm, ntiles, st);
+    if (qc == 2) return launch_latent_tc<2, 1>(p, um, rm, ntiles, st);
+    return launch_latent_tc<3, 1>(p, um, rm, ntiles, st);
+  }
+  if (qc == 1) return launch_latent_tc<1, 2>(p, um, rm, ntiles, st);
+  if (qc == 2) return launch_latent_tc<2, 2>(p, um, rm, ntiles, st);
+  return launch_latent_tc<3, 2>(p, um, rm, ntiles, st);
 }
 
 }  // extern "C"

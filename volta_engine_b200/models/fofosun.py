@@ -21,7 +21,7 @@ from .mixers import MIXERS, apply_linear, make_linear
 from .slot_state import SlotStates
 
 # CUDA sources whose kernels this model and its sampling launch
-KERNEL_SOURCES = ("gemm_tcgen05.cu", "gemv_rows.cu", "latent.cu", "linattn.cu", "mla.cu", "rowops.cu", "sampling.cu")
+KERNEL_SOURCES = ("gemm_bf16_wide.cu", "gemm_tcgen05.cu", "gemv_rows.cu", "latent.cu", "linattn.cu", "mla.cu", "rowops.cu", "sampling.cu")
 DTYPES = {"bf16": torch.bfloat16, "bfloat16": torch.bfloat16, "fp32": torch.float32, "float32": torch.float32}
 
 

@@ -520,6 +520,19 @@ def bf16_gemv_f32(W, x, out=None):
     return out
 
 
+GEMM_WIDE = os.environ.get("VOLTA_GEMM_WIDE", "1") != "0"
+
+
+def bf16_wide(T: int, N: int) -> bool:
+    """256 x 256 output tiles (csrc/cuda/gemm_bf16_wide.cu) where the grid still fills the GPU: a tile of twice the features
+    takes about 1.4 times as long as a 128 x 256 one."""
+    if T <= 128 or not GEMM_WIDE:
+        return False
+    tt = (T + 255) // 256
+    waves = lambda n: (n + 147) // 148
+    return 1.4 * waves((N + 255) // 256 * tt) < waves((N + 127) // 128 * tt)
+
+
 def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False):
     """out[t, n] = alpha * sum_k W[n,k] x[t,k] on tcgen05 (bf16 x bf16, fp32 accumulate)."""
     N, K = W.shape
@@ -527,7 +540,7 @@ def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False):
     if out is None:
         out = torch.empty(T, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     f32 = out.dtype == torch.float32
-    call("gemm_bf16", "plplplppliiifp", ptr(W), W.stride(0), ptr(x), x.stride(0), 0 if f32 else ptr(out),
+    call("gemm_bf16_wide" if bf16_wide(T, N) else "gemm_bf16", "plplplppliiifp", ptr(W), W.stride(0), ptr(x), x.stride(0), 0 if f32 else ptr(out),
          out.stride(0), ptr(out) if f32 else 0, ptr(residual), residual.stride(0) if residual is not None else 0,
          T, N, K, float(alpha), ptr(status_word(x.device)))
     return out
@@ -539,9 +552,6 @@ def gemm_f32(W, x):
     out = torch.empty(x.shape[0], N, dtype=torch.float32, device=x.device)
     call("gemm_f32", "plplpliii", ptr(W), W.stride(0), ptr(x), x.stride(0), ptr(out), N, x.shape[0], N, K)
     return out
-
-
-GEMM_WIDE = os.environ.get("VOLTA_GEMM_WIDE", "1") != "0"
 
 
 def gemm_w4a16(packed, sf_blocked, gscale, x, out=None, residual=None):

@@ -7,6 +7,7 @@ flash kernel; the all-32-bit form, and sizes outside the tensor-core kernels' ra
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 
 import torch
@@ -15,6 +16,8 @@ from .._lib import call, ptr
 from . import kernels as K
 
 PAGE = K.PAGE
+# prompt rows on the tcgen05 kernel where it applies; "mma" keeps the mma.sync kernel
+TC_PREFILL = os.environ.get("VOLTA_LATENT_PREFILL", "tc") != "mma"
 
 
 def _up(n: int, m: int) -> int:
@@ -54,6 +57,10 @@ class LatentSpec:
     def tc_prefill(self) -> bool:
         return (self.dim % 8 == 0 and self.rot % 8 == 0 and self.vdim % 8 == 0 and self.kv_rank % 8 == 0 and self.dim + self.rot <= 256
                 and self.vdim <= 256)
+
+    @property
+    def tcgen05(self) -> bool:
+        return self.tc_prefill and -(-self.dim // 64) - (-self.rot // 64) <= 3 and self.vdim <= 128 and self.scale > 0
 
     def dims(self, pool):
         return (self.heads, self.dim, self.rot, self.vdim, self.kv_rank, self.rot0, self.width, pool.shape[-1])
@@ -145,6 +152,11 @@ def _expanded(spec, q, kv, w_norm, ukv, b, cache, pool, out, r0):
     call("latent_gather", "pipippi" + "pii", ptr(pool), pool.shape[-1], ptr(table), table.shape[1], ptr(t.ctx_slot), ptr(t.ctx_base), t.ctx_slot.numel(),
          ptr(lat), spec.width, t.ctx_total)
     up = ukv.forward(lat[:, : spec.kv_rank])
+    if spec.tcgen05 and TC_PREFILL:
+        tf, tc, tb = t.wide_tiles
+        call("latent_prefill_tc", _D + "plplpil" + "ppppi" + "plfp", *D, ptr(qo), qo.stride(0), ptr(up), up.stride(0), ptr(lat), spec.width, t.ctx_total,
+             ptr(b.pos[r0:]), ptr(tf), ptr(tc), ptr(tb), tf.numel(), ptr(out[r0:]), out.stride(0), float(spec.scale), ptr(K.status_word(dev)))
+        return
     call("latent_prefill", _D + "plplpip" + "pppi" + "plf", *D, ptr(qo), qo.stride(0), ptr(up), up.stride(0), ptr(lat), spec.width, ptr(b.pos[r0:]),
          ptr(t.tile_first), ptr(t.tile_count), ptr(t.tile_base), t.tile_first.numel(), ptr(out[r0:]), out.stride(0), float(spec.scale))
 

@@ -36,6 +36,7 @@ class SegmentTable:
     tile_first: torch.Tensor | None  # tiles of at most 64 rows of one of these segments; rows counted from short_rows
     tile_count: torch.Tensor | None
     tile_base: torch.Tensor | None   # the segment's ctx_base
+    wide_tiles: tuple | None          # the same with at most 128 rows per tile: (first, count, base)
     chunk_seg: torch.Tensor | None   # chunks of at most CHUNK_ROWS rows of these segments: segment (0 = the first behind short_rows),
     chunk_first: torch.Tensor | None  # first row (in the batch) and rows
     chunk_count: torch.Tensor | None
@@ -61,10 +62,10 @@ class SegmentTable:
             k += 1
         rest = host[k:]
         short = rest[0][1] if rest else n
-        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 7), n_short=k)
+        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 8), n_short=k)
         if rest:
             base, total = [], 0
-            tf, tc, tb, cs, cf, cc, c0 = [], [], [], [], [], [], [0]
+            tf, tc, tb, cs, cf, cc, c0, wide = [], [], [], [], [], [], [0], []
             per = CHUNK_ROWS if n >= 1024 else CHUNK_ROWS // 2
             for g, (s, f, c, p0) in enumerate(rest):
                 base.append(total)
@@ -72,6 +73,7 @@ class SegmentTable:
                     tf.append(f + o - short)
                     tc.append(min(64, c - o))
                     tb.append(total)
+                wide += [(f + o - short, min(128, c - o), total) for o in range(0, c, 128)]
                 for o in range(0, c, per):
                     cs.append(g)
                     cf.append(f + o)
@@ -81,6 +83,7 @@ class SegmentTable:
             t.chunks, t.longest = len(cs), max(b - a for a, b in zip(c0, c0[1:]))
             t.ctx_slot, t.ctx_base, t.ctx_total = dev([h[0] for h in rest]), dev(base), total
             t.tile_first, t.tile_count, t.tile_base = dev(tf), dev(tc), dev(tb)
+            t.wide_tiles = tuple(dev(list(v)) for v in zip(*wide))
             t.chunk_seg, t.chunk_first, t.chunk_count, t.seg_chunk0 = dev(cs), dev(cf), dev(cc), dev(c0)
         return t
 

@@ -16,7 +16,7 @@ TABLE = {
     "embed": ("Embedding", P), "rope_store": ("RoPE + KV store", P), "gated_act": ("SwiGLU / GeGLU", P),
     "kv_quant_store": ("KV formats", P), "attention": ("Attention", P),
     "argmax": ("Sampling", P), "argmax2": ("Sampling", P), "topk": ("Sampling", P),
-    "gemm_bf16": ("Gemm", P), "gemm_w4a16": ("LinearNVFP4", P), "gemm_w4a16_wide": ("LinearNVFP4", P), "gemm_w4a4": ("LinearNVFP4", P),
+    "gemm_bf16": ("Gemm", P), "gemm_bf16_wide": ("Gemm", P), "gemm_w4a16": ("LinearNVFP4", P), "gemm_w4a16_wide": ("LinearNVFP4", P), "gemm_w4a4": ("LinearNVFP4", P),
     "gemm_grouped_bf16": ("MoE grouped GEMM", P), "gemm_grouped_w4a16": ("MoE grouped GEMM", P),
     "decode_w4a4": ("LinearNVFP4 decode", P), "decode_set_prefetch": ("LinearNVFP4 decode", P), "nvfp4_expand_rows": ("LinearNVFP4 decode", P),
     "nvfp4_gemv": ("LinearNVFP4 decode", P), "nvfp4_gemv_mma": ("LinearNVFP4 decode", P),
@@ -28,7 +28,7 @@ TABLE = {
     "mla_rope_store": ("MLALatent", P), "mla_absorb_q": ("MLALatent", P), "mla_decode": ("MLALatent", P),
     "mla_expand_out": ("MLALatent", P),
     "latent_rope_store": ("LatentAttention", P), "latent_absorb": ("LatentAttention", P), "latent_attn": ("LatentAttention", P),
-    "latent_expand": ("LatentAttention", P), "latent_gather": ("LatentAttention", P), "latent_prefill": ("LatentAttention", P),
+    "latent_expand": ("LatentAttention", P), "latent_gather": ("LatentAttention", P), "latent_prefill": ("LatentAttention", P), "latent_prefill_tc": ("LatentAttention", P),
     "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P), "linattn_chunk": ("LinearAttention", P),
     "embed_rows": ("RowOps (fp32 residual)", P), "dyt_rows": ("RowOps (fp32 residual)", P), "group_rms": ("RowOps (fp32 residual)", P),
     "polynorm": ("RowOps (fp32 residual)", P), "gemv_rows": ("LinearBF16 decode", P), "gemm_f32": ("Gemm (fp32)", P),
