@@ -6,6 +6,7 @@
 // 2..5 epilogue (TMEM lane = output feature, column = token). Rows and columns outside the matrices read as zero and are not
 // stored; K need not be a multiple of 64. Every wait is bounded.
 #include "common.cuh"
+#include "gemm_epilogue.cuh"
 #include "tmap.h"
 
 namespace ve {
@@ -95,32 +96,12 @@ gemm_bf16_wide_kernel(const WideBf16Params p, const __grid_constant__ CUtensorMa
     const bool ok = mbar_wait(&acc_full, 0);
     if (!ok) atomicExch(&s_fail, 1);
     tc_fence_after();
-    if (ok && !s_fail) {
-      const int q = warp & 3;                              // TMEM lane quarter this warp may touch
-#pragma unroll 1
-      for (int sub = 0; sub < 2; ++sub) {
-        const int n = n0 + sub * 128 + q * 32 + lane;
-#pragma unroll 1
-        for (int c0 = 0; c0 < 256; c0 += 32) {
-          if (t0 + c0 >= p.T) break;
-          uint32_t r[32];
-          tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + sub * 256 + c0, r);
-          tmem_ld_wait();
-          if (n < p.N) {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              const int t = t0 + c0 + j;
-              if (t < p.T) {
-                float v = __uint_as_float(r[j]) * p.alpha;
-                if (p.residual) v += bf2f(p.residual[(long)t * p.ldr + n]);
-                if (p.out_f32) p.out_f32[(long)t * p.ldo + n] = v;
-                else p.out[(long)t * p.ldo + n] = f2bf(v);
-              }
-            }
-          }
-        }
-      }
-    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");        // one answer for the four warps: they meet at barriers below
+    if (!*(volatile int*)&s_fail)
+      for (int sub = 0; sub < 2; ++sub)
+        if (n0 + sub * 128 < p.N)
+          store_tile<256>(smem, tmem_base + sub * 256, warp & 3, (warp - 2) * 32 + lane, n0 + sub * 128, t0,
+                          TileOut{p.N, p.T, p.alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr});
   }
   tc_fence_before();
   __syncthreads();

@@ -15,6 +15,7 @@
 // dequantisers during the main loop (MODE 1) and epilogue (TMEM -> registers -> global) at the end.
 // Every mbarrier wait is bounded; on expiry the kernel records a status code and drains.
 #include "common.cuh"
+#include "gemm_epilogue.cuh"
 #include "tmap.h"
 
 namespace ve {
@@ -94,6 +95,7 @@ gemm_kernel(const GemmParams p, const __grid_constant__ CUtensorMap amap, const 
   constexpr int TMEM_COLS = (ACC_COLS + SF_COLS) <= 32 ? 32 : (ACC_COLS + SF_COLS) <= 64 ? 64
                             : (ACC_COLS + SF_COLS) <= 128 ? 128 : (ACC_COLS + SF_COLS) <= 256 ? 256 : 512;
   static_assert(STAGE_BYTES % 1024 == 0, "stage must keep 1024 B alignment");
+  static_assert(STAGES * STAGE_BYTES >= BN * 528, "the output tile is staged in the operand ring");
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -268,28 +270,9 @@ gemm_kernel(const GemmParams p, const __grid_constant__ CUtensorMap amap, const 
     const bool ok = mbar_wait(&acc_full, 0);
     if (!ok) atomicExch(&s_fail, 1);
     tc_fence_after();
-    if (ok && !s_fail) {
-      const int q = warp & 3;  // TMEM lane quarter this warp may touch
-      const int n = n0 + q * 32 + lane;
-#pragma unroll 1
-      for (int c0 = 0; c0 < BN; c0 += 16) {
-        uint32_t r[16];
-        tmem_ld16(tmem_base + ((uint32_t)(q * 32) << 16) + c0, r);
-        tmem_ld_wait();
-        if (n < p.N) {
-#pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const int t = t0 + c0 + j;
-            if (t < t_end) {
-              float v = __uint_as_float(r[j]) * alpha;
-              if (p.residual) v += bf2f(p.residual[(long)t * p.ldr + n]);
-              if (p.out_f32) p.out_f32[(long)t * p.ldo + n] = v;
-              else p.out[(long)t * p.ldo + n] = f2bf(v);
-            }
-          }
-        }
-      }
-    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");        // one answer for the four warps: they meet at barriers below
+    if (!*(volatile int*)&s_fail)
+      store_tile<BN>(smem, tmem_base, warp & 3, etid, n0, t0, TileOut{p.N, t_end, alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr});
   }
   tc_fence_before();
   __syncthreads();

@@ -10,6 +10,7 @@
 // weight sub-tiles of each stage into swizzled bf16 and run the epilogue. Every wait is bounded.
 // Reference kernel family this replaces: src/kernels/cuda/nvfp4/skinny_kernels.cu:531-558 (fused WMMA GEMM / dequant + HGEMM).
 #include "common.cuh"
+#include "gemm_epilogue.cuh"
 #include "tmap.h"
 
 namespace ve {
@@ -157,31 +158,11 @@ gemm_w4a16_wide_kernel(const WideParams p, const __grid_constant__ CUtensorMap a
     const bool ok = mbar_wait(&acc_full, 0);
     if (!ok) atomicExch(&s_fail, 1);
     tc_fence_after();
-    if (ok && !s_fail) {
-      const int q = warp & 3;
-#pragma unroll 1
-      for (int sub = 0; sub < 2; ++sub) {
-        const int n = n0 + sub * 128 + q * 32 + lane;
-#pragma unroll 1
-        for (int c0 = 0; c0 < 256; c0 += 16) {
-          if (t0 + c0 >= p.T) break;
-          uint32_t r[16];
-          tmem_ld16(tmem_base + ((uint32_t)(q * 32) << 16) + sub * 256 + c0, r);
-          tmem_ld_wait();
-          if (n < p.N) {
-#pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const int t = t0 + c0 + j;
-              if (t < p.T) {
-                float v = __uint_as_float(r[j]) * p.alpha;
-                if (p.residual) v += bf2f(p.residual[(long)t * p.ldr + n]);
-                p.out[(long)t * p.ldo + n] = f2bf(v);
-              }
-            }
-          }
-        }
-      }
-    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");        // one answer for the four warps: they meet at barriers below
+    if (!*(volatile int*)&s_fail)
+      for (int sub = 0; sub < 2; ++sub)
+        store_tile<256>(smem, tmem_base + sub * 256, warp & 3, etid, n0 + sub * 128, t0,
+                        TileOut{p.N, p.T, p.alpha, p.out, nullptr, p.ldo, p.residual, p.ldr});
   }
   tc_fence_before();
   __syncthreads();

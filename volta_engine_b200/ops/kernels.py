@@ -525,12 +525,12 @@ GEMM_WIDE = os.environ.get("VOLTA_GEMM_WIDE", "1") != "0"
 
 def bf16_wide(T: int, N: int) -> bool:
     """256 x 256 output tiles (csrc/cuda/gemm_bf16_wide.cu) where the grid still fills the GPU: a tile of twice the features
-    takes about 1.4 times as long as a 128 x 256 one."""
+    takes about 1.75 times as long as a 128 x 256 one."""
     if T <= 128 or not GEMM_WIDE:
         return False
     tt = (T + 255) // 256
     waves = lambda n: (n + 147) // 148
-    return 1.4 * waves((N + 255) // 256 * tt) < waves((N + 127) // 128 * tt)
+    return 1.75 * waves((N + 255) // 256 * tt) < waves((N + 127) // 128 * tt)
 
 
 def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False):
