@@ -7,9 +7,9 @@
 //              3  x = PolyNorm of an fp32 row
 //   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual
 // The rows are the M side (16) of mma.sync.m16n8k16 and eight weight rows the N side. The order of k inside a product does
-// not matter, so a lane takes eight consecutive k of one weight row with one 16-byte load and uses them as the B operands of
-// two MMAs, the matching activations as the A operands: weights go from global memory to registers and are read once. The
-// first weights are requested before the programmatic dependency wait, so they arrive while the kernel in front finishes.
+// not matter, so a lane takes eight consecutive k of one weight row as 16 bytes and uses them as the B operands of two MMAs, the
+// matching activations as the A operands. Weights are read once; the first of them are requested before the programmatic
+// dependency wait, so they arrive while the kernel in front finishes.
 // gemm_f32 is the plain fp32 product of the all-32-bit form.
 #include "rowmath.cuh"
 
@@ -33,6 +33,12 @@ VE_DEVINL void rows_mma(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+VE_DEVINL void rows_out(const RowsArgs& a, int m, int n, float v) {
+  if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
+  else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
+  else a.out[m * a.ldo + n] = f2bf(v);
 }
 
 // Activations of the prologue forms -> bf16 rows in shared memory.
@@ -110,15 +116,121 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
   __syncthreads();
 }
 
-// 8 warps: R tiles of 8 weight rows x KS slices of k; units of 32 k, slice s takes units s, s + KS, ... CTAs are resident and walk
-// the groups of R tiles; the ring of requested weights (8 units per warp) runs on across groups. XM 0: all activations in shared
-// memory (made by the prologue, or copied), rows 8..15 only with HI. XM 1: they pass through shared memory in slabs of 8 units
-// per slice (many rows of a long k).
-template <int KS, int XM, bool HI>
-__global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
+// All activations in shared memory (made by the prologue, or copied). Resident CTAs (two per SM) walk tiles of eight weight rows; the
+// eight warps of a CTA share the k of a tile in units of 32 k. Every lane copies the 16-byte pieces it will use itself into a ring of its
+// own in shared memory (cp.async, groups of four units, DEPTH groups), so no barrier stands between the copies and their use and
+// nothing waits in order for younger loads. The first groups are requested before the dependency wait. HI: more than eight rows.
+template <int DEPTH, bool HI>
+__global__ void __launch_bounds__(256) gemv_ring_kernel(const RowsArgs a) {
+  constexpr int U = 4, GROUP = 8 * U * 512;               // bytes of one group of all warps
+  extern __shared__ __align__(16) uint8_t xs[];           // [M][pitch] activations, then [DEPTH][8 warps][U][32 lanes][16 B]
+  __shared__ float part[8][8][HI ? 16 : 8][8], red[3][33];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  uint8_t* ring = xs + a.M * a.pitch + (warp * U * 32 + lane) * 16;
+  const uint32_t ring_s = smem_u32(ring);
+  const int tiles = (a.N + 7) / 8, units = (a.K + 31) / 32, per_tile = (units + 8 * U - 1) / (8 * U);      // groups per tile
+  const int mine = (tiles - (int)blockIdx.x + (int)gridDim.x - 1) / (int)gridDim.x, total = mine * per_tile;
+  // unit of the group's j-th place: neighbours are halves of one 128-byte line of a weight row
+  auto unit_of = [&](int gi, int j) { return ((gi * (U / 2) + (j >> 1)) * 8 + warp) * 2 + (j & 1); };
+  int i_tile = blockIdx.x, i_g = 0, i_stage = 0, i_left = total;      // what is requested next
+  auto issue = [&]() {
+    if (i_left > 0) {
+      const __nv_bfloat16* wr = a.W + (long)min(i_tile * 8 + g, a.N - 1) * a.ldw + t * 8;
+#pragma unroll
+      for (int j = 0; j < U; ++j) {
+        const int u = unit_of(i_g, j);
+        const bool in = u * 32 + t * 8 < a.K;
+        const int n = in ? 16 : 0;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(ring_s + i_stage * GROUP + j * 512), "l"(in ? wr + u * 32 : a.W), "r"(n) : "memory");
+      }
+      --i_left;
+      if (++i_g == per_tile) {
+        i_g = 0;
+        i_tile += gridDim.x;
+      }
+      if (++i_stage == DEPTH) i_stage = 0;
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int d = 0; d < DEPTH - 1; ++d) issue();
+  grid_dep_wait();
+  grid_dep_launch();
+  if (a.pro) {
+    rows_prologue(a, xs, &red[0][0]);
+  } else {
+    const __nv_bfloat16* xg = reinterpret_cast<const __nv_bfloat16*>(a.x);
+    const int K32 = units * 32;
+    for (int i = tid; i < a.M * (K32 / 8); i += 256) {
+      const int m = i / (K32 / 8), k = (i % (K32 / 8)) * 8;
+      *reinterpret_cast<uint4*>(xs + m * a.pitch + k * 2) = k < a.K ? *reinterpret_cast<const uint4*>(xg + m * a.ldx + k) : make_uint4(0, 0, 0, 0);
+    }
+    __syncthreads();
+  }
+  float c[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+  const bool lo_in = g < a.M, hi_in = HI && g + 8 < a.M;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  const uint8_t* xlo = xs + g * a.pitch + t * 16;
+  int stage = 0, gi = 0, done = 0;                        // done: tiles finished
+  for (int it = 0; it < total; ++it) {
+    issue();                                              // into the stage the group in front was read from
+    asm volatile("cp.async.wait_group %0;" ::"n"(DEPTH - 1) : "memory");
+    uint4 w[U], lo[U], hi[U];
+#pragma unroll
+    for (int j = 0; j < U; ++j) {
+      const int u = unit_of(gi, j);
+      w[j] = *reinterpret_cast<const uint4*>(ring + stage * GROUP + j * 512);
+      lo[j] = lo_in && u < units ? *reinterpret_cast<const uint4*>(xlo + u * 64) : zero;
+      hi[j] = hi_in && u < units ? *reinterpret_cast<const uint4*>(xlo + 8 * a.pitch + u * 64) : zero;
+    }
+#pragma unroll
+    for (int j = 0; j < U; ++j) {
+      rows_mma(c[j & 1], lo[j].x, hi[j].x, lo[j].y, hi[j].y, w[j].x, w[j].y);
+      rows_mma(c[2 + (j & 1)], lo[j].z, hi[j].z, lo[j].w, hi[j].w, w[j].z, w[j].w);
+    }
+    if (++stage == DEPTH) stage = 0;
+    if (++gi < per_tile) continue;
+    gi = 0;
+    // The warps' sums of this tile go to one of eight buffers; the warps take turns adding them up while the others go on. A
+    // buffer comes round after eight tiles, and every warp has waited for all others once in between.
+    const int buf = done & 7, bar = 1 + buf;
+    float* pt = &part[buf][warp][0][0];
+    pt[g * 8 + 2 * t] = (c[0][0] + c[1][0]) + (c[2][0] + c[3][0]);
+    pt[g * 8 + 2 * t + 1] = (c[0][1] + c[1][1]) + (c[2][1] + c[3][1]);
+    if (HI) {
+      pt[(g + 8) * 8 + 2 * t] = (c[0][2] + c[1][2]) + (c[2][2] + c[3][2]);
+      pt[(g + 8) * 8 + 2 * t + 1] = (c[0][3] + c[1][3]) + (c[2][3] + c[3][3]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+    if (buf != warp) {
+      asm volatile("bar.arrive %0, 256;" ::"r"(bar) : "memory");
+    } else {
+      asm volatile("bar.sync %0, 256;" ::"r"(bar) : "memory");
+      const int n0 = (blockIdx.x + done * gridDim.x) * 8;
+      for (int i = lane; i < a.M * 8; i += 32) {
+        if (n0 + (i & 7) < a.N) {
+          float v = 0.f;
+#pragma unroll
+          for (int y = 0; y < 8; ++y) v += (&part[buf][y][0][0])[i];
+          rows_out(a, i >> 3, n0 + (i & 7), v);
+        }
+      }
+    }
+    ++done;
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+}
+
+// Rows whose activations do not fit: they pass through shared memory in slabs of eight units per slice of k. 8 warps: R tiles of 8
+// weight rows x KS slices of k, weights from global memory to registers (a ring of eight 16-byte loads per lane).
+template <int KS, bool HI>
+__global__ void __launch_bounds__(256, 3) gemv_slab_kernel(const RowsArgs a) {
   constexpr int R = 8 / KS, PF = 8, SLAB = KS * PF * 32, SP = SLAB * 2 + 64;
   extern __shared__ __align__(16) uint8_t xs[];
-  __shared__ float part[2][8][HI ? 16 : 8][8], red[3][33];
+  __shared__ float part[2][8][HI ? 16 : 8][8];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int ks = warp % KS, rt = warp / KS;
   const int units = (a.K + 31) / 32, batches = ((units + KS - 1) / KS + PF - 1) / PF;
@@ -149,20 +261,7 @@ __global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (XM == 0) {
-    if (a.pro) {
-      rows_prologue(a, xs, &red[0][0]);
-    } else {
-      const int K32 = units * 32;
-      for (int i = tid; i < a.M * (K32 / 8); i += 256) {
-        const int m = i / (K32 / 8), k = (i % (K32 / 8)) * 8;
-        *reinterpret_cast<uint4*>(xs + m * a.pitch + k * 2) = k < a.K ? *reinterpret_cast<const uint4*>(xg + m * a.ldx + k) : make_uint4(0, 0, 0, 0);
-      }
-      __syncthreads();
-    }
-  } else {
-    slab(0, 0);
-  }
+  slab(0, 0);
   int pb = 0, stage = 0;
   for (; grp < groups; grp += gridDim.x) {
     float c[4] = {0.f, 0.f, 0.f, 0.f};
@@ -170,15 +269,13 @@ __global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
       const bool last = b + 1 == batches;
       const int ngrp = last ? grp + gridDim.x : grp, nu = last ? ks : ks + (b + 1) * PF * KS;
       const __nv_bfloat16* wr = row_of(ngrp);
-      if (XM == 1) {
-        if (!last || ngrp < groups) {
-          slab(last ? 0 : b + 1, stage ^ 1);
-          asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-          asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
+      if (!last || ngrp < groups) {
+        slab(last ? 0 : b + 1, stage ^ 1);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+      } else {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
       }
+      __syncthreads();
 #pragma unroll
       for (int j = 0; j < PF; ++j) {
         const uint4 w = buf[j];
@@ -186,22 +283,15 @@ __global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
         const int u = ks + (b * PF + j) * KS;
         if (u < units) {
           uint4 lo = make_uint4(0, 0, 0, 0), hi = make_uint4(0, 0, 0, 0);
-          if (XM == 0) {
-            if (g < a.M) lo = *reinterpret_cast<const uint4*>(xs + g * a.pitch + u * 64 + t * 16);
-            if (HI && g + 8 < a.M) hi = *reinterpret_cast<const uint4*>(xs + (g + 8) * a.pitch + u * 64 + t * 16);
-          } else {
-            const uint8_t* p = xs + (stage * (HI ? 16 : 8) + g) * SP + (j * KS + ks) * 64 + t * 16;
-            lo = *reinterpret_cast<const uint4*>(p);
-            if (HI) hi = *reinterpret_cast<const uint4*>(p + 8 * SP);
-          }
+          const uint8_t* p = xs + (stage * (HI ? 16 : 8) + g) * SP + (j * KS + ks) * 64 + t * 16;
+          lo = *reinterpret_cast<const uint4*>(p);
+          if (HI) hi = *reinterpret_cast<const uint4*>(p + 8 * SP);
           rows_mma(c, lo.x, hi.x, lo.y, hi.y, w.x, w.y);
           rows_mma(c, lo.z, hi.z, lo.w, hi.w, w.z, w.w);
         }
       }
-      if (XM == 1) {
-        stage ^= 1;
-        __syncthreads();                                  // the slab behind may be overwritten now
-      }
+      stage ^= 1;
+      __syncthreads();                                    // the slab behind may be overwritten now
     }
     part[pb][warp][g][2 * t] = c[0];
     part[pb][warp][g][2 * t + 1] = c[1];
@@ -216,9 +306,7 @@ __global__ void __launch_bounds__(256, 3) gemv_rows_kernel(const RowsArgs a) {
       float v = 0.f;
 #pragma unroll
       for (int s = 0; s < KS; ++s) v += part[pb][r * KS + s][m][e];
-      if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
-      else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
-      else a.out[m * a.ldo + n] = f2bf(v);
+      rows_out(a, m, n, v);
     }
     pb ^= 1;                                              // (the other buffer's readers are done: they passed the barrier above)
   }
@@ -258,19 +346,41 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       if (t0 + tt + i < T && n0 + tn + j < N) out[(long)(t0 + tt + i) * ldo + n0 + tn + j] = acc[i][j];
 }
 
-template <int KS, int XM, bool HI>
-static int launch_rows(const RowsArgs& a, cudaStream_t st) {
-  constexpr int SP = KS * 8 * 32 * 2 + 64;
-  const int smem = XM ? 2 * (HI ? 16 : 8) * SP : a.M * a.pitch;
-  static int attr = 0;
-  if (smem > attr) {
-    cudaError_t e = cudaFuncSetAttribute(gemv_rows_kernel<KS, XM, HI>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return (int)e;
-    attr = smem;
-  }
+template <typename F>
+static int allow_smem(F kernel, int smem, int& have) {
+  if (smem <= have) return 0;
+  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e == cudaSuccess) have = smem;
+  return (int)e;
+}
+
+template <int DEPTH, bool HI>
+static int launch_ring_d(const RowsArgs& a, cudaStream_t st) {
+  const int smem = a.M * a.pitch + DEPTH * 16 * 1024, tiles = (a.N + 7) / 8;
+  static int have = 0;
+  const int rc = allow_smem(gemv_ring_kernel<DEPTH, HI>, smem, have);
+  if (rc) return rc;
+  const int ctas = !HI && (smem + 18 * 1024) * 2 <= 227 * 1024 ? 296 : 148;
+  launch_pdl(gemv_ring_kernel<DEPTH, HI>, dim3(tiles < ctas ? tiles : ctas), dim3(256), smem, st, a);
+  return (int)cudaGetLastError();
+}
+template <bool HI>
+static int launch_ring(const RowsArgs& a, cudaStream_t st) {
+  const int room = (95 * 1024 - a.M * a.pitch) / (16 * 1024);           // groups that fit in half of the SM's shared memory
+  if (room >= 5) return launch_ring_d<5, HI>(a, st);
+  if (room == 4) return launch_ring_d<4, HI>(a, st);
+  return launch_ring_d<3, HI>(a, st);
+}
+
+template <int KS, bool HI>
+static int launch_slab(const RowsArgs& a, cudaStream_t st) {
+  constexpr int smem = 2 * (HI ? 16 : 8) * (KS * 8 * 32 * 2 + 64);
+  static int have = 0;
+  const int rc = allow_smem(gemv_slab_kernel<KS, HI>, smem, have);
+  if (rc) return rc;
   const int groups = ((a.N + 7) / 8 + 8 / KS - 1) / (8 / KS);
   const int per = (smem + (HI ? 9 : 5) * 1024) * 3 <= 222 * 1024 ? 3 : (smem + (HI ? 9 : 5) * 1024) * 2 <= 222 * 1024 ? 2 : 1;
-  launch_pdl(gemv_rows_kernel<KS, XM, HI>, dim3(groups < 148 * per ? groups : 148 * per), dim3(256), smem, st, a);
+  launch_pdl(gemv_slab_kernel<KS, HI>, dim3(groups < 148 * per ? groups : 148 * per), dim3(256), smem, st, a);
   return (int)cudaGetLastError();
 }
 
@@ -297,16 +407,9 @@ int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, 
   } else if (kx != K || ldx % 8 || ((uintptr_t)x & 15)) {
     return cudaErrorInvalidValue;
   }
-  const int tiles = (N + 7) / 8, units = (K + 31) / 32;
-  if ((long)M * a.pitch <= 100 * 1024) {
-    // at least eight units per warp where k is long enough; otherwise fewer slices of k and more rows per group
-#define VE_GR(KS) (M <= 8 ? launch_rows<KS, 0, false>(a, st) : launch_rows<KS, 0, true>(a, st))
-    if (units >= 48 || tiles < 148) return VE_GR(8);
-    if (units >= 24) return VE_GR(4);
-    return VE_GR(2);
-#undef VE_GR
-  }
-#define VE_GR(KS) (M <= 8 ? launch_rows<KS, 1, false>(a, st) : launch_rows<KS, 1, true>(a, st))
+  if ((long)M * a.pitch <= 100 * 1024) return M <= 8 ? launch_ring<false>(a, st) : launch_ring<true>(a, st);
+  const int tiles = (N + 7) / 8;
+#define VE_GR(KS) (M <= 8 ? launch_slab<KS, false>(a, st) : launch_slab<KS, true>(a, st))
   if (tiles >= 4 * 120) return VE_GR(2);
   if (tiles >= 2 * 120) return VE_GR(4);
   return VE_GR(8);
