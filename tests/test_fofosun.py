@@ -225,3 +225,33 @@ def test_other_designs_are_refused(tmp_path):
     write_model(tmp_path, "eights")
     with pytest.raises(NotImplementedError):
         load_model(tmp_path, "cpu", quantize="nvfp4")
+
+
+def test_trace_run_says_which_models_it_does_not_run(tmp_path):
+    from volta_engine_b200.models.dense import DenseConfig
+    from volta_engine_b200.models.factory import kernel_sources, save_dense_checkpoint
+    from volta_engine_b200.tools import trace_run
+    save_dense_checkpoint(tmp_path / "d", DenseConfig.tiny())
+    args = ["--model", str(tmp_path / "d"), "--out", str(tmp_path), "--max-tokens", "128"]
+    assert trace_run.main(args + ["--dtype", "bfloat16"], stdin=io.StringIO(""), device="cpu") == 2
+    assert trace_run.main(args + ["--dtype", "float32"], stdin=io.StringIO(""), device="cpu") == 3
+    assert kernel_sources(tmp_path / "d") is None
+
+
+def test_a_model_names_the_sources_of_its_kernels(tmp_path):
+    """Every entry point the model's Python side calls is defined in the sources that a fresh checkout compiles for it."""
+    import re
+    from pathlib import Path
+    import volta_engine_b200
+    from volta_engine_b200.models.factory import kernel_sources
+    write_model(tmp_path, "eights")
+    part, names = kernel_sources(tmp_path)
+    root = Path(volta_engine_b200.__file__).parent
+    defined = set()
+    for n in names:
+        defined |= set(re.findall(r"^int ve_(\w+)\(", (root / "csrc" / "cuda" / n).read_text(), re.M))
+    called = set()
+    for f in ("ops/latent.py", "ops/linear_attn.py", "ops/rowops.py"):
+        called |= set(re.findall(r'call\("(\w+)"', (root / f).read_text()))
+    called |= {"gemm_bf16", "gemm_bf16_wide", "gemm_f32", "argmax", "argmax2", "topk"}
+    assert part == "fofosun" and called <= defined
