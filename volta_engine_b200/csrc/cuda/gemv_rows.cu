@@ -3,9 +3,11 @@
 //   y[m][n] = sum_k W[n][k] x[m][k],   m < 16
 //   prologue   0  x given in bf16
 //              1  x = tanh(alpha h) w + b of the fp32 residual h
-//              2  x = RMS norm over groups of columns of an fp32 row [* sigmoid(gate)]
+//              2  x = RMS norm over groups of columns of an fp32 row [* sigmoid(gate) or silu(gate)], behind columns taken as they are
 //              3  x = PolyNorm of an fp32 row
-//   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual
+//              4  x = layer norm (no shift) of the weighted sum of the fp32 residual streams
+//              5  x = clamped gated unit of an fp32 [gate | up] row
+//   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write)
 // The rows are the M side (16) of mma.sync.m16n8k16 and eight weight rows the N side. The order of k inside a product does
 // not matter, so a lane takes eight consecutive k of one weight row as 16 bytes and uses them as the B operands of two MMAs, the
 // matching activations as the A operands. Weights are read once; the first of them are requested before the programmatic
@@ -26,6 +28,9 @@ struct RowsArgs {
   const float* coef; float eps;
   float* out_f32; __nv_bfloat16* out; long ldo;
   float* h; long ldh; const float* scale;
+  const float* head; long ldhead; int k0;     // prologue 2: the first k0 columns of x, as they are
+  int silu;                         // prologue 2: activation of the gate
+  int streams; const float* hmix;   // streams > 0: h [M][streams][N], scale [streams]
   int pitch;                        // bytes per activation row in shared memory (prologue forms)
 };
 
@@ -36,7 +41,16 @@ VE_DEVINL void rows_mma(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_
 }
 
 VE_DEVINL void rows_out(const RowsArgs& a, int m, int n, float v) {
-  if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
+  if (a.streams) {
+    float* hp = a.h + m * a.ldh + n;
+    float x[kMaxStreams];
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; ++s) x[s] = s < a.streams ? hp[(long)s * a.N] : 0.f;
+    streams_write(x, a.streams, a.hmix, a.scale, v);
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; ++s)
+      if (s < a.streams) hp[(long)s * a.N] = x[s];
+  } else if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
   else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
   else a.out[m * a.ldo + n] = f2bf(v);
 }
@@ -54,7 +68,9 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
       for (int m = 0; m < a.M; ++m) put(m, k, dyt_of(src[m * a.ldx + k], a.alpha, wk, bk));
     }
   } else if (a.pro == 2) {
-    const int groups = a.kx / a.G;
+    const int groups = (a.kx - a.k0) / a.G;
+    for (int i = tid; i < a.k0; i += 256)
+      for (int m = 0; m < a.M; ++m) put(m, i, a.head[m * a.ldhead + i]);
     if (groups * a.M >= 8) {
       for (int p = warp; p < groups * a.M; p += 8) {
         const int m = p / groups, c0 = (p % groups) * a.G;
@@ -67,8 +83,8 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
         for (int i = lane; i < a.G; i += 32) {
           const int c = c0 + i;
           float v = src[m * a.ldx + c] * inv * a.w[c % a.wlen];
-          if (a.gate) v *= sigmoid_of(a.gate[m * a.ldg + c]);
-          put(m, c, v);
+          if (a.gate) v *= a.silu ? silu_of(a.gate[m * a.ldg + c]) : sigmoid_of(a.gate[m * a.ldg + c]);
+          put(m, a.k0 + c, v);
         }
       }
     } else {
@@ -83,11 +99,54 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
         for (int i = tid; i < a.G; i += 256) {
           const int c = c0 + i;
           float v = src[m * a.ldx + c] * inv * a.w[c % a.wlen];
-          if (a.gate) v *= sigmoid_of(a.gate[m * a.ldg + c]);
-          put(m, c, v);
+          if (a.gate) v *= a.silu ? silu_of(a.gate[m * a.ldg + c]) : sigmoid_of(a.gate[m * a.ldg + c]);
+          put(m, a.k0 + c, v);
         }
       }
     }
+  } else if (a.pro == 4) {
+    // sums of every row around its first column (so that a common offset does not cancel digits), one exchange for all rows
+    const int S = a.G;
+    float win[kMaxStreams];
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; ++s) win[s] = s < S ? a.coef[s] : 0.f;
+    auto read = [&](int m, int k) {
+      float u = 0.f;
+#pragma unroll
+      for (int s = 0; s < kMaxStreams; ++s)
+        if (s < S) u = fmaf(win[s], src[m * a.ldx + (long)s * a.kx + k], u);
+      return u;
+    };
+    for (int m = 0; m < a.M; ++m) {
+      const float c = read(m, 0);
+      float s1 = 0.f, s2 = 0.f;
+      for (int i = tid; i < a.kx; i += 256) {
+        const float d = read(m, i) - c;
+        s1 += d;
+        s2 = fmaf(d, d, s2);
+      }
+      s1 = warp_sum(s1);
+      s2 = warp_sum(s2);
+      if (lane == 0) {
+        red[(m * 8 + warp) * 2] = s1;
+        red[(m * 8 + warp) * 2 + 1] = s2;
+      }
+    }
+    __syncthreads();
+    for (int m = 0; m < a.M; ++m) {
+      const float c = read(m, 0), n = 1.f / (float)a.kx;
+      float s1 = 0.f, s2 = 0.f;
+#pragma unroll
+      for (int y = 0; y < 8; ++y) {
+        s1 += red[(m * 8 + y) * 2];
+        s2 += red[(m * 8 + y) * 2 + 1];
+      }
+      const float d = s1 * n, inv = 1.f / sqrtf(fmaxf(fmaf(-d, d, s2 * n), 0.f) + a.eps);
+      for (int i = tid; i < a.kx; i += 256) put(m, i, (read(m, i) - c - d) * inv * a.w[i]);
+    }
+  } else if (a.pro == 5) {
+    for (int m = 0; m < a.M; ++m)
+      for (int i = tid; i < a.kx; i += 256) put(m, i, clamped_glu_of(src[m * a.ldx + i], src[m * a.ldx + a.kx + i], a.alpha, a.eps));
   } else {
     for (int m = 0; m < a.M; ++m) {
       float s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -124,7 +183,7 @@ template <int DEPTH, bool HI>
 __global__ void __launch_bounds__(256) gemv_ring_kernel(const RowsArgs a) {
   constexpr int U = 4, GROUP = 8 * U * 512;               // bytes of one group of all warps
   extern __shared__ __align__(16) uint8_t xs[];           // [M][pitch] activations, then [DEPTH][8 warps][U][32 lanes][16 B]
-  __shared__ float part[8][8][HI ? 16 : 8][8], red[3][33];
+  __shared__ float part[8][8][HI ? 16 : 8][8], red[4][33];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   uint8_t* ring = xs + a.M * a.pitch + (warp * U * 32 + lane) * 16;
   const uint32_t ring_s = smem_u32(ring);
@@ -390,20 +449,25 @@ using namespace ve;
 
 extern "C" {
 
-// pro 0: x bf16 [M, K], M <= 16. pro 1..3: x fp32 [M, kx], M <= 8 and the activation rows fit in shared memory (else refused).
-// Exactly one of h, out_f32 and out is written.
+// pro 0: x bf16 [M, K], M <= 16. pro 1..5: x fp32, M <= 8 and the activation rows (kx columns) fit in shared memory (else refused).
+// pro 2 with k0 > 0: columns [0, k0) from head, the norm's columns behind them. pro 4: G streams of kx columns weighted by coef.
+// pro 5: 2 kx columns, alpha and (in eps) the limit. Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
+// with hmix [streams][streams] and scale [streams].
 int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, const void* x, long ldx, const void* w, const void* b, float alpha, int G,
                  int wlen, const void* gate, long ldg, const void* coef, float eps, void* out_f32, void* out, long ldo, void* h, long ldh, const void* scale,
-                 cudaStream_t st) {
+                 const void* head, long ldhead, int k0, int silu, int streams, const void* hmix, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
-  if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 3) return cudaErrorInvalidValue;
+  if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 5) return cudaErrorInvalidValue;
   RowsArgs a{(const __nv_bfloat16*)W, ldw, N, K, M, pro, kx, x, ldx, (const float*)w, (const float*)b, alpha, G, wlen, (const float*)gate, ldg,
-             (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale, 0};
+             (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale,
+             (const float*)head, ldhead, k0, silu, streams, (const float*)hmix, 0};
+  if (streams < 0 || streams > kMaxStreams || (streams && (!h || !hmix || !scale))) return cudaErrorInvalidValue;
   const int K32 = (K + 31) / 32 * 32;
   a.pitch = K32 * 2 + ((K32 * 2) % 128 == 0 ? 64 : 0);            // rows of a quad pair land in different halves of the banks
   if (pro) {
     if (M > 8 || (long)M * a.pitch > 100 * 1024) return cudaErrorInvalidValue;
-    if ((pro == 1 && (!w || !b || h)) || (pro == 2 && (!w || G < 1 || kx % G || wlen < 1)) || (pro == 3 && !coef)) return cudaErrorInvalidValue;
+    if ((pro == 1 && (!w || !b || h)) || (pro == 2 && (!w || G < 1 || k0 < 0 || k0 > kx || (kx - k0) % G || wlen < 1 || (k0 && !head))) ||
+        (pro == 3 && !coef) || (pro == 4 && (!w || !coef || G < 1 || G > kMaxStreams || h))) return cudaErrorInvalidValue;
   } else if (kx != K || ldx % 8 || ((uintptr_t)x & 15)) {
     return cudaErrorInvalidValue;
   }

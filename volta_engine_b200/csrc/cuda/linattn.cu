@@ -1,10 +1,13 @@
 // Linear attention with a decayed outer-product state, one fp32 state S [dk][dv] per (slot, head):
 //     S_t = diag(d_t) S_(t-1) + k_t v_t^T,      o_t = S_t^T q_t
-// Two ways to get decay and key from a projection row [ q (H dk) | x (H dk) | v (H dv) | ... ]:
+// Three ways to get decay and key from a projection row [ q (H dk) | x (H dk) | v (H dv) | ... ]:
 //   MODE 0  constant decay per head (table), k = silu(x), v = silu(v)                     ("lightning" attention)
 //   MODE 1  forget gate per channel: f = lower + (1 - lower) sigmoid(x + bias), d = f, k = 1 - f, v as projected   (HGRN2)
-// q = silu(q) in both. Gates, decays, states and outputs are fp32; the file is compiled without fast-math.
+//   MODE 2  decay per channel sigmoid(z)^(1 / tau) with z = W a + bias for a low-rank row a of the projection; k = x, v as projected,
+//           q scaled by a constant                                                        (gated linear attention)
+// q = silu(q) in modes 0 and 1. Gates, decays, states and outputs are fp32; the file is compiled without fast-math.
 //
+//   linattn_decay   the decays of mode 2 as rows (for the chunks; the stepped kernel forms its own)
 //   linattn_step    walks the rows of a segment in order with the state in registers (decode rows, short portions, and the
 //                   all-32-bit form). One CTA per (head, 32 value columns, segment).
 //   linattn_chunk   prompt portions, chunks of up to 128 rows in parallel: (a) every chunk's own contribution to the state,
@@ -27,11 +30,35 @@ struct LinArgs {
   const int* pos; const int* slot;
   const int* seg_first; const int* seg_count;   // null: one CTA row per batch row, the first row of a slot takes them all
   float* state;                                 // [slots][H][dk][dv]
-  const float* bias; const float* lower;        // MODE 1: [H dk] each
+  const float* bias; const float* lower;        // MODE 1: [H dk] each; MODE 2: bias
   const float* decay;                           // MODE 0: [H]
   float* o; long ldo;                           // [rows][H dv]
   int rows, H, dk, dv;
+  const float* w2; int rank, a_col;             // MODE 2: [H dk][rank], first column of the low-rank part in a projection row
+  float inv_tau, q_scale;
 };
+
+// sigmoid(z)^inv_tau through the logarithm of the sigmoid, which is exact on both sides
+VE_DEVINL float root_decay(float z, float inv_tau) { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau); }
+
+template <typename X>
+VE_DEVINL float lowrank_of(const X* __restrict__ a, const float* __restrict__ w, int rank, float z) {
+  float z1 = 0.f;
+  int r = 0;
+  if ((rank & 3) == 0) {
+    float z2 = 0.f, z3 = 0.f;
+    for (; r < rank; r += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(w + r);
+      z = fmaf(v.x, to_f(a[r]), z);
+      z1 = fmaf(v.y, to_f(a[r + 1]), z1);
+      z2 = fmaf(v.z, to_f(a[r + 2]), z2);
+      z3 = fmaf(v.w, to_f(a[r + 3]), z3);
+    }
+    return (z + z1) + (z2 + z3);
+  }
+  for (; r < rank; ++r) z = fmaf(w[r], to_f(a[r]), z);
+  return z;
+}
 
 // Rows of the segment that blockIdx.z stands for; -1 when there is nothing to do.
 VE_DEVINL int segment_of(const LinArgs& a, int z, int& count) {
@@ -84,19 +111,25 @@ __global__ void __launch_bounds__(256) linattn_step_kernel(const LinArgs a) {
   }
   const X* base = reinterpret_cast<const X*>(a.proj);
   const long oq = (long)h * a.dk + tid, okx = (long)(a.H + h) * a.dk + tid, ov = (long)2 * a.H * a.dk + (long)h * a.dv + col;
-  float rq = 0.f, rx = 0.f, rv = 0.f;
+  float rq = 0.f, rx = 0.f, rv = 0.f, rz = 0.f;
+  const float* w2 = MODE == 2 && tid < a.dk ? a.w2 + ((long)h * a.dk + tid) * a.rank : nullptr;
+  if (MODE == 2 && tid < a.dk) bias = a.bias[h * a.dk + tid];
   if (tid < a.dk) {
     rq = to_f(base[i * a.ld + oq]);
     rx = to_f(base[i * a.ld + okx]);
+    if (MODE == 2) rz = lowrank_of(base + i * a.ld + a.a_col, w2, a.rank, bias);
   }
   if (live) rv = to_f(base[i * a.ld + ov]);
   int b = 0, prev = -1;
   while (i >= 0) {
     if (tid < NK * 8) {
       const bool in = tid < a.dk;
-      sq[b][tid] = in ? silu_of(rq) : 0.f;
+      sq[b][tid] = in ? (MODE == 2 ? rq * a.q_scale : silu_of(rq)) : 0.f;
       if (MODE == 0) sk[b][tid] = in ? silu_of(rx) : 0.f;
-      else {
+      else if (MODE == 2) {
+        sk[b][tid] = in ? rx : 0.f;
+        sd[b][tid] = in ? root_decay(rz, a.inv_tau) : 0.f;
+      } else {
         const float z = rx + bias;
         sd[b][tid] = in ? fmaf(1.f - low, sigmoid_of(z), low) : 0.f;
         sk[b][tid] = in ? (1.f - low) * sigmoid_of(-z) : 0.f;
@@ -109,6 +142,7 @@ __global__ void __launch_bounds__(256) linattn_step_kernel(const LinArgs a) {
       if (tid < a.dk) {
         rq = to_f(base[nxt * a.ld + oq]);
         rx = to_f(base[nxt * a.ld + okx]);
+        if (MODE == 2) rz = lowrank_of(base + nxt * a.ld + a.a_col, w2, a.rank, bias);
       }
       if (live) rv = to_f(base[nxt * a.ld + ov]);
     }
@@ -156,6 +190,8 @@ struct LinChunkArgs {
   const float* bias; const float* lower; const float* decay;
   float* o; long ldo;
   int H, dk, dv, vec;                   // vec: 16-byte copies are aligned
+  const float* dec;                     // MODE 2: decays [rows][H dk]
+  float q_scale;
 };
 
 VE_DEVINL void la_ldsm_x4(uint32_t addr, uint32_t* r) {
@@ -182,16 +218,18 @@ VE_DEVINL void la_put(__nv_bfloat16* hi, __nv_bfloat16* lo, int at, float v) {
 }
 
 // grid (chunks, H), 128 threads. OUT false: pass (a), true: pass (c). DK, DV: padded widths (32, 64 or 128).
+// MODE 2 brings its decays as rows: they are staged beside the projections, and the block's own products read decays, keys and
+// queries where they were staged.
 template <int DK, int DV, int MODE, bool OUT>
 __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a) {
   constexpr int KP = DK + 8, VP = DV + 8;                 // bf16 row pitches: 16 bytes past a multiple of 64 (no ldmatrix conflicts)
   constexpr int MT = DV >= 64 ? DV / 64 : 1;              // 16-column tiles of the value width per warp
-  constexpr int NT = DK / 8, RAW = 2 * DK + DV;           // RAW: floats per staged row [q | x | v]
+  constexpr int NT = DK / 8, RAW = 2 * DK + DV + (MODE == 2 ? DK : 0);           // RAW: floats per staged row [q | x | v (| decay)]
   constexpr int CG = DK / 8;                              // channels per thread in the block's own products
   extern __shared__ __align__(16) uint8_t sm[];
   float* raw = reinterpret_cast<float*>(sm);              // [2][16][RAW]
   float* sf = raw + 2 * 16 * RAW;                         // [16][DK] decays
-  float* btot = sf + 16 * DK;                             // [DK]
+  float* btot = sf + (MODE == 2 ? 0 : 16 * DK);           // [DK]
   __nv_bfloat16* ksh = reinterpret_cast<__nv_bfloat16*>(btot + DK);   // [16][KP] decayed keys, two terms
   __nv_bfloat16* ksl = ksh + 16 * KP;
   __nv_bfloat16* vs = ksl + 16 * KP;                      // [16][VP]
@@ -218,6 +256,10 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
   float* cs = a.start + ((long)c * a.H + h) * a.dk * a.dv;
   const long oq = (long)h * a.dk, ox = (long)(a.H + h) * a.dk, ov = (long)2 * a.H * a.dk + (long)h * a.dv;
 
+  auto from = [&](int part, int row, int col) {           // where column col of a staged part lives
+    if (MODE == 2 && part == 3) return a.dec + ((long)(first + row) * a.H + h) * a.dk + col;
+    return a.proj + (long)(first + row) * a.ld + (part == 0 ? oq : part == 1 ? ox : ov) + col;
+  };
   // rows [16 b, 16 b + 16) of the chunk into raw buffer b & 1 (rows and columns that do not exist: zeros)
   auto stage = [&](int b) {
     float* dst = raw + (b & 1) * 16 * RAW;
@@ -225,18 +267,18 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
       constexpr int Q4 = RAW / 4;
       for (int i = tid; i < 16 * Q4; i += 128) {
         const int r = i / Q4, w = (i % Q4) * 4, row = b * 16 + r;
-        const int part = w < DK ? 0 : (w < 2 * DK ? 1 : 2), col = w - part * DK;
+        const int part = w < DK ? 0 : (w < 2 * DK ? 1 : (w < 2 * DK + DV ? 2 : 3)), col = part == 3 ? w - 2 * DK - DV : w - part * DK;
         const bool in = row < count && col < (part == 2 ? a.dv : a.dk) && (OUT || part != 0);
-        const float* src = a.proj + (in ? (long)(first + row) * a.ld + (part == 0 ? oq : part == 1 ? ox : ov) + col : 0);
+        const float* src = in ? from(part, row, col) : a.proj;
         const int n = in ? 16 : 0;
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * RAW + w)), "l"(src), "r"(n) : "memory");
       }
     } else {
       for (int i = tid; i < 16 * RAW; i += 128) {
         const int r = i / RAW, w = i % RAW, row = b * 16 + r;
-        const int part = w < DK ? 0 : (w < 2 * DK ? 1 : 2), col = w - part * DK;
+        const int part = w < DK ? 0 : (w < 2 * DK ? 1 : (w < 2 * DK + DV ? 2 : 3)), col = part == 3 ? w - 2 * DK - DV : w - part * DK;
         const bool in = row < count && col < (part == 2 ? a.dv : a.dk);
-        dst[i] = in ? a.proj[(long)(first + row) * a.ld + (part == 0 ? oq : part == 1 ? ox : ov) + col] : 0.f;
+        dst[i] = in ? *from(part, row, col) : 0.f;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -286,6 +328,9 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         if (MODE == 0) {
           f[i] = in ? head_decay : 1.f;
           k[i] = in ? silu_of(x) : 0.f;
+        } else if (MODE == 2) {
+          f[i] = in ? rw[i * RAW + 2 * DK + DV + tid] : 1.f;
+          k[i] = x;                                       // (zero where there is no row or channel)
         } else {
           const float z = x + bias, e = expf(-fabsf(z)), r = 1.f / (1.f + e);       // sigmoid(z) and sigmoid(-z)
           const float p = z >= 0.f ? r : e * r, n = z >= 0.f ? e * r : r;
@@ -294,10 +339,12 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         }
         run *= f[i];
         if (OUT) {
-          const float q = in ? silu_of(rw[i * RAW + tid]) : 0.f;
-          sf[i * DK + tid] = f[i];
-          sk[i * DK + tid] = k[i];
-          sq[i * DK + tid] = q;
+          const float q = MODE == 2 ? rw[i * RAW + tid] * a.q_scale : in ? silu_of(rw[i * RAW + tid]) : 0.f;
+          if (MODE != 2) {
+            sf[i * DK + tid] = f[i];
+            sk[i * DK + tid] = k[i];
+            sq[i * DK + tid] = q;
+          }
           la_put(qph, qpl, i * KP + tid, q * run);
         }
       }
@@ -321,6 +368,10 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
     if (OUT) {
       // ---- the block's own products in fp32: thread = (key row s, CG channels)
       const int s = tid & 15, c0 = (tid >> 4) * CG;
+      constexpr int OP = MODE == 2 ? RAW : DK;            // row pitch of the operands
+      const float* of = (MODE == 2 ? rw + 2 * DK + DV : sf) + c0;
+      const float* ok = (MODE == 2 ? rw + DK : sk) + c0;
+      const float* oqs = (MODE == 2 ? rw : sq) + c0;
       float w[CG], acc[16];
 #pragma unroll
       for (int j = 0; j < CG; ++j) w[j] = 0.f;
@@ -329,11 +380,11 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         float sum = 0.f;
 #pragma unroll
         for (int j = 0; j < CG; j += 4) {
-          const float4 f4 = *reinterpret_cast<const float4*>(sf + i * DK + c0 + j), q4 = *reinterpret_cast<const float4*>(sq + i * DK + c0 + j);
+          const float4 f4 = *reinterpret_cast<const float4*>(of + i * OP + j), q4 = *reinterpret_cast<const float4*>(oqs + i * OP + j);
           const float fv[4] = {f4.x, f4.y, f4.z, f4.w}, qv[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            w[j + e] = i == s ? sk[s * DK + c0 + j + e] : w[j + e] * fv[e];
+            w[j + e] = i == s ? ok[s * OP + j + e] : w[j + e] * fv[e];
             sum = fmaf(qv[e], w[j + e], sum);
           }
         }
@@ -368,7 +419,7 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         float v = 0.f;
 #pragma unroll
         for (int y = 0; y < 8; ++y) v += apart[(y * 16 + (i >> 4)) * 17 + (i & 15)];
-        la_put(ah, al, (i >> 4) * 24 + (i & 15), v);
+        la_put(ah, al, (i >> 4) * 24 + (i & 15), MODE == 2 ? v * a.q_scale : v);
       }
       __syncthreads();
       if (wlive) {
@@ -437,6 +488,37 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
   if (!OUT && ch) a.total[((long)c * a.H + h) * a.dk + tid] = prod;
 }
 
+// dec[row][c] = sigmoid(W a + bias)^inv_tau. 128 channels per CTA (their weight rows in shared memory), rows in steps of the grid.
+template <typename X>
+__global__ void __launch_bounds__(128) linattn_decay_kernel(const X* __restrict__ a, long lda, const float* __restrict__ w, const float* __restrict__ bias,
+                                                            float* __restrict__ dec, int rows, int C, int rank, float inv_tau) {
+  extern __shared__ float ws[];                           // [128][rank + 1]
+  grid_dep_wait();
+  grid_dep_launch();
+  const int c0 = blockIdx.x * 128, c = c0 + threadIdx.x;
+  for (int i = threadIdx.x; i < 128 * rank; i += 128) {
+    const int j = i / rank;
+    ws[j * (rank + 1) + i % rank] = c0 + j < C ? w[(long)c0 * rank + i] : 0.f;
+  }
+  __syncthreads();
+  if (c >= C) return;
+  const float b = bias[c];
+  const float* wr = ws + threadIdx.x * (rank + 1);
+  for (int r0 = blockIdx.y * 4; r0 < rows; r0 += gridDim.y * 4) {
+    float z[4] = {b, b, b, b};
+    const X* ar = a + (long)r0 * lda;
+    for (int r = 0; r < rank; ++r) {
+      const float v = wr[r];
+#pragma unroll
+      for (int y = 0; y < 4; ++y)
+        if (r0 + y < rows) z[y] = fmaf(v, to_f(ar[y * lda + r]), z[y]);
+    }
+#pragma unroll
+    for (int y = 0; y < 4; ++y)
+      if (r0 + y < rows) dec[(long)(r0 + y) * C + c] = root_decay(z[y], inv_tau);
+  }
+}
+
 // Contributions -> start states, segment by segment (segments of one chunk have neither). grid (element blocks, H, segments).
 __global__ void __launch_bounds__(256) linattn_scan_kernel(const LinChunkArgs a) {
   grid_dep_wait();
@@ -468,8 +550,8 @@ __global__ void __launch_bounds__(256) linattn_scan_kernel(const LinChunkArgs a)
 
 template <int DK, int DV, int MODE>
 static int launch_chunks(const LinChunkArgs& a, int chunks, int segs, int longest, cudaStream_t st) {
-  constexpr int base = (2 * 16 * (2 * DK + DV) + 17 * DK) * 4 + 2 * 16 * (DK + 8) * 2 + 16 * (DV + 8) * 2;
-  constexpr int full = base + 2 * 16 * (DK + 8) * 2 + 2 * 16 * 24 * 2 + 8 * 16 * 17 * 4 + 2 * 16 * DK * 4;
+  constexpr int base = (2 * 16 * ((MODE == 2 ? 3 : 2) * DK + DV) + (MODE == 2 ? 1 : 17) * DK) * 4 + 2 * 16 * (DK + 8) * 2 + 16 * (DV + 8) * 2;
+  constexpr int full = base + 2 * 16 * (DK + 8) * 2 + 2 * 16 * 24 * 2 + 8 * 16 * 17 * 4 + (MODE == 2 ? 0 : 2 * 16 * DK * 4);
   static_assert(full <= 227 * 1024, "shared memory budget");
   static bool attr_set = false;
   if (!attr_set) {
@@ -492,18 +574,19 @@ using namespace ve;
 
 extern "C" {
 
-// mode 0 / 1 as above (bias / lower or decay accordingly). x32: the projection rows are fp32 (else bf16). nseg > 0: segment
+// mode 0 / 1 / 2 as above (bias / lower, decay, or bias / w2 / rank / a_col / inv_tau / q_scale accordingly). x32: the projection rows are fp32 (else bf16). nseg > 0: segment
 // table; 0: segments from the slots of the rows (a few rows only: every CTA scans them).
 int ve_linattn_step(const void* proj, long ld, int x32, const void* pos, const void* slot, const void* seg_first, const void* seg_count, int nseg,
                     void* state, const void* bias, const void* lower, const void* decay, void* o, long ldo, int rows, int H, int dk, int dv,
-                    int mode, cudaStream_t st) {
+                    int mode, const void* w2, int rank, int a_col, float inv_tau, float q_scale, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (dk < 1 || dk > 256 || dv < 1 || H < 1 || (mode == 0 ? !decay : (!bias || !lower))) return cudaErrorInvalidValue;
+  if (dk < 1 || dk > 256 || dv < 1 || H < 1 || (mode == 0 ? !decay : mode == 1 ? !bias || !lower : !bias || !w2 || rank < 1)) return cudaErrorInvalidValue;
+  if (mode == 2 && rank % 4 == 0 && ((uintptr_t)w2 & 15)) return cudaErrorInvalidValue;
   LinArgs a{proj, ld, (const int*)pos, (const int*)slot, nseg > 0 ? (const int*)seg_first : nullptr, (const int*)seg_count, (float*)state,
-            (const float*)bias, (const float*)lower, (const float*)decay, (float*)o, ldo, rows, H, dk, dv};
+            (const float*)bias, (const float*)lower, (const float*)decay, (float*)o, ldo, rows, H, dk, dv, (const float*)w2, rank, a_col, inv_tau, q_scale};
   const dim3 grid(H, (dv + 31) / 32, nseg > 0 ? nseg : rows), block(32, 8);
 #define VE_LS(NK, X, MODE) launch_pdl(linattn_step_kernel<NK, X, MODE>, grid, block, 0, st, a)
-#define VE_LS_M(NK, X) do { if (mode == 0) VE_LS(NK, X, 0); else VE_LS(NK, X, 1); } while (0)
+#define VE_LS_M(NK, X) do { if (mode == 0) VE_LS(NK, X, 0); else if (mode == 1) VE_LS(NK, X, 1); else VE_LS(NK, X, 2); } while (0)
 #define VE_LS_X(NK) do { if (x32) VE_LS_M(NK, float); else VE_LS_M(NK, __nv_bfloat16); } while (0)
   if (dk <= 32) VE_LS_X(4);
   else if (dk <= 64) VE_LS_X(8);
@@ -515,19 +598,39 @@ int ve_linattn_step(const void* proj, long ld, int x32, const void* pos, const v
   VE_CHECK_LAUNCH();
 }
 
+// Decays of mode 2 for rows a [rows][rank] (pitch lda; fp32 when x32, else bf16), weights w [C][rank].
+int ve_linattn_decay(const void* a, long lda, int x32, const void* w, const void* bias, void* dec, int rows, int C, int rank, float inv_tau, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (C < 1 || rank < 1 || rank > 400) return cudaErrorInvalidValue;         // (the weight rows of 128 channels are in shared memory)
+  const int cx = (C + 127) / 128, ry = (rows + 3) / 4, most = (148 * 8 + cx - 1) / cx;
+  const dim3 grid(cx, ry < most ? ry : most);
+  const size_t smem = (size_t)128 * (rank + 1) * 4;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(linattn_decay_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_decay_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  if (x32) launch_pdl(linattn_decay_kernel<float>, grid, dim3(128), smem, st, (const float*)a, lda, (const float*)w, (const float*)bias, (float*)dec, rows, C, rank, inv_tau);
+  else launch_pdl(linattn_decay_kernel<__nv_bfloat16>, grid, dim3(128), smem, st, (const __nv_bfloat16*)a, lda, (const float*)w, (const float*)bias, (float*)dec,
+                  rows, C, rank, inv_tau);
+  VE_CHECK_LAUNCH();
+}
+
 // The chunked form over a table of chunks (chunk_count <= 128 rows each; a segment's chunks follow each other, all but its last
 // one a multiple of 16 rows): proj fp32, dk and dv <= 128. start / total: scratch (see LinChunkArgs); longest: most chunks of
 // any segment.
 int ve_linattn_chunk(const void* proj, long ld, const void* pos, const void* slot, const void* chunk_seg, const void* chunk_first, const void* chunk_count,
                      const void* seg_chunk0, int chunks, int segs, int longest, void* state, void* start, void* total, const void* bias, const void* lower,
-                     const void* decay, void* o, long ldo, int H, int dk, int dv, int mode, cudaStream_t st) {
+                     const void* decay, void* o, long ldo, int H, int dk, int dv, int mode, const void* dec, float q_scale, cudaStream_t st) {
   if (chunks <= 0) return 0;
-  if (dk < 1 || dk > 128 || dv < 1 || dv > 128 || H < 1 || segs < 1 || (mode == 0 ? !decay : (!bias || !lower))) return cudaErrorInvalidValue;
-  const int vec = !((uintptr_t)proj & 15) && ld % 4 == 0 && dk % 4 == 0 && dv % 4 == 0;
+  if (mode == 2 && !dec) return cudaErrorInvalidValue;
+  if (dk < 1 || dk > 128 || dv < 1 || dv > 128 || H < 1 || segs < 1 || (mode == 0 ? !decay : mode == 1 && (!bias || !lower))) return cudaErrorInvalidValue;
+  const int vec = !((uintptr_t)proj & 15) && ld % 4 == 0 && dk % 4 == 0 && dv % 4 == 0 && !((uintptr_t)dec & 15);
   LinChunkArgs a{(const float*)proj, ld, (const int*)pos, (const int*)slot, (const int*)chunk_seg, (const int*)chunk_first, (const int*)chunk_count,
                  (const int*)seg_chunk0, (float*)state, (float*)start, (float*)total, (const float*)bias, (const float*)lower, (const float*)decay,
-                 (float*)o, ldo, H, dk, dv, vec};
-#define VE_LC(DK, DV) return mode == 0 ? launch_chunks<DK, DV, 0>(a, chunks, segs, longest, st) : launch_chunks<DK, DV, 1>(a, chunks, segs, longest, st)
+                 (float*)o, ldo, H, dk, dv, vec, (const float*)dec, q_scale};
+#define VE_LC(DK, DV) return mode == 0 ? launch_chunks<DK, DV, 0>(a, chunks, segs, longest, st) : mode == 1 ? launch_chunks<DK, DV, 1>(a, chunks, segs, longest, st) \
+    : launch_chunks<DK, DV, 2>(a, chunks, segs, longest, st)
 #define VE_LC_V(DK) do { if (dv <= 32) VE_LC(DK, 32); if (dv <= 64) VE_LC(DK, 64); VE_LC(DK, 128); } while (0)
   if (dk <= 32) VE_LC_V(32);
   if (dk <= 64) VE_LC_V(64);

@@ -26,6 +26,30 @@ VE_DEVINL float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
 VE_DEVINL float silu_of(float z) { return z / (1.f + expf(-z)); }
 VE_DEVINL float dyt_of(float h, float alpha, float w, float b) { return fmaf(tanhf(alpha * h), w, b); }
 
+// Gated unit with both halves clamped: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1)
+VE_DEVINL float clamped_glu_of(float g, float u, float alpha, float limit) {
+  const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
+  return a / (1.f + expf(-alpha * a)) * (b + 1.f);
+}
+
+// Residual streams (at most kMaxStreams copies of a row): every stream anew from all old ones and a sublayer's result,
+// x_t <- sum_s mix[s][t] x_s + out[t] y; and what a sublayer reads, sum_s in[s] x_s.
+constexpr int kMaxStreams = 8;
+VE_DEVINL void streams_write(float* x, int S, const float* __restrict__ mix, const float* __restrict__ out, float y) {
+  float o[kMaxStreams];
+#pragma unroll
+  for (int s = 0; s < kMaxStreams; ++s) o[s] = s < S ? x[s] : 0.f;
+#pragma unroll
+  for (int t = 0; t < kMaxStreams; ++t)
+    if (t < S) {
+      float v = out[t] * y;
+#pragma unroll
+      for (int s = 0; s < kMaxStreams; ++s)
+        if (s < S) v = fmaf(mix[s * S + t], o[s], v);
+      x[t] = v;
+    }
+}
+
 // PolyNorm: sums of z^2, z^4, z^6 over a row, then c0 z / rms(z) + c1 z^2 / rms(z^2) + c2 z^3 / rms(z^3) + c3
 VE_DEVINL void poly_sums(float z, float& s1, float& s2, float& s3) {
   const float q = z * z, q2 = q * q;

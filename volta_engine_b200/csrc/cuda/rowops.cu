@@ -1,23 +1,47 @@
 // Row operators of decoders whose residual stream is fp32. Storage of activations is a template parameter (bf16, or fp32
 // for the all-32-bit form of a model); every operator computes in fp32. This file is compiled without fast-math: norms,
 // gates and angles follow the 32-bit definitions to rounding.
-//   embed_rows   out[r] = table[ids[r]] widened to fp32
+//   embed_rows   out[r] = table[ids[r]] widened to fp32 [+ sinusoidal position vector], once per residual stream
 //   dyt_rows     h += scale * part (optional, element-wise scale), out = tanh(alpha h) w + b        ("Dynamic Tanh" norm)
-//   group_rms    out = x / rms(x over groups of G columns) * w [* sigmoid(gate)]; w repeats with its own length
+//   stream_norm  residual streams rewritten from the old ones and a sublayer's result (optional), then the layer norm (no shift) of
+//                their weighted sum
+//   group_rms    out = x / rms(x over groups of G columns) * w [* sigmoid(gate) or silu(gate)]; w repeats with its own length
+//   clamped_glu  out = gated unit of [gate | up] rows with both halves clamped
 //   polynorm     out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3, N = division by the row's root mean square
 //   scale_add    h += scale * part
 #include "rowmath.cuh"
 
 namespace ve {
 
+// freq (optional, double): turns by half circles per position and column pair; column 2i gets the sine, 2i + 1 the cosine.
 template <typename T>
-__global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int H, int vocab) {
+__global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, const int* __restrict__ pos, const double* __restrict__ freq,
+                                  float* __restrict__ out, int H, int vocab, int S) {
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
   int id = ids[row];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
-  for (int i = threadIdx.x; i < H; i += blockDim.x) out[row * H + i] = to_f(table[(long)id * H + i]);
+  const T* src = table + (long)id * H;
+  float* dst = out + row * S * H;
+  if (!freq) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float v = to_f(src[i]);
+      for (int s = 0; s < S; ++s) dst[(long)s * H + i] = v;
+    }
+    return;
+  }
+  const double p = (double)pos[row];
+  for (int i = threadIdx.x * 2; i < H; i += blockDim.x * 2) {
+    const double t = p * freq[i >> 1];
+    float sn, cs;
+    sincospif((float)(t - 2.0 * rint(0.5 * t)), &sn, &cs);
+    const float v0 = to_f(src[i]) + sn, v1 = i + 1 < H ? to_f(src[i + 1]) + cs : 0.f;
+    for (int s = 0; s < S; ++s) {
+      dst[(long)s * H + i] = v0;
+      if (i + 1 < H) dst[(long)s * H + i + 1] = v1;
+    }
+  }
 }
 
 template <typename T>
@@ -68,10 +92,12 @@ __global__ void dyt_rows4_kernel(float* __restrict__ h, const T* __restrict__ pa
   }
 }
 
+VE_DEVINL float gate_of(float z, int silu) { return silu ? silu_of(z) : sigmoid_of(z); }
+
 // grid (rows, groups); x fp32 or T
 template <typename X, typename T>
 __global__ void group_rms_kernel(const X* __restrict__ x, long ldx, const float* __restrict__ w, int wlen, const X* __restrict__ gate,
-                                 long ldg, T* __restrict__ out, long ldo, int G, float eps) {
+                                 long ldg, int silu, T* __restrict__ out, long ldo, int G, float eps) {
   __shared__ float red[33];
   grid_dep_wait();
   grid_dep_launch();
@@ -87,8 +113,195 @@ __global__ void group_rms_kernel(const X* __restrict__ x, long ldx, const float*
   for (int i = threadIdx.x; i < G; i += blockDim.x) {
     const int c = c0 + i;
     float v = to_f(x[row * ldx + c]) * inv * w[c % wlen];
-    if (gate) v *= sigmoid_of(to_f(gate[row * ldg + c]));
+    if (gate) v *= gate_of(to_f(gate[row * ldg + c]), silu);
     out[row * ldo + c] = from_f<T>(v);
+  }
+}
+
+// Narrow groups (G <= 128 N4): one warp per group, the group in registers, four columns per lane and step (G, wlen, pitches and
+// bases multiples of four elements). groups = all groups of all rows.
+template <int N4, typename X, typename T>
+__global__ void __launch_bounds__(256) group_rms4_kernel(const X* __restrict__ x, long ldx, const float* __restrict__ w, int wlen, const X* __restrict__ gate,
+                                                         long ldg, int silu, T* __restrict__ out, long ldo, int G, int per_row, long groups, float eps) {
+  grid_dep_wait();
+  grid_dep_launch();
+  const int lane = threadIdx.x & 31;
+  for (long q = blockIdx.x * 8l + (threadIdx.x >> 5); q < groups; q += gridDim.x * 8l) {
+    const long row = q / per_row;
+    const int c0 = (int)(q - row * per_row) * G;
+    float4 v[N4], z[N4];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (j * 32 + lane) * 4;
+      v[j] = i < G ? load4(x + row * ldx + c0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (gate && i < G) z[j] = load4(gate + row * ldg + c0 + i);
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)G + eps);
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (j * 32 + lane) * 4;
+      if (i >= G) continue;
+      const float4 wv = *reinterpret_cast<const float4*>(w + (c0 + i) % wlen);
+      float4 o = make_float4(v[j].x * inv * wv.x, v[j].y * inv * wv.y, v[j].z * inv * wv.z, v[j].w * inv * wv.w);
+      if (gate) {
+        o.x *= gate_of(z[j].x, silu);
+        o.y *= gate_of(z[j].y, silu);
+        o.z *= gate_of(z[j].z, silu);
+        o.w *= gate_of(z[j].w, silu);
+      }
+      store4(out + row * ldo + c0 + i, o);
+    }
+  }
+}
+
+// h [rows][S][H]. One CTA per row.
+template <typename T>
+__global__ void __launch_bounds__(256) stream_norm_kernel(float* __restrict__ h, const T* __restrict__ part, long ldp, const float* __restrict__ mix,
+                                                          const float* __restrict__ wout, const float* __restrict__ win, const float* __restrict__ w,
+                                                          T* __restrict__ out, long ldo, int H, int S, float eps) {
+  __shared__ float red[33];
+  grid_dep_wait();
+  grid_dep_launch();
+  const long row = blockIdx.x;
+  float* hr = h + row * S * H;
+  auto read = [&](int i) {
+    float u = 0.f;
+    for (int s = 0; s < S; ++s) u = fmaf(win[s], hr[(long)s * H + i], u);
+    return u;
+  };
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    if (part) {
+      float x[kMaxStreams];
+#pragma unroll
+      for (int s = 0; s < kMaxStreams; ++s) x[s] = s < S ? hr[(long)s * H + i] : 0.f;
+      streams_write(x, S, mix, wout, to_f(part[row * ldp + i]));
+#pragma unroll
+      for (int s = 0; s < kMaxStreams; ++s)
+        if (s < S) hr[(long)s * H + i] = x[s];
+    }
+    if (out) sum += read(i);                              // (a thread reads what it wrote itself)
+  }
+  if (!out) return;
+  const float mean = block_sum(sum, red) / (float)H;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float d = read(i) - mean;
+    ss = fmaf(d, d, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) out[row * ldo + i] = from_f<T>((read(i) - mean) * inv * w[i]);
+}
+
+// The same on four columns per thread and step, the row in registers (H <= 1024 NV; H, pitches and bases multiples of four).
+template <int S, int NV, typename T>
+__global__ void __launch_bounds__(256) stream_norm4_kernel(float* __restrict__ h, const T* __restrict__ part, long ldp, const float* __restrict__ mix,
+                                                           const float* __restrict__ wout, const float* __restrict__ win, const float* __restrict__ w,
+                                                           T* __restrict__ out, long ldo, int H, float eps) {
+  __shared__ float red[33];
+  grid_dep_wait();
+  grid_dep_launch();
+  const long row = blockIdx.x;
+  float* hr = h + row * S * H;
+  float a[S][S], b[S], r[S];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+    r[s] = win[s];
+    b[s] = part ? wout[s] : 0.f;
+#pragma unroll
+    for (int t = 0; t < S; ++t) a[s][t] = part ? mix[s * S + t] : 0.f;
+  }
+  float4 u[NV];
+  float sum = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (j * 256 + threadIdx.x) * 4;
+    u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H) {
+      float4 x[S];
+#pragma unroll
+      for (int s = 0; s < S; ++s) x[s] = *reinterpret_cast<const float4*>(hr + (long)s * H + i);
+      if (part) {
+        const float4 p = load4(part + row * ldp + i);
+        float4 y[S];
+#pragma unroll
+        for (int t = 0; t < S; ++t) {
+          y[t] = make_float4(b[t] * p.x, b[t] * p.y, b[t] * p.z, b[t] * p.w);
+#pragma unroll
+          for (int s = 0; s < S; ++s) {
+            y[t].x = fmaf(a[s][t], x[s].x, y[t].x);
+            y[t].y = fmaf(a[s][t], x[s].y, y[t].y);
+            y[t].z = fmaf(a[s][t], x[s].z, y[t].z);
+            y[t].w = fmaf(a[s][t], x[s].w, y[t].w);
+          }
+          *reinterpret_cast<float4*>(hr + (long)t * H + i) = y[t];
+        }
+#pragma unroll
+        for (int s = 0; s < S; ++s) x[s] = y[s];
+      }
+#pragma unroll
+      for (int s = 0; s < S; ++s) {
+        u[j].x = fmaf(r[s], x[s].x, u[j].x);
+        u[j].y = fmaf(r[s], x[s].y, u[j].y);
+        u[j].z = fmaf(r[s], x[s].z, u[j].z);
+        u[j].w = fmaf(r[s], x[s].w, u[j].w);
+      }
+      sum += (u[j].x + u[j].y) + (u[j].z + u[j].w);
+    }
+  }
+  if (!out) return;
+  const float mean = block_sum(sum, red) / (float)H;
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    if ((j * 256 + threadIdx.x) * 4 < H) {
+      u[j].x -= mean;
+      u[j].y -= mean;
+      u[j].z -= mean;
+      u[j].w -= mean;
+      ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)H + eps);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (j * 256 + threadIdx.x) * 4;
+    if (i < H) {
+      const float4 wv = *reinterpret_cast<const float4*>(w + i);
+      store4(out + row * ldo + i, make_float4(u[j].x * inv * wv.x, u[j].y * inv * wv.y, u[j].z * inv * wv.z, u[j].w * inv * wv.w));
+    }
+  }
+}
+
+// z [rows][2 F]: gates, then ups.
+template <typename X, typename T>
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, float alpha, float limit) {
+  grid_dep_wait();
+  grid_dep_launch();
+  for (long q = blockIdx.x * 256l + threadIdx.x; q < total; q += gridDim.x * 256l) {
+    const long row = q / F;
+    const int i = (int)(q - row * F);
+    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + i]), to_f(z[row * ldz + F + i]), alpha, limit));
+  }
+}
+__global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* __restrict__ z, long ldz, __nv_bfloat16* __restrict__ out, long ldo, long total8,
+                                                           int F, float alpha, float limit) {
+  grid_dep_wait();
+  grid_dep_launch();
+  const int f8 = F >> 3;
+  for (long q = blockIdx.x * 256l + threadIdx.x; q < total8; q += gridDim.x * 256l) {
+    const long row = q / f8;
+    const int i = (int)(q - row * f8) * 8;
+    bf16x8 g = *reinterpret_cast<const bf16x8*>(z + row * ldz + i);
+    const bf16x8 u = *reinterpret_cast<const bf16x8*>(z + row * ldz + F + i);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 a = __bfloat1622float2(g.v[e]), b = __bfloat1622float2(u.v[e]);
+      g.v[e] = __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, alpha, limit), clamped_glu_of(a.y, b.y, alpha, limit));
+    }
+    *reinterpret_cast<bf16x8*>(out + row * ldo + i) = g;
   }
 }
 
@@ -157,11 +370,61 @@ using namespace ve;
 
 extern "C" {
 
-// f32: 1 = activations and tables fp32, 0 = bf16.
-int ve_embed_rows(const void* ids, const void* table, void* out, int rows, int H, int vocab, int f32, cudaStream_t st) {
+// f32: 1 = activations and tables fp32, 0 = bf16. out [rows][S][H]; pos and freq may be null.
+int ve_embed_rows(const void* ids, const void* table, const void* pos, const void* freq, void* out, int rows, int H, int vocab, int S, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (f32) launch_pdl(embed_rows_kernel<float>, dim3(rows), dim3(row_threads(H)), 0, st, (const int*)ids, (const float*)table, (float*)out, H, vocab);
-  else launch_pdl(embed_rows_kernel<__nv_bfloat16>, dim3(rows), dim3(row_threads(H)), 0, st, (const int*)ids, (const __nv_bfloat16*)table, (float*)out, H, vocab);
+  if (S < 1 || (freq && !pos)) return cudaErrorInvalidValue;
+#define VE_EM(T) launch_pdl(embed_rows_kernel<T>, dim3(rows), dim3(row_threads(H)), 0, st, (const int*)ids, (const T*)table, (const int*)pos, \
+    (const double*)freq, (float*)out, H, vocab, S)
+  if (f32) VE_EM(float);
+  else VE_EM(__nv_bfloat16);
+#undef VE_EM
+  VE_CHECK_LAUNCH();
+}
+
+// h [rows][S][H] contiguous fp32; part null: the streams stay; out null: only the streams are rewritten.
+int ve_stream_norm(void* h, const void* part, long ldp, const void* mix, const void* wout, const void* win, const void* w, void* out, long ldo, int rows,
+                   int H, int S, float eps, int f32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (S < 1 || S > kMaxStreams || (part && (!mix || !wout)) || (out && (!win || !w))) return cudaErrorInvalidValue;
+  const bool vec = !f32 && S <= 4 && H % 4 == 0 && H <= 8192 && win && (!part || ldp % 4 == 0) && (!out || ldo % 4 == 0) && !((uintptr_t)h & 15) &&
+                   !((uintptr_t)part & 7) && !((uintptr_t)w & 15) && !((uintptr_t)out & 7);
+#define VE_SN(S_, NV) launch_pdl(stream_norm4_kernel<S_, NV, __nv_bfloat16>, dim3(rows), dim3(256), 0, st, (float*)h, (const __nv_bfloat16*)part, ldp, \
+    (const float*)mix, (const float*)wout, (const float*)win, (const float*)w, (__nv_bfloat16*)out, ldo, H, eps)
+#define VE_SN_V(S_) do { if (H <= 1024) VE_SN(S_, 1); else if (H <= 2048) VE_SN(S_, 2); else if (H <= 4096) VE_SN(S_, 4); else VE_SN(S_, 8); } while (0)
+  if (vec) {
+    if (S == 1) VE_SN_V(1);
+    else if (S == 2) VE_SN_V(2);
+    else if (S == 3) VE_SN_V(3);
+    else VE_SN_V(4);
+    VE_CHECK_LAUNCH();
+  }
+#undef VE_SN_V
+#undef VE_SN
+#define VE_SN(T) launch_pdl(stream_norm_kernel<T>, dim3(rows), dim3(row_threads(H)), 0, st, (float*)h, (const T*)part, ldp, (const float*)mix, \
+    (const float*)wout, (const float*)win, (const float*)w, (T*)out, ldo, H, S, eps)
+  if (f32) VE_SN(float);
+  else VE_SN(__nv_bfloat16);
+#undef VE_SN
+  VE_CHECK_LAUNCH();
+}
+
+// z rows [gate F | up F], fp32 when x32, else of the activation type.
+int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, float alpha, float limit, int f32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (F < 1) return cudaErrorInvalidValue;
+  const bool vec = !f32 && !x32 && F % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && !((uintptr_t)z & 15) && !((uintptr_t)out & 15);
+  const long total = (long)rows * F / (vec ? 8 : 1), blocks = (total + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
+  if (vec) {
+    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, alpha, limit);
+    VE_CHECK_LAUNCH();
+  }
+#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, alpha, limit)
+  if (f32) VE_CG(float, float);
+  else if (x32) VE_CG(float, __nv_bfloat16);
+  else VE_CG(__nv_bfloat16, __nv_bfloat16);
+#undef VE_CG
   VE_CHECK_LAUNCH();
 }
 
@@ -186,17 +449,25 @@ int ve_dyt_rows(void* h, const void* part, long ldp, const void* scale, const vo
   VE_CHECK_LAUNCH();
 }
 
-// x (and gate) fp32 when x32, else of the activation type; cols = groups * G.
-int ve_group_rms(const void* x, long ldx, int x32, const void* w, int wlen, const void* gate, long ldg, void* out, long ldo, int rows, int cols,
+// x (and gate) fp32 when x32, else of the activation type; cols = groups * G. silu: the gate's activation is SiLU, else sigmoid.
+int ve_group_rms(const void* x, long ldx, int x32, const void* w, int wlen, const void* gate, long ldg, int silu, void* out, long ldo, int rows, int cols,
                  int G, float eps, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (G <= 0 || cols % G || wlen <= 0) return cudaErrorInvalidValue;
-  const dim3 grid(rows, cols / G), block(row_threads(G));
-#define VE_GR(X, T) launch_pdl(group_rms_kernel<X, T>, grid, block, 0, st, (const X*)x, ldx, (const float*)w, wlen, (const X*)gate, ldg, (T*)out, ldo, G, eps)
+  const int xa = x32 || f32 ? 15 : 7, oa = f32 ? 15 : 7;
+  const bool vec = G <= 512 && G % 4 == 0 && wlen % 4 == 0 && ldx % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && !((uintptr_t)x & xa) && !((uintptr_t)gate & xa) &&
+                   !((uintptr_t)out & oa) && !((uintptr_t)w & 15);
+  const long groups = (long)rows * (cols / G), blocks = (groups + 7) / 8;
+  const dim3 grid(rows, cols / G), block(row_threads(G)), grid4((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
+#define VE_GR4(N4, X, T) launch_pdl(group_rms4_kernel<N4, X, T>, grid4, dim3(256), 0, st, (const X*)x, ldx, (const float*)w, wlen, (const X*)gate, ldg, silu, \
+    (T*)out, ldo, G, cols / G, groups, eps)
+#define VE_GR(X, T) do { if (vec && G <= 128) VE_GR4(1, X, T); else if (vec) VE_GR4(4, X, T); \
+    else launch_pdl(group_rms_kernel<X, T>, grid, block, 0, st, (const X*)x, ldx, (const float*)w, wlen, (const X*)gate, ldg, silu, (T*)out, ldo, G, eps); } while (0)
   if (f32) VE_GR(float, float);
   else if (x32) VE_GR(float, __nv_bfloat16);
   else VE_GR(__nv_bfloat16, __nv_bfloat16);
 #undef VE_GR
+#undef VE_GR4
   VE_CHECK_LAUNCH();
 }
 

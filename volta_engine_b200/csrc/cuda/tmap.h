@@ -79,4 +79,35 @@ inline int make_tmap_2d(CUtensorMap* map, const void* base, CUtensorMapDataType 
   return 0;
 }
 
+// 3-D row-major tensor [outer, rows, cols]: outer pitch `outer_bytes`, row pitch `pitch_bytes`; box = [1, box_rows, box_cols]. The
+// same table, the key's fields carry both pitches.
+inline int make_tmap_3d(CUtensorMap* map, const void* base, CUtensorMapDataType dt, int elem_bytes, uint64_t outer, uint64_t rows, uint64_t cols,
+                        uint64_t outer_bytes, uint64_t pitch_bytes, uint32_t box_rows, uint32_t box_cols, CUtensorMapSwizzle swz) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (!fn) return (int)cudaErrorNotSupported;
+  if (((uintptr_t)base & 15) || (pitch_bytes & 15) || (outer_bytes & 15)) return (int)cudaErrorMisalignedAddress;
+  TmapKey key;
+  memset(&key, 0, sizeof(key));
+  key.base = base, key.rows = rows | (outer << 24), key.cols = cols | (pitch_bytes << 32), key.pitch = outer_bytes;
+  key.box_rows = box_rows, key.box_cols = box_cols, key.dt = (int)dt, key.elem_bytes = elem_bytes, key.swz = (int)swz, key.used = 2;
+  if (rows >> 24 || outer >> 40 || cols >> 32 || pitch_bytes >> 31) return (int)cudaErrorInvalidValue;
+  uint64_t h = (uint64_t)(uintptr_t)base * 0x9E3779B97F4A7C15ull;
+  h ^= (key.rows * 0xC2B2AE3D27D4EB4Full) ^ (key.cols << 17) ^ (outer_bytes << 29) ^ ((uint64_t)box_cols << 52) ^ 0x5bd1e995ull;
+  TmapSlot* slot = tmap_table() + ((h ^ (h >> 29)) & (kTmapSlots - 1));
+  if (memcmp(&slot->key, &key, sizeof(key)) == 0) {
+    memcpy(map, &slot->map, sizeof(CUtensorMap));
+    return 0;
+  }
+  cuuint64_t dims[3] = {cols, rows, outer};
+  cuuint64_t strides[2] = {pitch_bytes, outer_bytes};
+  cuuint32_t box[3] = {box_cols, box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(map, dt, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, swz, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return (int)cudaErrorInvalidValue;
+  slot->key = key;
+  memcpy(&slot->map, map, sizeof(CUtensorMap));
+  return 0;
+}
+
 }  // namespace ve

@@ -6,18 +6,21 @@ front, the layer scale and the residual add inside the linears' launches.
 """
 from __future__ import annotations
 
+import copy
+
 import torch
 
+from ..ops.gqa import GqaSpec, distance_bias, gqa_attend
 from ..ops.latent import LatentSpec, latent_rows
 from ..ops.linear import LinearBF16, LinearF32
 from ..ops.linear_attn import LinAttnSpec, LinAttnState, linattn_rows
 from ..ops.rowops import GroupRMS, gemv_rows
 
 
-def make_linear(src, names, device, dtype):
-    """One linear computing the stacked outputs of the tensors ``names``."""
+def make_linear(src, names, device, dtype, dim: int = 0):
+    """One linear computing the stacked outputs of the tensors ``names`` (``dim`` 1: the sum of their outputs on stacked inputs)."""
     names = [names] if isinstance(names, str) else names
-    w = torch.cat([src.tensor(n, device, dtype) for n in names], 0) if len(names) > 1 else src.tensor(names[0], device, dtype)
+    w = torch.cat([src.tensor(n, device, dtype) for n in names], dim) if len(names) > 1 else src.tensor(names[0], device, dtype)
     return LinearF32(w) if dtype == torch.float32 else LinearBF16(w)
 
 
@@ -28,25 +31,55 @@ def apply_linear(lin, x, out_f32: bool = False):
     return lin.forward(x, out_f32=out_f32)
 
 
-class LinearRecurrence:
-    """HGRN2 and lightning attention: one fused input projection [q | forget gate or k | v | gate], the decayed outer-product
-    recurrence, an RMS norm of its output (per head, or over all heads and gated), the output projection."""
-    cached = False
+class Mixer:
+    """What the decoder asks of a mixer beside ``rows`` and ``step``."""
+    cached = False                  # owns one layer of the paged cache (``cache_index``)
+    recurrent = False               # has a state per slot (``bind``, ``state``)
+    cache_index = -1
+    state = None
 
-    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
+    @staticmethod
+    def row_widths(m: dict) -> tuple[int, int]:
+        """Elements of a token's row in the key and in the value pool, from the mixer's sizes."""
+        return 0, 0
+
+    def linears(self):
+        return [self.in_proj, self.out]
+
+    def extra_bytes(self) -> int:
+        """Bytes of further matrices a decode step reads."""
+        return 0
+
+    def state_elements(self) -> int:
+        return 0
+
+
+class LinearRecurrence(Mixer):
+    """HGRN2, lightning attention and gated linear attention: one fused input projection [q | forget gate or k | v | gate | low-rank
+    decay], the decayed outer-product recurrence, an RMS norm of its output (per head, or over all heads; gated), the output
+    projection. ``out_scale``: a factor on what enters the output projection."""
+    recurrent = True
+    PARTS = {"hgrn2": ("q", "f", "v"), "lightning": ("q", "k", "v", "g"), "gated_linear_attention": ("q", "k", "v", "g", "a1")}
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype, linears: bool = True, out_scale: float = 1.0):
         H, dk, dv = int(m["heads"]), int(m["dim"]), int(m["vdim"])
         f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
-        self.gated = kind == "lightning"
+        self.parts = [p + n for n in self.PARTS[kind]]
+        self.gated = "g" in self.PARTS[kind]
         if kind == "lightning":
             decay = m["decay"] if isinstance(m["decay"], (list, tuple)) else [m["decay"]] * H
             self.spec = LinAttnSpec(H, dk, dv, decay=torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device))
             if self.spec.decay.numel() != H:
                 raise ValueError(f"{p}: {self.spec.decay.numel()} decays for {H} heads")
-        else:
+        elif kind == "hgrn2":
             self.spec = LinAttnSpec(H, dk, dv, lower=f32("lower"), bias=f32("f.b"))
-        self.in_proj = make_linear(src, [p + n for n in (("q", "k", "v", "g") if self.gated else ("q", "f", "v"))], device, dtype)
-        self.out = make_linear(src, p + "o", device, dtype)
-        self.norm = GroupRMS(f32("norm"), eps, 0 if self.gated else dv)
+        else:
+            self.spec = LinAttnSpec(H, dk, dv, bias=f32("a2.b"), w2=src.tensor(p + "a2", device, torch.float32).contiguous(), a_col=H * (2 * dk + 2 * dv),
+                                    tau=float(m["tau"]), q_scale=dk ** -0.5)
+        if linears:
+            self.in_proj = make_linear(src, self.parts, device, dtype)
+            self.out = make_linear(src, p + "o", device, dtype)
+        self.norm = GroupRMS(f32("norm") * out_scale, eps, 0 if kind == "lightning" else dv, silu=kind == "gated_linear_attention")
         self.dtype = dtype
         self.state: LinAttnState | None = None
 
@@ -55,28 +88,126 @@ class LinearRecurrence:
             self.state = LinAttnState(self.spec, kv.max_slots, kv.page_table.device)
         return self.state
 
-    def linears(self):
-        return [self.in_proj, self.out]
+    def state_elements(self) -> int:
+        return self.spec.heads * self.spec.dk * self.spec.dv
 
-    def _gate(self, proj):
-        return proj[:, self.spec.cols:] if self.gated else None
+    def extra_bytes(self) -> int:
+        return self.spec.w2.numel() * 4 if self.spec.w2 is not None else 0
+
+    def gate(self, proj):
+        return proj[:, self.spec.cols: self.spec.cols + self.spec.heads * self.spec.dv] if self.gated else None
+
+    def recur(self, proj, b, kv, journal, chunked: bool):
+        return linattn_rows(proj, b, self.bind(kv), self.spec, *journal, chunked=chunked)
 
     def rows(self, x, b, kv, journal=(None, None)):
         proj = apply_linear(self.in_proj, x, out_f32=True)         # gates and keys enter the recurrence unrounded
-        o = linattn_rows(proj, b, self.bind(kv), self.spec, *journal, chunked=self.dtype != torch.float32)
-        y = self.norm.rows(o, self.dtype, gate=self._gate(proj))
+        o = self.recur(proj, b, kv, journal, self.dtype != torch.float32)
+        return apply_linear(self.out, self.norm.rows(o, self.dtype, gate=self.gate(proj)))
+
+    def step(self, pro, residual, b, kv, journal=(None, None)):
+        proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
+        o = self.recur(proj, b, kv, journal, True)
+        gemv_rows(self.out, b.n, residual=residual, **self.norm.prologue(o, self.gate(proj)))
+
+
+class GroupedAttention(Mixer):
+    """Grouped-query softmax attention without rotation: normed queries and keys, a query temperature, a bias by distance and a sink;
+    one fused input projection [q | k | v]. ``out_scale`` as above."""
+    cached = True
+    PARTS = ("q", "k", "v")
+
+    @staticmethod
+    def row_widths(m: dict) -> tuple[int, int]:
+        return GqaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), 1.0).row_widths
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype, linears: bool = True, out_scale: float = 1.0):
+        f32 = lambda name: src.tensor(p + name, device, torch.float32).contiguous()
+        temp = m.get("q_temp") or {"coef": 0.0, "every": 0}
+        self.spec = GqaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), eps, q_norm=f32("q.norm"),
+                            k_norm=f32("k.norm"), temp_coef=float(temp["coef"]), temp_every=int(temp["every"]),
+                            bias=distance_bias(f32("rel"), int(m["bias_max"])), sink=f32("sink"), out_scale=out_scale)
+        self.parts = [p + n for n in self.PARTS]
+        if linears:
+            self.in_proj = make_linear(src, self.parts, device, dtype)
+            self.out = make_linear(src, p + "o", device, dtype)
+        self.dtype = dtype
+
+    def attend(self, proj, b, kv, out):
+        return gqa_attend(self.spec, proj, b, kv, kv.k[self.cache_index], kv.v[self.cache_index], out)
+
+    def _out(self, proj):
+        return torch.empty(proj.shape[0], self.spec.heads * self.spec.vdim, dtype=self.dtype, device=proj.device)
+
+    def rows(self, x, b, kv, journal=None):
+        proj = apply_linear(self.in_proj, x, out_f32=True)
+        return apply_linear(self.out, self.attend(proj, b, kv, self._out(proj)))
+
+    def step(self, pro, residual, b, kv, journal=None):
+        proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
+        gemv_rows(self.out, b.n, residual=residual, x=self.attend(proj, b, kv, self._out(proj)))
+
+
+class Parallel(Mixer):
+    """Grouped attention and gated linear attention side by side on the same rows: one input projection for both, and one output
+    projection over the two results put next to each other (each times its scale)."""
+    cached = recurrent = True
+
+    @staticmethod
+    def row_widths(m: dict) -> tuple[int, int]:
+        return GroupedAttention.row_widths(m["left"])
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
+        self.left = GroupedAttention("grouped_attention", m["left"], eps, src, p + "left.", device, dtype, False, float(m["left_scale"]))
+        self.right = LinearRecurrence("gated_linear_attention", m["right"], eps, src, p + "right.", device, dtype, False, float(m["right_scale"]))
+        self.in_proj = make_linear(src, self.left.parts + self.right.parts, device, dtype)
+        self.out = make_linear(src, [p + "left.o", p + "right.o"], device, dtype, dim=1)
+        self.k0 = self.left.spec.heads * self.left.spec.vdim         # columns of the left result
+        self.k1 = self.right.spec.heads * self.right.spec.dv
+        self.dtype = dtype
+
+    def __copy__(self):
+        new = object.__new__(Parallel)
+        new.__dict__.update(self.__dict__)
+        new.left, new.right = copy.copy(self.left), copy.copy(self.right)
+        return new
+
+    cache_index = property(lambda self: self.left.cache_index, lambda self, i: setattr(self.left, "cache_index", i))
+    state = property(lambda self: self.right.state, lambda self, s: setattr(self.right, "state", s))
+
+    def bind(self, kv):
+        return self.right.bind(kv)
+
+    def state_elements(self) -> int:
+        return self.right.state_elements()
+
+    def extra_bytes(self) -> int:
+        return self.right.extra_bytes()
+
+    def rows(self, x, b, kv, journal=(None, None)):
+        proj = apply_linear(self.in_proj, x, out_f32=True)
+        y = torch.empty(x.shape[0], self.k0 + self.k1, dtype=self.dtype, device=x.device)
+        self.left.attend(proj, b, kv, y[:, : self.k0])
+        pr = proj[:, self.left.spec.cols:]
+        o = self.right.recur(pr, b, kv, journal, self.dtype != torch.float32)
+        self.right.norm.rows(o, self.dtype, gate=self.right.gate(pr), out=y[:, self.k0:])
         return apply_linear(self.out, y)
 
     def step(self, pro, residual, b, kv, journal=(None, None)):
         proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
-        o = linattn_rows(proj, b, self.bind(kv), self.spec, *journal)
-        gemv_rows(self.out, b.n, residual=residual, **self.norm.prologue(o, self._gate(proj)) if self.gated else self.norm.prologue(o))
+        att = self.left.attend(proj, b, kv, torch.empty(b.n, self.k0, dtype=torch.float32, device=proj.device))
+        pr = proj[:, self.left.spec.cols:]
+        o = self.right.recur(pr, b, kv, journal, True)
+        gemv_rows(self.out, b.n, residual=residual, **self.right.norm.prologue(o, self.right.gate(pr), head=att))
 
 
-class LatentAttention:
+class LatentAttention(Mixer):
     """Multi-head attention over a low-rank latent per token, with a low-rank query and a rotated key part shared by the heads."""
-    cached = True                   # owns one layer of the paged cache (``cache_index``)
-    state = None
+    cached = True
+
+    @staticmethod
+    def row_widths(m: dict) -> tuple[int, int]:
+        return LatentSpec(1, 1, int(m["rot_dim"]), 1, int(m["kv_rank"]), 1.0, 1.0, 1e-5).width, 0
 
     def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
         rot = m["rot"]
@@ -97,7 +228,6 @@ class LatentAttention:
         self.q_norm = GroupRMS(f32("dq.norm"), eps)
         self.kv_norm = f32("dkv.norm")
         self.dtype = dtype
-        self.cache_index = -1
 
     def linears(self):
         return [self.down, self.uq, self.out]
@@ -120,4 +250,5 @@ class LatentAttention:
         gemv_rows(self.out, b.n, residual=residual, x=att)
 
 
-MIXERS = {"hgrn2": LinearRecurrence, "lightning": LinearRecurrence, "latent_attention": LatentAttention}
+MIXERS = {"hgrn2": LinearRecurrence, "lightning": LinearRecurrence, "latent_attention": LatentAttention,
+          "gated_linear_attention": LinearRecurrence, "grouped_attention": GroupedAttention, "parallel": Parallel}

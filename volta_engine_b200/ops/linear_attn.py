@@ -2,11 +2,13 @@
 
     S_t = diag(d_t) S_(t-1) + k_t v_t^T,     o_t = S_t^T q_t
 
-over projection rows [ q (heads dk) | x (heads dk) | v (heads dv) | ... ]; q = silu(q) and either
+over projection rows [ q (heads dk) | x (heads dk) | v (heads dv) | ... ] and one of
 
-  * ``decay`` given (lightning attention): d = decay[head], k = silu(x), v = silu(v), or
+  * ``decay`` given (lightning attention): d = decay[head], k = silu(x), v = silu(v), q = silu(q);
   * ``lower`` / ``bias`` given (HGRN2): the forget gate f = lower + (1 - lower) sigmoid(x + bias) per channel is the decay and
-    its complement 1 - f the key; v as projected.
+    its complement 1 - f the key; v as projected, q = silu(q);
+  * ``w2`` / ``bias`` given (gated linear attention): d = sigmoid(w2 a + bias)^(1 / tau) per channel from a low-rank part a of the
+    row (columns from ``a_col``); k = x and v as projected, q times ``q_scale``.
 
 A row at position 0 starts its slot from a zero state; rows of one slot inside a batch are consecutive positions in order.
 """
@@ -27,10 +29,23 @@ class LinAttnSpec:
     decay: torch.Tensor | None = None       # fp32 [heads]
     lower: torch.Tensor | None = None       # fp32 [heads * dk]
     bias: torch.Tensor | None = None        # fp32 [heads * dk]
+    w2: torch.Tensor | None = None          # fp32 [heads * dk, rank]
+    a_col: int = 0
+    tau: float = 1.0
+    q_scale: float = 1.0
 
     @property
     def mode(self) -> int:
-        return 0 if self.decay is not None else 1
+        return 0 if self.decay is not None else 2 if self.w2 is not None else 1
+
+    @property
+    def rank(self) -> int:
+        return self.w2.shape[1] if self.w2 is not None else 0
+
+    @property
+    def chunks(self) -> bool:
+        """The chunked kernels take these sizes."""
+        return self.dk <= 128 and self.dv <= 128 and self.rank <= 400
 
     @property
     def cols(self) -> int:
@@ -54,9 +69,13 @@ class LinAttnState:
         self.rec[slot].copy_(snap["rec"])
 
 
-def gates(x, spec: LinAttnSpec):
-    """fp32 rows of the second projection block -> (decay, key), each [rows, heads, dk]."""
-    n = x.shape[0]
+def gates(pf, spec: LinAttnSpec):
+    """fp32 projection rows -> (decay, key), each [rows, heads, dk]."""
+    n, D = pf.shape[0], spec.heads * spec.dk
+    x = pf[:, D: 2 * D]
+    if spec.mode == 2:
+        z = pf[:, spec.a_col: spec.a_col + spec.rank] @ spec.w2.t() + spec.bias
+        return torch.exp(torch.nn.functional.logsigmoid(z) / spec.tau).reshape(n, spec.heads, spec.dk), x.reshape(n, spec.heads, spec.dk)
     if spec.mode == 0:
         k = torch.nn.functional.silu(x).reshape(n, spec.heads, spec.dk)
         return spec.decay.reshape(1, spec.heads, 1).expand_as(k), k
@@ -70,8 +89,8 @@ def linattn_reference(proj, pos, slot, st: LinAttnState, spec: LinAttnSpec) -> t
     """CPU statement over the rows of a batch; updates ``st`` in place -> fp32 [rows, heads * dv]."""
     n, H, dk, dv = proj.shape[0], spec.heads, spec.dk, spec.dv
     pf = proj.float()
-    q = torch.nn.functional.silu(pf[:, : H * dk]).reshape(n, H, dk)
-    d, k = gates(pf[:, H * dk: 2 * H * dk], spec)
+    q = (pf[:, : H * dk] * spec.q_scale if spec.mode == 2 else torch.nn.functional.silu(pf[:, : H * dk])).reshape(n, H, dk)
+    d, k = gates(pf, spec)
     v = pf[:, 2 * H * dk: spec.cols].reshape(n, H, dv)
     if spec.mode == 0:
         v = torch.nn.functional.silu(v)
@@ -91,8 +110,9 @@ def linattn_reference(proj, pos, slot, st: LinAttnState, spec: LinAttnSpec) -> t
 def _step(proj, pos, slot, st, spec, o, rows, segs=None):
     x32 = 1 if proj.dtype == torch.float32 else 0
     first, count, n = segs if segs is not None else (None, None, 0)
-    call("linattn_step", "plipp" + "ppi" + "pppp" + "pliiiii", ptr(proj), proj.stride(0), x32, ptr(pos), ptr(slot), ptr(first), ptr(count), n,
-         ptr(st.rec), ptr(spec.bias), ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), rows, spec.heads, spec.dk, spec.dv, spec.mode)
+    call("linattn_step", "plipp" + "ppi" + "pppp" + "pliiiii" + "piiff", ptr(proj), proj.stride(0), x32, ptr(pos), ptr(slot), ptr(first), ptr(count), n,
+         ptr(st.rec), ptr(spec.bias), ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), rows, spec.heads, spec.dk, spec.dv, spec.mode,
+         ptr(spec.w2), spec.rank, spec.a_col, 1.0 / spec.tau, float(spec.q_scale))
 
 
 def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJournal | None = None, rows=None,
@@ -116,7 +136,7 @@ def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJourn
             journal.fn = lambda keep: _step(proj, pos, slot, st, spec, o2, keep)
         return o
     t = b.segments()
-    if not chunked or spec.dk > 128 or spec.dv > 128 or proj.dtype != torch.float32:
+    if not chunked or not spec.chunks or proj.dtype != torch.float32:
         _step(proj, pos, slot, st, spec, o, n, (t.first, t.count, t.n))
         return o
     if t.n_short:
@@ -125,7 +145,12 @@ def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJourn
         multi = t.longest > 1
         start = torch.empty((t.chunks, spec.heads, spec.dk, spec.dv) if multi else (1,), dtype=torch.float32, device=proj.device)
         total = torch.empty((t.chunks, spec.heads, spec.dk) if multi else (1,), dtype=torch.float32, device=proj.device)
-        call("linattn_chunk", "plpppppp" + "iii" + "ppp" + "pppp" + "liiii", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
+        dec = None
+        if spec.mode == 2:
+            dec = torch.empty(n, spec.heads * spec.dk, dtype=torch.float32, device=proj.device)
+            a = proj[:, spec.a_col:]
+            call("linattn_decay", "plippp" + "iiif", ptr(a), a.stride(0), 1, ptr(spec.w2), ptr(spec.bias), ptr(dec), n, spec.heads * spec.dk, spec.rank, 1.0 / spec.tau)
+        call("linattn_chunk", "plpppppp" + "iii" + "ppp" + "pppp" + "liiii" + "pf", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
              ptr(t.chunk_count), ptr(t.seg_chunk0), t.chunks, t.seg_chunk0.numel() - 1, t.longest, ptr(st.rec), ptr(start), ptr(total), ptr(spec.bias),
-             ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), spec.heads, spec.dk, spec.dv, spec.mode)
+             ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), spec.heads, spec.dk, spec.dv, spec.mode, ptr(dec), float(spec.q_scale))
     return o

@@ -51,12 +51,13 @@ class DynamicTanh:
 @dataclass
 class GroupRMS:
     """RMS norm over groups of ``group`` columns (0: the whole row) with a plain weight that repeats with its own length,
-    optionally times sigmoid(gate)."""
+    optionally times sigmoid(gate) (``silu``: times silu(gate))."""
     w: torch.Tensor           # fp32
     eps: float
     group: int = 0
+    silu: bool = False
 
-    def rows(self, x, out_dtype, gate=None):
+    def rows(self, x, out_dtype, gate=None, out=None):
         rows, cols = x.shape
         G = self.group or cols
         if not x.is_cuda:
@@ -64,16 +65,21 @@ class GroupRMS:
             v = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + self.eps)).reshape(rows, cols)
             v = v * self.w.repeat(cols // self.w.numel())
             if gate is not None:
-                v = v * torch.sigmoid(gate.float())
-            return v.to(out_dtype)
-        out = torch.empty(rows, cols, dtype=out_dtype, device=x.device)
+                v = v * (torch.nn.functional.silu(gate.float()) if self.silu else torch.sigmoid(gate.float()))
+            if out is None:
+                return v.to(out_dtype)
+            return out.copy_(v)
+        if out is None:
+            out = torch.empty(rows, cols, dtype=out_dtype, device=x.device)
         assert gate is None or gate.dtype == x.dtype
-        call("group_rms", "plipipl" + "pliiifi", ptr(x), x.stride(0), _f32(x), ptr(self.w), self.w.numel(), ptr(gate),
-             gate.stride(0) if gate is not None else 0, ptr(out), out.stride(0), rows, cols, G, float(self.eps), _f32(out))
+        call("group_rms", "plipipli" + "pliiifi", ptr(x), x.stride(0), _f32(x), ptr(self.w), self.w.numel(), ptr(gate),
+             gate.stride(0) if gate is not None else 0, int(self.silu), ptr(out), out.stride(0), rows, cols, G, float(self.eps), _f32(out))
         return out
 
-    def prologue(self, x, gate=None):
-        return {"pro": 2, "x": x, "w": self.w, "G": self.group or x.shape[1], "wlen": self.w.numel(), "gate": gate, "eps": self.eps}
+    def prologue(self, x, gate=None, head=None):
+        """``head``: fp32 columns in front of the normed ones, taken as they are."""
+        return {"pro": 2, "x": x, "w": self.w, "G": self.group or x.shape[1], "wlen": self.w.numel(), "gate": gate, "eps": self.eps,
+                "head": head, "silu": self.silu}
 
 
 @dataclass
@@ -96,13 +102,90 @@ class PolyNorm:
         return {"pro": 3, "x": z, "coef": self.coef, "eps": self.eps}
 
 
-def embed_rows(ids, table):
-    """-> fp32 [rows, H]."""
+@dataclass
+class ClampedGlu:
+    """Rows [gate | up]: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up clamped to +-limit."""
+    limit: float
+    alpha: float
+
+    def rows(self, z, out_dtype):
+        rows, F = z.shape[0], z.shape[1] // 2
+        if not z.is_cuda:
+            g, u = z[:, :F].float().clamp(max=self.limit), z[:, F:].float().clamp(-self.limit, self.limit)
+            return (g * torch.sigmoid(self.alpha * g) * (u + 1.0)).to(out_dtype)
+        out = torch.empty(rows, F, dtype=out_dtype, device=z.device)
+        call("clamped_glu", "plipliiffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, float(self.alpha), float(self.limit), _f32(out))
+        return out
+
+    def prologue(self, z):
+        return {"pro": 5, "x": z, "kx": z.shape[1] // 2, "alpha": self.alpha, "eps": self.limit}
+
+
+@dataclass
+class StreamWrite:
+    """How a sublayer's result y enters residual streams [rows, streams, H]: x_t <- sum_s mix[s, t] x_s + out[t] y."""
+    mix: torch.Tensor         # fp32 [streams, streams], [from, to]
+    out: torch.Tensor         # fp32 [streams]
+
+    def add(self, h, part):
+        h.copy_(torch.einsum("rsd,st->rtd", h, self.mix) + self.out[:, None] * part.float()[:, None, :])
+
+
+@dataclass
+class StreamNorm:
+    """Layer norm (weight, no shift) of the weighted sum of the residual streams [rows, streams, H]."""
+    w: torch.Tensor           # fp32 [H]
+    eps: float
+    read: torch.Tensor        # fp32 [streams]
+
+    def rows(self, h, out_dtype, part=None, write: StreamWrite | None = None):
+        """The streams rewritten with ``part`` (in place, optional), then the norm of what is read from them."""
+        rows, S, H = h.shape
+        if not h.is_cuda:
+            if part is not None:
+                write.add(h, part)
+            u = torch.einsum("rsd,s->rd", h, self.read)
+            u = u - u.mean(-1, keepdim=True)
+            return (u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + self.eps) * self.w).to(out_dtype)
+        out = torch.empty(rows, H, dtype=out_dtype, device=h.device)
+        call("stream_norm", "pplppppliiifi", ptr(h), ptr(part), part.stride(0) if part is not None else 0, ptr(write.mix) if part is not None else 0,
+             ptr(write.out) if part is not None else 0, ptr(self.read), ptr(self.w), ptr(out), out.stride(0), rows, H, S, float(self.eps), _f32(out))
+        return out
+
+    def prologue(self, h):
+        S, H = h.shape[1:]
+        return {"pro": 4, "x": h.view(h.shape[0], S * H), "kx": H, "w": self.w, "G": S, "coef": self.read, "eps": self.eps}
+
+
+class SinusoidalPositions:
+    """Position vectors: sine in column 2i, cosine in 2i + 1 of position * base^(-2i / width). Half circles per position are kept
+    in double, so that angles are exact at any position."""
+
+    def __init__(self, width: int, base: float, device):
+        i = torch.arange((width + 1) // 2, dtype=torch.float64)
+        self.width = width
+        self.freq = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / width)
+        self.half_turns = (self.freq / torch.pi).to(device)
+
+    def vectors(self, pos):
+        ang = pos.double()[:, None] * self.freq[None, :]
+        return torch.stack([ang.sin(), ang.cos()], -1).flatten(1)[:, : self.width].float()
+
+
+def embed_rows(ids, table, pos=None, positions: SinusoidalPositions | None = None, streams: int = 0):
+    """-> fp32 [rows, H]; with ``positions`` their vectors of ``pos`` are added; with ``streams`` the rows come that many times
+    ([rows, streams, H])."""
+    S = max(1, streams)
     if not table.is_cuda:
-        return table[ids.long()].float()
+        x = table[ids.long()].float()
+        if positions is not None:
+            x = x + positions.vectors(pos)
+        return x[:, None, :].repeat(1, S, 1) if streams else x
     V, H = table.shape
-    out = torch.empty(ids.numel(), H, dtype=torch.float32, device=table.device)
-    call("embed_rows", "pppiiii", ptr(ids), ptr(table), ptr(out), ids.numel(), H, V, _f32(table))
+    n = ids.numel()
+    out = torch.empty((n, S, H) if streams else (n, H), dtype=torch.float32, device=table.device)
+    call("embed_rows", "pppppiiiii", ptr(ids), ptr(table), ptr(pos) if positions is not None else 0, ptr(positions.half_turns) if positions is not None else 0,
+         ptr(out), n, H, V, S, _f32(table))
     return out
 
 
@@ -111,19 +194,26 @@ def fused_fits(lin, rows: int) -> bool:
     return rows <= FUSED_ROWS and rows * (lin.weight.shape[1] + 64) * 2 <= FUSED_SMEM
 
 
-def gemv_rows(lin, M: int, *, x, pro=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, out_f32=False, residual=None):
+def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, head=None, silu=False,
+              out_f32=False, residual=None):
     """A bf16 linear on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
-    ``residual`` = (h fp32, scale | None): h += scale * y in place; otherwise the product is returned."""
+    ``residual`` = (h fp32, scale | None): h += scale * y in place, (streams, StreamWrite): the streams rewritten in place; otherwise
+    the product is returned."""
     W = lin.weight
     N, K = W.shape
     dev = W.device
     if pro == 0 and x.shape[1] != K:              # weight rows padded to 16 bytes
         x = torch.nn.functional.pad(x, (0, K - x.shape[1]))
+    k0 = head.shape[1] if head is not None else 0
     out = None
     if residual is None:
         out = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=dev)
     h, scale = residual if residual is not None else (None, None)
-    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp", ptr(W), W.stride(0), N, K, M, pro, x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
+    streams, mix = 0, None
+    if isinstance(scale, StreamWrite):
+        streams, mix, scale = h.shape[1], scale.mix, scale.out
+    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiip", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
          float(alpha), G, wlen, ptr(gate), gate.stride(0) if gate is not None else 0, ptr(coef), float(eps),
-         ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, N, ptr(h), h.stride(0) if h is not None else 0, ptr(scale))
+         ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, N, ptr(h), h.stride(0) if h is not None else 0, ptr(scale),
+         ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), streams, ptr(mix))
     return out

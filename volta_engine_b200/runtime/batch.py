@@ -44,6 +44,15 @@ class SegmentTable:
     n_short: int = 0                  # leading segments that make up short_rows
     chunks: int = 0
     longest: int = 0                  # most chunks of any segment
+    by_tokens: dict = field(default_factory=dict)
+
+    def tiles(self, per: int):
+        """(first row in the batch, rows) of tiles of at most ``per`` rows over the segments behind ``short_rows``."""
+        t = self.by_tokens.get(per)
+        if t is None:
+            rows = [(f + o, min(per, c - o)) for _, f, c, _ in self.host[self.n_short:] for o in range(0, c, per)]
+            t = self.by_tokens[per] = tuple(torch.tensor(list(v), dtype=torch.int32).to(self.first.device, non_blocking=True) for v in zip(*rows))
+        return t
 
     @classmethod
     def build(cls, slots, pos, device):

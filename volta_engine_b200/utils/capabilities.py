@@ -29,8 +29,10 @@ TABLE = {
     "mla_expand_out": ("MLALatent", P),
     "latent_rope_store": ("LatentAttention", P), "latent_absorb": ("LatentAttention", P), "latent_attn": ("LatentAttention", P),
     "latent_expand": ("LatentAttention", P), "latent_gather": ("LatentAttention", P), "latent_prefill": ("LatentAttention", P), "latent_prefill_tc": ("LatentAttention", P),
-    "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P), "linattn_chunk": ("LinearAttention", P),
+    "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P), "linattn_chunk": ("LinearAttention", P), "linattn_decay": ("LinearAttention", P),
+    "gqa_store": ("GroupedAttention", P), "gqa_rows": ("GroupedAttention", P), "gqa_decode": ("GroupedAttention", P), "gqa_prefill": ("GroupedAttention", P),
     "embed_rows": ("RowOps (fp32 residual)", P), "dyt_rows": ("RowOps (fp32 residual)", P), "group_rms": ("RowOps (fp32 residual)", P),
+    "stream_norm": ("RowOps (fp32 residual)", P), "clamped_glu": ("RowOps (fp32 residual)", P),
     "polynorm": ("RowOps (fp32 residual)", P), "gemv_rows": ("LinearBF16 decode", P), "gemm_f32": ("Gemm (fp32)", P),
     "dsa_prep": ("DSA", P), "dsa_pool_update": ("DSA", P), "dsa_score": ("DSA / QSA", P), "dsa_select": ("DSA / QSA", P),
     "dsa_gather": ("DSA / QSA", P), "dsa_kpad": ("DSA / QSA", D), "qsa_prep": ("QSA", P), "qsa_pool_update": ("QSA", P),
