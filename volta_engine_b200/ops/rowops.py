@@ -148,7 +148,7 @@ class StreamNorm:
             u = u - u.mean(-1, keepdim=True)
             return (u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + self.eps) * self.w).to(out_dtype)
         out = torch.empty(rows, H, dtype=out_dtype, device=h.device)
-        call("stream_norm", "pplppppliiifi", ptr(h), ptr(part), part.stride(0) if part is not None else 0, ptr(write.mix) if part is not None else 0,
+        call("stream_norm", "pplpppppliiifi", ptr(h), ptr(part), part.stride(0) if part is not None else 0, ptr(write.mix) if part is not None else 0,
              ptr(write.out) if part is not None else 0, ptr(self.read), ptr(self.w), ptr(out), out.stride(0), rows, H, S, float(self.eps), _f32(out))
         return out
 
