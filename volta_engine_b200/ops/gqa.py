@@ -185,8 +185,12 @@ def gqa_attend(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
     view of any row pitch; fp32, or bf16 as the cache). ``kpool`` / ``vpool``: this layer's pages."""
     if not proj.is_cuda:
         return gqa_reference(spec, proj, b, cache, kpool, vpool, out)
-    n = proj.shape[0]
-    q = gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool)
+    return gqa_scores(spec, gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool), b, cache, kpool, vpool, out)
+
+
+def gqa_scores(spec: GqaSpec, q, b, cache, kpool, vpool, out):
+    """Attention of the queries of ``gqa_store`` over the cached rows."""
+    n = q.shape[0]
     if b.row_path or kpool.dtype == torch.float32 or not spec.tc_prefill or out.dtype != torch.bfloat16:
         _each_row(spec, q, b.pos, b.slot, cache, kpool, vpool, out)
         return out

@@ -49,7 +49,8 @@ def build(which: str, width: int, layers: int, dev, pages: int, slots: int, max_
     return model, model.make_cache(pages, slots, max_seq)
 
 
-def run_model(which: str, width: int, layers: int, dev, prompt_len: int, steps: int, warm: int, chunk: int) -> dict:
+def run_model(which: str, width: int, layers: int, dev, prompt_len: int, steps: int, warm: int, chunk: int, build=build) -> dict:
+    """Prefill and decode rates of one model. ``build(which, width, layers, device, pages, slots, max_seq)`` -> (model, cache)."""
     from .. import _lib
     from ..runtime.engine import Engine
     streams = 16
