@@ -1,26 +1,11 @@
-"""Small Fofosun configurations, engines and comparisons for the tests."""
+"""Small Fofosun configurations for the tests."""
 import json
 
-import pytest
 import torch
 
 import fofosun_plain as plain
+from listed_util import DEVICES, DTYPES, TOL, engine, off, one_thread, tokens  # noqa: F401
 from volta_engine_b200.models.fofosun import FofosunConfig, FofosunModel, RandomSource
-from volta_engine_b200.runtime.engine import Engine
-from volta_engine_b200.runtime.kv_cache import PagedKVCache
-
-DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]
-DTYPES = ["fp32", "bf16"]
-TOL = {"fp32": 1e-4, "bf16": 0.04}        # root mean square of the difference over that of the logits
-
-
-@pytest.fixture(autouse=True)
-def one_thread():
-    """The models are so small that a pool of threads only gets in its own way."""
-    n = torch.get_num_threads()
-    torch.set_num_threads(1)
-    yield
-    torch.set_num_threads(n)
 
 
 def hgrn2(heads, dim, vdim, ff=None):
@@ -99,22 +84,6 @@ def reference(name, tokens, seed=3):
     if key not in _want:
         _want[key] = plain.forward(CONFIGS[name], Weights(CONFIGS[name], seed).t, tokens)[0]
     return _want[key]
-
-
-def tokens(n, vocab, seed=0):
-    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def engine(model, pages=24, slots=4, max_seq=1024, **kw):
-    model.reset_states()
-    kv = PagedKVCache(model.kv_layers, 1, model.cfg.head_dim, pages, slots, max_seq, model.device, dtype=model.dtype, v_head_dim=8)
-    return Engine(model, kv, use_graphs=kw.pop("use_graphs", model.device.type == "cuda"), **kw)
-
-
-def off(got, want):
-    """Per row: root mean square of the difference over the root mean square of the wanted logits."""
-    g, w = got.double().cpu(), want.double()
-    return ((g - w).pow(2).mean(-1).sqrt() / w.pow(2).mean(-1).sqrt().mean()).max().item()
 
 
 def write_model(path, name, seed=3):

@@ -7,19 +7,9 @@ import pytest
 import torch
 
 from fofosun_util import CONFIGS, DEVICES, DTYPES, TOL, engine, make, off, one_thread, reference, tokens, write_model  # noqa: F401
+from listed_util import CUTS, run, schedule
 
 NAMES = list(CONFIGS)
-
-
-def run(eng, slot, toks, cuts, p0=0):
-    """Tokens of one sequence in portions of the given sizes -> logits of all of them."""
-    out, at = [], 0
-    for c in cuts:
-        part = toks[at:at + c]
-        out.append(eng.forward_segments([(slot, part, p0 + at, list(range(len(part))))]).float().clone())
-        at += c
-    assert at == len(toks)
-    return torch.cat(out)
 
 
 @pytest.mark.parametrize("device", DEVICES)
@@ -49,10 +39,6 @@ def test_residual_after_every_layer(device):
         assert (got - want).abs().max() < 2e-4 * want.abs().max()
 
 
-CUTS = {"one by one": [1] * 150, "twos": [2] * 75, "prompt then decode": [110] + [1] * 40, "around pages": [63, 1, 1, 63, 2, 20],
-        "short and long": [3, 17, 2, 64, 15, 16, 33], "halves": [75, 75]}
-
-
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["eights", "odd", "wide"])
@@ -68,31 +54,6 @@ def test_portions_and_decoding(name, dtype, device):
         assert off(run(eng, slot, toks, cuts), want) < TOL[dtype], what
         eng.kv.release(slot)                     # the next way of cutting gets used pages and a used state slot
     assert eng.kv.free_pages() == eng.kv.num_pages - 1
-
-
-def schedule(lengths, seed):
-    """Random steps over several requests: portions of some beside single tokens of others; at most four live at once."""
-    g = torch.Generator().manual_seed(seed)
-    left, live, steps = list(range(len(lengths))), [], []
-    done = [0] * len(lengths)
-    while left or live:
-        while left and len(live) < 4:
-            live.append(left.pop(0))
-        step, ended = [], []
-        for r in list(live):
-            if len(live) > 1 and torch.rand((), generator=g) < 0.2:
-                continue                         # left out of this step
-            rest = lengths[r] - done[r]
-            n = [1, 1, 2, 3, 16, 29, 64, 90][int(torch.randint(0, 8, (), generator=g))] if rest > 12 else 1
-            n = min(n, rest)
-            step.append((r, done[r], n))
-            done[r] += n
-            if done[r] == lengths[r]:
-                ended.append(r)
-        live = [r for r in live if r not in ended]
-        if step:
-            steps.append((step, ended))
-    return steps
 
 
 @pytest.mark.parametrize("device", DEVICES)

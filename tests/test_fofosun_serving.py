@@ -1,31 +1,16 @@
 """The Fofosun decoder under the scheduler: greedy generation against the plain statement, prompts and decode rows in one forward,
 sampling, speculation with rollback of the recurrent state, prefix snapshots, the launcher."""
-import json
-
 import pytest
 import torch
 
 import fofosun_plain as plain
 from fofosun_util import CONFIGS, DEVICES, Weights, engine, make, one_thread, tokens, write_model  # noqa: F401
-from volta_engine_b200.runtime.generator import Generator, Request
-from volta_engine_b200.runtime.options import Options
+from listed_util import generator, run_all, write_tokenizer
+from volta_engine_b200.runtime.generator import Request
 from volta_engine_b200.runtime.prefix_cache import PrefixCache
 from volta_engine_b200.runtime.sampling import SamplingParams
 
 NAME = "eights"
-
-
-class Tok:
-    eos_ids: list = []
-
-    def decode_bytes(self, ids, skip_special=False):
-        return bytes(i & 0x7F for i in ids)
-
-
-def generator(model, slots=3, pages=24, chunk=48, cache=None, **opt):
-    eng = engine(model, pages=pages, slots=slots, max_seq=512, prefill_chunk=chunk)
-    o = Options.resolve(dict({"max_slots": slots, "prefix_interval": 64, "loop_detect": False}, **opt), env={})
-    return Generator(eng, Tok(), o, prefix_cache=cache, eos_ids=[])
 
 
 def greedy(prompt, n):
@@ -35,22 +20,6 @@ def greedy(prompt, n):
     for _ in range(n):
         seq.append(int(plain.forward(cfg, w, seq)[0][-1].argmax()))
     return seq[len(prompt):]
-
-
-def run_all(gen, reqs):
-    """Submit everything, step until all are done -> token lists in order."""
-    out = [[] for _ in reqs]
-    left = [len(reqs)]
-    for i, r in enumerate(reqs):
-        r.on_text = lambda t, ids, lp, i=i: out[i].extend(ids)
-        r.on_finish = lambda reason, usage: left.__setitem__(0, left[0] - 1)
-        gen.submit(r)
-    for _ in range(2000):
-        if not left[0]:
-            break
-        gen.step()
-    assert not left[0]
-    return out
 
 
 def prompts():
@@ -164,18 +133,6 @@ def test_cancelled_requests_in_a_mixed_step():
         if len(done) == 3:
             break
     assert done == {0: "length", 1: "length", 2: "cancelled"}
-
-
-def write_tokenizer(d, vocab):
-    """A byte-level vocabulary of 256 pieces and no merges, enough for the launcher."""
-    alphabet = [chr(b) if 33 <= b < 127 or 161 <= b < 173 or 174 <= b < 256 else None for b in range(256)]
-    n = 0
-    for b in range(256):
-        if alphabet[b] is None:
-            alphabet[b] = chr(256 + n)
-            n += 1
-    (d / "tokenizer.json").write_text(json.dumps({"model": {"type": "BPE", "vocab": {c: i for i, c in enumerate(alphabet)}, "merges": []},
-                                                  "added_tokens": [], "pre_tokenizer": {"type": "ByteLevel"}}))
 
 
 def test_server_on_a_model_directory(tmp_path):

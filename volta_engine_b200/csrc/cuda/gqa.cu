@@ -17,6 +17,7 @@
 namespace ve {
 
 constexpr int kGPage = 64;
+constexpr int kGMinPages = 2;     // of a key split
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct GqaDims {
@@ -39,8 +40,8 @@ VE_DEVINL int page_of(const GqaRows& r, int slot, int kt) { return r.page_table[
 // proj row: [q (H d) | k (G d) | v (G dv) | ...]. grid (rows, ceil((H + 2 G) / 8)), a warp per head.
 template <typename X, typename T>
 __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const GqaRows rw, const X* __restrict__ proj, long ld, const float* __restrict__ wq,
-                                                        const float* __restrict__ wk, float eps, float coef, int every, T* __restrict__ qo,
-                                                        T* __restrict__ kpool, T* __restrict__ vpool) {
+                                                        const float* __restrict__ wk, float eps, float coef, int every, int vec,
+                                                        T* __restrict__ qo, T* __restrict__ kpool, T* __restrict__ vpool) {
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
@@ -58,6 +59,26 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
   }
   const int w = is_v ? n.dv : n.d, wide = is_v ? n.vw : n.kw;
   const float* wn = is_v ? nullptr : is_q ? wq : wk;
+  const float t = is_q && every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
+  if (vec) {                                // widths up to 256 in multiples of eight: four columns per lane and step, kept in registers
+    float4 v[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = (j * 32 + lane) * 4;
+      v[j] = i < w ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    const float g = wn ? t / sqrtf(warp_sum(ss) / (float)w + eps) : t;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = (j * 32 + lane) * 4;
+      if (i >= w) continue;
+      const float4 q = wn ? *reinterpret_cast<const float4*>(wn + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+      store4(dst + i, make_float4(v[j].x * g * q.x, v[j].y * g * q.y, v[j].z * g * q.z, v[j].w * g * q.w));
+    }
+    return;
+  }
   float f = 1.f;
   if (wn) {
     float ss = 0.f;
@@ -67,7 +88,6 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
     }
     f = 1.f / sqrtf(warp_sum(ss) / (float)w + eps);
   }
-  const float t = is_q && every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
   for (int i = lane; i < wide; i += 32) {
     float v = 0.f;
     if (i < w) {
@@ -156,6 +176,14 @@ VE_DEVINL uint32_t gq_pack(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&t);
 }
 
+template <typename O>
+VE_DEVINL void put_row(O* p, float4 v) {                  // four columns of an output row of any alignment
+  p[0] = from_f<O>(v.x);
+  p[1] = from_f<O>(v.y);
+  p[2] = from_f<O>(v.z);
+  p[3] = from_f<O>(v.w);
+}
+
 struct GqaDecode {
   GqaDims n;
   GqaRows rw;
@@ -191,7 +219,9 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       for (int i = tid; i < nh * n.dv; i += 128) out[row * ldo + (long)h0 * n.dv + i] = from_f<O>(0.f);
     return;
   }
-  const int p = a.rw.pos[row], pages = p / kGPage + 1, per = (pages + a.nsplit - 1) / a.nsplit;
+  // the grid does not know the position: a row takes as many of its splits as have at least kGMinPages pages
+  const int p = a.rw.pos[row], pages = p / kGPage + 1, per = max(kGMinPages, (pages + a.nsplit - 1) / a.nsplit), used = (pages + per - 1) / per;
+  if (z >= used) return;
   const int kt_begin = z * per, kt_end = min(pages, kt_begin + per);
   if (tid == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(&full[i], 1);
@@ -347,7 +377,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
         l = fmaf(ls[w * 16 + hr], f, l);
       }
     }
-    if (a.nsplit == 1) {
+    if (used == 1) {
       const float snk = sink_of(h0 + hr), top = fmaxf(m, snk), f = exp2f(m - top);
       const float den = fmaf(l, f, a.sc.sink ? exp2f(snk - top) : 0.f);
       out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * f / den * a.sc.out_scale);
@@ -357,11 +387,11 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       if (c == 0) a.lse[at] = l > 0.f ? m + log2f(l) : -FLT_MAX;
     }
   }
-  if (a.nsplit == 1) return;
+  if (used == 1) return;
   __threadfence();
   __syncthreads();
   int* tk = a.tickets + (long)blockIdx.x * n.G + kvh;
-  if (tid == 0) s_last = atomicAdd(tk, 1) == a.nsplit - 1;
+  if (tid == 0) s_last = atomicAdd(tk, 1) == used - 1;
   __syncthreads();
   if (!s_last) return;
   __threadfence();
@@ -369,7 +399,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
   float* sw = ms;                           // [16][64]
   for (int hr = warp; hr < nh; hr += 4) {
     const long at = (row * n.H + h0 + hr) * a.nsplit;
-    const float l0 = lane < a.nsplit ? __ldcg(a.lse + at + lane) : -FLT_MAX, l1 = lane + 32 < a.nsplit ? __ldcg(a.lse + at + lane + 32) : -FLT_MAX;
+    const float l0 = lane < used ? __ldcg(a.lse + at + lane) : -FLT_MAX, l1 = lane + 32 < used ? __ldcg(a.lse + at + lane + 32) : -FLT_MAX;
     const float snk = sink_of(h0 + hr), top = fmaxf(snk, warp_max(fmaxf(l0, l1)));
     const float w0 = l0 == -FLT_MAX ? 0.f : exp2f(l0 - top), w1 = l1 == -FLT_MAX ? 0.f : exp2f(l1 - top);
     const float den = warp_sum(w0 + w1) + (a.sc.sink ? exp2f(snk - top) : 0.f), inv = a.sc.out_scale / den;
@@ -377,13 +407,43 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
     sw[hr * 64 + lane + 32] = w1 * inv;
   }
   __syncthreads();
-  for (int i = tid; i < nh * n.dv; i += 128) {
-    const int hr = i / n.dv, c = i % n.dv;
-    const float* part = a.o_part + (row * n.H + h0 + hr) * a.nsplit * n.dv + c;
-    float acc = 0.f;
+  if (n.dv % 4 == 0) {
+    // four columns per thread; few columns: the splits are dealt to up to four thread groups
+    const int c4 = n.dv / 4, items = nh * c4, ng = items <= 32 ? 4 : items <= 64 ? 2 : 1, per = 128 / ng, y0 = tid / per;
+    float4* acc4 = reinterpret_cast<float4*>(sw + 16 * 64);
+    for (int i = tid % per; i < items; i += per) {
+      const int hr = i / c4, c = (i % c4) * 4;
+      const float* part = a.o_part + (row * n.H + h0 + hr) * a.nsplit * n.dv + c;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-    for (int y = 0; y < a.nsplit; ++y) acc = fmaf(sw[hr * 64 + y], __ldcg(part + (long)y * n.dv), acc);
-    out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc);
+      for (int y = y0; y < used; y += ng) {
+        const float4 x = __ldcg(reinterpret_cast<const float4*>(part + (long)y * n.dv));
+        const float f = sw[hr * 64 + y];
+        v = make_float4(fmaf(f, x.x, v.x), fmaf(f, x.y, v.y), fmaf(f, x.z, v.z), fmaf(f, x.w, v.w));
+      }
+      if (ng > 1) acc4[tid] = v;
+      else put_row(out + row * ldo + (long)(h0 + hr) * n.dv + c, v);
+    }
+    if (ng > 1) {
+      __syncthreads();
+      if (tid < items) {                    // (at most `per` items)
+        float4 v = acc4[tid];
+        for (int y = 1; y < ng; ++y) {
+          const float4 x = acc4[y * per + tid];
+          v = make_float4(v.x + x.x, v.y + x.y, v.z + x.z, v.w + x.w);
+        }
+        put_row(out + row * ldo + (long)(h0 + tid / c4) * n.dv + (tid % c4) * 4, v);
+      }
+    }
+  } else {
+    for (int i = tid; i < nh * n.dv; i += 128) {
+      const int hr = i / n.dv, c = i % n.dv;
+      const float* part = a.o_part + (row * n.H + h0 + hr) * a.nsplit * n.dv + c;
+      float acc = 0.f;
+#pragma unroll 8
+      for (int y = 0; y < used; ++y) acc = fmaf(sw[hr * 64 + y], __ldcg(part + (long)y * n.dv), acc);
+      out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc);
+    }
   }
   if (tid == 0) *tk = 0;
 }
@@ -434,7 +494,9 @@ int ve_gqa_store(VE_GDIMS, VE_GROWS, const void* proj, long ld, int x32, const v
   const GqaDims n = VE_GMAKE;
   if (!gdims_ok(n)) return cudaErrorInvalidValue;
   const dim3 grid(rows, (H + 2 * G + 7) / 8);
-#define VE_GS(X, T) launch_pdl(gqa_store_kernel<X, T>, grid, dim3(256), 0, st, n, VE_RMAKE, (const X*)proj, ld, (const float*)wq, (const float*)wk, eps, coef, every, \
+  const int vec = d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && kw == d && vw == dv && ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)wq & 15) &&
+                  !((uintptr_t)wk & 15);
+#define VE_GS(X, T) launch_pdl(gqa_store_kernel<X, T>, grid, dim3(256), 0, st, n, VE_RMAKE, (const X*)proj, ld, (const float*)wq, (const float*)wk, eps, coef, every, vec, \
     (T*)qo, (T*)kpool, (T*)vpool)
   if (f32) VE_GS(float, float);
   else if (x32) VE_GS(float, __nv_bfloat16);
@@ -481,12 +543,12 @@ int ve_gqa_decode(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpoo
 #undef VE_GD
 }
 
-// Tiles of at most 128 / (H / G) tokens of one sequence (rows tile_first .. + tile_count of the batch); kw <= 256, vw <= 128.
+// Tiles of at most 128 / (H / G) tokens of one sequence (rows tile_first .. + tile_count of the batch); kw <= 256, vw <= 128, scale > 0.
 int ve_gqa_prefill(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpool, const void* vpool, long pages, const void* tile_first, const void* tile_count,
                    int ntiles, void* out, long ldo, void* status, cudaStream_t st) {
   if (ntiles <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 128 || H / G > 128 || ((uintptr_t)q & 15) || (bias && L < 1)) return cudaErrorInvalidValue;
+  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 128 || H / G > 128 || !(scale > 0.f) || ((uintptr_t)q & 15) || (bias && L < 1)) return cudaErrorInvalidValue;
   CUtensorMap km, vm;
   int rc = pool_map(&km, kpool, pages, n, kw, kps);
   if (!rc) rc = pool_map(&vm, vpool, pages, n, vw, vps);

@@ -24,13 +24,19 @@ struct GqaTc {
   int* status;
 };
 
-constexpr int kGtRows = 128, kGtThreads = 320, kGtVs = 2;
+constexpr int kGtRows = 128, kGtThreads = 320;
 constexpr float kGtLazyLog2 = 8.f;
+
+// Page stages: a page's keys and values are requested in turn, and the values wait for the weights of their page; with four stages
+// the requests run far enough ahead that no product waits for memory.
+template <int DQC, int DVC> struct GtStages {
+  static constexpr int K = DQC > 3 ? 2 : 4, V = DQC > 3 && DVC > 1 ? 2 : 4;
+};
 
 template <int DQC, int DVC>
 __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc p, const __grid_constant__ CUtensorMap kmap,
                                                                     const __grid_constant__ CUtensorMap vmap) {
-  constexpr int KS = DQC > 3 ? 2 : 3, KB = DQC * 8192, VB = DVC * 8192, QC = kGtRows * 128, PB = kGtRows * 128, DV = DVC * 64;
+  constexpr int KS = GtStages<DQC, DVC>::K, VS = GtStages<DQC, DVC>::V, KB = DQC * 8192, VB = DVC * 8192, QC = kGtRows * 128, PB = kGtRows * 128, DV = DVC * 64;
   constexpr uint32_t TMEM_COLS = 512, O_COL = 256;       // S of stream t, buffer b at t * 128 + b * 64; O of stream t at 256 + t * DV
   const float NEG_INF = __int_as_float(0xff800000);
   grid_dep_wait();
@@ -39,9 +45,9 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(gt_smem) + 1023) & ~(uintptr_t)1023);
   uint8_t* q_s = smem;                                   // [DQC][128 rows][128 B]
   uint8_t* k_s = q_s + DQC * QC;                         // [KS][DQC][64 keys][128 B]
-  uint8_t* v_s = k_s + KS * KB;                          // [kGtVs][DVC][64 keys][128 B]
-  uint8_t* p_s = v_s + kGtVs * VB;                       // [2 streams][2 terms][128 rows][128 B]
-  __shared__ uint64_t kfull[KS], kempty[KS], vfull[kGtVs], vempty[kGtVs], s_full[2][2], p_full[2], pv_done[2];
+  uint8_t* v_s = k_s + KS * KB;                          // [VS][DVC][64 keys][128 B]
+  uint8_t* p_s = v_s + VS * VB;                       // [2 streams][2 terms][128 rows][128 B]
+  __shared__ uint64_t kfull[KS], kempty[KS], vfull[VS], vempty[VS], s_full[2][2], p_full[2], pv_done[2];
   __shared__ uint32_t tmem_holder;
   __shared__ int s_fail;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -54,7 +60,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       mbar_init(&kfull[i], 1);
       mbar_init(&kempty[i], 1);
     }
-    for (int i = 0; i < kGtVs; ++i) {
+    for (int i = 0; i < VS; ++i) {
       mbar_init(&vfull[i], 1);
       mbar_init(&vempty[i], 1);
     }
@@ -97,7 +103,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       prefetch_tmap(&kmap);
       prefetch_tmap(&vmap);
       for (int j = 0; j < n; ++j) {
-        const int ks = j % KS, vs = j % kGtVs, page = page_of(p.rw, slot, j);
+        const int ks = j % KS, vs = j % VS, page = page_of(p.rw, slot, j);
         if (j >= KS && !mbar_wait(&kempty[ks], ((j / KS) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
@@ -105,7 +111,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
         mbar_expect_tx(&kfull[ks], KB);
 #pragma unroll
         for (int c = 0; c < DQC; ++c) tma_load_3d(k_s + ks * KB + c * 8192, &kmap, &kfull[ks], c * 64, kvh * kGPage, page);
-        if (j >= kGtVs && !mbar_wait(&vempty[vs], ((j / kGtVs) - 1) & 1)) {
+        if (j >= VS && !mbar_wait(&vempty[vs], ((j / VS) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
         }
@@ -141,8 +147,8 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
         // the S buffer page j + 2 lands in was read by the softmax of page j - 2, which ended before its P arrived
         if (j + 2 < n) ok = issue_s(j + 2);
         if (!ok) break;
-        const int t = j & 1, i = j >> 1, vs = j % kGtVs;
-        ok = mbar_wait(&vfull[vs], (j / kGtVs) & 1) && mbar_wait(&p_full[t], i & 1);
+        const int t = j & 1, i = j >> 1, vs = j % VS;
+        ok = mbar_wait(&vfull[vs], (j / VS) & 1) && mbar_wait(&p_full[t], i & 1);
         if (!ok) break;
         tc_fence_after();
 #pragma unroll
@@ -177,13 +183,13 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       tmem_ld32(t_lane + strm * 128 + b * 64, reinterpret_cast<uint32_t*>(sv));
       tmem_ld32(t_lane + strm * 128 + b * 64 + 32, reinterpret_cast<uint32_t*>(sv) + 32);
       tmem_ld_wait();
-      if (p.sc.bias && __any_sync(0xffffffffu, r_pos - key0 - 63 < L1)) {
+      // far pages: the scores stay as they are and one addend per row stands for the bias; near pages: scaled, bias by distance
+      const bool near = p.sc.bias && __any_sync(0xffffffffu, r_pos - key0 - 63 < L1);
+      if (near) {
 #pragma unroll
         for (int e = 0; e < 64; ++e) sv[e] = fmaf(sv[e], scale2, tab[min(max(r_pos - key0 - e, 0), L1)] * kLog2e);
-      } else {
-#pragma unroll
-        for (int e = 0; e < 64; ++e) sv[e] = fmaf(sv[e], scale2, far);
       }
+      const float mul = near ? 1.f : scale2, add = near ? 0.f : far;
       if (!r_ok || key0 + 63 > r_pos) {
 #pragma unroll
         for (int e = 0; e < 64; ++e) sv[e] = r_ok && key0 + e <= r_pos ? sv[e] : NEG_INF;
@@ -196,7 +202,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
         mx2 = fmaxf(mx2, sv[e + 2]);
         mx3 = fmaxf(mx3, sv[e + 3]);
       }
-      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
+      const float mx = fmaf(fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)), mul, add);          // the scale is positive
       const bool grow = mx > m_ref + kGtLazyLog2;
       float alpha = 1.f;
       if (grow) {
@@ -221,11 +227,11 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       }
       l0 *= alpha;
       l1 *= alpha;
-      const float neg_m = m_ref == NEG_INF ? 0.f : -m_ref;
+      const float neg_m = add - (m_ref == NEG_INF ? 0.f : m_ref);
       uint32_t w[32], x[32];                             // leading terms and remainders
 #pragma unroll
       for (int e = 0; e < 32; ++e) {
-        const float p0 = ex2_approx(sv[2 * e] + neg_m), p1 = ex2_approx(sv[2 * e + 1] + neg_m);
+        const float p0 = ex2_approx(fmaf(sv[2 * e], mul, neg_m)), p1 = ex2_approx(fmaf(sv[2 * e + 1], mul, neg_m));
         l0 += p0;
         l1 += p1;
         w[e] = gq_pack(p0, p1);
@@ -306,7 +312,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
 
 template <int DQC, int DVC>
 static int launch_gqa_tc(const GqaTc& p, const CUtensorMap& km, const CUtensorMap& vm, int ntiles, cudaStream_t st) {
-  constexpr int smem = DQC * kGtRows * 128 + (DQC > 3 ? 2 : 3) * DQC * 8192 + kGtVs * DVC * 8192 + 4 * kGtRows * 128 + 1024;
+  constexpr int smem = DQC * kGtRows * 128 + GtStages<DQC, DVC>::K * DQC * 8192 + GtStages<DQC, DVC>::V * DVC * 8192 + 4 * kGtRows * 128 + 1024;
   static_assert(smem <= 227 * 1024 - 512, "shared memory budget");
   static bool attr = false;
   if (!attr) {

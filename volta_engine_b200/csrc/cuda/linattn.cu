@@ -488,34 +488,46 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
   if (!OUT && ch) a.total[((long)c * a.H + h) * a.dk + tid] = prod;
 }
 
-// dec[row][c] = sigmoid(W a + bias)^inv_tau. 128 channels per CTA (their weight rows in shared memory), rows in steps of the grid.
-template <typename X>
+// dec[row][c] = sigmoid(W a + bias)^inv_tau. grid (channels / 128, rows / kDecayRows): thread = channel, the low-rank rows in shared
+// memory, the channel's weights in registers (RK >= rank, a multiple of four) or, RK 0, in shared memory.
+constexpr int kDecayRows = 32;
+template <int RK, typename X>
 __global__ void __launch_bounds__(128) linattn_decay_kernel(const X* __restrict__ a, long lda, const float* __restrict__ w, const float* __restrict__ bias,
                                                             float* __restrict__ dec, int rows, int C, int rank, float inv_tau) {
-  extern __shared__ float ws[];                           // [128][rank + 1]
+  extern __shared__ __align__(16) float ds[];             // [kDecayRows][RP], then (RK 0) [128][rank + 1]
+  const int RP = RK ? RK : rank, c0 = blockIdx.x * 128, c = c0 + threadIdx.x, r0 = blockIdx.y * kDecayRows, n = min(kDecayRows, rows - r0);
+  float* ws = ds + kDecayRows * RP;
+  float wr[RK ? RK : 1];
+  if (RK) {
+#pragma unroll
+    for (int r = 0; r < RK; ++r) wr[r] = r < rank && c < C ? w[(long)c * rank + r] : 0.f;
+  } else {
+    for (int i = threadIdx.x; i < 128 * rank; i += 128) ws[(i / rank) * (rank + 1) + i % rank] = c0 + i / rank < C ? w[(long)c0 * rank + i] : 0.f;
+  }
   grid_dep_wait();
   grid_dep_launch();
-  const int c0 = blockIdx.x * 128, c = c0 + threadIdx.x;
-  for (int i = threadIdx.x; i < 128 * rank; i += 128) {
-    const int j = i / rank;
-    ws[j * (rank + 1) + i % rank] = c0 + j < C ? w[(long)c0 * rank + i] : 0.f;
+  for (int i = threadIdx.x; i < n * RP; i += 128) {
+    const int y = i / RP, r = i % RP;
+    ds[i] = r < rank ? to_f(a[(long)(r0 + y) * lda + r]) : 0.f;
   }
   __syncthreads();
   if (c >= C) return;
   const float b = bias[c];
-  const float* wr = ws + threadIdx.x * (rank + 1);
-  for (int r0 = blockIdx.y * 4; r0 < rows; r0 += gridDim.y * 4) {
-    float z[4] = {b, b, b, b};
-    const X* ar = a + (long)r0 * lda;
-    for (int r = 0; r < rank; ++r) {
-      const float v = wr[r];
+  for (int y = 0; y < n; ++y) {
+    float z = b, z1 = 0.f, z2 = 0.f, z3 = 0.f;
+    if (RK) {
 #pragma unroll
-      for (int y = 0; y < 4; ++y)
-        if (r0 + y < rows) z[y] = fmaf(v, to_f(ar[y * lda + r]), z[y]);
+      for (int r = 0; r < RK; r += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(ds + y * RK + r);
+        z = fmaf(wr[RK ? r : 0], v.x, z);
+        z1 = fmaf(wr[RK ? r + 1 : 0], v.y, z1);
+        z2 = fmaf(wr[RK ? r + 2 : 0], v.z, z2);
+        z3 = fmaf(wr[RK ? r + 3 : 0], v.w, z3);
+      }
+    } else {
+      for (int r = 0; r < rank; ++r) z = fmaf(ws[threadIdx.x * (rank + 1) + r], ds[y * rank + r], z);
     }
-#pragma unroll
-    for (int y = 0; y < 4; ++y)
-      if (r0 + y < rows) dec[(long)(r0 + y) * C + c] = root_decay(z[y], inv_tau);
+    dec[(long)(r0 + y) * C + c] = root_decay((z + z1) + (z2 + z3), inv_tau);
   }
 }
 
@@ -601,18 +613,22 @@ int ve_linattn_step(const void* proj, long ld, int x32, const void* pos, const v
 // Decays of mode 2 for rows a [rows][rank] (pitch lda; fp32 when x32, else bf16), weights w [C][rank].
 int ve_linattn_decay(const void* a, long lda, int x32, const void* w, const void* bias, void* dec, int rows, int C, int rank, float inv_tau, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (C < 1 || rank < 1 || rank > 400) return cudaErrorInvalidValue;         // (the weight rows of 128 channels are in shared memory)
-  const int cx = (C + 127) / 128, ry = (rows + 3) / 4, most = (148 * 8 + cx - 1) / cx;
-  const dim3 grid(cx, ry < most ? ry : most);
-  const size_t smem = (size_t)128 * (rank + 1) * 4;
-  if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(linattn_decay_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_decay_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-  }
-  if (x32) launch_pdl(linattn_decay_kernel<float>, grid, dim3(128), smem, st, (const float*)a, lda, (const float*)w, (const float*)bias, (float*)dec, rows, C, rank, inv_tau);
-  else launch_pdl(linattn_decay_kernel<__nv_bfloat16>, grid, dim3(128), smem, st, (const __nv_bfloat16*)a, lda, (const float*)w, (const float*)bias, (float*)dec,
-                  rows, C, rank, inv_tau);
+  if (C < 1 || rank < 1 || rank > 320) return cudaErrorInvalidValue;         // (weights of 128 channels in shared memory above 32)
+  const dim3 grid((C + 127) / 128, (rows + kDecayRows - 1) / kDecayRows);
+  const int rk = rank <= 16 ? 16 : rank <= 32 ? 32 : 0;
+  const size_t smem = (size_t)(kDecayRows * (rk ? rk : rank) + (rk ? 0 : 128 * (rank + 1))) * 4;
+#define VE_LD(RK, X) do { \
+    if (smem > 48 * 1024) { \
+      const cudaError_t e = cudaFuncSetAttribute(linattn_decay_kernel<RK, X>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) return (int)e; \
+    } \
+    launch_pdl(linattn_decay_kernel<RK, X>, grid, dim3(128), smem, st, (const X*)a, lda, (const float*)w, (const float*)bias, (float*)dec, rows, C, rank, inv_tau); \
+  } while (0)
+#define VE_LD_R(X) do { if (rk == 16) VE_LD(16, X); else if (rk == 32) VE_LD(32, X); else VE_LD(0, X); } while (0)
+  if (x32) VE_LD_R(float);
+  else VE_LD_R(__nv_bfloat16);
+#undef VE_LD_R
+#undef VE_LD
   VE_CHECK_LAUNCH();
 }
 

@@ -152,6 +152,7 @@ class ListedModel(SlotStates, DenseModel):
 
     def reset_states(self) -> None:
         """Forget the slots' states (an engine with another slot count is about to be built on this model)."""
+        self.journal_on = False
         for L in self.layers:
             L.mixer.state = None
         for name in ("_jsets", "_shadows"):

@@ -83,7 +83,7 @@ class GqaSpec:
 
     @property
     def tc_prefill(self) -> bool:
-        return self.kw <= 256 and self.vw <= 128 and self.group <= 128
+        return self.kw <= 256 and self.vw <= 128 and self.group <= 128 and self.scale > 0
 
     def temperature(self, pos):
         return 1.0 + self.temp_coef * torch.log(((pos + 1) // self.temp_every + 1).float()) if self.temp_every > 0 else torch.ones(pos.shape)
@@ -171,7 +171,7 @@ def _each_row(spec, q, pos, slot, cache, kpool, vpool, out):
              ptr(out), out.stride(0), o32, n, int(f32))
         return
     units = n * spec.kv_heads * ((spec.group + 15) // 16)
-    nsplit = max(1, min(64, 296 // units)) if units <= MAX_TICKETS else 1           # two CTAs per SM, whatever the position
+    nsplit = max(16, min(64, 148 // units)) if units <= MAX_TICKETS else 1          # a row takes as many of them as its position asks for
     part = lse = None
     if nsplit > 1:
         part = torch.empty(n, spec.heads, nsplit, spec.vdim, dtype=torch.float32, device=dev)

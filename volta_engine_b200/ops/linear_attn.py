@@ -45,7 +45,7 @@ class LinAttnSpec:
     @property
     def chunks(self) -> bool:
         """The chunked kernels take these sizes."""
-        return self.dk <= 128 and self.dv <= 128 and self.rank <= 400
+        return self.dk <= 128 and self.dv <= 128 and self.rank <= 320
 
     @property
     def cols(self) -> int:

@@ -124,6 +124,7 @@ class Engine:
                 b = BatchRows.make(ids, pos, [slot] * c, self.device, LOGITS_LAST if last else LOGITS_NONE, G,
                                    prefill=True)
             self._mm_rows(b, slot, start_pos + done, c, mm)
+            self._no_journal(c)
             logits = self.model.forward(b, self.kv)
             if last:
                 rows = logits.shape[0]
@@ -204,6 +205,11 @@ class Engine:
     def supports_journal(self) -> bool:
         """Models with recurrent state record verify blocks so that rejected rows can be taken back (``rollback``)."""
         return hasattr(self.model, "rollback_state")
+
+    def _no_journal(self, rows: int) -> None:
+        """Rows of a forward that nobody takes back (a short prompt portion would otherwise be recorded like the verify block in front)."""
+        if self.supports_journal:
+            self.model.begin_journal(False, rows)
 
     def rollback(self, slot: int, keep_rows: int) -> None:
         """After ``step(..., journal=True)`` over rows of ``slot``: keep the effect of the first ``keep_rows`` rows on the
@@ -320,6 +326,7 @@ class Engine:
             b = BatchRows.make(tokens, pos, [slot] * c, self.device, LOGITS_LAST if want_token else LOGITS_NONE, G,
                                prefill=True)
         self._mm_rows(b, slot, start_pos, c, mm)
+        self._no_journal(c)
         logits = self.model.forward(b, self.kv)
         if not want_token:
             return -1
@@ -363,8 +370,7 @@ class Engine:
             ids += toks
             pos += range(p0, p0 + len(toks))
             slots += [slot] * len(toks)
-        if self.supports_journal:
-            self.model.begin_journal(False, total)
+        self._no_journal(total)
         b = BatchRows.make(ids, pos, slots, self.device, LOGITS_ROWS if n_want else LOGITS_NONE, 1, prefill=False, nsplit=self._nsplit(total))
         if n_want:
             b.want = torch.tensor([at[i] + w for i, s in enumerate(segs) for w in s[3]], dtype=torch.int64).to(self.device, non_blocking=True)
