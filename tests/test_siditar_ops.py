@@ -313,7 +313,7 @@ def test_attention_of_a_mixed_batch(dtype, device):
 @pytest.mark.parametrize("H,G,d,dv", [(4, 1, 128, 128), (3, 3, 64, 64), (2, 1, 256, 128), (6, 2, 40, 72)])
 def test_prompt_of_many_pages_with_moving_references(H, G, d, dv):
     """Scores grow along the sequence, then fall: both streams, all ring stages and several query tiles."""
-    spec, W, m = attn_case(H, G, d, dv, B=32, D=200, seed=3, coef=3.0, every=100, scale=2.0 / d ** 0.5)
+    spec, W, m = attn_case(H, G, d, dv, B=32, D=200, seed=3, coef=1.0, every=100, scale=2.0 / d ** 0.5)
     T = 700
     x = rnd(T, spec.cols, seed=5).to(torch.bfloat16).float()
     want = plain.biased_attention(W, "", m, x.double(), spec.eps)
