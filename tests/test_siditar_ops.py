@@ -80,7 +80,12 @@ def test_clamped_gated_unit(rows, ff, limit, dtype, device):
     z[0, 0], z[0, ff] = -50.0, -50.0                                 # the gate has no lower bound, the other half has
     eye = torch.eye(ff, dtype=torch.float64)
     pick = {"gate": torch.cat([eye, 0 * eye], 1), "up": torch.cat([0 * eye, eye], 1), "down": eye}
-    close(ClampedGlu(limit, 1.702).rows(z.to(device), dtype), plain.clamped_ff(pick, "", {"limit": limit}, z.double()), dtype, f32=5e-6)
+    want = plain.clamped_ff(pick, "", {"limit": limit}, z.double())
+    close(ClampedGlu(limit, 1.702).rows(z.to(device), dtype), want, dtype, f32=5e-6)
+    if ff % 4 == 0:                                                  # the same with the halves in blocks, as a weight in blocks makes them
+        zb = (z.float() @ ClampedGlu.interleave(pick["gate"].float(), pick["up"].float()).t()).to(dtype)
+        assert not torch.equal(zb, z)
+        close(ClampedGlu(limit, 1.702, True).rows(zb.to(device), dtype), want, dtype, f32=5e-6)
 
 
 @pytest.mark.parametrize("device", DEVICES)
@@ -123,6 +128,15 @@ def test_decode_linear_with_prologues(N, K, M):
         y = v.float().to(torch.bfloat16).double() @ Wd.t()
         want = plain.write_streams(hs.double().transpose(0, 1), mix.double(), out.double(), y).transpose(0, 1)
         assert (hd.double().cpu() - want).abs().max() < 1e-2 * want.pow(2).mean().sqrt()
+    if N % 16 == 0:                                                   # the gated unit as the epilogue
+        x, w = rnd(M, 1, K, seed=13), rnd(K, seed=14)
+        n = StreamNorm(w.to(dev), 1e-5, torch.ones(1, device=dev))
+        blk = LinearBF16(ClampedGlu.interleave(W[:N // 2], W[N // 2:]).to(dev))
+        got = gemv_rows(blk, M, **n.prologue(x.to(dev)), **ClampedGlu(0.8, 1.702, True).epilogue())
+        z = plain.layer_norm(x[:, 0].double(), w.double(), 1e-5).float().to(torch.bfloat16).double() @ Wd.t()
+        eye = torch.eye(N // 2, dtype=torch.float64)
+        v = plain.clamped_ff({"gate": torch.cat([eye, 0 * eye], 1), "up": torch.cat([0 * eye, eye], 1), "down": eye}, "", {"limit": 0.8}, z)
+        assert got.shape == (M, N // 2) and (got.double().cpu() - v).abs().max() < 2e-2 * v.pow(2).mean().sqrt() + 2 ** -8 * v.abs().max()
     for G in (g for g in (8, 5, 1) if (K - 11) % g == 0 or K % 8 == 0):
         k0 = K % G + 2 * G
         a, x, gate, w = rnd(M, k0, seed=9), rnd(M, K - k0, seed=10), rnd(M, K - k0 + 2, seed=11)[:, 1:-1], rnd(G, seed=12)

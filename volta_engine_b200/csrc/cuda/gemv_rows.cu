@@ -7,7 +7,8 @@
 //              3  x = PolyNorm of an fp32 row
 //              4  x = layer norm (no shift) of the weighted sum of the fp32 residual streams
 //              5  x = clamped gated unit of an fp32 [gate | up] row
-//   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write)
+//   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write), or, for
+//              weight rows in blocks of [4 gate | 4 up], the clamped gated unit of the pairs in bf16 (half as many columns)
 // The rows are the M side (16) of mma.sync.m16n8k16 and eight weight rows the N side. The order of k inside a product does
 // not matter, so a lane takes eight consecutive k of one weight row as 16 bytes and uses them as the B operands of two MMAs, the
 // matching activations as the A operands. Weights are read once; the first of them are requested before the programmatic
@@ -30,6 +31,7 @@ struct RowsArgs {
   float* h; long ldh; const float* scale;
   const float* head; long ldhead; int k0;     // prologue 2: the first k0 columns of x, as they are
   int silu;                         // prologue 2: activation of the gate
+  int glu; float glu_alpha, glu_limit;
   int streams; const float* hmix;   // streams > 0: h [M][streams][N], scale [streams]
   int pitch;                        // bytes per activation row in shared memory (prologue forms)
 };
@@ -269,11 +271,17 @@ __global__ void __launch_bounds__(256) gemv_ring_kernel(const RowsArgs a) {
     } else {
       asm volatile("bar.sync %0, 256;" ::"r"(bar) : "memory");
       const int n0 = (blockIdx.x + done * gridDim.x) * 8;
-      for (int i = lane; i < a.M * 8; i += 32) {
-        if (n0 + (i & 7) < a.N) {
-          float v = 0.f;
+      for (int i0 = 0; i0 < a.M * 8; i0 += 32) {
+        const int i = i0 + lane;
+        const bool in = i < a.M * 8 && n0 + (i & 7) < a.N;
+        float v = 0.f;
+        if (in)
 #pragma unroll
           for (int y = 0; y < 8; ++y) v += (&part[buf][y][0][0])[i];
+        if (a.glu) {                                      // lanes e and e + 4 of a row hold a pair
+          const float u = __shfl_down_sync(0xffffffffu, v, 4);
+          if (in && (i & 7) < 4) a.out[(i >> 3) * a.ldo + n0 / 2 + (i & 3)] = f2bf(clamped_glu_of(v, u, a.glu_alpha, a.glu_limit));
+        } else if (in) {
           rows_out(a, i >> 3, n0 + (i & 7), v);
         }
       }
@@ -451,16 +459,18 @@ extern "C" {
 
 // pro 0: x bf16 [M, K], M <= 16. pro 1..5: x fp32, M <= 8 and the activation rows (kx columns) fit in shared memory (else refused).
 // pro 2 with k0 > 0: columns [0, k0) from head, the norm's columns behind them. pro 4: G streams of kx columns weighted by coef.
-// pro 5: 2 kx columns, alpha and (in eps) the limit. Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
+// pro 5: 2 kx columns, alpha and (in eps) the limit. glu: out bf16 [M][N / 2] (N a multiple of 8). Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
 // with hmix [streams][streams] and scale [streams].
 int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, const void* x, long ldx, const void* w, const void* b, float alpha, int G,
                  int wlen, const void* gate, long ldg, const void* coef, float eps, void* out_f32, void* out, long ldo, void* h, long ldh, const void* scale,
-                 const void* head, long ldhead, int k0, int silu, int streams, const void* hmix, cudaStream_t st) {
+                 const void* head, long ldhead, int k0, int silu, int glu, float glu_alpha, float glu_limit, int streams, const void* hmix,
+                 cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 5) return cudaErrorInvalidValue;
   RowsArgs a{(const __nv_bfloat16*)W, ldw, N, K, M, pro, kx, x, ldx, (const float*)w, (const float*)b, alpha, G, wlen, (const float*)gate, ldg,
              (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale,
-             (const float*)head, ldhead, k0, silu, streams, (const float*)hmix, 0};
+             (const float*)head, ldhead, k0, silu, glu, glu_alpha, glu_limit, streams, (const float*)hmix, 0};
+  if (glu && (!out || N % 8 || (long)M * ((K + 31) / 32 * 64 + 64) > 100 * 1024)) return cudaErrorInvalidValue;
   if (streams < 0 || streams > kMaxStreams || (streams && (!h || !hmix || !scale))) return cudaErrorInvalidValue;
   const int K32 = (K + 31) / 32 * 32;
   a.pitch = K32 * 2 + ((K32 * 2) % 128 == 0 ? 64 : 0);            // rows of a quad pair land in different halves of the banks

@@ -275,33 +275,43 @@ __global__ void __launch_bounds__(256) stream_norm4_kernel(float* __restrict__ h
   }
 }
 
-// z [rows][2 F]: gates, then ups.
+// z [rows][2 F]: gates, then ups (blk 0), or blocks of [4 gates | 4 ups].
 template <typename X, typename T>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, float alpha, float limit) {
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, int blk, float alpha,
+                                                          float limit) {
   grid_dep_wait();
   grid_dep_launch();
   for (long q = blockIdx.x * 256l + threadIdx.x; q < total; q += gridDim.x * 256l) {
     const long row = q / F;
-    const int i = (int)(q - row * F);
-    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + i]), to_f(z[row * ldz + F + i]), alpha, limit));
+    const int i = (int)(q - row * F), g = blk ? (i >> 2) * 8 + (i & 3) : i, u = blk ? g + 4 : F + i;
+    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + g]), to_f(z[row * ldz + u]), alpha, limit));
   }
 }
+VE_DEVINL __nv_bfloat162 clamped_glu2(__nv_bfloat162 g, __nv_bfloat162 u, float alpha, float limit) {
+  const float2 a = __bfloat1622float2(g), b = __bfloat1622float2(u);
+  return __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, alpha, limit), clamped_glu_of(a.y, b.y, alpha, limit));
+}
 __global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* __restrict__ z, long ldz, __nv_bfloat16* __restrict__ out, long ldo, long total8,
-                                                           int F, float alpha, float limit) {
+                                                           int F, int blk, float alpha, float limit) {
   grid_dep_wait();
   grid_dep_launch();
   const int f8 = F >> 3;
   for (long q = blockIdx.x * 256l + threadIdx.x; q < total8; q += gridDim.x * 256l) {
     const long row = q / f8;
     const int i = (int)(q - row * f8) * 8;
-    bf16x8 g = *reinterpret_cast<const bf16x8*>(z + row * ldz + i);
-    const bf16x8 u = *reinterpret_cast<const bf16x8*>(z + row * ldz + F + i);
+    const __nv_bfloat16* zr = z + row * ldz;
+    const bf16x8 a = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i : i)), b = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i + 8 : F + i));
+    bf16x8 o;
+    if (blk) {
+      o.v[0] = clamped_glu2(a.v[0], a.v[2], alpha, limit);
+      o.v[1] = clamped_glu2(a.v[1], a.v[3], alpha, limit);
+      o.v[2] = clamped_glu2(b.v[0], b.v[2], alpha, limit);
+      o.v[3] = clamped_glu2(b.v[1], b.v[3], alpha, limit);
+    } else {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float2 a = __bfloat1622float2(g.v[e]), b = __bfloat1622float2(u.v[e]);
-      g.v[e] = __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, alpha, limit), clamped_glu_of(a.y, b.y, alpha, limit));
+      for (int e = 0; e < 4; ++e) o.v[e] = clamped_glu2(a.v[e], b.v[e], alpha, limit);
     }
-    *reinterpret_cast<bf16x8*>(out + row * ldo + i) = g;
+    *reinterpret_cast<bf16x8*>(out + row * ldo + i) = o;
   }
 }
 
@@ -409,18 +419,18 @@ int ve_stream_norm(void* h, const void* part, long ldp, const void* mix, const v
   VE_CHECK_LAUNCH();
 }
 
-// z rows [gate F | up F], fp32 when x32, else of the activation type.
-int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, float alpha, float limit, int f32, cudaStream_t st) {
+// z rows [gate F | up F] (blk 0) or blocks of [4 gate | 4 up] (F a multiple of 4); fp32 when x32, else of the activation type.
+int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, int blk, float alpha, float limit, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (F < 1) return cudaErrorInvalidValue;
+  if (F < 1 || (blk && F % 4)) return cudaErrorInvalidValue;
   const bool vec = !f32 && !x32 && F % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && !((uintptr_t)z & 15) && !((uintptr_t)out & 15);
   const long total = (long)rows * F / (vec ? 8 : 1), blocks = (total + 255) / 256;
   const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
   if (vec) {
-    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, alpha, limit);
+    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, blk, alpha, limit);
     VE_CHECK_LAUNCH();
   }
-#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, alpha, limit)
+#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, blk, alpha, limit)
   if (f32) VE_CG(float, float);
   else if (x32) VE_CG(float, __nv_bfloat16);
   else VE_CG(__nv_bfloat16, __nv_bfloat16);

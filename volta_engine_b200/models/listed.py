@@ -8,7 +8,8 @@ slots, batches and the forward pass are here. A layer's parts are row operators 
   norm1, norm2     ``rows(h, dtype, part, write)``: the sublayer result in front enters the residual, then the norm of it;
                    ``prologue(h)``: the norm as the prologue of a decode linear
   write1, write2   how a sublayer's result enters the residual (an element-wise scale, or a StreamWrite)
-  up, act, down    the feed-forward: linear, row operator, linear
+  up, act, down    the feed-forward: linear, row operator, linear; in decode steps the operator is the epilogue of the first linear
+                   (``act.epilogue()``) or the prologue of the second
 """
 from __future__ import annotations
 
@@ -192,8 +193,9 @@ class ListedModel(SlotStates, DenseModel):
         for li, L in enumerate(self.layers):
             L.mixer.step(L.norm1.prologue(h), (h, L.write1), b, kv, self._journal(li, L, b, kv))
             if L.up is not None:
-                z = gemv_rows(L.up, b.n, out_f32=True, **L.norm2.prologue(h))
-                gemv_rows(L.down, b.n, residual=(h, L.write2), **L.act.prologue(z))
+                epi = L.act.epilogue()
+                z = gemv_rows(L.up, b.n, out_f32=epi is None, **L.norm2.prologue(h), **(epi or {}))
+                gemv_rows(L.down, b.n, residual=(h, L.write2), **(L.act.prologue(z) if epi is None else {"x": z}))
             if self.layer_tap is not None:
                 self.layer_tap.append(self.residual_rows(h))
         self.last_residual = h

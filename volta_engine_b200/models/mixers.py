@@ -17,10 +17,12 @@ from ..ops.linear_attn import LinAttnSpec, LinAttnState, linattn_rows
 from ..ops.rowops import GroupRMS, gemv_rows
 
 
-def make_linear(src, names, device, dtype, dim: int = 0):
-    """One linear computing the stacked outputs of the tensors ``names`` (``dim`` 1: the sum of their outputs on stacked inputs)."""
+def make_linear(src, names, device, dtype, dim: int = 0, join=None):
+    """One linear computing the stacked outputs of the tensors ``names`` (``dim`` 1: the sum of their outputs on stacked inputs;
+    ``join``: a function that makes one weight of them)."""
     names = [names] if isinstance(names, str) else names
-    w = torch.cat([src.tensor(n, device, dtype) for n in names], dim) if len(names) > 1 else src.tensor(names[0], device, dtype)
+    parts = [src.tensor(n, device, dtype) for n in names]
+    w = join(*parts) if join is not None else torch.cat(parts, dim) if len(parts) > 1 else parts[0]
     return LinearF32(w) if dtype == torch.float32 else LinearBF16(w)
 
 

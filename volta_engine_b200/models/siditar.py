@@ -53,8 +53,10 @@ class SiditarModel(ListedModel):
         L = ListedLayer(MIXERS[spec["type"]](spec["type"], spec["mixer"], eps, src, p + "mix.", dev, dt), norm(1), write(1))
         if spec.get("mlp") is not None:
             L.norm2, L.write2 = norm(2), write(2)
-            L.up, L.down = make_linear(src, [p + "mlp.gate", p + "mlp.up"], dev, dt), make_linear(src, p + "mlp.down", dev, dt)
-            L.act = ClampedGlu(float(spec["mlp"]["limit"]), GLU_ALPHA)
+            halves = [p + "mlp.gate", p + "mlp.up"]
+            blocks = int(spec["mlp"]["ff"]) % 8 == 0
+            L.up = make_linear(src, halves, dev, dt, join=ClampedGlu.interleave if blocks else None)
+            L.down, L.act = make_linear(src, p + "mlp.down", dev, dt), ClampedGlu(float(spec["mlp"]["limit"]), GLU_ALPHA, blocks)
         return L
 
     def embed_batch(self, b):

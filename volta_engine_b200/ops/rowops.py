@@ -98,26 +98,44 @@ class PolyNorm:
         call("polynorm", "plipplii" + "fi", ptr(z), z.stride(0), _f32(z), ptr(self.coef), ptr(out), out.stride(0), rows, F, float(self.eps), _f32(out))
         return out
 
+    def epilogue(self):
+        return None             # statistics over the whole row
+
     def prologue(self, z):
         return {"pro": 3, "x": z, "coef": self.coef, "eps": self.eps}
 
 
 @dataclass
 class ClampedGlu:
-    """Rows [gate | up]: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up clamped to +-limit."""
+    """Rows [gate | up]: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up clamped to +-limit. ``blocks``: the columns come
+    as blocks of [4 gate | 4 up] (``interleave`` reorders a weight for it), which a decode linear can finish in its epilogue."""
     limit: float
     alpha: float
+    blocks: bool = False
+
+    @staticmethod
+    def interleave(gate, up):
+        """Weights of the two halves [F, K] (F a multiple of 4) -> one weight whose outputs are in blocks."""
+        F, K = gate.shape
+        return torch.stack([gate.reshape(F // 4, 4, K), up.reshape(F // 4, 4, K)], 1).reshape(2 * F, K)
 
     def rows(self, z, out_dtype):
         rows, F = z.shape[0], z.shape[1] // 2
         if not z.is_cuda:
-            g, u = z[:, :F].float().clamp(max=self.limit), z[:, F:].float().clamp(-self.limit, self.limit)
+            v = z.float().reshape(rows, F // 4, 2, 4).transpose(1, 2).reshape(rows, 2 * F) if self.blocks else z.float()
+            g, u = v[:, :F].clamp(max=self.limit), v[:, F:].clamp(-self.limit, self.limit)
             return (g * torch.sigmoid(self.alpha * g) * (u + 1.0)).to(out_dtype)
         out = torch.empty(rows, F, dtype=out_dtype, device=z.device)
-        call("clamped_glu", "plipliiffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, float(self.alpha), float(self.limit), _f32(out))
+        call("clamped_glu", "plipliiiffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, int(self.blocks), float(self.alpha), float(self.limit),
+             _f32(out))
         return out
 
+    def epilogue(self):
+        """Operands of a decode linear that ends with this operator; None: it goes into the prologue of the next one."""
+        return {"glu": (self.alpha, self.limit)} if self.blocks else None
+
     def prologue(self, z):
+        assert not self.blocks
         return {"pro": 5, "x": z, "kx": z.shape[1] // 2, "alpha": self.alpha, "eps": self.limit}
 
 
@@ -195,8 +213,9 @@ def fused_fits(lin, rows: int) -> bool:
 
 
 def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, head=None, silu=False,
-              out_f32=False, residual=None):
+              glu=None, out_f32=False, residual=None):
     """A bf16 linear on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
+    ``glu`` = (alpha, limit): the clamped gated unit of its outputs, which come in blocks, in bf16.
     ``residual`` = (h fp32, scale | None): h += scale * y in place, (streams, StreamWrite): the streams rewritten in place; otherwise
     the product is returned."""
     W = lin.weight
@@ -207,13 +226,14 @@ def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wl
     k0 = head.shape[1] if head is not None else 0
     out = None
     if residual is None:
-        out = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=dev)
+        N_out = N // 2 if glu else N
+        out = torch.empty(M, N_out, dtype=torch.float32 if out_f32 else torch.bfloat16, device=dev)
     h, scale = residual if residual is not None else (None, None)
     streams, mix = 0, None
     if isinstance(scale, StreamWrite):
         streams, mix, scale = h.shape[1], scale.mix, scale.out
-    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiip", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
+    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiiffip", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
          float(alpha), G, wlen, ptr(gate), gate.stride(0) if gate is not None else 0, ptr(coef), float(eps),
-         ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, N, ptr(h), h.stride(0) if h is not None else 0, ptr(scale),
-         ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), streams, ptr(mix))
+         ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, out.stride(0) if out is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(scale),
+         ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), int(glu is not None), *(map(float, glu or (0.0, 0.0))), streams, ptr(mix))
     return out

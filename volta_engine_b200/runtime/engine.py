@@ -8,8 +8,9 @@ never depends on host arguments; attention grids are position independent.
 """
 from __future__ import annotations
 
+import contextlib
+import gc
 import os
-
 import time
 from dataclasses import dataclass
 
@@ -34,6 +35,19 @@ class GenStats:
     @property
     def decode_tok_s(self):
         return self.new_tokens / (self.decode_ms / 1e3) if self.decode_ms > 0 else 0.0
+
+
+@contextlib.contextmanager
+def no_collection():
+    """Keep the garbage collector out of a capture: a graph of an engine that is gone would be destroyed inside it, which ends the
+    capture with an error."""
+    on = gc.isenabled()
+    gc.disable()
+    try:
+        yield
+    finally:
+        if on:
+            gc.enable()
 
 
 class _Graph:
@@ -179,7 +193,7 @@ class Engine:
         else:
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
+            with no_collection(), torch.cuda.graph(graph):
                 g.logits = self._forward_static(rows, nsplit, topk)
             g.graph = graph
             graph.replay()

@@ -13,6 +13,7 @@ import torch
 
 from ..ops import kernels as K
 from .batch import BatchRows, LOGITS_ALL, MAX_GRAPH_ROWS
+from .engine import no_collection
 
 
 class MtpRunner:
@@ -170,7 +171,7 @@ class MtpRunner:
         else:
             torch.cuda.synchronize()
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
+            with no_collection(), torch.cuda.graph(g):
                 self._round_body(st, k, d)
             st["graph"] = g
             g.replay()

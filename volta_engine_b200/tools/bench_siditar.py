@@ -138,7 +138,7 @@ def run_kernels(width: int, dev) -> dict:
                 kb.add(f"linear prompt ({nm})", who, lambda: lin.forward(xi, out_f32=f32), lin.nbytes() + n * (lin.in_features * 2 + lin.out_features * (4 if f32 else 2)),
                        2.0 * n * lin.in_features * lin.out_features)
         else:
-            z, zo = torch.randn(1, L.up.out_features, device=dev), torch.randn(1, O[0].up.out_features, device=dev)
+            z, zo = torch.randn(1, L.down.in_features, device=dev).to(bf), torch.randn(1, O[0].up.out_features, device=dev)
             att, o = torch.randn(1, D, device=dev), torch.randn(1, D, device=dev)
             om = O[1].mixer
             po = torch.randn(1, om.in_proj.out_features, device=dev)
@@ -148,9 +148,9 @@ def run_kernels(width: int, dev) -> dict:
                                                                                             **mx.right.norm.prologue(o, mx.right.gate(pr), head=att)), mx.out.nbytes(), 0)
             kb.add("linear decode: output norm + out + residual", "fofosun", lambda: gemv_rows(om.out, 1, residual=(ho, O[1].write1),
                                                                                             **om.norm.prologue(o, om.gate(po))), om.out.nbytes(), 0)
-            kb.add("linear decode: norm + gate and up", "siditar", lambda: gemv_rows(L.up, 1, out_f32=True, **L.norm2.prologue(h)), L.up.nbytes(), 0)
+            kb.add("linear decode: norm + gate and up + activation", "siditar", lambda: gemv_rows(L.up, 1, **L.norm2.prologue(h), **L.act.epilogue()), L.up.nbytes(), 0)
             kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(O[0].up, 1, out_f32=True, **O[0].norm2.prologue(ho)), O[0].up.nbytes(), 0)
-            kb.add("linear decode: activation + down + residual", "siditar", lambda: gemv_rows(L.down, 1, residual=(h, L.write2), **L.act.prologue(z)), L.down.nbytes(), 0)
+            kb.add("linear decode: down + residual", "siditar", lambda: gemv_rows(L.down, 1, residual=(h, L.write2), x=z), L.down.nbytes(), 0)
             kb.add("linear decode: activation + down + residual", "fofosun", lambda: gemv_rows(O[0].down, 1, residual=(ho, O[0].write2), **O[0].act.prologue(zo)),
                    O[0].down.nbytes(), 0)
     return {"width": width, "prompt_rows": T, "context": ctx, "peaks": kb.pk, "kernels": kb.rows}
