@@ -139,8 +139,9 @@ def test_server_on_a_model_directory(tmp_path):
     from volta_engine_b200.server import cli
     write_model(tmp_path, NAME)
     write_tokenizer(tmp_path, CONFIGS[NAME]["vocab"])
-    cfg, _ = cli.resolve_config(["--model-dir", str(tmp_path), "--set", "max_slots=2", "--set", "max_seq=512", "--set", "kv_pool=1024", "--set", "dtype=fp32"], env={})
+    cfg, _ = cli.resolve_config(["--model-dir", str(tmp_path), "--port", "0", "--set", "max_slots=2", "--set", "max_seq=512", "--set", "kv_pool=1024", "--set", "dtype=fp32"], env={})
     srv, gen, eng = cli.build_server(cfg, "cpu")
     assert type(eng.model).__name__ == "FofosunModel" and eng.kv.k.dtype == torch.float32 and gen.mixed
     p = gen.tok.encode("a prompt")
     assert gen.generate(Request(list(p), max_tokens=6, ignore_eos=True))["tokens"] == greedy(p, 6)
+    srv.http.stop()

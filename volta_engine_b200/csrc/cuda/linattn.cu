@@ -513,6 +513,7 @@ __global__ void __launch_bounds__(128) linattn_decay_kernel(const X* __restrict_
   __syncthreads();
   if (c >= C) return;
   const float b = bias[c];
+#pragma unroll 4
   for (int y = 0; y < n; ++y) {
     float z = b, z1 = 0.f, z2 = 0.f, z3 = 0.f;
     if (RK) {
