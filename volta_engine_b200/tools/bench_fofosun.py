@@ -210,7 +210,7 @@ def run_kernels(width: int, dev) -> dict:
         h, x = torch.randn(n, width, device=dev), torch.randn(n, width, device=dev).to(bf)
         ly = mine.layers[0]
         if n > 1:
-            kb.add("add + norm prompt", "fofosun (fp32 residual)", lambda: ly.norm1.rows(h, bf, x, ly.ls1), n * width * 12, 0)
+            kb.add("add + norm prompt", "fofosun (fp32 residual)", lambda: ly.norm1.rows(h, bf, x, ly.write1), n * width * 12, 0)
             hb = h.to(bf)
             kb.add("add + norm prompt", "glm5 assembly", lambda: K.rmsnorm(x, L.attn_norm, 1e-5, 1.0, residual=hb), n * width * 8, 0)
             z = torch.randn(n, width * 6, device=dev).to(bf)
@@ -229,7 +229,7 @@ def run_kernels(width: int, dev) -> dict:
         else:
             z = torch.randn(1, width * 6, device=dev)
             kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(ly.up, 1, out_f32=True, **ly.norm2.prologue(h)), ly.up.nbytes(), 0)
-            kb.add("linear decode: activation + down + add", "fofosun", lambda: gemv_rows(ly.down, 1, residual=(h, ly.ls2), **ly.act.prologue(z)), ly.down.nbytes(), 0)
+            kb.add("linear decode: activation + down + add", "fofosun", lambda: gemv_rows(ly.down, 1, residual=(h, ly.write2), **ly.act.prologue(z)), ly.down.nbytes(), 0)
             kb.add("linear decode: in projection", "fofosun", lambda: gemv_rows(ly.mixer.in_proj, 1, out_f32=True, **ly.norm1.prologue(h)), ly.mixer.in_proj.nbytes(), 0)
             gul = other.layers[0].gate_up
             kb.add("linear decode: gate and up", "glm5 assembly (bf16)", lambda: gul.forward(x), gul.nbytes(), 0)
