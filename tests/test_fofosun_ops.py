@@ -366,12 +366,9 @@ def test_rotation_is_exact_at_far_positions(device):
     r.kv.k[1, 0].zero_()
     r.kv.k[1, 0, :, :, :16] = 0
     if device == "cpu":
-        a = base
-        from volta_engine_b200.ops.latent import _rotate
-        ang0 = torch.arange(6).double()[:, None] * spec.freq
-        ang1 = (torch.arange(6) + a).double()[:, None] * spec.freq
-        s0 = _rotate(q[:, 8:], ang0) @ _rotate(kv[:, 16:], ang0).t()
-        s1 = _rotate(q[:, 8:], ang1) @ _rotate(kv[:, 16:], ang1).t()
+        at = torch.arange(6)
+        s0 = spec.turn.turn(q[:, 8:], at) @ spec.turn.turn(kv[:, 16:], at).t()
+        s1 = spec.turn.turn(q[:, 8:], at + base) @ spec.turn.turn(kv[:, 16:], at + base).t()
         assert (s0 - s1).abs().max() < 1e-5
         return
     from volta_engine_b200._lib import call, ptr
@@ -382,8 +379,8 @@ def test_rotation_is_exact_at_far_positions(device):
         slot = torch.full((6,), 1, dtype=torch.int32, device="cuda")
         qo, kvd = torch.empty(6, 16, device="cuda"), kv.cuda()
         qd = q.cuda()
-        call("latent_rope_store", "iiiiiiii" + "plplpli" + "pp" + "pppip" + "ifi", *D, ptr(qd), 16, ptr(qo), 16, ptr(kvd), 24, 1, ptr(r.norm), ptr(spec.freq),
-             ptr(pos), ptr(slot), ptr(r.kv.page_table), r.kv.page_table.shape[1], ptr(r.kv.k[1]), 6, 1e-5, 1)
+        call("latent_rope_store", "iiiiiiii" + "plplplii" + "ppf" + "pppip" + "ifi", *D, ptr(qd), 16, ptr(qo), 16, ptr(kvd), 24, 1, 1, ptr(r.norm),
+             ptr(spec.turn.half_turns), 1.0, ptr(pos), ptr(slot), ptr(r.kv.page_table), r.kv.page_table.shape[1], ptr(r.kv.k[1]), 6, 1e-5, 1)
         page = 7 if p0 else 0
         off = p0 % 64
         qs.append(qo[:, 8:].cpu() @ r.kv.k[1, page, 0, off:off + 6, 16:24].cpu().t())

@@ -7,7 +7,8 @@
 //              3  x = PolyNorm of an fp32 row
 //              4  x = layer norm (no shift) of the weighted sum of the fp32 residual streams
 //              5  x = clamped gated unit of an fp32 [gate | up] row
-//   epilogue   store fp32 or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write), or, for
+//              6  x = h + RMS norm of a sublayer's result (fp32, optional), as it is or RMS normed; the sum is also stored
+//   epilogue   store fp32 (with a soft cap or without) or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write), or, for
 //              weight rows in blocks of [4 gate | 4 up], the clamped gated unit of the pairs in bf16 (half as many columns)
 // The rows are the M side (16) of mma.sync.m16n8k16 and eight weight rows the N side. The order of k inside a product does
 // not matter, so a lane takes eight consecutive k of one weight row as 16 bytes and uses them as the B operands of two MMAs, the
@@ -31,7 +32,10 @@ struct RowsArgs {
   float* h; long ldh; const float* scale;
   const float* head; long ldhead; int k0;     // prologue 2: the first k0 columns of x, as they are
   int silu;                         // prologue 2: activation of the gate
-  int glu; float glu_alpha, glu_limit;
+  int glu; Glu unit;                // epilogue (and prologue 5)
+  float cap;                        // > 0: soft cap of the fp32 output
+  const float* part; long ldpart; float* h_out;          // prologue 6: w normalises part, b the sum (null: none); h_out [M][kx]
+  int v4;                           // prologue 6: four columns at a time
   int streams; const float* hmix;   // streams > 0: h [M][streams][N], scale [streams]
   int pitch;                        // bytes per activation row in shared memory (prologue forms)
 };
@@ -53,8 +57,97 @@ VE_DEVINL void rows_out(const RowsArgs& a, int m, int n, float v) {
     for (int s = 0; s < kMaxStreams; ++s)
       if (s < a.streams) hp[(long)s * a.N] = x[s];
   } else if (a.h) a.h[m * a.ldh + n] = fmaf(v, a.scale ? a.scale[n] : 1.f, a.h[m * a.ldh + n]);
-  else if (a.out_f32) a.out_f32[m * a.ldo + n] = v;
+  else if (a.out_f32) a.out_f32[m * a.ldo + n] = a.cap > 0.f ? soft_cap_of(v, a.cap) : v;
   else a.out[m * a.ldo + n] = f2bf(v);
+}
+
+template <int V> struct Cols;
+template <> struct Cols<1> {
+  float v[1];
+  VE_DEVINL void load(const float* p) { v[0] = *p; }
+  VE_DEVINL void store(float* p) const { *p = v[0]; }
+  VE_DEVINL void store(__nv_bfloat16* p) const { *p = f2bf(v[0]); }
+};
+template <> struct Cols<4> {
+  float v[4];
+  VE_DEVINL void load(const float* p) {
+    const float4 t = load4(p);
+    v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+  }
+  VE_DEVINL void store(float* p) const { store4(p, make_float4(v[0], v[1], v[2], v[3])); }
+  VE_DEVINL void store(__nv_bfloat16* p) const { store4(p, make_float4(v[0], v[1], v[2], v[3])); }
+};
+
+// Prologue 6: one exchange between the warps for all rows and norm. The first CTA stores the sum.
+template <int V>
+VE_DEVINL void residual_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const float* h = reinterpret_cast<const float*>(a.x);
+  auto gather = [&](float s, int m, float* r) {
+    s = warp_sum(s);
+    if (lane == 0) r[m * 8 + warp] = s;
+  };
+  auto over = [&](int m, const float* r) {
+    float s = 0.f;
+#pragma unroll
+    for (int y = 0; y < 8; ++y) s += r[m * 8 + y];
+    return 1.f / sqrtf(s / (float)a.kx + a.eps);
+  };
+  auto sum = [&](int m, int i, float inv, Cols<V>& x) {
+    x.load(h + m * a.ldx + i);
+    if (!a.part) return;
+    Cols<V> y, w;
+    y.load(a.part + m * a.ldpart + i);
+    w.load(a.w + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x.v[e] = fmaf(y.v[e] * inv, w.v[e], x.v[e]);
+  };
+  if (a.part) {
+    for (int m = 0; m < a.M; ++m) {
+      float s = 0.f;
+#pragma unroll 4
+      for (int i = tid * V; i < a.kx; i += 256 * V) {
+        Cols<V> y;
+        y.load(a.part + m * a.ldpart + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s = fmaf(y.v[e], y.v[e], s);
+      }
+      gather(s, m, red);
+    }
+    __syncthreads();
+  }
+  if (a.b) {
+    for (int m = 0; m < a.M; ++m) {
+      const float inv = a.part ? over(m, red) : 0.f;
+      float s = 0.f;
+#pragma unroll 4
+      for (int i = tid * V; i < a.kx; i += 256 * V) {
+        Cols<V> x;
+        sum(m, i, inv, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s = fmaf(x.v[e], x.v[e], s);
+      }
+      gather(s, m, red + 64);
+    }
+    __syncthreads();
+  }
+  for (int m = 0; m < a.M; ++m) {
+    const float inv = a.part ? over(m, red) : 0.f, inv2 = a.b ? over(m, red + 64) : 1.f;
+    __nv_bfloat16* xr = reinterpret_cast<__nv_bfloat16*>(xs + m * a.pitch);
+#pragma unroll 4
+    for (int i = tid * V; i < a.kx; i += 256 * V) {
+      Cols<V> x;
+      sum(m, i, inv, x);
+      if (a.h_out && blockIdx.x == 0) x.store(a.h_out + (long)m * a.kx + i);
+      if (a.b) {
+        Cols<V> w;
+        w.load(a.b + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x.v[e] *= inv2 * w.v[e];
+      }
+      x.store(xr + i);
+    }
+  }
 }
 
 // Activations of the prologue forms -> bf16 rows in shared memory.
@@ -148,7 +241,10 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
     }
   } else if (a.pro == 5) {
     for (int m = 0; m < a.M; ++m)
-      for (int i = tid; i < a.kx; i += 256) put(m, i, clamped_glu_of(src[m * a.ldx + i], src[m * a.ldx + a.kx + i], a.alpha, a.eps));
+      for (int i = tid; i < a.kx; i += 256) put(m, i, clamped_glu_of(src[m * a.ldx + i], src[m * a.ldx + a.kx + i], a.unit));
+  } else if (a.pro == 6) {
+    if (a.v4) residual_prologue<4>(a, xs, red);
+    else residual_prologue<1>(a, xs, red);
   } else {
     for (int m = 0; m < a.M; ++m) {
       float s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -182,7 +278,7 @@ VE_DEVINL void rows_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
 // own in shared memory (cp.async, groups of four units, DEPTH groups), so no barrier stands between the copies and their use and
 // nothing waits in order for younger loads. The first groups are requested before the dependency wait. HI: more than eight rows.
 template <int DEPTH, bool HI>
-__global__ void __launch_bounds__(256) gemv_ring_kernel(const RowsArgs a) {
+__global__ void __launch_bounds__(256, 2) gemv_ring_kernel(const RowsArgs a) {
   constexpr int U = 4, GROUP = 8 * U * 512;               // bytes of one group of all warps
   extern __shared__ __align__(16) uint8_t xs[];           // [M][pitch] activations, then [DEPTH][8 warps][U][32 lanes][16 B]
   __shared__ float part[8][8][HI ? 16 : 8][8], red[4][33];
@@ -280,7 +376,7 @@ __global__ void __launch_bounds__(256) gemv_ring_kernel(const RowsArgs a) {
           for (int y = 0; y < 8; ++y) v += (&part[buf][y][0][0])[i];
         if (a.glu) {                                      // lanes e and e + 4 of a row hold a pair
           const float u = __shfl_down_sync(0xffffffffu, v, 4);
-          if (in && (i & 7) < 4) a.out[(i >> 3) * a.ldo + n0 / 2 + (i & 3)] = f2bf(clamped_glu_of(v, u, a.glu_alpha, a.glu_limit));
+          if (in && (i & 7) < 4) a.out[(i >> 3) * a.ldo + n0 / 2 + (i & 3)] = f2bf(clamped_glu_of(v, u, a.unit));
         } else if (in) {
           rows_out(a, i >> 3, n0 + (i & 7), v);
         }
@@ -457,19 +553,22 @@ using namespace ve;
 
 extern "C" {
 
-// pro 0: x bf16 [M, K], M <= 16. pro 1..5: x fp32, M <= 8 and the activation rows (kx columns) fit in shared memory (else refused).
+// pro 0: x bf16 [M, K], M <= 16. pro 1..6: x fp32, M <= 8 and the activation rows (kx columns) fit in shared memory (else refused).
 // pro 2 with k0 > 0: columns [0, k0) from head, the norm's columns behind them. pro 4: G streams of kx columns weighted by coef.
-// pro 5: 2 kx columns, alpha and (in eps) the limit. glu: out bf16 [M][N / 2] (N a multiple of 8). Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
+// pro 5: 2 kx columns, glu_alpha, glu_limit and glu_shift. pro 6: part fp32 (null: none) normed with w, the sum with b (null: not), stored to
+// h_out [M][kx] (null: not). cap > 0: soft cap of out_f32. glu: out bf16 [M][N / 2] (N a multiple of 8). Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
 // with hmix [streams][streams] and scale [streams].
 int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, const void* x, long ldx, const void* w, const void* b, float alpha, int G,
                  int wlen, const void* gate, long ldg, const void* coef, float eps, void* out_f32, void* out, long ldo, void* h, long ldh, const void* scale,
-                 const void* head, long ldhead, int k0, int silu, int glu, float glu_alpha, float glu_limit, int streams, const void* hmix,
-                 cudaStream_t st) {
+                 const void* head, long ldhead, int k0, int silu, int glu, float glu_alpha, float glu_limit, float glu_shift, int streams, const void* hmix,
+                 float cap, const void* part, long ldpart, void* h_out, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
-  if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 5) return cudaErrorInvalidValue;
+  if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 6) return cudaErrorInvalidValue;
   RowsArgs a{(const __nv_bfloat16*)W, ldw, N, K, M, pro, kx, x, ldx, (const float*)w, (const float*)b, alpha, G, wlen, (const float*)gate, ldg,
              (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale,
-             (const float*)head, ldhead, k0, silu, glu, glu_alpha, glu_limit, streams, (const float*)hmix, 0};
+             (const float*)head, ldhead, k0, silu, glu, Glu{glu_alpha, glu_limit, glu_shift}, cap, (const float*)part, ldpart, (float*)h_out,
+             kx % 4 == 0 && ldx % 4 == 0 && ldpart % 4 == 0 && !(((uintptr_t)x | (uintptr_t)part | (uintptr_t)w | (uintptr_t)b | (uintptr_t)h_out) & 15),
+             streams, (const float*)hmix, 0};
   if (glu && (!out || N % 8 || (long)M * ((K + 31) / 32 * 64 + 64) > 100 * 1024)) return cudaErrorInvalidValue;
   if (streams < 0 || streams > kMaxStreams || (streams && (!h || !hmix || !scale))) return cudaErrorInvalidValue;
   const int K32 = (K + 31) / 32 * 32;
@@ -477,7 +576,7 @@ int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, 
   if (pro) {
     if (M > 8 || (long)M * a.pitch > 100 * 1024) return cudaErrorInvalidValue;
     if ((pro == 1 && (!w || !b || h)) || (pro == 2 && (!w || G < 1 || k0 < 0 || k0 > kx || (kx - k0) % G || wlen < 1 || (k0 && !head))) ||
-        (pro == 3 && !coef) || (pro == 4 && (!w || !coef || G < 1 || G > kMaxStreams || h))) return cudaErrorInvalidValue;
+        (pro == 3 && !coef) || (pro == 6 && part && !w) || (pro == 4 && (!w || !coef || G < 1 || G > kMaxStreams || h))) return cudaErrorInvalidValue;
   } else if (kx != K || ldx % 8 || ((uintptr_t)x & 15)) {
     return cudaErrorInvalidValue;
   }

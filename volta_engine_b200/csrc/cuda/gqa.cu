@@ -1,10 +1,11 @@
 // Grouped-query softmax attention with its sizes and its score terms as parameters: query / key width and value width may differ and
-// need not be powers of two; optional RMS norm of queries and keys, query temperature by position, bias by distance (a table per
-// head whose last entry holds for everything farther), a sink (one more term of the denominator), a factor on the result.
+// need not be powers of two; optional rotary positions, then RMS norm (with or without a weight) of queries and keys, query temperature
+// by position, sliding window, bias by distance (a table per head whose last entry holds for everything farther), a sink (one more term
+// of the denominator), a factor on the result, a sigmoid gate on every element of it.
 //
 // Cache: a page of the pool is 64 tokens x row width; this layer sees it as [kv heads][64][kw] (values [kv heads][64][vw]) with kw, vw the
 // widths rounded up to 8 elements (pad columns are zero), so layers of unlike sizes share one pool.
-//   gqa_store    norms, temperature, queries as rows [heads][kw], keys and values into the cache
+//   gqa_store    rotation, norms, temperature, queries as rows [heads][kw], keys and values into the cache
 //   gqa_rows     one CTA per (row, head) on the CUDA cores: the all-32-bit form, and sizes outside the range of the others
 //   gqa_decode   decode rows: 16 query heads of a kv head x 64-key pages (TMA) on mma.sync, key splits over the grid, the split
 //                that ends last merges
@@ -13,6 +14,7 @@
 #include "rowmath.cuh"
 #include "tmap.h"
 #include <float.h>
+#include <limits.h>
 
 namespace ve {
 
@@ -29,7 +31,21 @@ struct GqaScore {
   const float* bias; int L;       // [H][L] by distance, entry L - 1 for everything from L - 1 on (null: none)
   const float* sink;              // [H] (null: none)
   float out_scale;
+  int window;                     // keys at distances below it are seen (INT_MAX: all in front)
+  const void* gate; long ldg;     // [rows][H dv] (null: none), fp32 (gate32) or bf16
+  int gate32, gatev;              // gatev: eight columns from a multiple of eight on are 16-byte aligned
 };
+struct GqaTurn {
+  const double* freq;             // half turns per position
+  int pairs;                      // 0: no rotation
+  float mul;
+  int neighbours;                 // pairs are columns (2 i, 2 i + 1), else (i, i + pairs)
+};
+VE_DEVINL float gate_at(const GqaScore& sc, long row, int c) {
+  if (!sc.gate) return 1.f;
+  const long at = row * sc.ldg + c;
+  return sigmoid_of(sc.gate32 ? reinterpret_cast<const float*>(sc.gate)[at] : to_f(reinterpret_cast<const __nv_bfloat16*>(sc.gate)[at]));
+}
 struct GqaRows {
   const int* pos; const int* slot; const int* page_table;
   int max_pages;
@@ -37,17 +53,23 @@ struct GqaRows {
 
 VE_DEVINL int page_of(const GqaRows& r, int slot, int kt) { return r.page_table[(long)slot * r.max_pages + kt]; }
 
-// proj row: [q (H d) | k (G d) | v (G dv) | ...]. grid (rows, ceil((H + 2 G) / 8)), a warp per head.
+// proj row: [q (H d) | k (G d) | v (G dv) | ...]. grid (rows, ceil((H + 2 G) / 8)), a warp per head. norm: queries and keys are divided by
+// their root mean square (behind the rotation), times wq / wk where given.
 template <typename X, typename T>
-__global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const GqaRows rw, const X* __restrict__ proj, long ld, const float* __restrict__ wq,
-                                                        const float* __restrict__ wk, float eps, float coef, int every, int vec,
+__global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const GqaRows rw, const X* __restrict__ proj, long ld, const GqaTurn tn, int norm,
+                                                        const float* __restrict__ wq, const float* __restrict__ wk, float eps, float coef, int every, int vec,
                                                         T* __restrict__ qo, T* __restrict__ kpool, T* __restrict__ vpool) {
+  __shared__ __align__(16) float cs[kMaxPairs], sn[kMaxPairs];
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
   const int item = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (item >= n.H + 2 * n.G) return;
   const int p = rw.pos[row], s = rw.slot[row];
+  if (tn.pairs) {
+    angle_row(p, tn.freq, tn.pairs, tn.mul, cs, sn);
+    __syncthreads();
+  }
+  if (item >= n.H + 2 * n.G) return;
   const bool is_q = item < n.H, is_v = item >= n.H + n.G;
   if (s < 0 && !is_q) return;
   const X* src = proj + row * ld + (is_v ? (long)(n.H + n.G) * n.d + (long)(item - n.H - n.G) * n.dv : (long)item * n.d);
@@ -57,8 +79,9 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
     const int page = page_of(rw, s, p / kGPage), at = p % kGPage;
     dst = is_v ? vpool + page * n.vps + ((long)(item - n.H - n.G) * kGPage + at) * n.vw : kpool + page * n.kps + ((long)(item - n.H) * kGPage + at) * n.kw;
   }
-  const int w = is_v ? n.dv : n.d, wide = is_v ? n.vw : n.kw;
+  const int w = is_v ? n.dv : n.d, wide = is_v ? n.vw : n.kw, turned = is_v ? 0 : 2 * tn.pairs;
   const float* wn = is_v ? nullptr : is_q ? wq : wk;
+  const bool nrm = norm && !is_v;
   const float t = is_q && every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
   if (vec) {                                // widths up to 256 in multiples of eight: four columns per lane and step, kept in registers
     float4 v[2];
@@ -67,9 +90,23 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
     for (int j = 0; j < 2; ++j) {
       const int i = (j * 32 + lane) * 4;
       v[j] = i < w ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < turned) {
+        if (tn.neighbours) {
+          const float2 c = *reinterpret_cast<const float2*>(cs + i / 2), z = *reinterpret_cast<const float2*>(sn + i / 2);
+          v[j] = make_float4(fmaf(v[j].x, c.x, -(v[j].y * z.x)), fmaf(v[j].y, c.x, v[j].x * z.x), fmaf(v[j].z, c.y, -(v[j].w * z.y)),
+                             fmaf(v[j].w, c.y, v[j].z * z.y));
+        } else {
+          const bool low = i < tn.pairs;
+          const int k = low ? i : i - tn.pairs;
+          const float4 c = *reinterpret_cast<const float4*>(cs + k), o = load4(src + (low ? i + tn.pairs : k));
+          float4 z = *reinterpret_cast<const float4*>(sn + k);
+          if (low) z = make_float4(-z.x, -z.y, -z.z, -z.w);
+          v[j] = make_float4(fmaf(v[j].x, c.x, o.x * z.x), fmaf(v[j].y, c.y, o.y * z.y), fmaf(v[j].z, c.z, o.z * z.z), fmaf(v[j].w, c.w, o.w * z.w));
+        }
+      }
       ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
     }
-    const float g = wn ? t / sqrtf(warp_sum(ss) / (float)w + eps) : t;
+    const float g = nrm ? t / sqrtf(warp_sum(ss) / (float)w + eps) : t;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int i = (j * 32 + lane) * 4;
@@ -79,11 +116,19 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
     }
     return;
   }
+  auto value = [&](int i) {
+    const float v = to_f(src[i]);
+    if (i >= turned) return v;
+    const bool low = tn.neighbours ? !(i & 1) : i < tn.pairs;
+    const int k = tn.neighbours ? i >> 1 : low ? i : i - tn.pairs, other = tn.neighbours ? i ^ 1 : low ? i + tn.pairs : k;
+    const float o = to_f(src[other]) * sn[k];
+    return fmaf(v, cs[k], low ? -o : o);
+  };
   float f = 1.f;
-  if (wn) {
+  if (nrm) {
     float ss = 0.f;
     for (int i = lane; i < w; i += 32) {
-      const float v = to_f(src[i]);
+      const float v = value(i);
       ss = fmaf(v, v, ss);
     }
     f = 1.f / sqrtf(warp_sum(ss) / (float)w + eps);
@@ -91,7 +136,7 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
   for (int i = lane; i < wide; i += 32) {
     float v = 0.f;
     if (i < w) {
-      v = to_f(src[i]) * f;
+      v = value(i) * f;
       if (wn) v *= wn[i];
       v *= t;
     }
@@ -120,7 +165,7 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const GqaDims n, const Gq
   float acc[NC], m = -FLT_MAX, l = 0.f;
 #pragma unroll
   for (int j = 0; j < NC; ++j) acc[j] = 0.f;
-  for (int key = warp; key <= p; key += 4) {
+  for (int key = max(0, p - sc.window + 1) + warp; key <= p; key += 4) {
     const int page = page_of(rw, s, key / kGPage);
     const T* kr = kpool + page * n.kps + ((long)g * kGPage + key % kGPage) * n.kw;
     const T* vr = vpool + page * n.vps + ((long)g * kGPage + key % kGPage) * n.vw;
@@ -156,7 +201,7 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const GqaDims n, const Gq
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) v += os[w * NC * 32 + i] * f[w];
-    orow[i] = from_f<O>(v / lt * sc.out_scale);
+    orow[i] = from_f<O>(v / lt * sc.out_scale * gate_at(sc, row, h * n.dv + i));
   }
 }
 
@@ -177,11 +222,11 @@ VE_DEVINL uint32_t gq_pack(float lo, float hi) {
 }
 
 template <typename O>
-VE_DEVINL void put_row(O* p, float4 v) {                  // four columns of an output row of any alignment
-  p[0] = from_f<O>(v.x);
-  p[1] = from_f<O>(v.y);
-  p[2] = from_f<O>(v.z);
-  p[3] = from_f<O>(v.w);
+VE_DEVINL void put_row(O* p, float4 v, const GqaScore& sc, long row, int c) {            // four columns (from c on) of an output row of any alignment
+  p[0] = from_f<O>(v.x * gate_at(sc, row, c));
+  p[1] = from_f<O>(v.y * gate_at(sc, row, c + 1));
+  p[2] = from_f<O>(v.z * gate_at(sc, row, c + 2));
+  p[3] = from_f<O>(v.w * gate_at(sc, row, c + 3));
 }
 
 struct GqaDecode {
@@ -220,9 +265,10 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
     return;
   }
   // the grid does not know the position: a row takes as many of its splits as have at least kGMinPages pages
-  const int p = a.rw.pos[row], pages = p / kGPage + 1, per = max(kGMinPages, (pages + a.nsplit - 1) / a.nsplit), used = (pages + per - 1) / per;
+  const int p = a.rw.pos[row], win = a.sc.window, kt0 = max(0, p - win + 1) / kGPage, pages = p / kGPage + 1 - kt0;
+  const int per = max(kGMinPages, (pages + a.nsplit - 1) / a.nsplit), used = (pages + per - 1) / per;
   if (z >= used) return;
-  const int kt_begin = z * per, kt_end = min(pages, kt_begin + per);
+  const int kt_begin = kt0 + z * per, kt_end = min(kt0 + pages, kt_begin + per);
   if (tid == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(&full[i], 1);
     mbar_fence_init();
@@ -294,7 +340,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       for (int e = 0; e < 4; ++e) {
         const int dist = p - (first + nt * 8 + 2 * t + (e & 1)), r = e >> 1;
         const float b = near ? tab[r][min(max(dist, 0), a.sc.L - 1)] * kLog2e : far[r];
-        const float v = dist >= 0 ? fmaf(sa[nt][e], scale2, b) : -FLT_MAX;
+        const float v = (unsigned)dist < (unsigned)win ? fmaf(sa[nt][e], scale2, b) : -FLT_MAX;
         sa[nt][e] = v;
         mx[r] = fmaxf(mx[r], v);
       }
@@ -380,7 +426,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
     if (used == 1) {
       const float snk = sink_of(h0 + hr), top = fmaxf(m, snk), f = exp2f(m - top);
       const float den = fmaf(l, f, a.sc.sink ? exp2f(snk - top) : 0.f);
-      out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * f / den * a.sc.out_scale);
+      out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * f / den * a.sc.out_scale * gate_at(a.sc, row, (h0 + hr) * n.dv + c));
     } else {
       const long at = (row * n.H + h0 + hr) * a.nsplit + z;
       a.o_part[at * n.dv + c] = l > 0.f ? acc / l : 0.f;
@@ -422,7 +468,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
         v = make_float4(fmaf(f, x.x, v.x), fmaf(f, x.y, v.y), fmaf(f, x.z, v.z), fmaf(f, x.w, v.w));
       }
       if (ng > 1) acc4[tid] = v;
-      else put_row(out + row * ldo + (long)(h0 + hr) * n.dv + c, v);
+      else put_row(out + row * ldo + (long)(h0 + hr) * n.dv + c, v, a.sc, row, (h0 + hr) * n.dv + c);
     }
     if (ng > 1) {
       __syncthreads();
@@ -432,7 +478,8 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
           const float4 x = acc4[y * per + tid];
           v = make_float4(v.x + x.x, v.y + x.y, v.z + x.z, v.w + x.w);
         }
-        put_row(out + row * ldo + (long)(h0 + tid / c4) * n.dv + (tid % c4) * 4, v);
+        const int c = (h0 + tid / c4) * n.dv + (tid % c4) * 4;
+        put_row(out + row * ldo + c, v, a.sc, row, c);
       }
     }
   } else {
@@ -442,7 +489,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       float acc = 0.f;
 #pragma unroll 8
       for (int y = 0; y < used; ++y) acc = fmaf(sw[hr * 64 + y], __ldcg(part + (long)y * n.dv), acc);
-      out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc);
+      out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * gate_at(a.sc, row, (h0 + hr) * n.dv + c));
     }
   }
   if (tid == 0) *tk = 0;
@@ -474,8 +521,12 @@ using namespace ve;
 #define VE_GMAKE GqaDims{H, G, d, dv, kw, vw, kps, vps}
 #define VE_GROWS const void* pos, const void* slot, const void* page_table, int max_pages
 #define VE_RMAKE GqaRows{(const int*)pos, (const int*)slot, (const int*)page_table, max_pages}
-#define VE_GSCORE float scale, const void* bias, int L, const void* sink, float out_scale
-#define VE_SMAKE GqaScore{scale, (const float*)bias, L, (const float*)sink, out_scale}
+#define VE_GSCORE float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32
+#define VE_SMAKE gscore(scale, bias, L, sink, out_scale, window, gate, ldg, gate32, dv)
+static GqaScore gscore(float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32, int dv) {
+  return GqaScore{scale, (const float*)bias, L, (const float*)sink, out_scale, window > 0 ? window : INT_MAX, gate, ldg, gate32,
+                  dv % 8 == 0 && ldg % 8 == 0 && !((uintptr_t)gate & 15)};
+}
 static bool gdims_ok(const GqaDims& n) {
   return n.G > 0 && n.H > 0 && n.H % n.G == 0 && n.d > 0 && n.dv > 0 && n.kw >= n.d && n.vw >= n.dv && n.kps >= (long)n.G * 64 * n.kw && n.vps >= (long)n.G * 64 * n.vw;
 }
@@ -487,17 +538,19 @@ static int pool_map(CUtensorMap* m, const void* pool, long pages, const GqaDims&
 
 extern "C" {
 
-// proj rows fp32 when x32 (else bf16); f32: queries and pools fp32 (else bf16). wq, wk null: no norm; every 0: no temperature.
-int ve_gqa_store(VE_GDIMS, VE_GROWS, const void* proj, long ld, int x32, const void* wq, const void* wk, float eps, float coef, int every, void* qo, void* kpool,
-                 void* vpool, int rows, int f32, cudaStream_t st) {
+// proj rows fp32 when x32 (else bf16); f32: queries and pools fp32 (else bf16). pairs 0: no rotation; norm 0: no norm, else wq and wk are its
+// weights (null: none); every 0: no temperature.
+int ve_gqa_store(VE_GDIMS, VE_GROWS, const void* proj, long ld, int x32, const void* freq, int pairs, float mul, int neighbours, int norm, const void* wq,
+                 const void* wk, float eps, float coef, int every, void* qo, void* kpool, void* vpool, int rows, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n)) return cudaErrorInvalidValue;
+  if (!gdims_ok(n) || pairs < 0 || pairs > kMaxPairs || 2 * pairs > d || (pairs && !freq)) return cudaErrorInvalidValue;
   const dim3 grid(rows, (H + 2 * G + 7) / 8);
+  const GqaTurn tn{(const double*)freq, pairs, mul, neighbours};
   const int vec = d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && kw == d && vw == dv && ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)wq & 15) &&
-                  !((uintptr_t)wk & 15);
-#define VE_GS(X, T) launch_pdl(gqa_store_kernel<X, T>, grid, dim3(256), 0, st, n, VE_RMAKE, (const X*)proj, ld, (const float*)wq, (const float*)wk, eps, coef, every, vec, \
-    (T*)qo, (T*)kpool, (T*)vpool)
+                  !((uintptr_t)wk & 15) && pairs % (neighbours ? 2 : 4) == 0;
+#define VE_GS(X, T) launch_pdl(gqa_store_kernel<X, T>, grid, dim3(256), 0, st, n, VE_RMAKE, (const X*)proj, ld, tn, norm, (const float*)wq, (const float*)wk, eps, coef, \
+    every, vec, (T*)qo, (T*)kpool, (T*)vpool)
   if (f32) VE_GS(float, float);
   else if (x32) VE_GS(float, __nv_bfloat16);
   else VE_GS(__nv_bfloat16, __nv_bfloat16);

@@ -7,7 +7,8 @@
 //     the pages' by the tensor map); keys and values have rings of their own (a key page is free as soon as its scores are done);
 //   * a bias by distance is added to the scaled scores: one value per row for pages far enough back, a table look-up otherwise;
 //   * the softmax weights enter the second product as two bf16 terms (value and remainder), so they keep 32-bit quality;
-//   * the sink joins the sums in the epilogue.
+//   * with a sliding window the pages in front of the first token's window are not visited;
+//   * the sink joins the sums in the epilogue, the gate multiplies the result there.
 // Every wait is bounded; on expiry the CTA records a status code, skips its stores and frees its TMEM.
 #pragma once
 
@@ -33,6 +34,30 @@ template <int DQC, int DVC> struct GtStages {
   static constexpr int K = DQC > 3 ? 2 : 4, V = DQC > 3 && DVC > 1 ? 2 : 4;
 };
 
+// Gates of eight columns from c on, of which `live` exist.
+VE_DEVINL void gate8(const GqaScore& sc, long row, int c, int live, float* g) {
+  if (!sc.gate) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = 1.f;
+  } else if (sc.gatev) {
+    const long at = row * sc.ldg + c;
+    float4 x, y;
+    if (sc.gate32) {
+      x = load4(reinterpret_cast<const float*>(sc.gate) + at);
+      y = load4(reinterpret_cast<const float*>(sc.gate) + at + 4);
+    } else {
+      const uint4 v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(sc.gate) + at);
+      x = make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+      y = make_float4(__uint_as_float(v.z << 16), __uint_as_float(v.z & 0xffff0000u), __uint_as_float(v.w << 16), __uint_as_float(v.w & 0xffff0000u));
+    }
+    g[0] = sigmoid_of(x.x); g[1] = sigmoid_of(x.y); g[2] = sigmoid_of(x.z); g[3] = sigmoid_of(x.w);
+    g[4] = sigmoid_of(y.x); g[5] = sigmoid_of(y.y); g[6] = sigmoid_of(y.z); g[7] = sigmoid_of(y.w);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = e < live ? gate_at(sc, row, c + e) : 0.f;
+  }
+}
+
 template <int DQC, int DVC>
 __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc p, const __grid_constant__ CUtensorMap kmap,
                                                                     const __grid_constant__ CUtensorMap vmap) {
@@ -54,7 +79,8 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
   const int tile = gridDim.x - 1 - blockIdx.x, kvh = blockIdx.y, hpg = p.n.H / p.n.G;      // late tiles (many keys) first
   const int first = p.tile_first[tile], count = p.tile_count[tile], slot = p.rw.slot[first];
   if (slot < 0 || count <= 0) return;
-  const int n = p.rw.pos[first + count - 1] / kGPage + 1;               // pages
+  const int win = p.sc.window, kt0 = max(0, p.rw.pos[first] - win + 1) / kGPage;        // first page a row sees
+  const int n = p.rw.pos[first + count - 1] / kGPage + 1 - kt0;         // pages
   if (tid == 0) {
     for (int i = 0; i < KS; ++i) {
       mbar_init(&kfull[i], 1);
@@ -103,7 +129,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       prefetch_tmap(&kmap);
       prefetch_tmap(&vmap);
       for (int j = 0; j < n; ++j) {
-        const int ks = j % KS, vs = j % VS, page = page_of(p.rw, slot, j);
+        const int ks = j % KS, vs = j % VS, page = page_of(p.rw, slot, kt0 + j);
         if (j >= KS && !mbar_wait(&kempty[ks], ((j / KS) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
@@ -175,7 +201,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
     bool ok = true;
     uint8_t* prow = p_s + strm * 2 * PB + r * 128;
     for (int i = 0; i < n_mine; ++i) {
-      const int b = i & 1, key0 = (2 * i + strm) * 64;
+      const int b = i & 1, key0 = (kt0 + 2 * i + strm) * 64;
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[strm][b], (i >> 1) & 1));
       if (!ok) break;
       tc_fence_after();
@@ -190,9 +216,9 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
         for (int e = 0; e < 64; ++e) sv[e] = fmaf(sv[e], scale2, tab[min(max(r_pos - key0 - e, 0), L1)] * kLog2e);
       }
       const float mul = near ? 1.f : scale2, add = near ? 0.f : far;
-      if (!r_ok || key0 + 63 > r_pos) {
+      if (!r_ok || key0 + 63 > r_pos || r_pos - key0 >= win) {
 #pragma unroll
-        for (int e = 0; e < 64; ++e) sv[e] = r_ok && key0 + e <= r_pos ? sv[e] : NEG_INF;
+        for (int e = 0; e < 64; ++e) sv[e] = r_ok && (unsigned)(r_pos - key0 - e) < (unsigned)win ? sv[e] : NEG_INF;
       }
       float mx0 = sv[0], mx1 = sv[1], mx2 = sv[2], mx3 = sv[3];
 #pragma unroll
@@ -283,6 +309,8 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
           const int col = c0 + q4 * 8;
           if (col >= p.n.dv) continue;
           uint32_t w[4];
+          float gt[8];
+          gate8(p.sc, r_tok, r_head * p.n.dv + col, p.n.dv - col, gt);
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float a = __uint_as_float(ov[q4 * 8 + 2 * e]) * f0, c = __uint_as_float(ov[q4 * 8 + 2 * e + 1]) * f0;
@@ -290,7 +318,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
               a = fmaf(__uint_as_float(ow[q4 * 8 + 2 * e]), f1, a);
               c = fmaf(__uint_as_float(ow[q4 * 8 + 2 * e + 1]), f1, c);
             }
-            w[e] = gq_pack(a, c);
+            w[e] = gq_pack(a * gt[2 * e], c * gt[2 * e + 1]);
           }
           if (p.vec) *reinterpret_cast<uint4*>(orow + col) = make_uint4(w[0], w[1], w[2], w[3]);
           else

@@ -10,11 +10,13 @@
 //   latent_prefill  prompt rows against expanded keys / values: mma.sync flash attention, 64 rows x 64 keys; scores and
 //                   weights keep 32-bit quality (weights enter the second product as two bf16 terms). On tcgen05 (latent_tc.cuh)
 //                   where plain + rotated width are at most three chunks of 64 columns and the values two, else on mma.sync
-// Angles are formed in double from a frequency table, so they are exact at any position. No fast-math in this file.
-// Neighbouring dimensions (2i, 2i + 1) form a rotation pair.
+// A sliding window hides keys at distances from it on; prompt rows then expand only the cached rows that some row of their portion sees.
+// Angles come from a table of half turns per position in double, so they are exact at any position; sine and cosine may carry a factor.
+// No fast-math in this file. Neighbouring dimensions (2i, 2i + 1) form a rotation pair.
 #include "rowmath.cuh"
 #include "tmap.h"
 #include <float.h>
+#include <limits.h>
 
 namespace ve {
 
@@ -24,9 +26,13 @@ struct LatentDims {
   int H, d, rot, dv, kr;     // heads, unrotated / rotated query width, value width, latent width
   int rot0, W, pitch;        // column of the rotated part, row width written by this layer, pool row pitch
 };
+struct LatentTurn {
+  const double* freq;        // half turns per position
+  float mul;                 // factor on sine and cosine
+};
 
-template <typename T>
-VE_DEVINL void store_latent_row(const LatentDims& n, const float* __restrict__ kv, const float* __restrict__ w, const float* cs, const float* sn,
+template <typename K, typename T>
+VE_DEVINL void store_latent_row(const LatentDims& n, const K* __restrict__ kv, const float* __restrict__ w, const float* cs, const float* sn,
                                 T* __restrict__ dst, float eps, float* red) {
   float ss = 0.f;
   for (int i = threadIdx.x; i < n.kr; i += blockDim.x) {
@@ -47,15 +53,6 @@ VE_DEVINL void store_latent_row(const LatentDims& n, const float* __restrict__ k
   }
 }
 
-VE_DEVINL void angles(int pos, const double* __restrict__ freq, int pairs, float* cs, float* sn) {
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    double s, c;
-    sincos((double)pos * freq[i], &s, &c);
-    cs[i] = (float)c;
-    sn[i] = (float)s;
-  }
-}
-
 template <typename T>
 VE_DEVINL T* cache_row(T* pool, const LatentDims& n, const int* page_table, int max_pages, int slot, int pos) {
   const int page = page_table[(long)slot * max_pages + pos / kLPage];
@@ -63,9 +60,9 @@ VE_DEVINL T* cache_row(T* pool, const LatentDims& n, const int* page_table, int 
 }
 
 // Prompt rows: grid (rows). q [rows][H (d + rot)] of type X -> qo of type T (may be the same memory when X = T).
-template <typename X, typename T>
-__global__ void __launch_bounds__(256) latent_rope_store_kernel(const LatentDims n, const X* q, long ldq, T* qo, long ldqo, const float* __restrict__ kv,
-                                                                long ldkv, const float* __restrict__ w, const double* __restrict__ freq,
+template <typename X, typename K, typename T>
+__global__ void __launch_bounds__(256) latent_rope_store_kernel(const LatentDims n, const X* q, long ldq, T* qo, long ldqo, const K* __restrict__ kv,
+                                                                long ldkv, const float* __restrict__ w, const LatentTurn tn,
                                                                 const int* __restrict__ pos, const int* __restrict__ slot,
                                                                 const int* __restrict__ page_table, int max_pages, T* __restrict__ pool, float eps) {
   __shared__ float red[33], cs[128], sn[128];
@@ -74,7 +71,7 @@ __global__ void __launch_bounds__(256) latent_rope_store_kernel(const LatentDims
   const long row = blockIdx.x;
   const int p = pos[row], s = slot[row];
   if (s < 0) return;
-  angles(p, freq, n.rot / 2, cs, sn);
+  angle_row(p, tn.freq, n.rot / 2, tn.mul, cs, sn);
   __syncthreads();
   const int hw = n.d + n.rot;
   if (qo) {
@@ -105,9 +102,9 @@ __global__ void __launch_bounds__(256) latent_rope_store_kernel(const LatentDims
 
 // Decode rows: grid (rows, H + 1, nz). Block y < H: latent columns [z * cols, ...) of head y's absorbed query (z = 0: also the
 // rotated part); block y == H (z == 0): the cache row. 128 threads = 16 groups over d x 8 lanes over columns (VEC each).
-template <int VEC, typename X, typename T>
-__global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentDims n, const X* __restrict__ q, long ldq, const float* __restrict__ kv, long ldkv,
-                                                            const float* __restrict__ w, const T* __restrict__ w_uk, const double* __restrict__ freq,
+template <int VEC, typename X, typename K, typename T>
+__global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentDims n, const X* __restrict__ q, long ldq, const K* __restrict__ kv, long ldkv,
+                                                            const float* __restrict__ w, const T* __restrict__ w_uk, const LatentTurn tn,
                                                             const int* __restrict__ pos, const int* __restrict__ slot,
                                                             const int* __restrict__ page_table, int max_pages, T* __restrict__ pool,
                                                             T* __restrict__ q_abs, int qw, float eps) {
@@ -119,7 +116,7 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentDims n, 
   const int h = blockIdx.y, z = blockIdx.z, tid = threadIdx.x;
   const int p = pos[row], s = slot[row];
   if (s < 0 || (h == n.H && z > 0)) return;
-  if (z == 0) angles(p, freq, n.rot / 2, cs, sn);
+  if (z == 0) angle_row(p, tn.freq, n.rot / 2, tn.mul, cs, sn);
   if (h == n.H) {
     __syncthreads();
     store_latent_row(n, kv + row * ldkv, w, cs, sn, cache_row(pool, n, page_table, max_pages, s, p), eps, red);
@@ -178,7 +175,7 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentDims n, 
 template <int NC, typename T>
 __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims n, const T* __restrict__ q_abs, int qw, const int* __restrict__ pos,
                                                           const int* __restrict__ slot, const int* __restrict__ page_table, int max_pages,
-                                                          const T* __restrict__ pool, float scale, float* __restrict__ o_lat) {
+                                                          const T* __restrict__ pool, float scale, int window, float* __restrict__ o_lat) {
   extern __shared__ float sm[];             // [qw] query, then [4][NC * 32] outputs
   __shared__ float sm_m[4], sm_l[4];
   grid_dep_wait();
@@ -192,7 +189,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentDims n, co
   float acc[NC], m = -FLT_MAX, l = 0.f;
 #pragma unroll
   for (int j = 0; j < NC; ++j) acc[j] = 0.f;
-  for (int key = warp; key <= p; key += 4) {
+  for (int key = max(0, p - window + 1) + warp; key <= p; key += 4) {
     const int page = page_table[(long)s * max_pages + key / kLPage];
     const T* kr = pool + ((long)page * kLPage + key % kLPage) * n.pitch;
     float c[NC], dot = 0.f;
@@ -294,9 +291,10 @@ __global__ void __launch_bounds__(512) latent_expand_kernel(const LatentDims n, 
   }
 }
 
-// rows [0, n) of out [n][W]: src_row[i] = slot * 2^32 + position is resolved through the page table. grid (rows), 16-byte pieces.
+// rows [0, total) of out [total][W]: cached rows of seg_slot[g] from position seg_start[g] on stand from row seg_base[g] on. 16-byte pieces.
 __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, int pitch, const int* __restrict__ page_table, int max_pages,
-                                     const int* __restrict__ seg_slot, const int* __restrict__ seg_base, int nseg, __nv_bfloat16* __restrict__ out,
+                                     const int* __restrict__ seg_slot, const int* __restrict__ seg_base, const int* __restrict__ seg_start, int nseg,
+                                     __nv_bfloat16* __restrict__ out,
                                      int W, int total) {
   grid_dep_wait();
   grid_dep_launch();
@@ -305,7 +303,7 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, int
     const int r = (int)(i / per), c = (int)(i % per) * 8;
     int g = 0;
     while (g + 1 < nseg && seg_base[g + 1] <= r) ++g;
-    const int key = r - seg_base[g];
+    const int key = seg_start[g] + r - seg_base[g];
     const int page = page_table[(long)seg_slot[g] * max_pages + key / kLPage];
     *reinterpret_cast<uint4*>(out + (long)r * W + c) = *reinterpret_cast<const uint4*>(pool + ((long)page * kLPage + key % kLPage) * pitch + c);
   }
@@ -337,7 +335,9 @@ struct LatentPrefill {
   const __nv_bfloat16* up; long ldu;       // [keys][H d | H dv], expanded from the gathered latents
   const __nv_bfloat16* lat; int W;         // [keys][W], gathered cache rows (the rotated part is read)
   const int* pos;
-  const int* tile_first; const int* tile_count; const int* tile_base;   // query tiles; tile_base = first key row of the sequence
+  const int* tile_first; const int* tile_count; const int* tile_base;   // query tiles; tile_base = first key row of the sequence,
+  const int* tile_key0;                    // which is this position
+  int window;
   __nv_bfloat16* out; long ldo;            // [rows][H dv]
   float scale_log2;
 };
@@ -354,7 +354,9 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentPrefill
   const LatentDims& n = p.n;
   const int tile = gridDim.x - 1 - blockIdx.x, h = blockIdx.y;          // late tiles (many keys) first
   const int first = p.tile_first[tile], count = p.tile_count[tile];
-  const long kbase = p.tile_base[tile];
+  const int win = p.window, skip = max(0, p.pos[first] - win + 1 - p.tile_key0[tile]) / 64 * 64;      // key rows that no row of the tile sees
+  const int key0 = p.tile_key0[tile] + skip;
+  const long kbase = p.tile_base[tile] + skip;
   const int hw = n.d + n.rot;
   for (int i = tid; i < 2 * STAGE / 16; i += 128) *reinterpret_cast<uint4*>(lsm + i * 16) = make_uint4(0, 0, 0, 0);   // pad columns stay zero
   int r_row[2], r_pos[2];
@@ -366,7 +368,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentPrefill
     r_row[e] = first + (r_ok[e] ? r : 0);
     r_pos[e] = p.pos[r_row[e]];
   }
-  const int keys = p.pos[first + count - 1] + 1, nkt = (keys + 63) / 64;
+  const int keys = p.pos[first + count - 1] + 1 - key0, nkt = (keys + 63) / 64;
   uint32_t qf[DQ / 16][4];
 #pragma unroll
   for (int kk = 0; kk < DQ / 16; ++kk)
@@ -407,7 +409,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentPrefill
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    if (w_live && kt * 64 <= w_last) {
+    if (w_live && key0 + kt * 64 <= w_last) {
       const uint32_t kb = sbase + (kt & 1) * STAGE, vb = kb + 64 * KP;
       float sacc[8][4];
 #pragma unroll
@@ -427,8 +429,8 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentPrefill
       for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int key = kt * 64 + nt * 8 + 2 * t + (e & 1);
-          const float v = key <= r_pos[e >> 1] ? sacc[nt][e] * p.scale_log2 : -FLT_MAX;
+          const int dist = r_pos[e >> 1] - (key0 + kt * 64 + nt * 8 + 2 * t + (e & 1));
+          const float v = (unsigned)dist < (unsigned)win ? sacc[nt][e] * p.scale_log2 : -FLT_MAX;
           sacc[nt][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -519,53 +521,51 @@ static bool ldims_ok(const LatentDims& n) {
 
 extern "C" {
 
-// kv rows are fp32. x32: q rows are fp32 (else bf16); f32: q_out, pool fp32 (else bf16). q_out null: only the cache row is written.
-int ve_latent_rope_store(VE_LDIMS, const void* q, long ldq, void* qo, long ldqo, const void* kv, long ldkv, int x32, const void* w, const void* freq,
-                         const void* pos, const void* slot, const void* page_table, int max_pages, void* pool, int rows, float eps, int f32, cudaStream_t st) {
+// x32, kv32: q, kv rows are fp32 (else bf16); f32: q, kv, q_out, pool fp32 (else bf16). q_out null: only the cache row is written.
+int ve_latent_rope_store(VE_LDIMS, const void* q, long ldq, void* qo, long ldqo, const void* kv, long ldkv, int x32, int kv32, const void* w,
+                         const void* freq, float mul, const void* pos, const void* slot, const void* page_table, int max_pages, void* pool, int rows, float eps, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const LatentDims n = VE_LMAKE;
   if (!ldims_ok(n)) return cudaErrorInvalidValue;
-#define VE_RS(X, T) launch_pdl(latent_rope_store_kernel<X, T>, dim3(rows), dim3(256), 0, st, n, (const X*)q, ldq, (T*)qo, ldqo, (const float*)kv, ldkv, \
-    (const float*)w, (const double*)freq, (const int*)pos, (const int*)slot, (const int*)page_table, max_pages, (T*)pool, eps)
-  if (f32) VE_RS(float, float);
-  else if (x32) VE_RS(float, __nv_bfloat16);
-  else VE_RS(__nv_bfloat16, __nv_bfloat16);
+  const LatentTurn tn{(const double*)freq, mul};
+#define VE_RS(X, K, T) launch_pdl(latent_rope_store_kernel<X, K, T>, dim3(rows), dim3(256), 0, st, n, (const X*)q, ldq, (T*)qo, ldqo, (const K*)kv, ldkv, \
+    (const float*)w, tn, (const int*)pos, (const int*)slot, (const int*)page_table, max_pages, (T*)pool, eps)
+  if (f32) VE_RS(float, float, float);
+  else if (x32) VE_RS(float, float, __nv_bfloat16);
+  else if (kv32) VE_RS(__nv_bfloat16, float, __nv_bfloat16);
+  else VE_RS(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
 #undef VE_RS
   VE_CHECK_LAUNCH();
 }
 
 // q_abs [rows][H][qw] (qw >= rot0 + rot; columns outside the latent and the rotated part are written as zero).
-int ve_latent_absorb(VE_LDIMS, const void* q, long ldq, const void* kv, long ldkv, int x32, const void* w, const void* w_uk, const void* freq,
-                     const void* pos, const void* slot, const void* page_table, int max_pages, void* pool, void* q_abs, int qw, int rows, float eps,
+int ve_latent_absorb(VE_LDIMS, const void* q, long ldq, const void* kv, long ldkv, int x32, int kv32, const void* w, const void* w_uk,
+                     const void* freq, float mul, const void* pos, const void* slot, const void* page_table, int max_pages, void* pool, void* q_abs, int qw, int rows, float eps,
                      int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const LatentDims n = VE_LMAKE;
   if (!ldims_ok(n) || qw < rot0 + rot) return cudaErrorInvalidValue;
   const bool al = !((uintptr_t)w_uk & 15);
-#define VE_AB(V, X, T) launch_pdl(latent_absorb_kernel<V, X, T>, dim3(rows, H + 1, (kr + 8 * V - 1) / (8 * V)), dim3(128), 0, st, n, (const X*)q, ldq, \
-    (const float*)kv, ldkv, (const float*)w, (const T*)w_uk, (const double*)freq, (const int*)pos, (const int*)slot, (const int*)page_table, max_pages, \
-    (T*)pool, (T*)q_abs, qw, eps)
-  if (f32) {
-    if (al && kr % 4 == 0) VE_AB(4, float, float);
-    else VE_AB(1, float, float);
-  } else if (x32) {
-    if (al && kr % 8 == 0) VE_AB(8, float, __nv_bfloat16);
-    else VE_AB(1, float, __nv_bfloat16);
-  } else {
-    if (al && kr % 8 == 0) VE_AB(8, __nv_bfloat16, __nv_bfloat16);
-    else VE_AB(1, __nv_bfloat16, __nv_bfloat16);
-  }
+  const LatentTurn tn{(const double*)freq, mul};
+#define VE_AB(V, X, K, T) launch_pdl(latent_absorb_kernel<V, X, K, T>, dim3(rows, H + 1, (kr + 8 * V - 1) / (8 * V)), dim3(128), 0, st, n, (const X*)q, ldq, \
+    (const K*)kv, ldkv, (const float*)w, (const T*)w_uk, tn, (const int*)pos, (const int*)slot, (const int*)page_table, max_pages, (T*)pool, (T*)q_abs, qw, eps)
+#define VE_AB_V(V, X, K, T) do { if (al && kr % V == 0) VE_AB(V, X, K, T); else VE_AB(1, X, K, T); } while (0)
+  if (f32) VE_AB_V(4, float, float, float);
+  else if (x32) VE_AB_V(8, float, float, __nv_bfloat16);
+  else if (kv32) VE_AB_V(8, __nv_bfloat16, float, __nv_bfloat16);
+  else VE_AB_V(8, __nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
+#undef VE_AB_V
 #undef VE_AB
   VE_CHECK_LAUNCH();
 }
 
 int ve_latent_attn(VE_LDIMS, const void* q_abs, int qw, const void* pos, const void* slot, const void* page_table, int max_pages, const void* pool,
-                   float scale, void* o_lat, int rows, int f32, cudaStream_t st) {
+                   float scale, int window, void* o_lat, int rows, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const LatentDims n = VE_LMAKE;
   if (!ldims_ok(n) || kr > 1024 || qw > 4096) return cudaErrorInvalidValue;
 #define VE_LA(NC, T) launch_pdl(latent_attn_kernel<NC, T>, dim3(rows, H), dim3(128), (size_t)(qw + 4 * NC * 32) * 4, st, n, (const T*)q_abs, qw, (const int*)pos, \
-    (const int*)slot, (const int*)page_table, max_pages, (const T*)pool, scale, (float*)o_lat)
+    (const int*)slot, (const int*)page_table, max_pages, (const T*)pool, scale, window > 0 ? window : INT_MAX, (float*)o_lat)
 #define VE_LA_T(T) do { if (kr <= 128) VE_LA(4, T); else if (kr <= 256) VE_LA(8, T); else if (kr <= 512) VE_LA(16, T); else VE_LA(32, T); } while (0)
   if (f32) VE_LA_T(float);
   else VE_LA_T(__nv_bfloat16);
@@ -594,27 +594,29 @@ int ve_latent_expand(VE_LDIMS, const void* o_part, const void* lse, int nsplit, 
   VE_CHECK_LAUNCH();
 }
 
-// seg_base [nseg]: first output row of every sequence (ascending); rows [seg_base[g], seg_base[g + 1]) are its positions 0, 1, ...
-int ve_latent_gather(const void* pool, int pitch, const void* page_table, int max_pages, const void* seg_slot, const void* seg_base, int nseg, void* out,
-                     int W, int total, cudaStream_t st) {
+// seg_base [nseg]: first output row of every sequence (ascending); rows [seg_base[g], seg_base[g + 1]) are its positions seg_start[g], + 1, ...
+int ve_latent_gather(const void* pool, int pitch, const void* page_table, int max_pages, const void* seg_slot, const void* seg_base, const void* seg_start,
+                     int nseg, void* out, int W, int total, cudaStream_t st) {
   if (total <= 0) return 0;
   if (W % 8 || pitch % 8 || W > pitch || nseg < 1) return cudaErrorInvalidValue;
   const long items = (long)total * (W / 8);
   const long blocks = (items + 255) / 256;
   launch_pdl(latent_gather_kernel, dim3((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), 0, st, (const __nv_bfloat16*)pool, pitch,
-             (const int*)page_table, max_pages, (const int*)seg_slot, (const int*)seg_base, nseg, (__nv_bfloat16*)out, W, total);
+             (const int*)page_table, max_pages, (const int*)seg_slot, (const int*)seg_base, (const int*)seg_start, nseg, (__nv_bfloat16*)out, W, total);
   VE_CHECK_LAUNCH();
 }
 
 // Widths d, rot and dv multiples of 8, d + rot <= 256, dv <= 256; all bases and pitches 16-byte aligned (bf16).
 int ve_latent_prefill(VE_LDIMS, const void* q, long ldq, const void* up, long ldu, const void* lat, int lat_w, const void* pos, const void* tile_first,
-                      const void* tile_count, const void* tile_base, int ntiles, void* out, long ldo, float scale, cudaStream_t st) {
+                      const void* tile_count, const void* tile_base, const void* tile_key0, int ntiles, int window, void* out, long ldo, float scale,
+                      cudaStream_t st) {
   if (ntiles <= 0) return 0;
   const LatentDims n = VE_LMAKE;
   if (!ldims_ok(n) || d % 8 || rot % 8 || dv % 8 || rot0 % 8 || lat_w % 8 || ldq % 8 || ldu % 8 || ldo % 2 || d + rot > 256 || dv > 256 ||
       ((uintptr_t)up & 15) || ((uintptr_t)lat & 15) || ((uintptr_t)q & 3) || ((uintptr_t)out & 3)) return cudaErrorInvalidValue;
   LatentPrefill p{n, (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)up, ldu, (const __nv_bfloat16*)lat, lat_w, (const int*)pos, (const int*)tile_first,
-                  (const int*)tile_count, (const int*)tile_base, (__nv_bfloat16*)out, ldo, scale * 1.4426950408889634f};
+                  (const int*)tile_count, (const int*)tile_base, (const int*)tile_key0, window > 0 ? window : INT_MAX, (__nv_bfloat16*)out, ldo,
+                  scale * 1.4426950408889634f};
   const int q_w = d + rot;
   if (dv <= 64) {
     if (q_w <= 64) return launch_latent_prefill<64, 64>(p, ntiles, st);
@@ -632,8 +634,8 @@ int ve_latent_prefill(VE_LDIMS, const void* q, long ldq, const void* up, long ld
 // The same on tcgen05: tiles of at most 128 rows; d and rot in at most three chunks of 64 columns together, dv <= 128. up
 // [up_rows][...] and lat [up_rows][lat_w] are read through tensor maps.
 int ve_latent_prefill_tc(VE_LDIMS, const void* q, long ldq, const void* up, long ldu, const void* lat, int lat_w, long up_rows, const void* pos,
-                         const void* tile_first, const void* tile_count, const void* tile_base, int ntiles, void* out, long ldo, float scale, void* status,
-                         cudaStream_t st) {
+                         const void* tile_first, const void* tile_count, const void* tile_base, const void* tile_key0, int ntiles, int window, void* out,
+                         long ldo, float scale, void* status, cudaStream_t st) {
   if (ntiles <= 0) return 0;
   const LatentDims n = VE_LMAKE;
   const int uc = (d + 63) / 64, qc = uc + (rot + 63) / 64, vc = (dv + 63) / 64;
@@ -644,8 +646,8 @@ int ve_latent_prefill_tc(VE_LDIMS, const void* q, long ldq, const void* up, long
   if (rc) return rc;
   rc = make_tmap_2d(&rm, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, up_rows, lat_w, (uint64_t)lat_w * 2, 64, 64, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
-  LatentTc p{n, (const __nv_bfloat16*)q, ldq, (const int*)pos, (const int*)tile_first, (const int*)tile_count, (const int*)tile_base, (__nv_bfloat16*)out, ldo,
-             scale * 1.4426950408889634f, uc, (int*)status};
+  LatentTc p{n, (const __nv_bfloat16*)q, ldq, (const int*)pos, (const int*)tile_first, (const int*)tile_count, (const int*)tile_base,
+             (const int*)tile_key0, window > 0 ? window : INT_MAX, (__nv_bfloat16*)out, ldo, scale * 1.4426950408889634f, uc, (int*)status};
   if (vc == 1) {
     if (qc == 1) return launch_latent_tc<1, 1>(p, um, rm, ntiles, st);
     if (qc == 2) return launch_latent_tc<2, 1>(p, um, rm, ntiles, st);

@@ -6,7 +6,8 @@
 //   * query and key are DQC chunks of 64 columns (plain part, then rotated part; pad columns of the query are zero), the key's
 //     rotated part comes from the cached rows and is shared by the heads; values are DVC chunks;
 //   * the softmax weights enter the second product as two bf16 terms (value and remainder), so they keep 32-bit quality;
-//   * keys and values have rings of their own (a key tile is free as soon as its scores are done).
+//   * keys and values have rings of their own (a key tile is free as soon as its scores are done);
+//   * with a sliding window the key tiles in front of the first row's window are not visited.
 // Every wait is bounded; on expiry the CTA records a status code, skips its stores and frees its TMEM.
 #pragma once
 
@@ -17,6 +18,8 @@ struct LatentTc {
   const __nv_bfloat16* q; long ldq;        // [rows][H (d + rot)], rotated
   const int* pos;
   const int* tile_first; const int* tile_count; const int* tile_base;
+  const int* tile_key0;                    // position of the key row tile_base
+  int window;
   __nv_bfloat16* out; long ldo;
   float scale_log2;
   int uc;                                  // chunks of the plain part
@@ -45,8 +48,10 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
   __shared__ int s_fail;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int tile = gridDim.x - 1 - blockIdx.x, h = blockIdx.y;          // late tiles (many keys) first
-  const int first = p.tile_first[tile], count = p.tile_count[tile], kbase = p.tile_base[tile];
-  const int n = p.pos[first + count - 1] / kLPage + 1;                  // key tiles
+  const int first = p.tile_first[tile], count = p.tile_count[tile], win = p.window;
+  const int skip = max(0, p.pos[first] - win + 1 - p.tile_key0[tile]) / kLPage * kLPage;      // key rows that no row of the tile sees
+  const int kbase = p.tile_base[tile] + skip, kpos = p.tile_key0[tile] + skip;                // first key row and its position
+  const int n = (p.pos[first + count - 1] - kpos) / kLPage + 1;         // key tiles
   if (tid == 0) {
     for (int i = 0; i < kLtKs; ++i) {
       mbar_init(&kfull[i], 1);
@@ -170,7 +175,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
     bool ok = true;
     uint8_t* prow = p_s + strm * 2 * PB + r * 128;
     for (int i = 0; i < n_mine; ++i) {
-      const int b = i & 1, key0 = (2 * i + strm) * 64;
+      const int b = i & 1, key0 = kpos + (2 * i + strm) * 64;
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[strm][b], (i >> 1) & 1));
       if (!ok) break;
       tc_fence_after();
@@ -178,9 +183,9 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
       tmem_ld32(t_lane + strm * 128 + b * 64, reinterpret_cast<uint32_t*>(sv));
       tmem_ld32(t_lane + strm * 128 + b * 64 + 32, reinterpret_cast<uint32_t*>(sv) + 32);
       tmem_ld_wait();
-      if (!r_ok || key0 + 63 > r_pos) {
+      if (!r_ok || key0 + 63 > r_pos || r_pos - key0 >= win) {
 #pragma unroll
-        for (int e = 0; e < 64; ++e) sv[e] = r_ok && key0 + e <= r_pos ? sv[e] : NEG_INF;
+        for (int e = 0; e < 64; ++e) sv[e] = r_ok && (unsigned)(r_pos - key0 - e) < (unsigned)win ? sv[e] : NEG_INF;
       }
       float mx0 = sv[0], mx1 = sv[1], mx2 = sv[2], mx3 = sv[3];
 #pragma unroll

@@ -15,6 +15,7 @@
 #include "common.cuh"
 #include "tmap.h"
 #include <float.h>
+#include <limits.h>
 
 namespace ve {
 
@@ -117,6 +118,7 @@ struct MlaParams {
   float scale_log2;
   int* status;
   int row;                      // cache row width in elements (a multiple of 64) where it is not a template constant
+  int window;                   // keys at distances below it are seen (INT_MAX: all in front)
 };
 
 VE_DEVINL void m_ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
@@ -160,9 +162,10 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
   const int s = p.slot ? p.slot[tok] : 0;
   if (s < 0) return;
   const int ps = p.pos[tok];
-  const int ntile_all = ps / kMlaPage + 1;
+  const int win = P2 ? p.window : INT_MAX;
+  const int kt0 = P2 ? max(0, ps - win + 1) / kMlaPage : 0, ntile_all = ps / kMlaPage + 1 - kt0;
   const int tps = (ntile_all + p.nsplit - 1) / p.nsplit;
-  const int kt_begin = z * tps, kt_end = min(ntile_all, kt_begin + tps);
+  const int kt_begin = kt0 + z * tps, kt_end = min(kt0 + ntile_all, kt_begin + tps);
 
   if (tid == 0) {
     mbar_init(&full[0], 1);
@@ -224,7 +227,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p, cons
       for (int e = 0; e < 4; ++e) {
         const int row = g + (e >> 1) * 8, key_l = warp * 16 + nt * 8 + 2 * t + (e & 1);
         const int key = kt * kMlaPage + key_l;
-        ss[row * kSPitch + key_l] = key <= ps ? sacc[nt][e] * p.scale_log2 : -FLT_MAX;
+        ss[row * kSPitch + key_l] = (unsigned)(ps - key) < (unsigned)win ? sacc[nt][e] * p.scale_log2 : -FLT_MAX;
       }
     __syncthreads();
     // ---- every warp: softmax statistics of its two rows over all 64 keys, P fragments
@@ -392,6 +395,7 @@ int ve_mla_decode(const void* q_abs, void* o_lat, void* o_part, void* lse_part, 
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = (int*)status;
   p.row = kLatRow;
+  p.window = INT_MAX;
   CUtensorMap kmap;
   int rc = make_tmap_2d(&kmap, pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)pool_pages * kMlaPage, kLatRow,
                         (uint64_t)kLatRow * 2, kMlaPage, 64, CU_TENSOR_MAP_SWIZZLE_128B);
@@ -418,7 +422,7 @@ int ve_mla_decode(const void* q_abs, void* o_lat, void* o_part, void* lse_part, 
 // [rows, heads, nsplit, lat rounded up to 64 * {1, 2, 4, 8}] and lse_part (log2 units); a split without keys leaves
 // lse = -FLT_MAX. The merge is part of latent_expand.
 int ve_latent_decode(const void* q_abs, void* o_part, void* lse_part, const void* pos, const void* slot, const void* page_table, int max_pages,
-                     void* pool, long pool_pages, int pitch, int row, int lat, int rows, int heads, int nsplit, float scale, void* status,
+                     void* pool, long pool_pages, int pitch, int row, int lat, int rows, int heads, int nsplit, float scale, int window, void* status,
                      cudaStream_t st) {
   if (rows <= 0) return 0;
   const int nb = lat <= 64 ? 1 : lat <= 128 ? 2 : lat <= 256 ? 4 : 8;
@@ -436,6 +440,7 @@ int ve_latent_decode(const void* q_abs, void* o_part, void* lse_part, const void
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = (int*)status;
   p.row = row;
+  p.window = window > 0 ? window : INT_MAX;
   CUtensorMap kmap;
   int rc = make_tmap_2d(&kmap, pool, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)pool_pages * kMlaPage, pitch, (uint64_t)pitch * 2, kMlaPage, 64,
                         CU_TENSOR_MAP_SWIZZLE_128B);

@@ -26,10 +26,27 @@ VE_DEVINL float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
 VE_DEVINL float silu_of(float z) { return z / (1.f + expf(-z)); }
 VE_DEVINL float dyt_of(float h, float alpha, float w, float b) { return fmaf(tanhf(alpha * h), w, b); }
 
-// Gated unit with both halves clamped: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1)
-VE_DEVINL float clamped_glu_of(float g, float u, float alpha, float limit) {
-  const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
-  return a / (1.f + expf(-alpha * a)) * (b + 1.f);
+// Gated unit with both halves clamped: min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + shift).
+// alpha 1, an infinite limit and shift 0 make it silu(g) u.
+struct Glu { float alpha, limit, shift; };
+VE_DEVINL float clamped_glu_of(float g, float u, const Glu& c) {
+  const float a = fminf(g, c.limit), b = fminf(fmaxf(u, -c.limit), c.limit);
+  return a / (1.f + expf(-c.alpha * a)) * (b + c.shift);
+}
+
+VE_DEVINL float soft_cap_of(float v, float cap) { return cap * tanhf(v / cap); }
+
+// Sine and cosine (times mul) of a position's angles, by the threads of a block into shared memory. freq: half turns per position, in
+// double; the angle is reduced to one turn before it is rounded.
+constexpr int kMaxPairs = 256;
+VE_DEVINL void angle_row(int pos, const double* __restrict__ freq, int pairs, float mul, float* cs, float* sn) {
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const double t = (double)pos * freq[i];
+    float s, c;
+    sincospif((float)(t - 2.0 * rint(0.5 * t)), &s, &c);
+    cs[i] = c * mul;
+    sn[i] = s * mul;
+  }
 }
 
 // Residual streams (at most kMaxStreams copies of a row): every stream anew from all old ones and a sublayer's result,

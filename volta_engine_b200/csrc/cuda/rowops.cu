@@ -1,12 +1,14 @@
 // Row operators of decoders whose residual stream is fp32. Storage of activations is a template parameter (bf16, or fp32
 // for the all-32-bit form of a model); every operator computes in fp32. This file is compiled without fast-math: norms,
 // gates and angles follow the 32-bit definitions to rounding.
-//   embed_rows   out[r] = table[ids[r]] widened to fp32 [+ sinusoidal position vector], once per residual stream
+//   embed_rows   out[r] = table[ids[r]] widened to fp32, times a scale [+ sinusoidal position vector], once per residual stream
 //   dyt_rows     h += scale * part (optional, element-wise scale), out = tanh(alpha h) w + b        ("Dynamic Tanh" norm)
 //   stream_norm  residual streams rewritten from the old ones and a sublayer's result (optional), then the layer norm (no shift) of
 //                their weighted sum
 //   group_rms    out = x / rms(x over groups of G columns) * w [* sigmoid(gate) or silu(gate)]; w repeats with its own length
+//   residual_norm  h += RMS norm of a sublayer's result (or of the weighted sum of a token's routed results), out = h or its RMS norm
 //   clamped_glu  out = gated unit of [gate | up] rows with both halves clamped
+//   soft_cap     x = cap tanh(x / cap)
 //   polynorm     out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3, N = division by the row's root mean square
 //   scale_add    h += scale * part
 #include "rowmath.cuh"
@@ -16,7 +18,7 @@ namespace ve {
 // freq (optional, double): turns by half circles per position and column pair; column 2i gets the sine, 2i + 1 the cosine.
 template <typename T>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ table, const int* __restrict__ pos, const double* __restrict__ freq,
-                                  float* __restrict__ out, int H, int vocab, int S) {
+                                  float* __restrict__ out, int H, int vocab, int S, float scale) {
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
@@ -26,7 +28,7 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restri
   float* dst = out + row * S * H;
   if (!freq) {
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float v = to_f(src[i]);
+      const float v = to_f(src[i]) * scale;
       for (int s = 0; s < S; ++s) dst[(long)s * H + i] = v;
     }
     return;
@@ -36,7 +38,7 @@ __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restri
     const double t = p * freq[i >> 1];
     float sn, cs;
     sincospif((float)(t - 2.0 * rint(0.5 * t)), &sn, &cs);
-    const float v0 = to_f(src[i]) + sn, v1 = i + 1 < H ? to_f(src[i + 1]) + cs : 0.f;
+    const float v0 = fmaf(to_f(src[i]), scale, sn), v1 = i + 1 < H ? fmaf(to_f(src[i + 1]), scale, cs) : 0.f;
     for (int s = 0; s < S; ++s) {
       dst[(long)s * H + i] = v0;
       if (i + 1 < H) dst[(long)s * H + i + 1] = v1;
@@ -275,24 +277,142 @@ __global__ void __launch_bounds__(256) stream_norm4_kernel(float* __restrict__ h
   }
 }
 
+// One sublayer result per row: rows of `part`, or (top > 0) sum_k rw[row][k] part[inv ? inv[row top + k] : row top + k].
+struct ResultRows {
+  const int* inv; const float* rw; int top;
+};
+// h [rows][H]. One CTA per row. wa null: no result; wo null: the residual itself; out null: only the residual.
+template <typename T>
+__global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ h, const T* __restrict__ part, long ldp, const ResultRows rr,
+                                                            const float* __restrict__ wa, const float* __restrict__ wo, T* __restrict__ out, long ldo, int H,
+                                                            float eps) {
+  __shared__ float red[33];
+  grid_dep_wait();
+  grid_dep_launch();
+  const long row = blockIdx.x;
+  float* hr = h + row * H;
+  auto result = [&](int i) {
+    if (!rr.top) return to_f(part[row * ldp + i]);
+    float v = 0.f;
+    for (int k = 0; k < rr.top; ++k) {
+      const long r = row * rr.top + k;
+      v = fmaf(rr.rw[r], to_f(part[(rr.inv ? rr.inv[r] : r) * ldp + i]), v);
+    }
+    return v;
+  };
+  float inv = 0.f, s = 0.f;
+  if (wa) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float v = result(i);
+      s = fmaf(v, v, s);
+    }
+    inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
+    s = 0.f;
+  }
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float v = hr[i];
+    if (wa) {
+      v = fmaf(result(i) * inv, wa[i], v);
+      hr[i] = v;
+    }
+    if (!out) continue;
+    if (!wo) out[row * ldo + i] = from_f<T>(v);
+    s = fmaf(v, v, s);
+  }
+  if (!out || !wo) return;
+  inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) out[row * ldo + i] = from_f<T>(hr[i] * inv * wo[i]);      // (a thread reads what it wrote itself)
+}
+
+// The same on four columns per thread and step, the row in registers (H <= 1024 NV; H, pitches and bases multiples of four).
+template <int NV, typename T>
+__global__ void __launch_bounds__(256) residual_norm4_kernel(float* __restrict__ h, const T* __restrict__ part, long ldp, const ResultRows rr,
+                                                             const float* __restrict__ wa, const float* __restrict__ wo, T* __restrict__ out, long ldo, int H,
+                                                             float eps) {
+  __shared__ float red[33];
+  grid_dep_wait();
+  grid_dep_launch();
+  const long row = blockIdx.x;
+  float* hr = h + row * H;
+  float4 y[NV], x[NV];
+  float s = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (j * 256 + threadIdx.x) * 4;
+    x[j] = i < H ? load4(hr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    y[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (wa && !rr.top && i < H) y[j] = load4(part + row * ldp + i);
+  }
+  if (wa) {
+    for (int k = 0; k < rr.top; ++k) {
+      const long r = row * rr.top + k;
+      const T* pr = part + (rr.inv ? rr.inv[r] : r) * ldp;
+      const float f = rr.rw[r];
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const int i = (j * 256 + threadIdx.x) * 4;
+        if (i < H) {
+          const float4 v = load4(pr + i);
+          y[j] = make_float4(fmaf(f, v.x, y[j].x), fmaf(f, v.y, y[j].y), fmaf(f, v.z, y[j].z), fmaf(f, v.w, y[j].w));
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < NV; ++j) s += (y[j].x * y[j].x + y[j].y * y[j].y) + (y[j].z * y[j].z + y[j].w * y[j].w);
+    const float inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
+    s = 0.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = (j * 256 + threadIdx.x) * 4;
+      if (i < H) {
+        const float4 w = load4(wa + i);
+        x[j] = make_float4(fmaf(y[j].x * inv, w.x, x[j].x), fmaf(y[j].y * inv, w.y, x[j].y), fmaf(y[j].z * inv, w.z, x[j].z), fmaf(y[j].w * inv, w.w, x[j].w));
+        store4(hr + i, x[j]);
+      }
+    }
+  }
+  if (!out) return;
+  float inv = 1.f;
+  if (wo) {
+#pragma unroll
+    for (int j = 0; j < NV; ++j) s += (x[j].x * x[j].x + x[j].y * x[j].y) + (x[j].z * x[j].z + x[j].w * x[j].w);
+    inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
+  }
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (j * 256 + threadIdx.x) * 4;
+    if (i >= H) continue;
+    if (wo) {
+      const float4 w = load4(wo + i);
+      x[j] = make_float4(x[j].x * inv * w.x, x[j].y * inv * w.y, x[j].z * inv * w.z, x[j].w * inv * w.w);
+    }
+    store4(out + row * ldo + i, x[j]);
+  }
+}
+
+__global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ x, long n, float cap) {
+  grid_dep_wait();
+  grid_dep_launch();
+  for (long i = blockIdx.x * 256l + threadIdx.x; i < n; i += gridDim.x * 256l) x[i] = soft_cap_of(x[i], cap);
+}
+
 // z [rows][2 F]: gates, then ups (blk 0), or blocks of [4 gates | 4 ups].
 template <typename X, typename T>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, int blk, float alpha,
-                                                          float limit) {
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, int blk, const Glu u) {
   grid_dep_wait();
   grid_dep_launch();
   for (long q = blockIdx.x * 256l + threadIdx.x; q < total; q += gridDim.x * 256l) {
     const long row = q / F;
-    const int i = (int)(q - row * F), g = blk ? (i >> 2) * 8 + (i & 3) : i, u = blk ? g + 4 : F + i;
-    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + g]), to_f(z[row * ldz + u]), alpha, limit));
+    const int i = (int)(q - row * F), g = blk ? (i >> 2) * 8 + (i & 3) : i, up = blk ? g + 4 : F + i;
+    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + g]), to_f(z[row * ldz + up]), u));
   }
 }
-VE_DEVINL __nv_bfloat162 clamped_glu2(__nv_bfloat162 g, __nv_bfloat162 u, float alpha, float limit) {
+VE_DEVINL __nv_bfloat162 clamped_glu2(__nv_bfloat162 g, __nv_bfloat162 u, const Glu& c) {
   const float2 a = __bfloat1622float2(g), b = __bfloat1622float2(u);
-  return __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, alpha, limit), clamped_glu_of(a.y, b.y, alpha, limit));
+  return __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, c), clamped_glu_of(a.y, b.y, c));
 }
 __global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* __restrict__ z, long ldz, __nv_bfloat16* __restrict__ out, long ldo, long total8,
-                                                           int F, int blk, float alpha, float limit) {
+                                                           int F, int blk, const Glu u) {
   grid_dep_wait();
   grid_dep_launch();
   const int f8 = F >> 3;
@@ -303,13 +423,13 @@ __global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* 
     const bf16x8 a = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i : i)), b = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i + 8 : F + i));
     bf16x8 o;
     if (blk) {
-      o.v[0] = clamped_glu2(a.v[0], a.v[2], alpha, limit);
-      o.v[1] = clamped_glu2(a.v[1], a.v[3], alpha, limit);
-      o.v[2] = clamped_glu2(b.v[0], b.v[2], alpha, limit);
-      o.v[3] = clamped_glu2(b.v[1], b.v[3], alpha, limit);
+      o.v[0] = clamped_glu2(a.v[0], a.v[2], u);
+      o.v[1] = clamped_glu2(a.v[1], a.v[3], u);
+      o.v[2] = clamped_glu2(b.v[0], b.v[2], u);
+      o.v[3] = clamped_glu2(b.v[1], b.v[3], u);
     } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o.v[e] = clamped_glu2(a.v[e], b.v[e], alpha, limit);
+      for (int e = 0; e < 4; ++e) o.v[e] = clamped_glu2(a.v[e], b.v[e], u);
     }
     *reinterpret_cast<bf16x8*>(out + row * ldo + i) = o;
   }
@@ -381,11 +501,12 @@ using namespace ve;
 extern "C" {
 
 // f32: 1 = activations and tables fp32, 0 = bf16. out [rows][S][H]; pos and freq may be null.
-int ve_embed_rows(const void* ids, const void* table, const void* pos, const void* freq, void* out, int rows, int H, int vocab, int S, int f32, cudaStream_t st) {
+int ve_embed_rows(const void* ids, const void* table, const void* pos, const void* freq, void* out, int rows, int H, int vocab, int S, float scale, int f32,
+                  cudaStream_t st) {
   if (rows <= 0) return 0;
   if (S < 1 || (freq && !pos)) return cudaErrorInvalidValue;
 #define VE_EM(T) launch_pdl(embed_rows_kernel<T>, dim3(rows), dim3(row_threads(H)), 0, st, (const int*)ids, (const T*)table, (const int*)pos, \
-    (const double*)freq, (float*)out, H, vocab, S)
+    (const double*)freq, (float*)out, H, vocab, S, scale)
   if (f32) VE_EM(float);
   else VE_EM(__nv_bfloat16);
 #undef VE_EM
@@ -419,18 +540,51 @@ int ve_stream_norm(void* h, const void* part, long ldp, const void* mix, const v
   VE_CHECK_LAUNCH();
 }
 
-// z rows [gate F | up F] (blk 0) or blocks of [4 gate | 4 up] (F a multiple of 4); fp32 when x32, else of the activation type.
-int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, int blk, float alpha, float limit, int f32, cudaStream_t st) {
+// h [rows][H] contiguous fp32 += RMS norm of the result * wa (wa null: no result); out = h, or its RMS norm * wo (null: not normed; out null: no
+// output). top > 0: a row's result is the sum of rw [rows][top] times rows inv [rows][top] (null: in order) of part.
+int ve_residual_norm(void* h, const void* part, long ldp, const void* inv, const void* rw, int top, const void* wa, const void* wo, void* out, long ldo, int rows,
+                     int H, float eps, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
+  if (H < 1 || top < 0 || (wa && !part) || (top && !rw) || (!wa && !out)) return cudaErrorInvalidValue;
+  const ResultRows rr{(const int*)inv, (const float*)rw, wa ? top : 0};
+  const bool vec = !f32 && H % 4 == 0 && H <= 8192 && ldp % 4 == 0 && ldo % 4 == 0 && !(((uintptr_t)h | (uintptr_t)wa | (uintptr_t)wo) & 15) &&
+                   !(((uintptr_t)part | (uintptr_t)out) & 7);
+  if (f32) launch_pdl(residual_norm_kernel<float>, dim3(rows), dim3(256), 0, st, (float*)h, (const float*)part, ldp, rr, (const float*)wa, (const float*)wo,
+                      (float*)out, ldo, H, eps);
+  else if (!vec) launch_pdl(residual_norm_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, (float*)h, (const __nv_bfloat16*)part, ldp, rr, (const float*)wa,
+                            (const float*)wo, (__nv_bfloat16*)out, ldo, H, eps);
+#define VE_RN(NV) launch_pdl(residual_norm4_kernel<NV, __nv_bfloat16>, dim3(rows), dim3(256), 0, st, (float*)h, (const __nv_bfloat16*)part, ldp, rr, \
+    (const float*)wa, (const float*)wo, (__nv_bfloat16*)out, ldo, H, eps)
+  else if (H <= 1024) VE_RN(1);
+  else if (H <= 2048) VE_RN(2);
+  else if (H <= 4096) VE_RN(4);
+  else VE_RN(8);
+#undef VE_RN
+  VE_CHECK_LAUNCH();
+}
+
+int ve_soft_cap(void* x, long n, float cap, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return cudaErrorInvalidValue;
+  const long blocks = (n + 255) / 256;
+  launch_pdl(soft_cap_kernel, dim3((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), 0, st, (float*)x, n, cap);
+  VE_CHECK_LAUNCH();
+}
+
+// z rows [gate F | up F] (blk 0) or blocks of [4 gate | 4 up] (F a multiple of 4); fp32 when x32, else of the activation type.
+int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, int blk, float alpha, float limit, float shift, int f32,
+                   cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const Glu u{alpha, limit, shift};
   if (F < 1 || (blk && F % 4)) return cudaErrorInvalidValue;
   const bool vec = !f32 && !x32 && F % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && !((uintptr_t)z & 15) && !((uintptr_t)out & 15);
   const long total = (long)rows * F / (vec ? 8 : 1), blocks = (total + 255) / 256;
   const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
   if (vec) {
-    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, blk, alpha, limit);
+    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, blk, u);
     VE_CHECK_LAUNCH();
   }
-#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, blk, alpha, limit)
+#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, blk, u)
   if (f32) VE_CG(float, float);
   else if (x32) VE_CG(float, __nv_bfloat16);
   else VE_CG(__nv_bfloat16, __nv_bfloat16);

@@ -13,6 +13,7 @@ from dataclasses import dataclass
 import torch
 
 from ..ops.rowops import DynamicTanh, PolyNorm, embed_rows
+from .feed_forward import DenseFF
 from .listed import ListedConfig, ListedLayer, ListedModel, RandomTensors, save_listed
 from .mixers import MIXERS, make_linear
 
@@ -42,8 +43,7 @@ class FofosunModel(ListedModel):
         L = ListedLayer(MIXERS[spec["type"]](spec["type"], spec["mixer"], eps, src, p + "mix.", dev, dt), DynamicTanh.load(src, p + "norm1", dev), f32(p + "ls1"))
         if spec.get("mlp") is not None:
             L.norm2, L.write2 = DynamicTanh.load(src, p + "norm2", dev), f32(p + "ls2")
-            L.up, L.down = make_linear(src, p + "mlp.up", dev, dt), make_linear(src, p + "mlp.down", dev, dt)
-            L.act = PolyNorm(f32(p + "mlp.act"), eps)
+            L.ff = DenseFF(make_linear(src, p + "mlp.up", dev, dt), PolyNorm(f32(p + "mlp.act"), eps), make_linear(src, p + "mlp.down", dev, dt))
         return L
 
     def embed_batch(self, b):

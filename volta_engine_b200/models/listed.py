@@ -1,15 +1,15 @@
 """Decoders whose configuration lists its layers one by one: every layer has a token mixer of its own type and sizes
-(:mod:`.mixers`) and an optional feed-forward, with a norm in front of each and an fp32 residual. A range of layers may run several
-times in a row with the same weights; every pass has its own cache layer and state.
+(:mod:`.mixers`) and an optional feed-forward, with a norm in front of each (or behind it, on its result) and an fp32 residual. A range
+of layers may run several times in a row with the same weights; every pass has its own cache layer and state.
 
 A design supplies the parts (:meth:`ListedModel.load_layer`, ``load_ends``, ``embed_batch``); loading order, cache layers, state
 slots, batches and the forward pass are here. A layer's parts are row operators of :mod:`..ops.rowops`:
 
   norm1, norm2     ``rows(h, dtype, part, write)``: the sublayer result in front enters the residual, then the norm of it;
                    ``prologue(h)``: the norm as the prologue of a decode linear
-  write1, write2   how a sublayer's result enters the residual (an element-wise scale, or a StreamWrite)
-  up, act, down    the feed-forward: linear, row operator, linear; in decode steps the operator is the epilogue of the first linear
-                   (``act.epilogue()``) or the prologue of the second
+  write1, write2   how a sublayer's result enters the residual (an element-wise scale, a StreamWrite, or a NormedWrite: that one needs
+                   whole rows, so the reader behind adds the result)
+  ff               the feed-forward (:mod:`.feed_forward`)
 """
 from __future__ import annotations
 
@@ -20,8 +20,8 @@ from pathlib import Path
 
 import torch
 
-from ..ops.rowops import fused_fits, gemv_rows
-from ..runtime.batch import BatchRows
+from ..ops.rowops import RoutedRows, fused_fits, gemv_rows, soft_cap_
+from ..runtime.batch import LOGITS_ALL, BatchRows
 from .dense import DenseConfig, DenseModel
 from .mixers import MIXERS, apply_linear
 from .slot_state import SlotStates
@@ -37,13 +37,13 @@ class ListedConfig(DenseConfig):
     residual: str = "fp32"
 
     @classmethod
-    def listed(cls, c: dict, **kw):
-        """The fields every design of this form has."""
+    def listed(cls, c: dict, feed_forwards=("dense",), **kw):
+        """The fields every design of this form has. ``feed_forwards``: the kinds the design has."""
         layers = [dict(L) for L in c["layers"]]
         for i, L in enumerate(layers):
             if L["type"] not in MIXERS:
                 raise NotImplementedError(f"layer {i}: no mixer {L['type']!r} in this build")
-            if L.get("mlp") is not None and L["mlp"].get("kind", "dense") != "dense":
+            if L.get("mlp") is not None and L["mlp"].get("kind", "dense") not in feed_forwards:
                 raise NotImplementedError(f"layer {i}: no feed-forward {L['mlp']['kind']!r} in this build")
         lp = c.get("loop")
         loop = (int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else (0, 0, 1)
@@ -51,7 +51,7 @@ class ListedConfig(DenseConfig):
             raise ValueError(f"loop over layers {loop[0]} .. {loop[1]} of {len(layers)}, {loop[2]} times")
         widths = [MIXERS[L["type"]].row_widths(L["mixer"]) for L in layers]
         return cls(n_layers=len(layers), hidden=int(c["width"]), vocab=int(c["vocab"]), rms_eps=float(c["norm"]["eps"]), layers=layers, loop=loop,
-                   n_q=1, n_kv=1, ffn=max([int(L["mlp"]["ff"]) for L in layers if L.get("mlp") is not None] or [1]), quant="bf16",
+                   n_q=1, n_kv=1, ffn=max([int((L["mlp"].get("expert") or L["mlp"])["ff"]) for L in layers if L.get("mlp") is not None] or [1]), quant="bf16",
                    head_dim=max([k for k, _ in widths] + [0]) or 64, v_width=max([v for _, v in widths] + [8]), **kw)
 
     def runs(self) -> list:
@@ -61,17 +61,51 @@ class ListedConfig(DenseConfig):
 
 
 class ListedLayer:
-    __slots__ = ("mixer", "norm1", "write1", "norm2", "write2", "up", "act", "down")
+    __slots__ = ("mixer", "norm1", "write1", "norm2", "write2", "ff")
 
     def __init__(self, mixer, norm1, write1):
         self.mixer, self.norm1, self.write1 = mixer, norm1, write1
-        self.norm2 = self.write2 = self.up = self.act = self.down = None
+        self.norm2 = self.write2 = self.ff = None
 
     def again(self) -> "ListedLayer":
         """Another pass of this layer: the same weights, a cache layer and a state of its own."""
         L = copy.copy(self)
         L.mixer = copy.copy(self.mixer)
         return L
+
+
+def read_rows(norm, h, dtype, part, write):
+    """``norm.rows``; results of a routed feed-forward are summed in front of norms that do not sum them."""
+    if isinstance(part, RoutedRows) and not getattr(norm, "takes_routed", False):
+        part = part.tensor()
+    return norm.rows(h, dtype, part, write)
+
+
+class StepResidual:
+    """The residual of a decode step whose linears carry norms and updates, with a result that the next reader adds to it."""
+
+    def __init__(self, h):
+        self.h, self.part, self.write = h, None, None
+
+    def read(self, norm) -> dict:
+        """Operands of a linear that reads the residual through ``norm``."""
+        if self.part is None:
+            return norm.prologue(self.h)
+        pro = norm.prologue(self.h, self.part, self.write)
+        self.h, self.part = pro["h_out"], None
+        return pro
+
+    def put(self, write):
+        """-> ``finish(linear, **operands)``: the linear whose result enters the residual through ``write``."""
+        def finish(lin, **pro):
+            if getattr(write, "deferred", False):
+                self.later(gemv_rows(lin, self.h.shape[0], out_f32=True, **pro), write)
+            else:
+                gemv_rows(lin, self.h.shape[0], residual=(self.h, write), **pro)
+        return finish
+
+    def later(self, part, write):
+        self.part, self.write = part, write
 
 
 class ListedModel(SlotStates, DenseModel):
@@ -129,20 +163,21 @@ class ListedModel(SlotStates, DenseModel):
         pass
 
     @staticmethod
-    def _layer_bytes(layers) -> int:
+    def _layer_bytes(layers, step: bool) -> int:
         n = 0
         for L in layers:
             n += sum(lin.nbytes() for lin in L.mixer.linears()) + L.mixer.extra_bytes()
-            if L.up is not None:
-                n += L.up.nbytes() + L.down.nbytes()
+            if L.ff is not None:
+                n += L.ff.nbytes(step)
         return n
 
     def decode_bytes_per_token(self) -> int:
-        """Weight bytes a decode step reads (a looped layer's once per pass)."""
-        return self.lm_head.nbytes() + self._layer_bytes(self.layers)
+        """Weight bytes a decode step of one row reads (a looped layer's once per pass)."""
+        return self.lm_head.nbytes() + self._layer_bytes(self.layers, True)
 
     def weight_bytes(self) -> int:
-        return self.lm_head.nbytes() + self._layer_bytes(self.own_layers) + self.embed.numel() * self.embed.element_size()
+        tied = self.lm_head.weight.data_ptr() == self.embed.data_ptr()
+        return self.lm_head.nbytes() + self._layer_bytes(self.own_layers, False) + (0 if tied else self.embed.numel() * self.embed.element_size())
 
     # ------------------------------------------------------------------------------------------ state slots
     def _states(self, kv) -> list:
@@ -175,38 +210,47 @@ class ListedModel(SlotStates, DenseModel):
             return self._forward_fused(b, kv, h)
         dt, part, write = self.dtype, None, None
         for li, L in enumerate(self.layers):
-            x = L.norm1.rows(h, dt, part, write)
+            x = read_rows(L.norm1, h, dt, part, write)
             part, write = L.mixer.rows(x, b, kv, self._journal(li, L, b, kv)), L.write1
-            if L.up is not None:
-                x = L.norm2.rows(h, dt, part, write)
-                z = apply_linear(L.up, x, out_f32=b.row_path)
-                part, write = apply_linear(L.down, L.act.rows(z, dt)), L.write2
+            if L.ff is not None:
+                x = read_rows(L.norm2, h, dt, part, write)
+                part, write = L.ff.rows(x, b), L.write2
             if self.layer_tap is not None:
                 self.layer_tap.append(self.residual_rows(h, part, write))
-        x = self.final_norm.rows(h, dt, part, write)
+        x = read_rows(self.final_norm, h, dt, part, write)
         self.last_hidden, self.last_residual = x, h
         x = b.select_logits(x)
-        return None if x is None else apply_linear(self.lm_head, x, out_f32=True)
+        return None if x is None else self.capped(apply_linear(self.lm_head, x, out_f32=True))
+
+    def capped(self, logits):
+        return soft_cap_(logits, self.cfg.logit_softcap) if self.cfg.logit_softcap > 0 else logits
 
     def _forward_fused(self, b: BatchRows, kv, h):
         """A few decode rows: norms, activations and residual updates ride in the linears' launches."""
+        res = StepResidual(h)
         for li, L in enumerate(self.layers):
-            L.mixer.step(L.norm1.prologue(h), (h, L.write1), b, kv, self._journal(li, L, b, kv))
-            if L.up is not None:
-                epi = L.act.epilogue()
-                z = gemv_rows(L.up, b.n, out_f32=epi is None, **L.norm2.prologue(h), **(epi or {}))
-                gemv_rows(L.down, b.n, residual=(h, L.write2), **(L.act.prologue(z) if epi is None else {"x": z}))
+            L.mixer.step(res.read(L.norm1), res.put(L.write1), b, kv, self._journal(li, L, b, kv))
+            if L.ff is not None:
+                L.ff.step(res, L.norm2, L.write2, b)
             if self.layer_tap is not None:
-                self.layer_tap.append(self.residual_rows(h))
-        self.last_residual = h
-        h = b.select_logits(h)
-        return None if h is None else gemv_rows(self.lm_head, h.shape[0], out_f32=True, **self.final_norm.prologue(h))
+                self.layer_tap.append(self.residual_rows(res.h, res.part, res.write))
+        if res.part is not None and b.logits != LOGITS_ALL:          # the head reads some of the rows
+            self.final_norm.rows(res.h, torch.float32, res.part, res.write)
+            res.part = None
+        pro = res.read(self.final_norm)
+        self.last_residual = res.h
+        if b.logits != LOGITS_ALL:
+            h = b.select_logits(res.h)
+            if h is None:
+                return None
+            pro = self.final_norm.prologue(h)
+        return gemv_rows(self.lm_head, pro["x"].shape[0], out_f32=True, cap=self.cfg.logit_softcap, **pro)
 
     def _widest(self):
         """The linear with the longest input rows of those that take a prologue."""
         w = getattr(self, "_widest_lin", None)
         if w is None:
-            lins = [self.lm_head] + [x for L in self.own_layers for x in (*L.mixer.linears(), L.up, L.down) if x is not None]
+            lins = [self.lm_head] + [x for L in self.own_layers for x in (*L.mixer.linears(), *(L.ff.linears() if L.ff is not None else ()))]
             w = self._widest_lin = max(lins, key=lambda x: x.weight.shape[1])
         return w
 

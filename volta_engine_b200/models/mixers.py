@@ -1,6 +1,6 @@
 """Token mixers of decoders whose ``config.json`` lists its layers one by one, each with its own mixer type and sizes. A mixer
 reads normed rows and returns the rows of its output projection; ``step`` is the same on a few decode rows with the norm in
-front, the layer scale and the residual add inside the linears' launches.
+front, the layer scale and the residual add inside the linears' launches (``finish(linear, **operands)`` runs the last one).
 
 ``MIXERS`` maps the type names to classes; a class takes (mixer sizes, eps, tensor source, name prefix, device, dtype).
 """
@@ -14,6 +14,7 @@ from ..ops.gqa import GqaSpec, distance_bias, gqa_attend
 from ..ops.latent import LatentSpec, latent_rows
 from ..ops.linear import LinearBF16, LinearF32
 from ..ops.linear_attn import LinAttnSpec, LinAttnState, linattn_rows
+from ..ops.rotary import Rotation
 from ..ops.rowops import GroupRMS, gemv_rows
 
 
@@ -31,6 +32,16 @@ def apply_linear(lin, x, out_f32: bool = False):
     if x.is_cuda and isinstance(lin, LinearBF16) and x.shape[0] <= 16:
         return gemv_rows(lin, x.shape[0], x=x, out_f32=out_f32)
     return lin.forward(x, out_f32=out_f32)
+
+
+def window_of(m: dict) -> int:
+    """Size of a mixer's sliding window (0: none)."""
+    mask = m.get("mask")
+    if not mask:
+        return 0
+    if int(mask["size"]) < 1:
+        raise ValueError(f"a window of {mask['size']} keys")
+    return int(mask["size"])
 
 
 class Mixer:
@@ -107,10 +118,10 @@ class LinearRecurrence(Mixer):
         o = self.recur(proj, b, kv, journal, self.dtype != torch.float32)
         return apply_linear(self.out, self.norm.rows(o, self.dtype, gate=self.gate(proj)))
 
-    def step(self, pro, residual, b, kv, journal=(None, None)):
+    def step(self, pro, finish, b, kv, journal=(None, None)):
         proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
         o = self.recur(proj, b, kv, journal, True)
-        gemv_rows(self.out, b.n, residual=residual, **self.norm.prologue(o, self.gate(proj)))
+        finish(self.out, **self.norm.prologue(o, self.gate(proj)))
 
 
 class GroupedAttention(Mixer):
@@ -145,9 +156,31 @@ class GroupedAttention(Mixer):
         proj = apply_linear(self.in_proj, x, out_f32=True)
         return apply_linear(self.out, self.attend(proj, b, kv, self._out(proj)))
 
-    def step(self, pro, residual, b, kv, journal=None):
+    def step(self, pro, finish, b, kv, journal=None):
         proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
-        gemv_rows(self.out, b.n, residual=residual, x=self.attend(proj, b, kv, self._out(proj)))
+        finish(self.out, x=self.attend(proj, b, kv, self._out(proj)))
+
+
+class WindowedAttention(GroupedAttention):
+    """Grouped-query softmax attention with rotary positions, queries and keys brought to unit root mean square behind them, a sliding
+    window, a sink, and a sigmoid gate on the result; one fused input projection [q | k | v | gate]."""
+    PARTS = ("q", "k", "v", "g")
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
+        rot = m.get("rot")
+        self.spec = GqaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), eps, unit=True, gated=True,
+                            sink=src.tensor(p + "sink", device, torch.float32).reshape(-1).contiguous(), window=window_of(m),
+                            rot=Rotation.from_config(rot, False).bind(device) if rot else None)
+        if rot and self.spec.rot.dims > self.spec.dim:
+            raise ValueError(f"{p}: {self.spec.rot.dims} rotated columns of {self.spec.dim}")
+        self.parts = [p + n for n in self.PARTS]
+        self.in_proj = make_linear(src, self.parts, device, dtype)
+        self.out = make_linear(src, p + "o", device, dtype)
+        self.dtype = dtype
+
+    def rows(self, x, b, kv, journal=None):
+        proj = apply_linear(self.in_proj, x, out_f32=b.row_path)
+        return apply_linear(self.out, self.attend(proj, b, kv, self._out(proj)))
 
 
 class Parallel(Mixer):
@@ -195,62 +228,69 @@ class Parallel(Mixer):
         self.right.norm.rows(o, self.dtype, gate=self.right.gate(pr), out=y[:, self.k0:])
         return apply_linear(self.out, y)
 
-    def step(self, pro, residual, b, kv, journal=(None, None)):
+    def step(self, pro, finish, b, kv, journal=(None, None)):
         proj = gemv_rows(self.in_proj, b.n, out_f32=True, **pro)
         att = self.left.attend(proj, b, kv, torch.empty(b.n, self.k0, dtype=torch.float32, device=proj.device))
         pr = proj[:, self.left.spec.cols:]
         o = self.right.recur(pr, b, kv, journal, True)
-        gemv_rows(self.out, b.n, residual=residual, **self.right.norm.prologue(o, self.right.gate(pr), head=att))
+        finish(self.out, **self.right.norm.prologue(o, self.right.gate(pr), head=att))
 
 
 class LatentAttention(Mixer):
-    """Multi-head attention over a low-rank latent per token, with a low-rank query and a rotated key part shared by the heads."""
+    """Multi-head attention over a low-rank latent per token and a rotated key part shared by the heads, with a sliding window or
+    without. Queries come from a normed low-rank projection, or (no ``q_rank``) straight from the input: then one fused input
+    projection [q | latent and rotated part]."""
     cached = True
 
     @staticmethod
     def row_widths(m: dict) -> tuple[int, int]:
-        return LatentSpec(1, 1, int(m["rot_dim"]), 1, int(m["kv_rank"]), 1.0, 1.0, 1e-5).width, 0
+        return LatentSpec(1, 1, int(m["rot_dim"]), 1, int(m["kv_rank"]), 1.0, 2.0, 1e-5).width, 0
 
     def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
         rot = m["rot"]
         if int(rot["dims"]) != int(m["rot_dim"]):
             raise ValueError(f"{p}: the rotated part is turned as a whole")
         self.spec = LatentSpec(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]),
-                               float(rot["base"]), eps).bind(device)
-        self.q_rank = int(m["q_rank"])
+                               float(rot["base"]), eps, rot.get("scaling"), window_of(m)).bind(device)
         f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
-        self.down = make_linear(src, [p + "dq", p + "dkv"], device, dtype)
-        self.uq = make_linear(src, p + "uq", device, dtype)
+        self.q_rank = int(m.get("q_rank") or 0)
+        self.split = self.q_rank or self.spec.heads * (self.spec.dim + self.spec.rot)        # columns in front of the latent
+        self.down = make_linear(src, [p + ("dq" if self.q_rank else "q"), p + "dkv"], device, dtype)
+        self.uq = make_linear(src, p + "uq", device, dtype) if self.q_rank else None
         self.w_uk = src.tensor(p + "uk", device, dtype).contiguous()
         self.w_uv = src.tensor(p + "uv", device, dtype).contiguous()
         self.ukv = LinearBF16(torch.cat([self.w_uk, self.w_uv], 0)) if dtype != torch.float32 else None
         if self.ukv is not None and self.ukv.weight.shape[1] == self.spec.kv_rank:      # one copy: the absorbed form reads slices of the stacked weight
             self.w_uk, self.w_uv = self.ukv.weight[: self.w_uk.shape[0]], self.ukv.weight[self.w_uk.shape[0]:]
         self.out = make_linear(src, p + "o", device, dtype)
-        self.q_norm = GroupRMS(f32("dq.norm"), eps)
+        self.q_norm = GroupRMS(f32("dq.norm"), eps) if self.q_rank else None
         self.kv_norm = f32("dkv.norm")
         self.dtype = dtype
 
     def linears(self):
-        return [self.down, self.uq, self.out]
+        return [x for x in (self.down, self.uq, self.out) if x is not None]
 
     def extra_bytes(self) -> int:
         return (self.w_uk.numel() + self.w_uv.numel()) * self.w_uk.element_size()
 
     def _attend(self, q, a, b, kv):
-        return latent_rows(self.spec, q, a[:, self.q_rank:], self.kv_norm, self.w_uk, self.w_uv, self.ukv, b, kv, kv.k[self.cache_index])
+        return latent_rows(self.spec, q, a[:, self.split:], self.kv_norm, self.w_uk, self.w_uv, self.ukv, b, kv, kv.k[self.cache_index])
 
     def rows(self, x, b, kv, journal=None):
-        a = apply_linear(self.down, x, out_f32=True)
-        q = apply_linear(self.uq, self.q_norm.rows(a[:, : self.q_rank], self.dtype), out_f32=x.shape[0] <= 16)
+        few = x.shape[0] <= 16
+        if self.uq is None:
+            a = apply_linear(self.down, x, out_f32=few)
+            q = a[:, : self.split]
+        else:
+            a = apply_linear(self.down, x, out_f32=True)
+            q = apply_linear(self.uq, self.q_norm.rows(a[:, : self.q_rank], self.dtype), out_f32=few)
         return apply_linear(self.out, self._attend(q, a, b, kv))
 
-    def step(self, pro, residual, b, kv, journal=None):
+    def step(self, pro, finish, b, kv, journal=None):
         a = gemv_rows(self.down, b.n, out_f32=True, **pro)
-        q = gemv_rows(self.uq, b.n, out_f32=True, **self.q_norm.prologue(a[:, : self.q_rank]))
-        att = self._attend(q, a, b, kv)
-        gemv_rows(self.out, b.n, residual=residual, x=att)
+        q = a[:, : self.split] if self.uq is None else gemv_rows(self.uq, b.n, out_f32=True, **self.q_norm.prologue(a[:, : self.q_rank]))
+        finish(self.out, x=self._attend(q, a, b, kv))
 
 
 MIXERS = {"hgrn2": LinearRecurrence, "lightning": LinearRecurrence, "latent_attention": LatentAttention,
-          "gated_linear_attention": LinearRecurrence, "grouped_attention": GroupedAttention, "parallel": Parallel}
+          "gated_linear_attention": LinearRecurrence, "grouped_attention": GroupedAttention, "parallel": Parallel, "attention": WindowedAttention}

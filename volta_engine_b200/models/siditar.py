@@ -14,6 +14,7 @@ from dataclasses import dataclass
 import torch
 
 from ..ops.rowops import ClampedGlu, SinusoidalPositions, StreamNorm, StreamWrite, embed_rows
+from .feed_forward import DenseFF
 from .listed import ListedConfig, ListedLayer, ListedModel, RandomTensors, save_listed
 from .mixers import MIXERS, make_linear
 
@@ -53,10 +54,7 @@ class SiditarModel(ListedModel):
         L = ListedLayer(MIXERS[spec["type"]](spec["type"], spec["mixer"], eps, src, p + "mix.", dev, dt), norm(1), write(1))
         if spec.get("mlp") is not None:
             L.norm2, L.write2 = norm(2), write(2)
-            halves = [p + "mlp.gate", p + "mlp.up"]
-            blocks = int(spec["mlp"]["ff"]) % 8 == 0
-            L.up = make_linear(src, halves, dev, dt, join=ClampedGlu.interleave if blocks else None)
-            L.down, L.act = make_linear(src, p + "mlp.down", dev, dt), ClampedGlu(float(spec["mlp"]["limit"]), GLU_ALPHA, blocks)
+            L.ff = DenseFF.gated(src, p + "mlp.", ClampedGlu(float(spec["mlp"]["limit"]), GLU_ALPHA), dev, dt)
         return L
 
     def embed_batch(self, b):

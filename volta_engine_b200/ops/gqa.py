@@ -1,6 +1,6 @@
-"""Grouped-query softmax attention with its sizes and score terms as parameters (csrc/cuda/gqa.cu): RMS norm of queries and keys,
-query temperature by position, bias by distance, sink, unlike query / key and value widths. Positions enter through the temperature
-and the bias only.
+"""Grouped-query softmax attention with its sizes and score terms as parameters (csrc/cuda/gqa.cu): rotary positions, RMS norm of
+queries and keys behind them (with or without a weight), query temperature by position, sliding window, bias by distance, sink, output
+gate, unlike query / key and value widths.
 
 The paged cache's rows are as wide as the widest layer needs (``row_widths``); a layer sees a page as [kv heads, 64, width].
 
@@ -16,6 +16,7 @@ import torch
 
 from .._lib import call, ptr
 from . import kernels as K
+from .rotary import Rotation
 
 PAGE = K.PAGE
 MAX_TICKETS = 1 << 16
@@ -60,6 +61,10 @@ class GqaSpec:
     bias: torch.Tensor | None = None          # fp32 [heads, L] (distance_bias)
     sink: torch.Tensor | None = None          # fp32 [heads]: log of one more term of the denominator
     out_scale: float = 1.0                    # factor on the result
+    rot: Rotation | None = None               # of queries and keys, in front of their norm
+    unit: bool = False                        # queries and keys are normed without a weight
+    window: int = 0                           # a key is seen at distances below it (0: all in front)
+    gated: bool = False                       # columns behind the values: the result is multiplied with their sigmoid
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
@@ -69,8 +74,16 @@ class GqaSpec:
 
     @property
     def cols(self) -> int:
-        """Columns of a projection row [q | k | v]."""
+        """Columns of a projection row [q | k | v | gate]."""
+        return self.gate_col + (self.heads * self.vdim if self.gated else 0)
+
+    @property
+    def gate_col(self) -> int:
         return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+
+    def gate(self, proj):
+        """The gate's columns of projection rows."""
+        return proj[:, self.gate_col: self.cols] if self.gated else None
 
     @property
     def row_widths(self) -> tuple[int, int]:
@@ -89,8 +102,11 @@ class GqaSpec:
         return 1.0 + self.temp_coef * torch.log(((pos + 1) // self.temp_every + 1).float()) if self.temp_every > 0 else torch.ones(pos.shape)
 
 
-def _norm(v, w, eps):
-    return v if w is None else v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w
+def _norm(v, w, unit, eps):
+    if w is None and not unit:
+        return v
+    v = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+    return v if w is None else v * w
 
 
 def gqa_reference(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
@@ -98,10 +114,12 @@ def gqa_reference(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
     n, H, G, d, dv = proj.shape[0], spec.heads, spec.kv_heads, spec.dim, spec.vdim
     dt = kpool.dtype
     pf = proj.float()
-    q = _norm(pf[:, : H * d].reshape(n, H, d), spec.q_norm, spec.eps) * spec.temperature(b.pos)[:, None, None]
+    turn = (lambda x: spec.rot.turn(x, b.pos)) if spec.rot is not None else (lambda x: x)
+    q = _norm(turn(pf[:, : H * d].reshape(n, H, d)), spec.q_norm, spec.unit, spec.eps) * spec.temperature(b.pos)[:, None, None]
     q = q.to(dt).float()
-    k = _norm(pf[:, H * d: (H + G) * d].reshape(n, G, d), spec.k_norm, spec.eps)
-    v = pf[:, (H + G) * d: spec.cols].reshape(n, G, dv)
+    k = _norm(turn(pf[:, H * d: (H + G) * d].reshape(n, G, d)), spec.k_norm, spec.unit, spec.eps)
+    v = pf[:, (H + G) * d: spec.gate_col].reshape(n, G, dv)
+    gate = torch.sigmoid(spec.gate(pf)) if spec.gated else None
     kp = kpool.reshape(kpool.shape[0], -1)[:, : G * PAGE * spec.kw].view(-1, G, PAGE, spec.kw)
     vp = vpool.reshape(vpool.shape[0], -1)[:, : G * PAGE * spec.vw].view(-1, G, PAGE, spec.vw)
     rows = [(i, int(b.slot[i]), int(b.pos[i])) for i in range(n)]
@@ -114,16 +132,18 @@ def gqa_reference(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
         if s < 0:
             out[i] = 0
             continue
-        pgs = cache.page_table[s, : p // PAGE + 1].long()
-        ks = kp[pgs].transpose(1, 2).reshape(-1, G, spec.kw)[: p + 1, :, :d].float()
-        vs = vp[pgs].transpose(1, 2).reshape(-1, G, spec.vw)[: p + 1, :, :dv].float()
+        a = max(0, p - spec.window + 1) if spec.window else 0          # first key it sees
+        pgs, o = cache.page_table[s, a // PAGE: p // PAGE + 1].long(), a // PAGE * PAGE
+        ks = kp[pgs].transpose(1, 2).reshape(-1, G, spec.kw)[a - o: p + 1 - o, :, :d].float()
+        vs = vp[pgs].transpose(1, 2).reshape(-1, G, spec.vw)[a - o: p + 1 - o, :, :dv].float()
         sc = torch.einsum("gud,jgd->guj", q[i].reshape(G, spec.group, d), ks).reshape(H, -1) * spec.scale
         if spec.bias is not None:
-            sc = sc + spec.bias[:, (p - torch.arange(p + 1)).clamp(max=spec.bias.shape[1] - 1)]
+            sc = sc + spec.bias[:, (p - torch.arange(a, p + 1)).clamp(max=spec.bias.shape[1] - 1)]
         if spec.sink is not None:
             sc = torch.cat([sc, spec.sink[:, None]], 1)
-        pr = torch.softmax(sc, -1)[:, : p + 1].reshape(G, spec.group, -1)
-        out[i] = (torch.einsum("guj,jgv->guv", pr, vs) * spec.out_scale).reshape(-1).to(out.dtype)
+        pr = torch.softmax(sc, -1)[:, : p + 1 - a].reshape(G, spec.group, -1)
+        r = (torch.einsum("guj,jgv->guv", pr, vs) * spec.out_scale).reshape(-1)
+        out[i] = (r if gate is None else r * gate[i]).to(out.dtype)
     return out
 
 
@@ -137,7 +157,7 @@ def _ticket_words(dev):
     return t
 
 
-_D, _R, _S = "iiiiiill", "pppi", "fpipf"
+_D, _R, _S = "iiiiiill", "pppi", "fpipfipli"
 
 
 def _dims(spec, kpool, vpool):
@@ -148,58 +168,63 @@ def _rows(pos, slot, cache):
     return (ptr(pos), ptr(slot), ptr(cache.page_table), cache.page_table.shape[1])
 
 
-def _score(spec):
-    return (float(spec.scale), ptr(spec.bias), spec.bias.shape[1] if spec.bias is not None else 0, ptr(spec.sink), float(spec.out_scale))
+def _score(spec, gate):
+    return (float(spec.scale), ptr(spec.bias), spec.bias.shape[1] if spec.bias is not None else 0, ptr(spec.sink), float(spec.out_scale), spec.window,
+            ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.dtype == torch.float32))
 
 
 def gqa_store(spec: GqaSpec, proj, pos, slot, cache, kpool, vpool):
-    """Norms, temperature, cache rows -> queries [rows, heads, kw] of the cache's type."""
+    """Rotation, norms, temperature, cache rows -> queries [rows, heads, kw] of the cache's type."""
     n, f32 = proj.shape[0], kpool.dtype == torch.float32
     q = torch.empty(n, spec.heads, spec.kw, dtype=kpool.dtype, device=proj.device)
-    call("gqa_store", _D + _R + "pli" + "ppffi" + "pppii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), ptr(proj), proj.stride(0),
-         int(proj.dtype == torch.float32), ptr(spec.q_norm), ptr(spec.k_norm), float(spec.eps), float(spec.temp_coef), int(spec.temp_every), ptr(q), ptr(kpool),
+    rot = spec.rot
+    call("gqa_store", _D + _R + "pli" + "pifi" + "ippffi" + "pppii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), ptr(proj), proj.stride(0),
+         int(proj.dtype == torch.float32), ptr(rot.half_turns) if rot is not None else 0, rot.pairs if rot is not None else 0, rot.mul if rot is not None else 1.0,
+         int(rot is not None and rot.neighbours), int(spec.unit or spec.q_norm is not None or spec.k_norm is not None), ptr(spec.q_norm), ptr(spec.k_norm), float(spec.eps), float(spec.temp_coef), int(spec.temp_every), ptr(q), ptr(kpool),
          ptr(vpool), n, int(f32))
     return q
 
 
-def _each_row(spec, q, pos, slot, cache, kpool, vpool, out):
+def _each_row(spec, q, gate, pos, slot, cache, kpool, vpool, out):
     """Every row by itself: the split-key kernel, or the CUDA-core one."""
     n, dev, f32 = q.shape[0], q.device, kpool.dtype == torch.float32
     o32 = int(out.dtype == torch.float32)
     if f32 or not spec.tc_decode:
-        call("gqa_rows", _D + _R + _S + "ppp" + "pliii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec), ptr(q), ptr(kpool), ptr(vpool),
+        call("gqa_rows", _D + _R + _S + "ppp" + "pliii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate), ptr(q), ptr(kpool), ptr(vpool),
              ptr(out), out.stride(0), o32, n, int(f32))
         return
     units = n * spec.kv_heads * ((spec.group + 15) // 16)
-    nsplit = max(16, min(64, 148 // units)) if units <= MAX_TICKETS else 1          # a row takes as many of them as its position asks for
+    nsplit = max(16, min(64, 148 // units)) if units <= MAX_TICKETS else 1          # a row takes as many of them as its position asks for,
+    if spec.window:                                                                 # each at least two pages
+        nsplit = max(1, min(nsplit, ((spec.window + PAGE - 2) // PAGE + 2) // 2))
     part = lse = None
     if nsplit > 1:
         part = torch.empty(n, spec.heads, nsplit, spec.vdim, dtype=torch.float32, device=dev)
         lse = torch.empty(n, spec.heads, nsplit, dtype=torch.float32, device=dev)
-    call("gqa_decode", _D + _R + _S + "pppl" + "pppi" + "pliip", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec), ptr(q), ptr(kpool), ptr(vpool),
+    call("gqa_decode", _D + _R + _S + "pppl" + "pppi" + "pliip", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate), ptr(q), ptr(kpool), ptr(vpool),
          kpool.shape[0], ptr(part), ptr(lse), ptr(_ticket_words(dev)), nsplit, ptr(out), out.stride(0), o32, n, ptr(K.status_word(dev)))
 
 
 def gqa_attend(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
-    """All rows of batch ``b``: ``proj`` rows start with [q | k | v] as projected; the result goes to ``out`` [rows, heads * vdim] (a
+    """All rows of batch ``b``: ``proj`` rows start with [q | k | v | gate] as projected; the result goes to ``out`` [rows, heads * vdim] (a
     view of any row pitch; fp32, or bf16 as the cache). ``kpool`` / ``vpool``: this layer's pages."""
     if not proj.is_cuda:
         return gqa_reference(spec, proj, b, cache, kpool, vpool, out)
-    return gqa_scores(spec, gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool), b, cache, kpool, vpool, out)
+    return gqa_scores(spec, gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool), b, cache, kpool, vpool, out, spec.gate(proj))
 
 
-def gqa_scores(spec: GqaSpec, q, b, cache, kpool, vpool, out):
-    """Attention of the queries of ``gqa_store`` over the cached rows."""
+def gqa_scores(spec: GqaSpec, q, b, cache, kpool, vpool, out, gate=None):
+    """Attention of the queries of ``gqa_store`` over the cached rows. ``gate``: the gate's columns as projected."""
     n = q.shape[0]
     if b.row_path or kpool.dtype == torch.float32 or not spec.tc_prefill or out.dtype != torch.bfloat16:
-        _each_row(spec, q, b.pos, b.slot, cache, kpool, vpool, out)
+        _each_row(spec, q, gate, b.pos, b.slot, cache, kpool, vpool, out)
         return out
     t = b.segments()
     r0 = t.short_rows
     if r0:
-        _each_row(spec, q[:r0], b.pos[:r0], b.slot[:r0], cache, kpool, vpool, out[:r0])
+        _each_row(spec, q[:r0], None if gate is None else gate[:r0], b.pos[:r0], b.slot[:r0], cache, kpool, vpool, out[:r0])
     if r0 < n:
         tf, tc = t.tiles(128 // spec.group)
-        call("gqa_prefill", _D + _R + _S + "pppl" + "ppi" + "plp", *_dims(spec, kpool, vpool), *_rows(b.pos, b.slot, cache), *_score(spec), ptr(q), ptr(kpool),
+        call("gqa_prefill", _D + _R + _S + "pppl" + "ppi" + "plp", *_dims(spec, kpool, vpool), *_rows(b.pos, b.slot, cache), *_score(spec, gate), ptr(q), ptr(kpool),
              ptr(vpool), kpool.shape[0], ptr(tf), ptr(tc), tf.numel(), ptr(out), out.stride(0), ptr(K.status_word(q.device)))
     return out

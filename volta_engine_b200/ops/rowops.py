@@ -6,6 +6,7 @@ in fp32.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -107,11 +108,26 @@ class PolyNorm:
 
 @dataclass
 class ClampedGlu:
-    """Rows [gate | up]: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up clamped to +-limit. ``blocks``: the columns come
+    """Rows [gate | up]: g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = up clamped to +-limit. ``blocks``: the columns come
     as blocks of [4 gate | 4 up] (``interleave`` reorders a weight for it), which a decode linear can finish in its epilogue."""
     limit: float
     alpha: float
     blocks: bool = False
+    shift: float = 1.0
+
+    @classmethod
+    def silu(cls, blocks: bool = False):
+        """silu(gate) * up."""
+        return cls(math.inf, 1.0, blocks, 0.0)
+
+    @property
+    def constants(self) -> tuple:
+        return float(self.alpha), float(self.limit), float(self.shift)
+
+    def of(self, g, u):
+        """CPU statement on fp32 halves."""
+        g = g.clamp(max=self.limit)
+        return g * torch.sigmoid(self.alpha * g) * (u.clamp(-self.limit, self.limit) + self.shift)
 
     @staticmethod
     def interleave(gate, up):
@@ -123,20 +139,18 @@ class ClampedGlu:
         rows, F = z.shape[0], z.shape[1] // 2
         if not z.is_cuda:
             v = z.float().reshape(rows, F // 4, 2, 4).transpose(1, 2).reshape(rows, 2 * F) if self.blocks else z.float()
-            g, u = v[:, :F].clamp(max=self.limit), v[:, F:].clamp(-self.limit, self.limit)
-            return (g * torch.sigmoid(self.alpha * g) * (u + 1.0)).to(out_dtype)
+            return self.of(v[:, :F], v[:, F:]).to(out_dtype)
         out = torch.empty(rows, F, dtype=out_dtype, device=z.device)
-        call("clamped_glu", "plipliiiffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, int(self.blocks), float(self.alpha), float(self.limit),
-             _f32(out))
+        call("clamped_glu", "plipliiifffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, int(self.blocks), *self.constants, _f32(out))
         return out
 
     def epilogue(self):
         """Operands of a decode linear that ends with this operator; None: it goes into the prologue of the next one."""
-        return {"glu": (self.alpha, self.limit)} if self.blocks else None
+        return {"glu": self.constants} if self.blocks else None
 
     def prologue(self, z):
         assert not self.blocks
-        return {"pro": 5, "x": z, "kx": z.shape[1] // 2, "alpha": self.alpha, "eps": self.limit}
+        return {"pro": 5, "x": z, "kx": z.shape[1] // 2, "unit": self.constants}
 
 
 @dataclass
@@ -175,6 +189,68 @@ class StreamNorm:
         return {"pro": 4, "x": h.view(h.shape[0], S * H), "kx": H, "w": self.w, "G": S, "coef": self.read, "eps": self.eps}
 
 
+@dataclass
+class RoutedRows:
+    """Results of a routed feed-forward that are not summed yet: a row's result is sum_k w[row, k] d[inv[row, k]]."""
+    d: torch.Tensor           # [routes, H]
+    inv: torch.Tensor         # int32 [rows, top]
+    w: torch.Tensor           # fp32 [rows, top]
+
+    def tensor(self):
+        rows, top = self.w.shape
+        return torch.einsum("rk,rkh->rh", self.w, self.d[self.inv.long().reshape(-1)].reshape(rows, top, -1).float()).to(self.d.dtype)
+
+
+@dataclass
+class NormedWrite:
+    """How a sublayer's result enters the residual behind a norm of its own: h += RMS norm(y) * w (a factor on it is part of w).
+    Needs the whole row of y, so the linear that makes y cannot add it; the reader behind does (``ResidualNorm``)."""
+    w: torch.Tensor           # fp32 [H]
+    eps: float
+    deferred = True
+
+    def add(self, h, part):
+        p = (part.tensor() if isinstance(part, RoutedRows) else part).float()
+        h += p / torch.sqrt(p.pow(2).mean(-1, keepdim=True) + self.eps) * self.w
+
+
+@dataclass
+class ResidualNorm:
+    """What is read of an fp32 residual whose sublayers norm their results: the residual itself (``w`` None) or its RMS norm."""
+    w: torch.Tensor | None
+    eps: float
+    takes_routed = True
+
+    def rows(self, h, out_dtype, part=None, write: NormedWrite | None = None):
+        """The result in front enters the residual (in place, optional), then what is read of it."""
+        rows, H = h.shape
+        if not h.is_cuda:
+            if part is not None:
+                write.add(h, part)
+            v = h if self.w is None else h / torch.sqrt(h.pow(2).mean(-1, keepdim=True) + self.eps) * self.w
+            return v.to(out_dtype)
+        assert part is None or write.eps == self.eps
+        out = torch.empty(rows, H, dtype=out_dtype, device=h.device)
+        d, inv, w, top = (part.d, part.inv, part.w, part.w.shape[1]) if isinstance(part, RoutedRows) else (part, None, None, 0)
+        call("residual_norm", "pplppippplii" + "fi", ptr(h), ptr(d), d.stride(0) if d is not None else 0, ptr(inv), ptr(w), top,
+             ptr(write.w) if part is not None else 0, ptr(self.w), ptr(out), out.stride(0), rows, H, float(self.eps), _f32(out))
+        return out
+
+    def prologue(self, h, part=None, write: NormedWrite | None = None):
+        """``h_out``: the residual with ``part`` (fp32) in it, stored by the linear."""
+        assert part is None or write.eps == self.eps
+        return {"pro": 6, "x": h, "part": part, "w": write.w if part is not None else None, "b": self.w, "eps": self.eps,
+                "h_out": torch.empty(h.shape, dtype=torch.float32, device=h.device) if part is not None else None}
+
+
+def soft_cap_(x, cap: float):
+    """x <- cap tanh(x / cap), in place (fp32)."""
+    if not x.is_cuda:
+        return x.copy_(cap * torch.tanh(x / cap))
+    call("soft_cap", "plf", ptr(x), x.numel(), float(cap))
+    return x
+
+
 class SinusoidalPositions:
     """Position vectors: sine in column 2i, cosine in 2i + 1 of position * base^(-2i / width). Half circles per position are kept
     in double, so that angles are exact at any position."""
@@ -190,20 +266,20 @@ class SinusoidalPositions:
         return torch.stack([ang.sin(), ang.cos()], -1).flatten(1)[:, : self.width].float()
 
 
-def embed_rows(ids, table, pos=None, positions: SinusoidalPositions | None = None, streams: int = 0):
-    """-> fp32 [rows, H]; with ``positions`` their vectors of ``pos`` are added; with ``streams`` the rows come that many times
+def embed_rows(ids, table, pos=None, positions: SinusoidalPositions | None = None, streams: int = 0, scale: float = 1.0):
+    """-> fp32 [rows, H], times ``scale``; with ``positions`` their vectors of ``pos`` are added; with ``streams`` the rows come that many times
     ([rows, streams, H])."""
     S = max(1, streams)
     if not table.is_cuda:
-        x = table[ids.long()].float()
+        x = table[ids.long()].float() * scale
         if positions is not None:
             x = x + positions.vectors(pos)
         return x[:, None, :].repeat(1, S, 1) if streams else x
     V, H = table.shape
     n = ids.numel()
     out = torch.empty((n, S, H) if streams else (n, H), dtype=torch.float32, device=table.device)
-    call("embed_rows", "pppppiiiii", ptr(ids), ptr(table), ptr(pos) if positions is not None else 0, ptr(positions.half_turns) if positions is not None else 0,
-         ptr(out), n, H, V, S, _f32(table))
+    call("embed_rows", "pppppiiiifi", ptr(ids), ptr(table), ptr(pos) if positions is not None else 0, ptr(positions.half_turns) if positions is not None else 0,
+         ptr(out), n, H, V, S, float(scale), _f32(table))
     return out
 
 
@@ -213,9 +289,9 @@ def fused_fits(lin, rows: int) -> bool:
 
 
 def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, head=None, silu=False,
-              glu=None, out_f32=False, residual=None):
+              glu=None, unit=None, part=None, h_out=None, cap=0.0, out_f32=False, residual=None):
     """A bf16 linear on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
-    ``glu`` = (alpha, limit): the clamped gated unit of its outputs, which come in blocks, in bf16.
+    ``glu`` = (alpha, limit, shift): the clamped gated unit of its outputs, which come in blocks, in bf16. ``cap``: soft cap of fp32 outputs.
     ``residual`` = (h fp32, scale | None): h += scale * y in place, (streams, StreamWrite): the streams rewritten in place; otherwise
     the product is returned."""
     W = lin.weight
@@ -232,8 +308,9 @@ def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wl
     streams, mix = 0, None
     if isinstance(scale, StreamWrite):
         streams, mix, scale = h.shape[1], scale.mix, scale.out
-    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiiffip", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
+    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiifffip" + "fplp", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
          float(alpha), G, wlen, ptr(gate), gate.stride(0) if gate is not None else 0, ptr(coef), float(eps),
          ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, out.stride(0) if out is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(scale),
-         ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), int(glu is not None), *(map(float, glu or (0.0, 0.0))), streams, ptr(mix))
+         ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), int(glu is not None), *(glu or unit or (0.0, 0.0, 0.0)), streams, ptr(mix),
+         float(cap), ptr(part), part.stride(0) if part is not None else 0, ptr(h_out))
     return out

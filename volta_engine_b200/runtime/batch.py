@@ -23,6 +23,18 @@ LONG_SEGMENT = 16      # portions of at least this many rows take the prompt ker
 
 
 @dataclass
+class Contexts:
+    """Contexts of segments, one after the other: per segment its slot, the first row of its context and that row's position; ``tiles``
+    of at most 64 or 128 rows of one segment: (first row, counted from the table's ``short_rows``; rows; first row of the segment's
+    context; that row's position)."""
+    slot: torch.Tensor
+    base: torch.Tensor
+    start: torch.Tensor
+    total: int
+    tiles: dict
+
+
+@dataclass
 class SegmentTable:
     """Runs of consecutive rows of one slot inside a batch that is known on the host. Device tables are int32."""
     n: int                          # segments
@@ -30,13 +42,6 @@ class SegmentTable:
     count: torch.Tensor             # [n] rows
     host: list                      # [(slot, first row, rows, first position)]
     short_rows: int                 # leading rows that belong to segments shorter than LONG_SEGMENT
-    ctx_slot: torch.Tensor | None   # per segment behind those rows: its slot and the first row of its context when the contexts
-    ctx_base: torch.Tensor | None   # (positions 0 .. last) of these segments are laid out one after the other
-    ctx_total: int
-    tile_first: torch.Tensor | None  # tiles of at most 64 rows of one of these segments; rows counted from short_rows
-    tile_count: torch.Tensor | None
-    tile_base: torch.Tensor | None   # the segment's ctx_base
-    wide_tiles: tuple | None          # the same with at most 128 rows per tile: (first, count, base)
     chunk_seg: torch.Tensor | None   # chunks of at most CHUNK_ROWS rows of these segments: segment (0 = the first behind short_rows),
     chunk_first: torch.Tensor | None  # first row (in the batch) and rows
     chunk_count: torch.Tensor | None
@@ -44,14 +49,35 @@ class SegmentTable:
     n_short: int = 0                  # leading segments that make up short_rows
     chunks: int = 0
     longest: int = 0                  # most chunks of any segment
-    by_tokens: dict = field(default_factory=dict)
+    made: dict = field(default_factory=dict)
+
+    def _dev(self, v):
+        return torch.tensor(list(v), dtype=torch.int32).to(self.first.device, non_blocking=True)
+
+    def context(self, window: int = 0) -> "Contexts":
+        """What the segments behind ``short_rows`` see (a sliding window: none of their rows sees further back), laid out one after
+        the other."""
+        t = self.made.get(("context", window))
+        if t is None:
+            rest = self.host[self.n_short:]
+            start = [max(0, p0 - window + 1) if window else 0 for _, _, _, p0 in rest]
+            base, total = [], 0
+            for a, (_, _, c, p0) in zip(start, rest):
+                base.append(total)
+                total += p0 + c - a
+            tiles = {}
+            for per in (64, 128):
+                rows = [(f + o - self.short_rows, min(per, c - o), z, a) for a, z, (_, f, c, _) in zip(start, base, rest) for o in range(0, c, per)]
+                tiles[per] = tuple(self._dev(v) for v in zip(*rows))
+            t = self.made["context", window] = Contexts(self._dev([h[0] for h in rest]), self._dev(base), self._dev(start), total, tiles)
+        return t
 
     def tiles(self, per: int):
         """(first row in the batch, rows) of tiles of at most ``per`` rows over the segments behind ``short_rows``."""
-        t = self.by_tokens.get(per)
+        t = self.made.get(per)
         if t is None:
             rows = [(f + o, min(per, c - o)) for _, f, c, _ in self.host[self.n_short:] for o in range(0, c, per)]
-            t = self.by_tokens[per] = tuple(torch.tensor(list(v), dtype=torch.int32).to(self.first.device, non_blocking=True) for v in zip(*rows))
+            t = self.made[per] = tuple(self._dev(v) for v in zip(*rows))
         return t
 
     @classmethod
@@ -71,28 +97,17 @@ class SegmentTable:
             k += 1
         rest = host[k:]
         short = rest[0][1] if rest else n
-        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 2), 0, *([None] * 8), n_short=k)
+        t = cls(len(host), dev([h[1] for h in host]), dev([h[2] for h in host]), host, short, *([None] * 4), n_short=k)
         if rest:
-            base, total = [], 0
-            tf, tc, tb, cs, cf, cc, c0, wide = [], [], [], [], [], [], [0], []
+            cs, cf, cc, c0 = [], [], [], [0]
             per = CHUNK_ROWS if n >= 1024 else CHUNK_ROWS // 2
             for g, (s, f, c, p0) in enumerate(rest):
-                base.append(total)
-                for o in range(0, c, 64):
-                    tf.append(f + o - short)
-                    tc.append(min(64, c - o))
-                    tb.append(total)
-                wide += [(f + o - short, min(128, c - o), total) for o in range(0, c, 128)]
                 for o in range(0, c, per):
                     cs.append(g)
                     cf.append(f + o)
                     cc.append(min(per, c - o))
                 c0.append(len(cs))
-                total += p0 + c
             t.chunks, t.longest = len(cs), max(b - a for a, b in zip(c0, c0[1:]))
-            t.ctx_slot, t.ctx_base, t.ctx_total = dev([h[0] for h in rest]), dev(base), total
-            t.tile_first, t.tile_count, t.tile_base = dev(tf), dev(tc), dev(tb)
-            t.wide_tiles = tuple(dev(list(v)) for v in zip(*wide))
             t.chunk_seg, t.chunk_first, t.chunk_count, t.seg_chunk0 = dev(cs), dev(cf), dev(cc), dev(c0)
         return t
 

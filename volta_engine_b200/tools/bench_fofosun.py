@@ -215,21 +215,21 @@ def run_kernels(width: int, dev) -> dict:
             kb.add("add + norm prompt", "glm5 assembly", lambda: K.rmsnorm(x, L.attn_norm, 1e-5, 1.0, residual=hb), n * width * 8, 0)
             z = torch.randn(n, width * 6, device=dev).to(bf)
             gu = torch.randn(n, width * 8, device=dev).to(bf)
-            kb.add("activation prompt", "polynorm", lambda: ly.act.rows(z, bf), 2 * z.numel() * 2, 0)
+            kb.add("activation prompt", "polynorm", lambda: ly.ff.act.rows(z, bf), 2 * z.numel() * 2, 0)
             kb.add("activation prompt", "glm5 assembly", lambda: K.gated_act(gu, width * 4), gu.numel() * 3, 0)
             orow = torch.randn(n, D, device=dev)
             kb.add("output norm prompt", "hgrn2", lambda: mine.layers[0].mixer.norm.rows(orow, bf), n * D * 6, 0)
             zz = torch.randn(n, D, device=dev).to(bf)
             ob, nw = torch.empty(n, D, device=dev, dtype=bf), torch.ones(128, device=dev)
             kb.add("output norm prompt", "kda", lambda: call("kda_gated_norm", "pplppiiif", ptr(orow), ptr(zz), zz.stride(0), ptr(nw), ptr(ob), n, H, 128, 1e-5), n * D * 8, 0)
-            for lin, nm in ((ly.up, "up"), (ly.mixer.out, "out")):
+            for lin, nm in ((ly.ff.up, "up"), (ly.mixer.out, "out")):
                 xi = torch.randn(n, lin.in_features, device=dev).to(bf)
                 kb.add(f"linear prompt ({nm})", "shared kernel", lambda: lin.forward(xi), lin.nbytes() + n * (lin.in_features + lin.out_features) * 2,
                        2.0 * n * lin.in_features * lin.out_features)
         else:
             z = torch.randn(1, width * 6, device=dev)
-            kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(ly.up, 1, out_f32=True, **ly.norm2.prologue(h)), ly.up.nbytes(), 0)
-            kb.add("linear decode: activation + down + add", "fofosun", lambda: gemv_rows(ly.down, 1, residual=(h, ly.write2), **ly.act.prologue(z)), ly.down.nbytes(), 0)
+            kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(ly.ff.up, 1, out_f32=True, **ly.norm2.prologue(h)), ly.ff.up.nbytes(), 0)
+            kb.add("linear decode: activation + down + add", "fofosun", lambda: gemv_rows(ly.ff.down, 1, residual=(h, ly.write2), **ly.ff.act.prologue(z)), ly.ff.down.nbytes(), 0)
             kb.add("linear decode: in projection", "fofosun", lambda: gemv_rows(ly.mixer.in_proj, 1, out_f32=True, **ly.norm1.prologue(h)), ly.mixer.in_proj.nbytes(), 0)
             gul = other.layers[0].gate_up
             kb.add("linear decode: gate and up", "glm5 assembly (bf16)", lambda: gul.forward(x), gul.nbytes(), 0)

@@ -121,11 +121,11 @@ def run_kernels(width: int, dev) -> dict:
             x = torch.randn(n, width, device=dev).to(bf)
             kb.add("residual + norm prompt", f"siditar ({S} streams, layer norm)", lambda: L.norm1.rows(h, bf, x, L.write1), n * width * (8 * S + 4), 0)
             kb.add("residual + norm prompt", "fofosun (Dynamic Tanh)", lambda: O[0].norm1.rows(ho, bf, x, O[0].write1), n * width * 12, 0)
-            ff = L.down.in_features
-            z, zo = torch.randn(n, 2 * ff, device=dev).to(bf), torch.randn(n, O[0].down.in_features, device=dev).to(bf)
-            kb.add("activation prompt", "siditar (clamped gated unit)", lambda: L.act.rows(z, bf), n * ff * 6, 0)
+            ff = L.ff.down.in_features
+            z, zo = torch.randn(n, 2 * ff, device=dev).to(bf), torch.randn(n, O[0].ff.down.in_features, device=dev).to(bf)
+            kb.add("activation prompt", "siditar (clamped gated unit)", lambda: L.ff.act.rows(z, bf), n * ff * 6, 0)
             kb.add("activation prompt", "dense (SwiGLU)", lambda: K.gated_act(z, ff), n * ff * 6, 0)
-            kb.add("activation prompt", "fofosun (PolyNorm)", lambda: O[0].act.rows(zo, bf), zo.numel() * 4, 0)
+            kb.add("activation prompt", "fofosun (PolyNorm)", lambda: O[0].ff.act.rows(zo, bf), zo.numel() * 4, 0)
             o, y = torch.randn(n, D, device=dev), torch.empty(n, 2 * D, dtype=bf, device=dev)
             gate = mx.right.gate(pr)
             kb.add("output norm prompt", "siditar (gate in fp32)", lambda: mx.right.norm.rows(o, bf, gate=gate, out=y[:, D:]), n * D * 10, 0)
@@ -133,12 +133,12 @@ def run_kernels(width: int, dev) -> dict:
             po = torch.randn(n, om.in_proj.out_features, device=dev)
             kb.add("output norm prompt", "fofosun (lightning)", lambda: om.norm.rows(o, bf, gate=om.gate(po)), n * D * 10, 0)
             for who, lin, nm, f32 in (("siditar", mx.in_proj, "in projection", True), ("fofosun", om.in_proj, "in projection", True), ("siditar", mx.out, "out", False),
-                                      ("fofosun", om.out, "out", False), ("siditar", L.up, "gate and up", False), ("fofosun", O[0].up, "up", False)):
+                                      ("fofosun", om.out, "out", False), ("siditar", L.ff.up, "gate and up", False), ("fofosun", O[0].ff.up, "up", False)):
                 xi = torch.randn(n, lin.in_features, device=dev).to(bf)
                 kb.add(f"linear prompt ({nm})", who, lambda: lin.forward(xi, out_f32=f32), lin.nbytes() + n * (lin.in_features * 2 + lin.out_features * (4 if f32 else 2)),
                        2.0 * n * lin.in_features * lin.out_features)
         else:
-            z, zo = torch.randn(1, L.down.in_features, device=dev).to(bf), torch.randn(1, O[0].up.out_features, device=dev)
+            z, zo = torch.randn(1, L.ff.down.in_features, device=dev).to(bf), torch.randn(1, O[0].ff.up.out_features, device=dev)
             att, o = torch.randn(1, D, device=dev), torch.randn(1, D, device=dev)
             om = O[1].mixer
             po = torch.randn(1, om.in_proj.out_features, device=dev)
@@ -148,11 +148,11 @@ def run_kernels(width: int, dev) -> dict:
                                                                                             **mx.right.norm.prologue(o, mx.right.gate(pr), head=att)), mx.out.nbytes(), 0)
             kb.add("linear decode: output norm + out + residual", "fofosun", lambda: gemv_rows(om.out, 1, residual=(ho, O[1].write1),
                                                                                             **om.norm.prologue(o, om.gate(po))), om.out.nbytes(), 0)
-            kb.add("linear decode: norm + gate and up + activation", "siditar", lambda: gemv_rows(L.up, 1, **L.norm2.prologue(h), **L.act.epilogue()), L.up.nbytes(), 0)
-            kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(O[0].up, 1, out_f32=True, **O[0].norm2.prologue(ho)), O[0].up.nbytes(), 0)
-            kb.add("linear decode: down + residual", "siditar", lambda: gemv_rows(L.down, 1, residual=(h, L.write2), x=z), L.down.nbytes(), 0)
-            kb.add("linear decode: activation + down + residual", "fofosun", lambda: gemv_rows(O[0].down, 1, residual=(ho, O[0].write2), **O[0].act.prologue(zo)),
-                   O[0].down.nbytes(), 0)
+            kb.add("linear decode: norm + gate and up + activation", "siditar", lambda: gemv_rows(L.ff.up, 1, **L.norm2.prologue(h), **L.ff.act.epilogue()), L.ff.up.nbytes(), 0)
+            kb.add("linear decode: norm + up", "fofosun", lambda: gemv_rows(O[0].ff.up, 1, out_f32=True, **O[0].norm2.prologue(ho)), O[0].ff.up.nbytes(), 0)
+            kb.add("linear decode: down + residual", "siditar", lambda: gemv_rows(L.ff.down, 1, residual=(h, L.write2), x=z), L.ff.down.nbytes(), 0)
+            kb.add("linear decode: activation + down + residual", "fofosun", lambda: gemv_rows(O[0].ff.down, 1, residual=(ho, O[0].write2), **O[0].ff.act.prologue(zo)),
+                   O[0].ff.down.nbytes(), 0)
     return {"width": width, "prompt_rows": T, "context": ctx, "peaks": kb.pk, "kernels": kb.rows}
 
 

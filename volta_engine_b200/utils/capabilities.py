@@ -33,6 +33,7 @@ TABLE = {
     "gqa_store": ("GroupedAttention", P), "gqa_rows": ("GroupedAttention", P), "gqa_decode": ("GroupedAttention", P), "gqa_prefill": ("GroupedAttention", P),
     "embed_rows": ("RowOps (fp32 residual)", P), "dyt_rows": ("RowOps (fp32 residual)", P), "group_rms": ("RowOps (fp32 residual)", P),
     "stream_norm": ("RowOps (fp32 residual)", P), "clamped_glu": ("RowOps (fp32 residual)", P),
+    "residual_norm": ("RowOps (fp32 residual)", P), "soft_cap": ("RowOps (fp32 residual)", P),
     "polynorm": ("RowOps (fp32 residual)", P), "gemv_rows": ("LinearBF16 decode", P), "gemm_f32": ("Gemm (fp32)", P),
     "dsa_prep": ("DSA", P), "dsa_pool_update": ("DSA", P), "dsa_score": ("DSA / QSA", P), "dsa_select": ("DSA / QSA", P),
     "dsa_gather": ("DSA / QSA", P), "dsa_kpad": ("DSA / QSA", D), "qsa_prep": ("QSA", P), "qsa_pool_update": ("QSA", P),
@@ -41,6 +42,7 @@ TABLE = {
     "dsv4_index_key_store": ("DSV4", P), "dsv4_index_q": ("DSV4", P), "dsv4_candidates": ("DSV4", P), "dsv4_select": ("DSV4", P),
     "dsv4_gather": ("DSV4", D), "dsv4_q_prep": ("DSV4", D), "dsv4_attn_out": ("DSV4", P), "dsv4_woa": ("DSV4", P), "dsv4_engram_gate": ("Engram", P), "dsv4_engram_ids": ("Engram", P),
     "router_select": ("MoERouter", P), "nvfp4_moe_gemv": ("MoE", P), "moe_combine": ("MoE", P), "moe_sort": ("MoE", P),
+    "route_rows": ("RoutedFF", P), "routed_up": ("RoutedFF", P), "routed_down": ("RoutedFF", P),
     "moe_gather": ("MoE", P), "cpu_post": ("CpuExperts", D), "cpu_wait_add": ("CpuExperts", D),
     "cpu_mailbox_bytes": ("CpuExperts", D),
     "gdn_prepare": ("GDN", P), "gdn_recurrent": ("GDN", P), "gdn_gated_norm": ("GDN", P),
