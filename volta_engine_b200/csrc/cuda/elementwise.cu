@@ -286,6 +286,7 @@ int ve_rmsnorm_heads(void* x, const void* w, int rows, int heads, int hd, long r
                      cudaStream_t st) {
   const int warps = rows * heads;
   if (warps <= 0) return 0;
+  if (!x || !w) return cudaErrorInvalidValue;
   rmsnorm_heads_kernel<<<(warps + 7) / 8, 256, 0, st>>>((__nv_bfloat16*)x, (const __nv_bfloat16*)w, rows, heads, hd,
                                                         row_stride, eps, wbias);
   VE_CHECK_LAUNCH();

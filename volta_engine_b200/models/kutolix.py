@@ -27,7 +27,6 @@ EXPERT_ALPHA = 1.702
 
 @dataclass
 class KutolixConfig(ListedConfig):
-    embed_scale: float = 1.0
     residual_mult: float = 1.0
     model_type: str = "kutolix"
 

@@ -153,6 +153,9 @@ class MoEModel(DenseModel):
             self._init_attention(L, rnd, search)
             L.attn_norm, L.ffn_norm = nw.clone(), nw.clone()
             L.q_norm = L.k_norm = None
+            if cfg.qk_norm:
+                L.q_norm = torch.ones(cfg.head_dim, device=dev, dtype=torch.bfloat16) * (1.0 - cfg.norm_bias)
+                L.k_norm = L.q_norm.clone()
             L.gate_up = L.down = None
             L.dense_ffn = li < cfg.first_dense_layers
             if L.dense_ffn:
