@@ -109,7 +109,6 @@ class StepResidual:
 
 
 class ListedModel(SlotStates, DenseModel):
-    prefix_resume = "kv+state"
     supports_mixed = True           # prompt portions and decode rows of several sequences run in one forward
     kv_layers = 0
     kv_v_dim = 8
@@ -122,6 +121,11 @@ class ListedModel(SlotStates, DenseModel):
         self.vocab_pad = self.vocab_local = cfg.vocab
         self.kv_v_dim = cfg.v_width
         self.layer_tap = None       # a list that receives the residual after every layer run (tests, inspection)
+
+    @property
+    def prefix_resume(self) -> str:
+        """What a prefix snapshot holds: the paged cache, and the slot's state where a layer has one."""
+        return "kv+state" if any(L.mixer.recurrent for L in self.layers) else "kv"
 
     # ------------------------------------------------------------------------------------------ what a design supplies
     def load_ends(self, src) -> None:
