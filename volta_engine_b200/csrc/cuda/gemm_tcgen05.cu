@@ -169,8 +169,8 @@ gemm_kernel(const GemmParams p, const __grid_constant__ CUtensorMap amap, const 
           bulk_load(st + A_RAW + B_BYTES, p.sfa + (sf_tile * nkt + kt) * 2048, 2048, &full[s]);
 #pragma unroll
           for (int b = 0; b < NB128; ++b)
-            bulk_load(st + A_RAW + B_BYTES + SFA_BYTES + b * 2048,
-                      p.sfb + ((size_t)(blockIdx.y * NB128 + b) * nkt + kt) * 2048, 2048, &full[s]);
+            bulk_load(st + A_RAW + B_BYTES + SFA_BYTES + b * 2048,      // (a tile may end in front of its last 128 rows)
+                      p.sfb + ((size_t)min((int)blockIdx.y * NB128 + b, (p.T - 1) / 128) * nkt + kt) * 2048, 2048, &full[s]);
         }
       }
     }
