@@ -413,7 +413,7 @@ def experts_case(r, width, ff, limit, seed=0):
 
 
 EXP = [(Router(16, 3, 2, 1), 104, 40, 0.6), (Router(7, 2), 75, 19, 1.1), (Router(64, 8, 8, 4), 256, 96, 1.5), (Router(5, 4, 5, 4), 33, 130, 0.3), (Router(3, 3), 512, 8, 7.0),
-       (Router(1, 1), 64, 64, 1.0), (Router(40, 1, 8, 1), 136, 264, 2.0)]
+       (Router(1, 1), 64, 64, 1.0), (Router(40, 1, 8, 1), 136, 264, 2.0), (Router(9, 8, 3, 3), 24, 6272, 1.0)]
 
 
 @pytest.mark.parametrize("device", DEVICES)

@@ -6,7 +6,8 @@
 //   * query and key are DQC chunks of 64 columns (plain part, then rotated part; pad columns of the query are zero), the key's
 //     rotated part comes from the cached rows and is shared by the heads; values are DVC chunks;
 //   * the softmax weights enter the second product as two bf16 terms (value and remainder), so they keep 32-bit quality;
-//   * keys and values have rings of their own (a key tile is free as soon as its scores are done);
+//   * keys and values have rings and loaders of their own (a key tile is free as soon as its scores are done, and its successor is not
+//     requested behind values that wait for their weights): warps 0 and 10;
 //   * with a sliding window the key tiles in front of the first row's window are not visited.
 // Every wait is bounded; on expiry the CTA records a status code, skips its stores and frees its TMEM.
 #pragma once
@@ -26,7 +27,7 @@ struct LatentTc {
   int* status;
 };
 
-constexpr int kLtRows = 128, kLtThreads = 320, kLtKs = 3, kLtVs = 2;
+constexpr int kLtRows = 128, kLtThreads = 352, kLtKs = 3, kLtVs = 2;
 constexpr float kLtLazyLog2 = 8.f;
 
 template <int DQC, int DVC>
@@ -76,9 +77,9 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
   }
   // a softmax thread owns one row of one stream: TMEM lane = 32 * (warp % 4) + lane, stream = (warp - 2) / 4
   const int r = (warp & 3) * 32 + lane, strm = warp >= 6 ? 1 : 0;
-  const bool r_ok = warp >= 2 && r < count;
+  const bool soft = warp >= 2 && warp < 10, r_ok = soft && r < count;
   const int r_tok = first + (r_ok ? r : 0), r_pos = p.pos[r_tok];
-  if (warp >= 2) {
+  if (soft) {
     // the two streams' threads of a row share its 16-byte pieces of Q
     const __nv_bfloat16* src = p.q + (long)r_tok * p.ldq + (long)h * (p.n.d + p.n.rot);
 #pragma unroll
@@ -98,12 +99,12 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
   const uint32_t tmem_base = tmem_holder;
 
   if (warp == 0) {
-    // ------------------------------------------------------------------ key and value loads
+    // ------------------------------------------------------------------ key loads
     if (elect_one()) {
       prefetch_tmap(&upmap);
       prefetch_tmap(&rotmap);
       for (int j = 0; j < n; ++j) {
-        const int ks = j % kLtKs, vs = j % kLtVs, row = kbase + j * 64;
+        const int ks = j % kLtKs, row = kbase + j * 64;
         if (j >= kLtKs && !mbar_wait(&kempty[ks], ((j / kLtKs) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
@@ -114,6 +115,13 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
           if (c < p.uc) tma_load_2d(k_s + ks * KB + c * 8192, &upmap, &kfull[ks], h * p.n.d + c * 64, row);
           else tma_load_2d(k_s + ks * KB + c * 8192, &rotmap, &kfull[ks], p.n.rot0 + (c - p.uc) * 64, row);
         }
+      }
+    }
+  } else if (warp == 10) {
+    // ------------------------------------------------------------------ value loads
+    if (elect_one()) {
+      for (int j = 0; j < n; ++j) {
+        const int vs = j % kLtVs, row = kbase + j * 64;
         if (j >= kLtVs && !mbar_wait(&vempty[vs], ((j / kLtVs) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
@@ -253,7 +261,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_prefill_tc_kernel(const 
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  if (warp >= 2 && !s_fail) {
+  if (soft && !s_fail) {
     // ------------------------------------------------------------------ merge of the two streams and output
     const uint32_t t_lane = tmem_base + ((uint32_t)((warp & 3) * 32) << 16);
     const float* ml0 = reinterpret_cast<const float*>(p_s);

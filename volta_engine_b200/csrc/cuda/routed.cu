@@ -226,26 +226,29 @@ struct RoutedDown {
   long lda, ldw, ldo;
 };
 
-// grid (CTAs, rows), 256 threads, a warp per output column. Dynamic shared memory: [top][ff rounded up to 16 bytes] of T.
-template <typename T, typename O>
+// grid (CTAs, rows), 256 threads, a warp per output column. STAGED: activations in dynamic shared memory [top][ff rounded up to 16 bytes] of
+// T; else they are read where they are (rows of whole 16-byte pieces).
+template <bool STAGED, typename T, typename O>
 __global__ void __launch_bounds__(256) routed_down_kernel(const RoutedDown a, const T* __restrict__ act, const T* __restrict__ W, O* __restrict__ out) {
   constexpr int V = 16 / sizeof(T), U = 4;
   extern __shared__ __align__(16) uint8_t dsm[];
   __shared__ int s_id[kMaxTop];
   __shared__ float s_w[kMaxTop];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, F = (a.ff + V - 1) / V * V;
-  T* as = reinterpret_cast<T*>(dsm);
   const long row = blockIdx.y;
+  const T* as = STAGED ? reinterpret_cast<const T*>(dsm) : act + row * a.top * a.lda;
+  const long pitch = STAGED ? F : a.lda;
   grid_dep_wait();
   grid_dep_launch();
   if (tid < a.top) {
     s_id[tid] = a.ids[row * a.top + tid];
     s_w[tid] = a.weights[row * a.top + tid];
   }
-  for (int i = tid; i < a.top * F; i += 256) {
-    const int k = i / F, f = i - k * F;
-    as[i] = f < a.ff ? act[(row * a.top + k) * a.lda + f] : from_f<T>(0.f);
-  }
+  if (STAGED)
+    for (int i = tid; i < a.top * F; i += 256) {
+      const int k = i / F, f = i - k * F;
+      reinterpret_cast<T*>(dsm)[i] = f < a.ff ? act[(row * a.top + k) * a.lda + f] : from_f<T>(0.f);
+    }
   __syncthreads();
   for (int n = blockIdx.x * 8 + warp; n < a.N; n += gridDim.x * 8) {
     float acc = 0.f;
@@ -258,7 +261,7 @@ __global__ void __launch_bounds__(256) routed_down_kernel(const RoutedDown a, co
           p[j] = k0 + j < a.top ? __ldcs(reinterpret_cast<const uint4*>(W + ((long)s_id[k0 + j] * a.N + n) * a.ldw + f)) : make_uint4(0, 0, 0, 0);
 #pragma unroll
         for (int j = 0; j < U; ++j)
-          if (k0 + j < a.top) dot16(p[j], as + (k0 + j) * F + f, d[j]);
+          if (k0 + j < a.top) dot16(p[j], as + (k0 + j) * pitch + f, d[j]);
       }
 #pragma unroll
       for (int j = 0; j < U; ++j)
@@ -295,11 +298,16 @@ template <typename T, typename O>
 static int launch_routed_down(const RoutedDown& a, const void* act, const void* W, void* out, int rows, cudaStream_t st) {
   constexpr int V = 16 / sizeof(T);
   const size_t smem = (size_t)a.top * ((a.ff + V - 1) / V * V) * sizeof(T);
-  static size_t have = 0;
-  const int rc = routed_smem(routed_down_kernel<T, O>, smem, have);
-  if (rc) return rc;
   const int chunks = (a.N + 7) / 8, room = rows >= 592 ? 1 : 592 / rows, per = (chunks + room - 1) / room;
-  launch_pdl(routed_down_kernel<T, O>, dim3((chunks + per - 1) / per, rows), dim3(256), smem, st, a, (const T*)act, (const T*)W, (O*)out);
+  const dim3 grid((chunks + per - 1) / per, rows);
+  if (smem > 96 * 1024 && a.ff % V == 0 && a.lda % V == 0 && !((uintptr_t)act & 15)) {
+    launch_pdl(routed_down_kernel<false, T, O>, grid, dim3(256), 0, st, a, (const T*)act, (const T*)W, (O*)out);
+    return (int)cudaGetLastError();
+  }
+  static size_t have = 0;
+  const int rc = routed_smem(routed_down_kernel<true, T, O>, smem, have);
+  if (rc) return rc;
+  launch_pdl(routed_down_kernel<true, T, O>, grid, dim3(256), smem, st, a, (const T*)act, (const T*)W, (O*)out);
   return (int)cudaGetLastError();
 }
 
