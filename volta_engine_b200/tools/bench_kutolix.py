@@ -209,6 +209,8 @@ def run_kernels(width: int, dev) -> dict:
             kb.add("experts decode", "moe (NVFP4)", theirs, live * per_expert * 0.5625, 0)
             kb.add("linear decode: residual + norm + router", "kutolix", lambda: gemv_rows(E.router, 1, out_f32=True, **A.norm2.prologue(res, part, A.write1)),
                    E.router.nbytes(), 0)
+            mr = moe.layers[0].router
+            kb.add("linear decode: residual + norm + router", "moe (router alone)", lambda: mr.forward(xr, out_f32=True), mr.nbytes(), 0)
     return {"width": width, "prompt_rows": T, "context": ctx, "window": WINDOW, "peaks": kb.pk, "kernels": kb.rows}
 
 
