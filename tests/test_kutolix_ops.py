@@ -355,7 +355,7 @@ def test_latent_prompt_of_many_key_tiles(H, d, rot, dv, kr, window):
 
 
 # ------------------------------------------------------------------------------------------ routers and experts
-ROUTERS = [Router(16, 3, 2, 1), Router(12, 5, 3, 2), Router(7, 2), Router(40, 1, 8, 1), Router(64, 8, 8, 4), Router(5, 4, 5, 4), Router(6, 6, 2, 2), Router(300, 20, 10, 3),
+ROUTERS = [Router(18, 4, 3, 1), Router(12, 5, 3, 2), Router(7, 2), Router(40, 1, 8, 1), Router(64, 8, 8, 4), Router(5, 4, 5, 4), Router(6, 6, 2, 2), Router(300, 20, 10, 3),
            Router(1, 1), Router(1024, 32, 64, 7)]
 
 
@@ -412,7 +412,7 @@ def experts_case(r, width, ff, limit, seed=0):
     return W, {"expert": {"limit": limit}, "router": as_config(r)}, pack
 
 
-EXP = [(Router(16, 3, 2, 1), 104, 40, 0.6), (Router(7, 2), 75, 19, 1.1), (Router(64, 8, 8, 4), 256, 96, 1.5), (Router(5, 4, 5, 4), 33, 130, 0.3), (Router(3, 3), 512, 8, 7.0),
+EXP = [(Router(18, 4, 3, 1), 104, 40, 0.6), (Router(7, 2), 75, 19, 1.1), (Router(64, 8, 8, 4), 256, 88, 1.4), (Router(5, 4, 5, 4), 33, 130, 0.3), (Router(3, 3), 512, 8, 7.0),
        (Router(1, 1), 64, 64, 1.0), (Router(40, 1, 8, 1), 136, 264, 2.0), (Router(9, 8, 3, 3), 24, 6272, 1.0)]
 
 
