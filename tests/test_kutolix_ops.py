@@ -65,7 +65,7 @@ def test_rotations(rot, neighbours, device):
             kv = PagedKVCache(1, 1, spec.kw, 2, 1, 64, torch.device(device), dtype=torch.float32, v_head_dim=8)
             proj = torch.nn.functional.pad(v.reshape(len(pos), -1), (0, wide + 8)).to(device)
             hidden = torch.full((len(pos),), -1, dtype=torch.int32, device=device)                    # rows of no slot: queries only
-            got = gqa_store(spec, proj, pos.to(device), hidden, kv, kv.k[0], kv.v[0])[:, :, :wide].cpu()
+            got = gqa_store(spec, proj, pos.to(device), hidden, kv, kv.k[0], kv.v[0])[0][:, :, :wide].cpu()
         assert (got.double() - want).abs().max() < 4e-6 * mul
 
 

@@ -30,7 +30,7 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr", "-diag-suppress", "177,550",
 ]
 # sources whose results follow the 32-bit definitions of exp / tanh / division to rounding
-PRECISE = {"routed.cu", "rowops.cu", "linattn.cu", "latent.cu", "gemv_rows.cu", "gqa.cu"}
+PRECISE = {"routed.cu", "rowops.cu", "linattn.cu", "latent.cu", "gemv_rows.cu", "gqa.cu", "mingru.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-pthread", "-Wall", "-Wno-unused-function"]
 
 

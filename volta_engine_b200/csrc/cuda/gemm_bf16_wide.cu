@@ -20,6 +20,7 @@ struct WideBf16Params {
   const __nv_bfloat16* residual;
   long ldr;
   int* status;
+  const float* bias;
 };
 
 constexpr int WB_SUB = 128 * 128, WB_B = 256 * 128, WB_STAGE = 2 * WB_SUB + WB_B, WB_STAGES = 3;
@@ -101,7 +102,7 @@ gemm_bf16_wide_kernel(const WideBf16Params p, const __grid_constant__ CUtensorMa
       for (int sub = 0; sub < 2; ++sub)
         if (n0 + sub * 128 < p.N)
           store_tile<256>(smem, tmem_base + sub * 256, warp & 3, (warp - 2) * 32 + lane, n0 + sub * 128, t0,
-                          TileOut{p.N, p.T, p.alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr});
+                          TileOut{p.N, p.T, p.alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr, p.bias});
   }
   tc_fence_before();
   __syncthreads();
@@ -118,9 +119,9 @@ using namespace ve;
 
 extern "C" {
 
-// Arguments as ve_gemm_bf16: W [N, K] (pitch ldw), X [T, K] (pitch ldx), pitches multiples of 8 elements; out bf16 or out_f32.
+// Arguments as ve_gemm_bf16: W [N, K] (pitch ldw), X [T, K] (pitch ldx), pitches multiples of 8 elements; out bf16 or out_f32; bias fp32 [N] or null.
 int ve_gemm_bf16_wide(const void* W, long ldw, const void* X, long ldx, void* out, long ldo, void* out_f32, const void* residual, long ldr, int T, int N,
-                      int K, float alpha, void* status, cudaStream_t st) {
+                      int K, float alpha, const void* bias, void* status, cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
   if (K < 1) return cudaErrorInvalidValue;
   CUtensorMap amap, bmap;
@@ -134,7 +135,7 @@ int ve_gemm_bf16_wide(const void* W, long ldw, const void* X, long ldx, void* ou
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
-  WideBf16Params p{N, T, K, alpha, (__nv_bfloat16*)out, (float*)out_f32, ldo, (const __nv_bfloat16*)residual, ldr, (int*)status};
+  WideBf16Params p{N, T, K, alpha, (__nv_bfloat16*)out, (float*)out_f32, ldo, (const __nv_bfloat16*)residual, ldr, (int*)status, (const float*)bias};
   gemm_bf16_wide_kernel<<<dim3((N + 255) / 256, (T + 255) / 256), 192, WB_SMEM, st>>>(p, amap, bmap);
   return (int)cudaGetLastError();
 }

@@ -14,6 +14,7 @@ struct TileOut {
   long ldo;
   const __nv_bfloat16* residual;    // optional, added before rounding
   long ldr;
+  const float* bias;                // optional [N], added before rounding
 };
 
 // Called by four warps (etid 0..127, `quarter` = the TMEM lane quarter of the calling warp) once the accumulator is complete and the
@@ -23,6 +24,7 @@ VE_DEVINL void store_tile(uint8_t* stage, uint32_t tmem, int quarter, int etid, 
   const int lane = etid & 31, col = quarter * 32 + lane;
   const int rows = min(COLS, o.t_end - t0);
   const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
+  const float b = o.bias && n0 + col < o.N ? o.bias[n0 + col] : 0.f;
 #pragma unroll 1
   for (int c0 = 0; c0 < rows; c0 += 16) {
     uint32_t r[16];
@@ -30,13 +32,13 @@ VE_DEVINL void store_tile(uint8_t* stage, uint32_t tmem, int quarter, int etid, 
     tmem_ld_wait();
     if (o.out_f32) {
 #pragma unroll
-      for (int j = 0; j < 16; ++j) reinterpret_cast<float*>(stage + (c0 + j) * 528)[col] = __uint_as_float(r[j]) * o.alpha;
+      for (int j = 0; j < 16; ++j) reinterpret_cast<float*>(stage + (c0 + j) * 528)[col] = fmaf(__uint_as_float(r[j]), o.alpha, b);
     } else if (o.residual) {          // the sum is rounded once: keep the product in fp32 until the residual is added
 #pragma unroll
-      for (int j = 0; j < 16; ++j) reinterpret_cast<float*>(stage + (c0 + j) * 528)[col] = __uint_as_float(r[j]) * o.alpha;
+      for (int j = 0; j < 16; ++j) reinterpret_cast<float*>(stage + (c0 + j) * 528)[col] = fmaf(__uint_as_float(r[j]), o.alpha, b);
     } else {
 #pragma unroll
-      for (int j = 0; j < 16; ++j) reinterpret_cast<__nv_bfloat16*>(stage + (c0 + j) * 272)[col] = f2bf(__uint_as_float(r[j]) * o.alpha);
+      for (int j = 0; j < 16; ++j) reinterpret_cast<__nv_bfloat16*>(stage + (c0 + j) * 272)[col] = f2bf(fmaf(__uint_as_float(r[j]), o.alpha, b));
     }
   }
   asm volatile("bar.sync 1, 128;" ::: "memory");

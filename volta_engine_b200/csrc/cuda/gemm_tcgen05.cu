@@ -37,6 +37,7 @@ struct GemmParams {
   int n_per_expert;           // rows of one expert inside the stacked weight
   const float* alpha_tab;     // per-expert tensor scale (null: alpha)
   int n_tiles;                // grid.y of the grouped form
+  const float* bias;          // optional [N] (plain bf16 form)
 };
 
 template <int MODE>
@@ -272,7 +273,7 @@ gemm_kernel(const GemmParams p, const __grid_constant__ CUtensorMap amap, const 
     tc_fence_after();
     asm volatile("bar.sync 1, 128;" ::: "memory");        // one answer for the four warps: they meet at barriers below
     if (!*(volatile int*)&s_fail)
-      store_tile<BN>(smem, tmem_base, warp & 3, etid, n0, t0, TileOut{p.N, t_end, alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr});
+      store_tile<BN>(smem, tmem_base, warp & 3, etid, n0, t0, TileOut{p.N, t_end, alpha, p.out, p.out_f32, p.ldo, p.residual, p.ldr, p.bias});
   }
   tc_fence_before();
   __syncthreads();
@@ -325,9 +326,9 @@ using namespace ve;
 
 extern "C" {
 
-// bf16 weights W [N, K] (row pitch ldw elements), bf16 activations X [T, K] (pitch ldx).
+// bf16 weights W [N, K] (row pitch ldw elements), bf16 activations X [T, K] (pitch ldx), bias fp32 [N] or null.
 int ve_gemm_bf16(const void* W, long ldw, const void* X, long ldx, void* out, long ldo, void* out_f32,
-                 const void* residual, long ldr, int T, int N, int K, float alpha, void* status, cudaStream_t st) {
+                 const void* residual, long ldr, int T, int N, int K, float alpha, const void* bias, void* status, cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
   const int bn = pick_bn(T);
   CUtensorMap amap, bmap;
@@ -339,6 +340,7 @@ int ve_gemm_bf16(const void* W, long ldw, const void* X, long ldx, void* out, lo
   if (rc) return rc;
   GemmParams p{N, T, K, alpha, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)residual, ldr, (float*)out_f32,
                nullptr, nullptr, (int*)status};
+  p.bias = (const float*)bias;
   return dispatch_gemm<0>(p, amap, bmap, bn, st);
 }
 

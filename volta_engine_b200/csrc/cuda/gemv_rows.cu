@@ -8,7 +8,8 @@
 //              4  x = layer norm (no shift) of the weighted sum of the fp32 residual streams
 //              5  x = clamped gated unit of an fp32 [gate | up] row
 //              6  x = h + RMS norm of a sublayer's result (fp32, optional), as it is or RMS normed; the sum is also stored
-//   epilogue   store fp32 (with a soft cap or without) or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write), or, for
+//              (the row that enters the product can be stored too, in bf16)
+//   epilogue   add a bias (optional), then store fp32 (with a soft cap or without) or bf16, or h += scale * y on the fp32 residual, or the residual streams rewritten (streams_write), or, for
 //              weight rows in blocks of [4 gate | 4 up], the clamped gated unit of the pairs in bf16 (half as many columns)
 // The rows are the M side (16) of mma.sync.m16n8k16 and eight weight rows the N side. The order of k inside a product does
 // not matter, so a lane takes eight consecutive k of one weight row as 16 bytes and uses them as the B operands of two MMAs, the
@@ -35,6 +36,8 @@ struct RowsArgs {
   int glu; Glu unit;                // epilogue (and prologue 5)
   float cap;                        // > 0: soft cap of the fp32 output
   const float* part; long ldpart; float* h_out;          // prologue 6: w normalises part, b the sum (null: none); h_out [M][kx]
+  __nv_bfloat16* x_out;             // prologue 6: the rows that enter the product, [M][kx] (null: not stored)
+  const float* bias;                // [N] (null: none)
   int v4;                           // prologue 6: four columns at a time
   int streams; const float* hmix;   // streams > 0: h [M][streams][N], scale [streams]
   int pitch;                        // bytes per activation row in shared memory (prologue forms)
@@ -146,6 +149,7 @@ VE_DEVINL void residual_prologue(const RowsArgs& a, uint8_t* xs, float* red) {
         for (int e = 0; e < V; ++e) x.v[e] *= inv2 * w.v[e];
       }
       x.store(xr + i);
+      if (a.x_out && blockIdx.x == 0) x.store(a.x_out + (long)m * a.kx + i);
     }
   }
 }
@@ -374,6 +378,7 @@ __global__ void __launch_bounds__(256, 2) gemv_ring_kernel(const RowsArgs a) {
         if (in)
 #pragma unroll
           for (int y = 0; y < 8; ++y) v += (&part[buf][y][0][0])[i];
+        if (in && a.bias) v += a.bias[n0 + (i & 7)];
         if (a.glu) {                                      // lanes e and e + 4 of a row hold a pair
           const float u = __shfl_down_sync(0xffffffffu, v, 4);
           if (in && (i & 7) < 4) a.out[(i >> 3) * a.ldo + n0 / 2 + (i & 3)] = f2bf(clamped_glu_of(v, u, a.unit));
@@ -469,15 +474,16 @@ __global__ void __launch_bounds__(256, 3) gemv_slab_kernel(const RowsArgs a) {
       float v = 0.f;
 #pragma unroll
       for (int s = 0; s < KS; ++s) v += part[pb][r * KS + s][m][e];
+      if (a.bias) v += a.bias[n];
       rows_out(a, m, n, v);
     }
     pb ^= 1;                                              // (the other buffer's readers are done: they passed the barrier above)
   }
 }
 
-// out[t][n] = sum_k W[n][k] x[t][k], fp32 throughout. 64 x 64 tiles, 16 k per step, 4 x 4 outputs per thread.
+// out[t][n] = sum_k W[n][k] x[t][k] (+ bias[n]), fp32 throughout. 64 x 64 tiles, 16 k per step, 4 x 4 outputs per thread.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ W, long ldw, const float* __restrict__ x, long ldx, float* __restrict__ out,
-                                                       long ldo, int T, int N, int K) {
+                                                       long ldo, int T, int N, int K, const float* __restrict__ bias) {
   __shared__ float sw[16][65], sx[16][65];
   const int tid = threadIdx.x, n0 = blockIdx.x * 64, t0 = blockIdx.y * 64, tn = (tid & 15) * 4, tt = (tid >> 4) * 4;
   grid_dep_wait();
@@ -506,7 +512,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (t0 + tt + i < T && n0 + tn + j < N) out[(long)(t0 + tt + i) * ldo + n0 + tn + j] = acc[i][j];
+      if (t0 + tt + i < T && n0 + tn + j < N) out[(long)(t0 + tt + i) * ldo + n0 + tn + j] = bias ? acc[i][j] + bias[n0 + tn + j] : acc[i][j];
 }
 
 template <typename F>
@@ -556,18 +562,18 @@ extern "C" {
 // pro 0: x bf16 [M, K], M <= 16. pro 1..6: x fp32, M <= 8 and the activation rows (kx columns) fit in shared memory (else refused).
 // pro 2 with k0 > 0: columns [0, k0) from head, the norm's columns behind them. pro 4: G streams of kx columns weighted by coef.
 // pro 5: 2 kx columns, glu_alpha, glu_limit and glu_shift. pro 6: part fp32 (null: none) normed with w, the sum with b (null: not), stored to
-// h_out [M][kx] (null: not). cap > 0: soft cap of out_f32. glu: out bf16 [M][N / 2] (N a multiple of 8). Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
+// h_out [M][kx] (null: not), what enters the product to x_out [M][kx] (null: not). bias fp32 [N] (null: none). cap > 0: soft cap of out_f32. glu: out bf16 [M][N / 2] (N a multiple of 8). Exactly one of h, out_f32 and out is written; streams > 0: h [M][streams][N]
 // with hmix [streams][streams] and scale [streams].
 int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, const void* x, long ldx, const void* w, const void* b, float alpha, int G,
                  int wlen, const void* gate, long ldg, const void* coef, float eps, void* out_f32, void* out, long ldo, void* h, long ldh, const void* scale,
                  const void* head, long ldhead, int k0, int silu, int glu, float glu_alpha, float glu_limit, float glu_shift, int streams, const void* hmix,
-                 float cap, const void* part, long ldpart, void* h_out, cudaStream_t st) {
+                 float cap, const void* part, long ldpart, void* h_out, void* x_out, const void* bias, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 || ldw % 8 || ((uintptr_t)W & 15) || M > 16 || kx > K || kx < 1 || pro < 0 || pro > 6) return cudaErrorInvalidValue;
   RowsArgs a{(const __nv_bfloat16*)W, ldw, N, K, M, pro, kx, x, ldx, (const float*)w, (const float*)b, alpha, G, wlen, (const float*)gate, ldg,
              (const float*)coef, eps, (float*)out_f32, (__nv_bfloat16*)out, ldo, (float*)h, ldh, (const float*)scale,
-             (const float*)head, ldhead, k0, silu, glu, Glu{glu_alpha, glu_limit, glu_shift}, cap, (const float*)part, ldpart, (float*)h_out,
-             kx % 4 == 0 && ldx % 4 == 0 && ldpart % 4 == 0 && !(((uintptr_t)x | (uintptr_t)part | (uintptr_t)w | (uintptr_t)b | (uintptr_t)h_out) & 15),
+             (const float*)head, ldhead, k0, silu, glu, Glu{glu_alpha, glu_limit, glu_shift}, cap, (const float*)part, ldpart, (float*)h_out, (__nv_bfloat16*)x_out, (const float*)bias,
+             kx % 4 == 0 && ldx % 4 == 0 && ldpart % 4 == 0 && !(((uintptr_t)x | (uintptr_t)part | (uintptr_t)w | (uintptr_t)b | (uintptr_t)h_out | (uintptr_t)x_out) & 15),
              streams, (const float*)hmix, 0};
   if (glu && (!out || N % 8 || (long)M * ((K + 31) / 32 * 64 + 64) > 100 * 1024)) return cudaErrorInvalidValue;
   if (streams < 0 || streams > kMaxStreams || (streams && (!h || !hmix || !scale))) return cudaErrorInvalidValue;
@@ -589,9 +595,9 @@ int ve_gemv_rows(const void* W, long ldw, int N, int K, int M, int pro, int kx, 
 #undef VE_GR
 }
 
-int ve_gemm_f32(const void* W, long ldw, const void* x, long ldx, void* out, long ldo, int T, int N, int K, cudaStream_t st) {
+int ve_gemm_f32(const void* W, long ldw, const void* x, long ldx, void* out, long ldo, int T, int N, int K, const void* bias, cudaStream_t st) {
   if (T <= 0 || N <= 0) return 0;
-  launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (T + 63) / 64), dim3(256), 0, st, (const float*)W, ldw, (const float*)x, ldx, (float*)out, ldo, T, N, K);
+  launch_pdl(gemm_f32_kernel, dim3((N + 63) / 64, (T + 63) / 64), dim3(256), 0, st, (const float*)W, ldw, (const float*)x, ldx, (float*)out, ldo, T, N, K, (const float*)bias);
   VE_CHECK_LAUNCH();
 }
 

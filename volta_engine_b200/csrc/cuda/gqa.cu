@@ -1,7 +1,9 @@
 // Grouped-query softmax attention with its sizes and its score terms as parameters: query / key width and value width may differ and
-// need not be powers of two; optional rotary positions, then RMS norm (with or without a weight) of queries and keys, query temperature
-// by position, sliding window, bias by distance (a table per head whose last entry holds for everything farther), a sink (one more term
-// of the denominator), a factor on the result, a sigmoid gate on every element of it.
+// need not be powers of two; optional rotary positions and RMS norm (with or without a weight, behind the rotation or in front of it) of
+// queries and keys, query temperature by position, a factor per query head, a soft cap of the scores, a sliding window (with or without the
+// first tokens of the sequence in sight), bias by distance (a table per head whose last entry holds for everything farther), a sink (one
+// more term of the denominator), a factor on the result, a sigmoid gate on every element of it. Values may be rotated by their position
+// too: they are cached so, and the result is turned back by the query's position.
 //
 // Cache: a page of the pool is 64 tokens x row width; this layer sees it as [kv heads][64][kw] (values [kv heads][64][vw]) with kw, vw the
 // widths rounded up to 8 elements (pad columns are zero), so layers of unlike sizes share one pool.
@@ -34,12 +36,18 @@ struct GqaScore {
   int window;                     // keys at distances below it are seen (INT_MAX: all in front)
   const void* gate; long ldg;     // [rows][H dv] (null: none), fp32 (gate32) or bf16
   int gate32, gatev;              // gatev: eight columns from a multiple of eight on are 16-byte aligned
+  int keep;                       // keys at positions below it are seen at any distance
+  float cap;                      // > 0: scores are cap tanh(score / cap), in front of the bias
+  const float2* back; int bpairs; // [rows][bpairs] cosines and sines that the result is turned back by (null: not turned)
+  int bneigh;                     // pairs are columns (2 i, 2 i + 1), else (i, i + bpairs)
 };
 struct GqaTurn {
   const double* freq;             // half turns per position
   int pairs;                      // 0: no rotation
   float mul;
   int neighbours;                 // pairs are columns (2 i, 2 i + 1), else (i, i + pairs)
+  const double* vfreq; int vpairs;     // of the values (0: not turned), pairs as above
+  float2* back;                   // [rows][vpairs]: cosine and sine of the values' angles (null: not stored)
 };
 VE_DEVINL float gate_at(const GqaScore& sc, long row, int c) {
   if (!sc.gate) return 1.f;
@@ -51,24 +59,48 @@ struct GqaRows {
   int max_pages;
 };
 
+// Column c of a result turned back, from it and the other column of its pair.
+VE_DEVINL int back_partner(const GqaScore& sc, int c) { return sc.bneigh ? c ^ 1 : c < sc.bpairs ? c + sc.bpairs : c - sc.bpairs; }
+VE_DEVINL float turned_back(const GqaScore& sc, long row, int c, float own, float other) {
+  const float2 a = sc.back[row * sc.bpairs + (sc.bneigh ? c >> 1 : c < sc.bpairs ? c : c - sc.bpairs)];
+  const bool low = sc.bneigh ? !(c & 1) : c < sc.bpairs;
+  return fmaf(own, a.x, low ? other * a.y : -(other * a.y));
+}
+// Four neighbouring columns (from a multiple of four on) whose pairs are neighbours.
+VE_DEVINL float4 turned_back4(const GqaScore& sc, long row, int c, float4 v) {
+  const float2 a = sc.back[row * sc.bpairs + (c >> 1)], b = sc.back[row * sc.bpairs + (c >> 1) + 1];
+  return make_float4(fmaf(v.x, a.x, v.y * a.y), fmaf(v.y, a.x, -(v.x * a.y)), fmaf(v.z, b.x, v.w * b.y), fmaf(v.w, b.x, -(v.z * b.y)));
+}
+
+// Pages of a row or a tile: those of the first tokens, then those from the first window on.
+struct GqaPages {
+  int front, from;                // pages 0 .. front - 1, then from, from + 1, ...
+  VE_DEVINL GqaPages(const GqaScore& sc, int pos) : from(max(0, pos - sc.window + 1) / kGPage) { front = min(from, (sc.keep + kGPage - 1) / kGPage); }
+  VE_DEVINL int of(int i) const { return i < front ? i : from + i - front; }
+  VE_DEVINL int count(int last) const { return front + last / kGPage + 1 - from; }      // last: the last position that is seen
+};
+VE_DEVINL bool sees(const GqaScore& sc, int dist, int key) { return (unsigned)dist < (unsigned)sc.window || (key < sc.keep && dist >= 0); }
+
 VE_DEVINL int page_of(const GqaRows& r, int slot, int kt) { return r.page_table[(long)slot * r.max_pages + kt]; }
 
 // proj row: [q (H d) | k (G d) | v (G dv) | ...]. grid (rows, ceil((H + 2 G) / 8)), a warp per head. norm: queries and keys are divided by
-// their root mean square (behind the rotation), times wq / wk where given.
+// their root mean square, times wq / wk where given, behind the rotation (1) or in front of it (2). hmul: factors of the query heads.
 template <typename X, typename T>
 __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const GqaRows rw, const X* __restrict__ proj, long ld, const GqaTurn tn, int norm,
-                                                        const float* __restrict__ wq, const float* __restrict__ wk, float eps, float coef, int every, int vec,
+                                                        const float* __restrict__ wq, const float* __restrict__ wk, float eps, float coef, int every,
+                                                        const float* __restrict__ hmul, int vec,
                                                         T* __restrict__ qo, T* __restrict__ kpool, T* __restrict__ vpool) {
-  __shared__ __align__(16) float cs[kMaxPairs], sn[kMaxPairs];
+  __shared__ __align__(16) float qcs[kMaxPairs], qsn[kMaxPairs], vcs[kMaxPairs], vsn[kMaxPairs];
   grid_dep_wait();
   grid_dep_launch();
   const long row = blockIdx.x;
   const int item = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const int p = rw.pos[row], s = rw.slot[row];
-  if (tn.pairs) {
-    angle_row(p, tn.freq, tn.pairs, tn.mul, cs, sn);
-    __syncthreads();
-  }
+  if (tn.pairs) angle_row(p, tn.freq, tn.pairs, tn.mul, qcs, qsn);
+  if (tn.vpairs) angle_row(p, tn.vfreq, tn.vpairs, 1.f, vcs, vsn);
+  if (tn.pairs | tn.vpairs) __syncthreads();
+  if (tn.back && blockIdx.y == 0)
+    for (int i = threadIdx.x; i < tn.vpairs; i += 256) tn.back[row * tn.vpairs + i] = make_float2(vcs[i], vsn[i]);
   if (item >= n.H + 2 * n.G) return;
   const bool is_q = item < n.H, is_v = item >= n.H + n.G;
   if (s < 0 && !is_q) return;
@@ -79,26 +111,41 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
     const int page = page_of(rw, s, p / kGPage), at = p % kGPage;
     dst = is_v ? vpool + page * n.vps + ((long)(item - n.H - n.G) * kGPage + at) * n.vw : kpool + page * n.kps + ((long)(item - n.H) * kGPage + at) * n.kw;
   }
-  const int w = is_v ? n.dv : n.d, wide = is_v ? n.vw : n.kw, turned = is_v ? 0 : 2 * tn.pairs;
+  const int w = is_v ? n.dv : n.d, wide = is_v ? n.vw : n.kw, pairs = is_v ? tn.vpairs : tn.pairs, turned = 2 * pairs;
+  const float *cs = is_v ? vcs : qcs, *sn = is_v ? vsn : qsn;
   const float* wn = is_v ? nullptr : is_q ? wq : wk;
-  const bool nrm = norm && !is_v;
-  const float t = is_q && every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
+  const bool nrm = norm && !is_v, before = nrm && norm == 2;
+  float t = is_q && every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
+  if (is_q && hmul) t *= hmul[item];
   if (vec) {                                // widths up to 256 in multiples of eight: four columns per lane and step, kept in registers
     float4 v[2];
-    float ss = 0.f;
+    float ss = 0.f, f = 1.f;
+    auto normed = [&](float4 x, int i) {    // columns from i on, normed in front of the rotation
+      if (!before) return x;
+      const float4 q = wn ? *reinterpret_cast<const float4*>(wn + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+      return make_float4(x.x * f * q.x, x.y * f * q.y, x.z * f * q.z, x.w * f * q.w);
+    };
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int i = (j * 32 + lane) * 4;
       v[j] = i < w ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    if (before) f = 1.f / sqrtf(warp_sum(ss) / (float)w + eps);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = (j * 32 + lane) * 4;
+      if (i < w) v[j] = normed(v[j], i);
       if (i < turned) {
         if (tn.neighbours) {
           const float2 c = *reinterpret_cast<const float2*>(cs + i / 2), z = *reinterpret_cast<const float2*>(sn + i / 2);
           v[j] = make_float4(fmaf(v[j].x, c.x, -(v[j].y * z.x)), fmaf(v[j].y, c.x, v[j].x * z.x), fmaf(v[j].z, c.y, -(v[j].w * z.y)),
                              fmaf(v[j].w, c.y, v[j].z * z.y));
         } else {
-          const bool low = i < tn.pairs;
-          const int k = low ? i : i - tn.pairs;
-          const float4 c = *reinterpret_cast<const float4*>(cs + k), o = load4(src + (low ? i + tn.pairs : k));
+          const bool low = i < pairs;
+          const int k = low ? i : i - pairs, other = low ? i + pairs : k;
+          const float4 c = *reinterpret_cast<const float4*>(cs + k), o = normed(load4(src + other), other);
           float4 z = *reinterpret_cast<const float4*>(sn + k);
           if (low) z = make_float4(-z.x, -z.y, -z.z, -z.w);
           v[j] = make_float4(fmaf(v[j].x, c.x, o.x * z.x), fmaf(v[j].y, c.y, o.y * z.y), fmaf(v[j].z, c.z, o.z * z.z), fmaf(v[j].w, c.w, o.w * z.w));
@@ -106,29 +153,30 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
       }
       ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
     }
-    const float g = nrm ? t / sqrtf(warp_sum(ss) / (float)w + eps) : t;
+    const float g = nrm && !before ? t / sqrtf(warp_sum(ss) / (float)w + eps) : t;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int i = (j * 32 + lane) * 4;
       if (i >= w) continue;
-      const float4 q = wn ? *reinterpret_cast<const float4*>(wn + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+      const float4 q = wn && !before ? *reinterpret_cast<const float4*>(wn + i) : make_float4(1.f, 1.f, 1.f, 1.f);
       store4(dst + i, make_float4(v[j].x * g * q.x, v[j].y * g * q.y, v[j].z * g * q.z, v[j].w * g * q.w));
     }
     return;
   }
+  float f = 1.f;
+  auto raw = [&](int i) { return before ? to_f(src[i]) * f * (wn ? wn[i] : 1.f) : to_f(src[i]); };
   auto value = [&](int i) {
-    const float v = to_f(src[i]);
+    const float v = raw(i);
     if (i >= turned) return v;
-    const bool low = tn.neighbours ? !(i & 1) : i < tn.pairs;
-    const int k = tn.neighbours ? i >> 1 : low ? i : i - tn.pairs, other = tn.neighbours ? i ^ 1 : low ? i + tn.pairs : k;
-    const float o = to_f(src[other]) * sn[k];
+    const bool low = tn.neighbours ? !(i & 1) : i < pairs;
+    const int k = tn.neighbours ? i >> 1 : low ? i : i - pairs, other = tn.neighbours ? i ^ 1 : low ? i + pairs : k;
+    const float o = raw(other) * sn[k];
     return fmaf(v, cs[k], low ? -o : o);
   };
-  float f = 1.f;
   if (nrm) {
     float ss = 0.f;
     for (int i = lane; i < w; i += 32) {
-      const float v = value(i);
+      const float v = before ? to_f(src[i]) : value(i);
       ss = fmaf(v, v, ss);
     }
     f = 1.f / sqrtf(warp_sum(ss) / (float)w + eps);
@@ -136,8 +184,11 @@ __global__ void __launch_bounds__(256) gqa_store_kernel(const GqaDims n, const G
   for (int i = lane; i < wide; i += 32) {
     float v = 0.f;
     if (i < w) {
-      v = value(i) * f;
-      if (wn) v *= wn[i];
+      v = value(i);
+      if (!before) {
+        v *= f;
+        if (wn) v *= wn[i];
+      }
       v *= t;
     }
     dst[i] = from_f<T>(v);
@@ -165,7 +216,9 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const GqaDims n, const Gq
   float acc[NC], m = -FLT_MAX, l = 0.f;
 #pragma unroll
   for (int j = 0; j < NC; ++j) acc[j] = 0.f;
-  for (int key = max(0, p - sc.window + 1) + warp; key <= p; key += 4) {
+  const int begin = max(0, p - sc.window + 1), front = min(sc.keep, begin), total = front + p + 1 - begin;      // first tokens, then the window
+  for (int i = warp; i < total; i += 4) {
+    const int key = i < front ? i : begin + i - front;
     const int page = page_of(rw, s, key / kGPage);
     const T* kr = kpool + page * n.kps + ((long)g * kGPage + key % kGPage) * n.kw;
     const T* vr = vpool + page * n.vps + ((long)g * kGPage + key % kGPage) * n.vw;
@@ -174,6 +227,7 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const GqaDims n, const Gq
     for (int j = 0; j < NC; ++j) v[j] = j * 32 + lane < n.dv ? to_f(vr[j * 32 + lane]) : 0.f;
     for (int i = lane; i < n.d; i += 32) dot = fmaf(to_f(kr[i]), sm[i], dot);
     dot = warp_sum(dot) * sc.scale;
+    if (sc.cap > 0.f) dot = soft_cap_of(dot, sc.cap);
     if (sc.bias) dot += sc.bias[(long)h * sc.L + min(p - key, sc.L - 1)];
     const float mn = fmaxf(m, dot), corr = m == -FLT_MAX ? 0.f : expf(m - mn), e = expf(dot - mn);
     m = mn;
@@ -197,11 +251,16 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const GqaDims n, const Gq
     f[w] = sm_m[w] == -FLT_MAX ? 0.f : expf(sm_m[w] - mx);
     lt += sm_l[w] * f[w];
   }
-  for (int i = threadIdx.x; i < n.dv; i += 128) {
+  auto sum = [&](int i) {
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) v += os[w * NC * 32 + i] * f[w];
-    orow[i] = from_f<O>(v / lt * sc.out_scale * gate_at(sc, row, h * n.dv + i));
+    return v / lt;
+  };
+  for (int i = threadIdx.x; i < n.dv; i += 128) {
+    float v = sum(i);
+    if (sc.back) v = turned_back(sc, row, i, v, sum(back_partner(sc, i)));
+    orow[i] = from_f<O>(v * sc.out_scale * gate_at(sc, row, h * n.dv + i));
   }
 }
 
@@ -221,8 +280,10 @@ VE_DEVINL uint32_t gq_pack(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&t);
 }
 
+// Four columns (from a multiple of four on; c counts over all heads) of an output row of any alignment.
 template <typename O>
-VE_DEVINL void put_row(O* p, float4 v, const GqaScore& sc, long row, int c) {            // four columns (from c on) of an output row of any alignment
+VE_DEVINL void put_row(O* p, float4 v, const GqaScore& sc, long row, int c, int dv) {
+  if (sc.back) v = turned_back4(sc, row, c % dv, v);
   p[0] = from_f<O>(v.x * gate_at(sc, row, c));
   p[1] = from_f<O>(v.y * gate_at(sc, row, c + 1));
   p[2] = from_f<O>(v.z * gate_at(sc, row, c + 2));
@@ -265,17 +326,19 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
     return;
   }
   // the grid does not know the position: a row takes as many of its splits as have at least kGMinPages pages
-  const int p = a.rw.pos[row], win = a.sc.window, kt0 = max(0, p - win + 1) / kGPage, pages = p / kGPage + 1 - kt0;
+  const int p = a.rw.pos[row];
+  const GqaPages pg(a.sc, p);
+  const int pages = pg.count(p);
   const int per = max(kGMinPages, (pages + a.nsplit - 1) / a.nsplit), used = (pages + per - 1) / per;
   if (z >= used) return;
-  const int kt_begin = kt0 + z * per, kt_end = min(kt0 + pages, kt_begin + per);
+  const int kt_begin = z * per, kt_end = min(pages, kt_begin + per);      // (places in the list of pages)
   if (tid == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(&full[i], 1);
     mbar_fence_init();
   }
   __syncthreads();
   auto issue = [&](int kt, int stage) {
-    const int page = page_of(a.rw, s, kt);
+    const int page = page_of(a.rw, s, pg.of(kt));
     uint8_t* kb = smem + stage * STG;
     mbar_expect_tx(&full[stage], STG);
 #pragma unroll
@@ -298,7 +361,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       qf[kk][e] = ok && c < n.kw ? *reinterpret_cast<const uint32_t*>(qr + c) : 0u;
       qf[kk][2 + e] = ok && c + 8 < n.kw ? *reinterpret_cast<const uint32_t*>(qr + c + 8) : 0u;
     }
-  const float scale2 = a.sc.scale * kLog2e;
+  const float scale2 = a.sc.scale * kLog2e, cap2 = a.sc.cap * kLog2e, to_cap = a.sc.cap > 0.f ? a.sc.scale / a.sc.cap : 0.f;
   const float* tab[2] = {a.sc.bias + (long)head[0] * a.sc.L, a.sc.bias + (long)head[1] * a.sc.L};
   float far[2] = {0.f, 0.f};
   if (a.sc.bias) {
@@ -331,7 +394,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       gq_mma(sa[0], qf[kk], b0, b1);
       gq_mma(sa[1], qf[kk], b2, b3);
     }
-    const int first = kt * kGPage + key0;
+    const int first = pg.of(kt) * kGPage + key0;
     const bool near = a.sc.bias && p - (first + 15) < a.sc.L - 1;
     float mx[2] = {-FLT_MAX, -FLT_MAX};
 #pragma unroll
@@ -340,7 +403,8 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       for (int e = 0; e < 4; ++e) {
         const int dist = p - (first + nt * 8 + 2 * t + (e & 1)), r = e >> 1;
         const float b = near ? tab[r][min(max(dist, 0), a.sc.L - 1)] * kLog2e : far[r];
-        const float v = (unsigned)dist < (unsigned)win ? fmaf(sa[nt][e], scale2, b) : -FLT_MAX;
+        const float x = a.sc.cap > 0.f ? fmaf(tanhf(sa[nt][e] * to_cap), cap2, b) : fmaf(sa[nt][e], scale2, b);
+        const float v = sees(a.sc, dist, p - dist) ? x : -FLT_MAX;
         sa[nt][e] = v;
         mx[r] = fmaxf(mx[r], v);
       }
@@ -410,8 +474,8 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
   __syncthreads();
   auto sink_of = [&](int h) { return a.sc.sink ? a.sc.sink[h] * kLog2e : -FLT_MAX; };
   for (int i = tid; i < nh * n.dv; i += 128) {
-    const int hr = i / n.dv, c = i % n.dv;
-    float m = -FLT_MAX, acc = 0.f, l = 0.f;
+    const int hr = i / n.dv, c = i % n.dv, c2 = a.sc.back && used == 1 ? back_partner(a.sc, c) : c;
+    float m = -FLT_MAX, acc = 0.f, acc2 = 0.f, l = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, ms[w * 16 + hr]);
 #pragma unroll
@@ -420,10 +484,12 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
       if (mw != -FLT_MAX) {
         const float f = exp2f(mw - m);
         acc = fmaf(os[(w * 16 + hr) * DV + c], f, acc);
+        acc2 = fmaf(os[(w * 16 + hr) * DV + c2], f, acc2);
         l = fmaf(ls[w * 16 + hr], f, l);
       }
     }
     if (used == 1) {
+      if (a.sc.back) acc = turned_back(a.sc, row, c, acc, acc2);
       const float snk = sink_of(h0 + hr), top = fmaxf(m, snk), f = exp2f(m - top);
       const float den = fmaf(l, f, a.sc.sink ? exp2f(snk - top) : 0.f);
       out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * f / den * a.sc.out_scale * gate_at(a.sc, row, (h0 + hr) * n.dv + c));
@@ -453,7 +519,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
     sw[hr * 64 + lane + 32] = w1 * inv;
   }
   __syncthreads();
-  if (n.dv % 4 == 0) {
+  if (n.dv % 4 == 0 && (!a.sc.back || a.sc.bneigh)) {
     // four columns per thread; few columns: the splits are dealt to up to four thread groups
     const int c4 = n.dv / 4, items = nh * c4, ng = items <= 32 ? 4 : items <= 64 ? 2 : 1, per = 128 / ng, y0 = tid / per;
     float4* acc4 = reinterpret_cast<float4*>(sw + 16 * 64);
@@ -468,7 +534,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
         v = make_float4(fmaf(f, x.x, v.x), fmaf(f, x.y, v.y), fmaf(f, x.z, v.z), fmaf(f, x.w, v.w));
       }
       if (ng > 1) acc4[tid] = v;
-      else put_row(out + row * ldo + (long)(h0 + hr) * n.dv + c, v, a.sc, row, (h0 + hr) * n.dv + c);
+      else put_row(out + row * ldo + (long)(h0 + hr) * n.dv + c, v, a.sc, row, (h0 + hr) * n.dv + c, n.dv);
     }
     if (ng > 1) {
       __syncthreads();
@@ -479,16 +545,21 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaDecode a, O* _
           v = make_float4(v.x + x.x, v.y + x.y, v.z + x.z, v.w + x.w);
         }
         const int c = (h0 + tid / c4) * n.dv + (tid % c4) * 4;
-        put_row(out + row * ldo + c, v, a.sc, row, c);
+        put_row(out + row * ldo + c, v, a.sc, row, c, n.dv);
       }
     }
   } else {
     for (int i = tid; i < nh * n.dv; i += 128) {
       const int hr = i / n.dv, c = i % n.dv;
       const float* part = a.o_part + (row * n.H + h0 + hr) * a.nsplit * n.dv + c;
-      float acc = 0.f;
+      auto sum = [&](int off) {
+        float acc = 0.f;
 #pragma unroll 8
-      for (int y = 0; y < used; ++y) acc = fmaf(sw[hr * 64 + y], __ldcg(part + (long)y * n.dv), acc);
+        for (int y = 0; y < used; ++y) acc = fmaf(sw[hr * 64 + y], __ldcg(part + (long)y * n.dv + off), acc);
+        return acc;
+      };
+      float acc = sum(0);
+      if (a.sc.back) acc = turned_back(a.sc, row, c, acc, sum(back_partner(a.sc, c) - c));
       out[row * ldo + (long)(h0 + hr) * n.dv + c] = from_f<O>(acc * gate_at(a.sc, row, (h0 + hr) * n.dv + c));
     }
   }
@@ -521,11 +592,13 @@ using namespace ve;
 #define VE_GMAKE GqaDims{H, G, d, dv, kw, vw, kps, vps}
 #define VE_GROWS const void* pos, const void* slot, const void* page_table, int max_pages
 #define VE_RMAKE GqaRows{(const int*)pos, (const int*)slot, (const int*)page_table, max_pages}
-#define VE_GSCORE float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32
-#define VE_SMAKE gscore(scale, bias, L, sink, out_scale, window, gate, ldg, gate32, dv)
-static GqaScore gscore(float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32, int dv) {
+#define VE_GSCORE float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32, int keep, float cap, \
+    const void* back, int bpairs, int bneigh
+#define VE_SMAKE gscore(scale, bias, L, sink, out_scale, window, gate, ldg, gate32, dv, keep, cap, back, bpairs, bneigh)
+static GqaScore gscore(float scale, const void* bias, int L, const void* sink, float out_scale, int window, const void* gate, long ldg, int gate32, int dv,
+                       int keep, float cap, const void* back, int bpairs, int bneigh) {
   return GqaScore{scale, (const float*)bias, L, (const float*)sink, out_scale, window > 0 ? window : INT_MAX, gate, ldg, gate32,
-                  dv % 8 == 0 && ldg % 8 == 0 && !((uintptr_t)gate & 15)};
+                  dv % 8 == 0 && ldg % 8 == 0 && !((uintptr_t)gate & 15), window > 0 && keep > 0 ? keep : 0, cap, (const float2*)back, bpairs, bneigh};
 }
 static bool gdims_ok(const GqaDims& n) {
   return n.G > 0 && n.H > 0 && n.H % n.G == 0 && n.d > 0 && n.dv > 0 && n.kw >= n.d && n.vw >= n.dv && n.kps >= (long)n.G * 64 * n.kw && n.vps >= (long)n.G * 64 * n.vw;
@@ -538,19 +611,20 @@ static int pool_map(CUtensorMap* m, const void* pool, long pages, const GqaDims&
 
 extern "C" {
 
-// proj rows fp32 when x32 (else bf16); f32: queries and pools fp32 (else bf16). pairs 0: no rotation; norm 0: no norm, else wq and wk are its
-// weights (null: none); every 0: no temperature.
+// proj rows fp32 when x32 (else bf16); f32: queries and pools fp32 (else bf16). pairs 0: no rotation; norm 0: no norm, 1: behind the rotation, 2: in
+// front of it, wq and wk are its weights (null: none); every 0: no temperature; hmul: factors of the query heads (null: none); vpairs: 0, or dv / 2
+// pairs of value columns, whose angles are stored to back [rows][vpairs][2] (null: not).
 int ve_gqa_store(VE_GDIMS, VE_GROWS, const void* proj, long ld, int x32, const void* freq, int pairs, float mul, int neighbours, int norm, const void* wq,
-                 const void* wk, float eps, float coef, int every, void* qo, void* kpool, void* vpool, int rows, int f32, cudaStream_t st) {
+                 const void* wk, float eps, float coef, int every, const void* hmul, const void* vfreq, int vpairs, void* back, void* qo, void* kpool, void* vpool, int rows, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n) || pairs < 0 || pairs > kMaxPairs || 2 * pairs > d || (pairs && !freq)) return cudaErrorInvalidValue;
+  if (!gdims_ok(n) || pairs < 0 || pairs > kMaxPairs || 2 * pairs > d || (pairs && !freq) || (vpairs && (2 * vpairs != dv || vpairs > kMaxPairs || !vfreq))) return cudaErrorInvalidValue;
   const dim3 grid(rows, (H + 2 * G + 7) / 8);
-  const GqaTurn tn{(const double*)freq, pairs, mul, neighbours};
+  const GqaTurn tn{(const double*)freq, pairs, mul, neighbours, (const double*)vfreq, vpairs, (float2*)back};
   const int vec = d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && kw == d && vw == dv && ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)wq & 15) &&
-                  !((uintptr_t)wk & 15) && pairs % (neighbours ? 2 : 4) == 0;
+                  !((uintptr_t)wk & 15) && pairs % (neighbours ? 2 : 4) == 0 && vpairs % (neighbours ? 2 : 4) == 0;
 #define VE_GS(X, T) launch_pdl(gqa_store_kernel<X, T>, grid, dim3(256), 0, st, n, VE_RMAKE, (const X*)proj, ld, tn, norm, (const float*)wq, (const float*)wk, eps, coef, \
-    every, vec, (T*)qo, (T*)kpool, (T*)vpool)
+    every, (const float*)hmul, vec, (T*)qo, (T*)kpool, (T*)vpool)
   if (f32) VE_GS(float, float);
   else if (x32) VE_GS(float, __nv_bfloat16);
   else VE_GS(__nv_bfloat16, __nv_bfloat16);
@@ -562,7 +636,7 @@ int ve_gqa_store(VE_GDIMS, VE_GROWS, const void* proj, long ld, int x32, const v
 int ve_gqa_rows(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpool, const void* vpool, void* out, long ldo, int o32, int rows, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n) || kw > 2048 || dv > 1024 || (bias && L < 1) || (f32 && !o32)) return cudaErrorInvalidValue;
+  if (!gdims_ok(n) || kw > 2048 || dv > 1024 || (bias && L < 1) || (f32 && !o32) || (back && 2 * bpairs != dv)) return cudaErrorInvalidValue;
 #define VE_GR(NC, T, O) launch_pdl(gqa_rows_kernel<NC, T, O>, dim3(rows, H), dim3(128), (size_t)(kw + 4 * NC * 32) * 4, st, n, VE_RMAKE, VE_SMAKE, (const T*)q, \
     (const T*)kpool, (const T*)vpool, (O*)out, ldo)
 #define VE_GR_T(T, O) do { if (dv <= 64) VE_GR(2, T, O); else if (dv <= 128) VE_GR(4, T, O); else if (dv <= 256) VE_GR(8, T, O); else VE_GR(32, T, O); } while (0)
@@ -579,7 +653,7 @@ int ve_gqa_decode(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpoo
                   void* out, long ldo, int o32, int rows, void* status, cudaStream_t st) {
   if (rows <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 256 || nsplit < 1 || nsplit > 64 || (bias && L < 1) || (nsplit > 1 && (!o_part || !lse || !tickets)))
+  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 256 || nsplit < 1 || nsplit > 64 || (bias && L < 1) || (back && 2 * bpairs != dv) || (nsplit > 1 && (!o_part || !lse || !tickets)))
     return cudaErrorInvalidValue;
   CUtensorMap km, vm;
   int rc = pool_map(&km, kpool, pages, n, kw, kps);
@@ -596,12 +670,14 @@ int ve_gqa_decode(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpoo
 #undef VE_GD
 }
 
-// Tiles of at most 128 / (H / G) tokens of one sequence (rows tile_first .. + tile_count of the batch); kw <= 256, vw <= 128, scale > 0.
+// Tiles of at most 128 / (H / G) tokens of one sequence (rows tile_first .. + tile_count of the batch); kw <= 256, vw <= 128, scale > 0, pairs of
+// columns that the result is turned back in are neighbours.
 int ve_gqa_prefill(VE_GDIMS, VE_GROWS, VE_GSCORE, const void* q, const void* kpool, const void* vpool, long pages, const void* tile_first, const void* tile_count,
                    int ntiles, void* out, long ldo, void* status, cudaStream_t st) {
   if (ntiles <= 0) return 0;
   const GqaDims n = VE_GMAKE;
-  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 128 || H / G > 128 || !(scale > 0.f) || ((uintptr_t)q & 15) || (bias && L < 1)) return cudaErrorInvalidValue;
+  if (!gdims_ok(n) || kw % 8 || vw % 8 || kw > 256 || vw > 128 || H / G > 128 || !(scale > 0.f) || ((uintptr_t)q & 15) || (bias && L < 1) ||
+      (back && (2 * bpairs != dv || !bneigh))) return cudaErrorInvalidValue;
   CUtensorMap km, vm;
   int rc = pool_map(&km, kpool, pages, n, kw, kps);
   if (!rc) rc = pool_map(&vm, vpool, pages, n, vw, vps);

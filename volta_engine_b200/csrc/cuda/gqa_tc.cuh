@@ -7,8 +7,9 @@
 //     the pages' by the tensor map); keys and values have rings of their own (a key page is free as soon as its scores are done);
 //   * a bias by distance is added to the scaled scores: one value per row for pages far enough back, a table look-up otherwise;
 //   * the softmax weights enter the second product as two bf16 terms (value and remainder), so they keep 32-bit quality;
-//   * with a sliding window the pages in front of the first token's window are not visited;
-//   * the sink joins the sums in the epilogue, the gate multiplies the result there.
+//   * with a sliding window the pages between the first tokens that stay in sight and the first token's window are not visited;
+//   * a soft cap bends the scores in front of the bias (an exponential each and a quarter of a reciprocal: cap2_of4);
+//   * the sink joins the sums in the epilogue, the result is turned back and gated there.
 // Every wait is bounded; on expiry the CTA records a status code, skips its stores and frees its TMEM.
 #pragma once
 
@@ -58,6 +59,18 @@ VE_DEVINL void gate8(const GqaScore& sc, long row, int c, int live, float* g) {
   }
 }
 
+// Four capped scores in log2 units: cap2 tanh(s to_cap) with tanh(x) = 1 - 2 / (1 + exp(2 x)); to2 = 2 log2(e) to_cap. One reciprocal serves
+// the four (the exponents are held below 30, where the quotient is far below the last digit of one).
+VE_DEVINL void cap2_of4(float* s, float to2, float cap2) {
+  const float a = 1.f + ex2_approx(fminf(s[0] * to2, 30.f)), b = 1.f + ex2_approx(fminf(s[1] * to2, 30.f));
+  const float c = 1.f + ex2_approx(fminf(s[2] * to2, 30.f)), d = 1.f + ex2_approx(fminf(s[3] * to2, 30.f));
+  const float ab = a * b, cd = c * d, r = -2.f * cap2 * rcp_approx(ab * cd), rab = r * cd, rcd = r * ab;
+  s[0] = fmaf(rab, b, cap2);
+  s[1] = fmaf(rab, a, cap2);
+  s[2] = fmaf(rcd, d, cap2);
+  s[3] = fmaf(rcd, c, cap2);
+}
+
 template <int DQC, int DVC>
 __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc p, const __grid_constant__ CUtensorMap kmap,
                                                                     const __grid_constant__ CUtensorMap vmap) {
@@ -79,8 +92,9 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
   const int tile = gridDim.x - 1 - blockIdx.x, kvh = blockIdx.y, hpg = p.n.H / p.n.G;      // late tiles (many keys) first
   const int first = p.tile_first[tile], count = p.tile_count[tile], slot = p.rw.slot[first];
   if (slot < 0 || count <= 0) return;
-  const int win = p.sc.window, kt0 = max(0, p.rw.pos[first] - win + 1) / kGPage;        // first page a row sees
-  const int n = p.rw.pos[first + count - 1] / kGPage + 1 - kt0;         // pages
+  const int win = p.sc.window;
+  const GqaPages pg(p.sc, p.rw.pos[first]);
+  const int n = pg.count(p.rw.pos[first + count - 1]);                  // pages
   if (tid == 0) {
     for (int i = 0; i < KS; ++i) {
       mbar_init(&kfull[i], 1);
@@ -129,7 +143,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       prefetch_tmap(&kmap);
       prefetch_tmap(&vmap);
       for (int j = 0; j < n; ++j) {
-        const int ks = j % KS, vs = j % VS, page = page_of(p.rw, slot, kt0 + j);
+        const int ks = j % KS, vs = j % VS, page = page_of(p.rw, slot, pg.of(j));
         if (j >= KS && !mbar_wait(&kempty[ks], ((j / KS) - 1) & 1)) {
           atomicExch(&s_fail, 1);
           break;
@@ -193,7 +207,9 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
     const uint32_t t_lane = tmem_base + ((uint32_t)((warp & 3) * 32) << 16);
     const uint32_t o_col = O_COL + strm * DV;
     const int n_mine = (n - strm + 1) >> 1;
-    const float scale2 = p.sc.scale * kLog2e;
+    const bool capped = p.sc.cap > 0.f;
+    const float cap2 = p.sc.cap * kLog2e, to2 = capped ? 2.f * kLog2e * p.sc.scale / p.sc.cap : 0.f;
+    const float scale2 = capped ? 1.f : p.sc.scale * kLog2e;           // of what is in sv behind the cap
     const float* tab = p.sc.bias + (long)r_head * p.sc.L;
     const int L1 = p.sc.bias ? p.sc.L - 1 : 0;
     const float far = p.sc.bias ? tab[L1] * kLog2e : 0.f;
@@ -201,7 +217,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
     bool ok = true;
     uint8_t* prow = p_s + strm * 2 * PB + r * 128;
     for (int i = 0; i < n_mine; ++i) {
-      const int b = i & 1, key0 = (kt0 + 2 * i + strm) * 64;
+      const int b = i & 1, key0 = pg.of(2 * i + strm) * 64;
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[strm][b], (i >> 1) & 1));
       if (!ok) break;
       tc_fence_after();
@@ -209,6 +225,10 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       tmem_ld32(t_lane + strm * 128 + b * 64, reinterpret_cast<uint32_t*>(sv));
       tmem_ld32(t_lane + strm * 128 + b * 64 + 32, reinterpret_cast<uint32_t*>(sv) + 32);
       tmem_ld_wait();
+      if (capped) {
+#pragma unroll
+        for (int e = 0; e < 64; e += 4) cap2_of4(sv + e, to2, cap2);
+      }
       // far pages: the scores stay as they are and one addend per row stands for the bias; near pages: scaled, bias by distance
       const bool near = p.sc.bias && __any_sync(0xffffffffu, r_pos - key0 - 63 < L1);
       if (near) {
@@ -218,7 +238,7 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
       const float mul = near ? 1.f : scale2, add = near ? 0.f : far;
       if (!r_ok || key0 + 63 > r_pos || r_pos - key0 >= win) {
 #pragma unroll
-        for (int e = 0; e < 64; ++e) sv[e] = r_ok && (unsigned)(r_pos - key0 - e) < (unsigned)win ? sv[e] : NEG_INF;
+        for (int e = 0; e < 64; ++e) sv[e] = r_ok && sees(p.sc, r_pos - key0 - e, key0 + e) ? sv[e] : NEG_INF;
       }
       float mx0 = sv[0], mx1 = sv[1], mx2 = sv[2], mx3 = sv[3];
 #pragma unroll
@@ -317,6 +337,13 @@ __global__ void __launch_bounds__(kGtThreads, 1) gqa_prefill_kernel(const GqaTc 
             if (n > 1) {
               a = fmaf(__uint_as_float(ow[q4 * 8 + 2 * e]), f1, a);
               c = fmaf(__uint_as_float(ow[q4 * 8 + 2 * e + 1]), f1, c);
+            }
+            if (p.sc.back) {                             // (only pairs that exist: the last columns of eight may not)
+              const int m = (col >> 1) + e;
+              const float2 z = m < p.sc.bpairs ? p.sc.back[(long)r_tok * p.sc.bpairs + m] : make_float2(0.f, 0.f);
+              const float x = fmaf(a, z.x, c * z.y);
+              c = fmaf(c, z.x, -(a * z.y));
+              a = x;
             }
             w[e] = gq_pack(a * gt[2 * e], c * gt[2 * e + 1]);
           }

@@ -1,11 +1,12 @@
 // Linear attention with a decayed outer-product state, one fp32 state S [dk][dv] per (slot, head):
 //     S_t = diag(d_t) S_(t-1) + k_t v_t^T,      o_t = S_t^T q_t
 // Three ways to get decay and key from a projection row [ q (H dk) | x (H dk) | v (H dv) | ... ]:
-//   MODE 0  constant decay per head (table), k = silu(x), v = silu(v)                     ("lightning" attention)
+//   MODE 0  constant decay per head (table), k = silu(x), v = silu(v)                     ("lightning" attention), or with `plain` k = x,
+//           v as projected, q scaled by a constant                                        (retention)
 //   MODE 1  forget gate per channel: f = lower + (1 - lower) sigmoid(x + bias), d = f, k = 1 - f, v as projected   (HGRN2)
 //   MODE 2  decay per channel sigmoid(z)^(1 / tau) with z = W a + bias for a low-rank row a of the projection; k = x, v as projected,
 //           q scaled by a constant                                                        (gated linear attention)
-// q = silu(q) in modes 0 and 1. Gates, decays, states and outputs are fp32; the file is compiled without fast-math.
+// q = silu(q) in modes 0 (but for `plain`) and 1. Gates, decays, states and outputs are fp32; the file is compiled without fast-math.
 //
 //   linattn_decay   the decays of mode 2 as rows (for the chunks; the stepped kernel forms its own)
 //   linattn_step    walks the rows of a segment in order with the state in registers (decode rows, short portions, and the
@@ -22,6 +23,7 @@
 // A segment whose first row is at position 0 starts from a zero state. Segments come from a host table (first row, row count)
 // or, without one, from the slots of the rows themselves (rows of one slot are consecutive positions in order).
 #include "rowmath.cuh"
+#include "slot_rows.cuh"
 
 namespace ve {
 
@@ -36,6 +38,7 @@ struct LinArgs {
   int rows, H, dk, dv;
   const float* w2; int rank, a_col;             // MODE 2: [H dk][rank], first column of the low-rank part in a projection row
   float inv_tau, q_scale;
+  int plain;                                    // MODE 0: operands as projected, q scaled
 };
 
 // sigmoid(z)^inv_tau through the logarithm of the sigmoid, which is exact on both sides
@@ -58,27 +61,6 @@ VE_DEVINL float lowrank_of(const X* __restrict__ a, const float* __restrict__ w,
   }
   for (; r < rank; ++r) z = fmaf(w[r], to_f(a[r]), z);
   return z;
-}
-
-// Rows of the segment that blockIdx.z stands for; -1 when there is nothing to do.
-VE_DEVINL int segment_of(const LinArgs& a, int z, int& count) {
-  if (a.seg_first) {
-    count = a.seg_count[z];
-    return count > 0 ? a.seg_first[z] : -1;
-  }
-  const int s = a.slot[z];
-  if (s < 0) return -1;
-  for (int i = 0; i < z; ++i)
-    if (a.slot[i] == s) return -1;
-  count = -1;                                   // rows of the slot are found while walking
-  return z;
-}
-VE_DEVINL int next_row(const LinArgs& a, int i, int left) {
-  if (a.seg_first) return left > 1 ? i + 1 : -1;
-  const int s = a.slot[i];
-  for (int j = i + 1; j < a.rows; ++j)
-    if (a.slot[j] == s) return j;
-  return -1;
 }
 
 // block (32, 8): lane = value column, y = key group (channels y, y + 8, ...); NK channels per thread.
@@ -104,6 +86,7 @@ __global__ void __launch_bounds__(256) linattn_step_kernel(const LinArgs a) {
     S[j] = (!fresh && live && k < a.dk) ? st[(long)k * a.dv] : 0.f;
   }
   const float head_decay = MODE == 0 ? a.decay[h] : 0.f;
+  const bool plain = MODE == 0 && a.plain;
   float bias = 0.f, low = 0.f;
   if (MODE == 1 && tid < a.dk) {
     bias = a.bias[h * a.dk + tid];
@@ -124,8 +107,8 @@ __global__ void __launch_bounds__(256) linattn_step_kernel(const LinArgs a) {
   while (i >= 0) {
     if (tid < NK * 8) {
       const bool in = tid < a.dk;
-      sq[b][tid] = in ? (MODE == 2 ? rq * a.q_scale : silu_of(rq)) : 0.f;
-      if (MODE == 0) sk[b][tid] = in ? silu_of(rx) : 0.f;
+      sq[b][tid] = in ? (MODE == 2 || plain ? rq * a.q_scale : silu_of(rq)) : 0.f;
+      if (MODE == 0) sk[b][tid] = in ? (plain ? rx : silu_of(rx)) : 0.f;
       else if (MODE == 2) {
         sk[b][tid] = in ? rx : 0.f;
         sd[b][tid] = in ? root_decay(rz, a.inv_tau) : 0.f;
@@ -135,7 +118,7 @@ __global__ void __launch_bounds__(256) linattn_step_kernel(const LinArgs a) {
         sk[b][tid] = in ? (1.f - low) * sigmoid_of(-z) : 0.f;
       }
     }
-    const float v = MODE == 0 ? silu_of(rv) : rv;
+    const float v = MODE == 0 && !plain ? silu_of(rv) : rv;
     const int nxt = next_row(a, i, left);
     --left;
     if (nxt >= 0) {
@@ -192,6 +175,7 @@ struct LinChunkArgs {
   int H, dk, dv, vec;                   // vec: 16-byte copies are aligned
   const float* dec;                     // MODE 2: decays [rows][H dk]
   float q_scale;
+  int plain;                            // as above
 };
 
 VE_DEVINL void la_ldsm_x4(uint32_t addr, uint32_t* r) {
@@ -303,6 +287,7 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
       }
   const bool ch = tid < a.dk;
   const float head_decay = MODE == 0 ? a.decay[h] : 0.f;
+  const bool plain = MODE == 0 && a.plain;
   float bias = 0.f, low = 0.f, prod = 1.f;
   if (MODE == 1 && ch) {
     bias = a.bias[h * a.dk + tid];
@@ -327,7 +312,7 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         const bool in = ch && i < live;                   // rows behind the end: decay one, key zero
         if (MODE == 0) {
           f[i] = in ? head_decay : 1.f;
-          k[i] = in ? silu_of(x) : 0.f;
+          k[i] = in ? (plain ? x : silu_of(x)) : 0.f;
         } else if (MODE == 2) {
           f[i] = in ? rw[i * RAW + 2 * DK + DV + tid] : 1.f;
           k[i] = x;                                       // (zero where there is no row or channel)
@@ -339,7 +324,7 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
         }
         run *= f[i];
         if (OUT) {
-          const float q = MODE == 2 ? rw[i * RAW + tid] * a.q_scale : in ? silu_of(rw[i * RAW + tid]) : 0.f;
+          const float q = MODE == 2 || plain ? rw[i * RAW + tid] * a.q_scale : in ? silu_of(rw[i * RAW + tid]) : 0.f;
           if (MODE != 2) {
             sf[i * DK + tid] = f[i];
             sk[i * DK + tid] = k[i];
@@ -360,7 +345,7 @@ __global__ void __launch_bounds__(128) linattn_chunk_kernel(const LinChunkArgs a
     for (int i = tid; i < 16 * DV; i += 128) {
       const int r = i / DV, v = i % DV;
       const float x = rw[r * RAW + 2 * DK + v];
-      vs[r * VP + v] = f2bf(MODE == 0 ? silu_of(x) : x);
+      vs[r * VP + v] = f2bf(MODE == 0 && !plain ? silu_of(x) : x);
     }
     __syncthreads();
     float o[MT * 2][4];
@@ -587,16 +572,16 @@ using namespace ve;
 
 extern "C" {
 
-// mode 0 / 1 / 2 as above (bias / lower, decay, or bias / w2 / rank / a_col / inv_tau / q_scale accordingly). x32: the projection rows are fp32 (else bf16). nseg > 0: segment
+// mode 0 / 1 / 2 as above (bias / lower, decay, or bias / w2 / rank / a_col / inv_tau / q_scale accordingly; plain: q_scale too). x32: the projection rows are fp32 (else bf16). nseg > 0: segment
 // table; 0: segments from the slots of the rows (a few rows only: every CTA scans them).
 int ve_linattn_step(const void* proj, long ld, int x32, const void* pos, const void* slot, const void* seg_first, const void* seg_count, int nseg,
                     void* state, const void* bias, const void* lower, const void* decay, void* o, long ldo, int rows, int H, int dk, int dv,
-                    int mode, const void* w2, int rank, int a_col, float inv_tau, float q_scale, cudaStream_t st) {
+                    int mode, const void* w2, int rank, int a_col, float inv_tau, float q_scale, int plain, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (dk < 1 || dk > 256 || dv < 1 || H < 1 || (mode == 0 ? !decay : mode == 1 ? !bias || !lower : !bias || !w2 || rank < 1)) return cudaErrorInvalidValue;
   if (mode == 2 && rank % 4 == 0 && ((uintptr_t)w2 & 15)) return cudaErrorInvalidValue;
   LinArgs a{proj, ld, (const int*)pos, (const int*)slot, nseg > 0 ? (const int*)seg_first : nullptr, (const int*)seg_count, (float*)state,
-            (const float*)bias, (const float*)lower, (const float*)decay, (float*)o, ldo, rows, H, dk, dv, (const float*)w2, rank, a_col, inv_tau, q_scale};
+            (const float*)bias, (const float*)lower, (const float*)decay, (float*)o, ldo, rows, H, dk, dv, (const float*)w2, rank, a_col, inv_tau, q_scale, plain};
   const dim3 grid(H, (dv + 31) / 32, nseg > 0 ? nseg : rows), block(32, 8);
 #define VE_LS(NK, X, MODE) launch_pdl(linattn_step_kernel<NK, X, MODE>, grid, block, 0, st, a)
 #define VE_LS_M(NK, X) do { if (mode == 0) VE_LS(NK, X, 0); else if (mode == 1) VE_LS(NK, X, 1); else VE_LS(NK, X, 2); } while (0)
@@ -638,14 +623,14 @@ int ve_linattn_decay(const void* a, long lda, int x32, const void* w, const void
 // any segment.
 int ve_linattn_chunk(const void* proj, long ld, const void* pos, const void* slot, const void* chunk_seg, const void* chunk_first, const void* chunk_count,
                      const void* seg_chunk0, int chunks, int segs, int longest, void* state, void* start, void* total, const void* bias, const void* lower,
-                     const void* decay, void* o, long ldo, int H, int dk, int dv, int mode, const void* dec, float q_scale, cudaStream_t st) {
+                     const void* decay, void* o, long ldo, int H, int dk, int dv, int mode, const void* dec, float q_scale, int plain, cudaStream_t st) {
   if (chunks <= 0) return 0;
   if (mode == 2 && !dec) return cudaErrorInvalidValue;
   if (dk < 1 || dk > 128 || dv < 1 || dv > 128 || H < 1 || segs < 1 || (mode == 0 ? !decay : mode == 1 && (!bias || !lower))) return cudaErrorInvalidValue;
   const int vec = !((uintptr_t)proj & 15) && ld % 4 == 0 && dk % 4 == 0 && dv % 4 == 0 && !((uintptr_t)dec & 15);
   LinChunkArgs a{(const float*)proj, ld, (const int*)pos, (const int*)slot, (const int*)chunk_seg, (const int*)chunk_first, (const int*)chunk_count,
                  (const int*)seg_chunk0, (float*)state, (float*)start, (float*)total, (const float*)bias, (const float*)lower, (const float*)decay,
-                 (float*)o, ldo, H, dk, dv, vec, (const float*)dec, q_scale};
+                 (float*)o, ldo, H, dk, dv, vec, (const float*)dec, q_scale, plain};
 #define VE_LC(DK, DV) return mode == 0 ? launch_chunks<DK, DV, 0>(a, chunks, segs, longest, st) : mode == 1 ? launch_chunks<DK, DV, 1>(a, chunks, segs, longest, st) \
     : launch_chunks<DK, DV, 2>(a, chunks, segs, longest, st)
 #define VE_LC_V(DK) do { if (dv <= 32) VE_LC(DK, 32); if (dv <= 64) VE_LC(DK, 64); VE_LC(DK, 128); } while (0)

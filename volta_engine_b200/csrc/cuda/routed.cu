@@ -1,9 +1,10 @@
 // Routed feed-forwards (mixture of experts) of decoders with an fp32 residual, weights in bf16 (or fp32 for the all-32-bit form):
-//   route_rows   scores = softmax over all experts, in fp32; experts come in equal groups of neighbours, only the best groups stay open (a
+//   route_rows   scores = softmax over all experts or the sigmoid of every logit, in fp32; experts come in equal groups of neighbours, only the best groups stay open (a
 //                group's score: its best member, or the sum of its two best); the best open experts with their scores as weights
 //                (optionally renormalised, times a factor); ties go to the lower index
-//   routed_up    a few rows: routing, then gate and up rows of the chosen experts and the clamped gated unit
-//   routed_down  a few rows: sum over a row's experts of weight * W_down a
+//   routed_up    a few rows: routing, then gate and up rows of the chosen experts and the clamped gated unit (optionally of the input times the
+//                weight: the weight then multiplies both products in front of the unit)
+//   routed_down  a few rows: sum over a row's experts of weight * W_down a (or, behind weighted inputs, of W_down a), stored or added to the residual
 // Prompt rows sort their routes by expert (moe.cu) and run the grouped tensor-core GEMM. Expert weights: gate_up [E][2 ff][ldg] (gate rows,
 // then up rows), down [E][N][ldd]; row pitches are multiples of 16 bytes, pad columns are zero. No fast-math in this file.
 #include "rowmath.cuh"
@@ -15,6 +16,7 @@ struct Router {
   int E, top, groups, keep;
   int best2;                     // a group's score is the sum of its two best members
   int renorm; float factor;
+  int sigmoid;                   // of every logit by itself, instead of the softmax
 };
 constexpr int kMaxExperts = 1024, kMaxTop = 32, kRoutedRows = 8;
 
@@ -43,15 +45,19 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
     sc[e] = l;
     m = fmaxf(m, l);
   }
-  m = warp_max(m);
-  float s = 0.f;
-  for (int e = lane; e < r.E; e += 32) {
-    const float v = expf(sc[e] - m);
-    sc[e] = v;
-    s += v;
+  if (r.sigmoid) {
+    for (int e = lane; e < r.E; e += 32) sc[e] = sigmoid_of(sc[e]);
+  } else {
+    m = warp_max(m);
+    float s = 0.f;
+    for (int e = lane; e < r.E; e += 32) {
+      const float v = expf(sc[e] - m);
+      sc[e] = v;
+      s += v;
+    }
+    s = warp_sum(s);
+    for (int e = lane; e < r.E; e += 32) sc[e] /= s;
   }
-  s = warp_sum(s);
-  for (int e = lane; e < r.E; e += 32) sc[e] /= s;
   __syncwarp();
   if (r.keep < r.groups) {
     float* gs = sc + r.E;
@@ -164,6 +170,7 @@ struct RoutedUp {
   long ldx, ldw, lda;
   Glu unit;
   int* ids; float* weights;                // written by the first CTA of a group
+  int wx;                                  // the weight multiplies what the expert reads
 };
 
 // grid (CTAs, row groups), 256 threads. X: rows as they are given (rounded to T). A warp makes one column of a route: gate and up row, lanes
@@ -216,14 +223,18 @@ __global__ void __launch_bounds__(256, 3) routed_up_kernel(const RoutedUp a, con
     }
     g = warp_sum(g);
     u = warp_sum(u);
-    if (lane == 0) out[((long)row0 * top + route) * a.lda + o] = from_f<T>(clamped_glu_of(g, u, a.unit));
+    if (lane == 0) {
+      const float f = a.wx ? s_w[m][route - m * top] : 1.f;
+      out[((long)row0 * top + route) * a.lda + o] = from_f<T>(clamped_glu_of(g * f, u * f, a.unit));
+    }
   }
 }
 
 struct RoutedDown {
-  const int* ids; const float* weights;
+  const int* ids; const float* weights;    // weights null: all one
   int top, N, ff;
   long lda, ldw, ldo;
+  int add;                                 // out (fp32) is added to
 };
 
 // grid (CTAs, rows), 256 threads, a warp per output column. STAGED: activations in dynamic shared memory [top][ff rounded up to 16 bytes] of
@@ -242,7 +253,7 @@ __global__ void __launch_bounds__(256) routed_down_kernel(const RoutedDown a, co
   grid_dep_launch();
   if (tid < a.top) {
     s_id[tid] = a.ids[row * a.top + tid];
-    s_w[tid] = a.weights[row * a.top + tid];
+    s_w[tid] = a.weights ? a.weights[row * a.top + tid] : 1.f;
   }
   if (STAGED)
     for (int i = tid; i < a.top * F; i += 256) {
@@ -268,7 +279,7 @@ __global__ void __launch_bounds__(256) routed_down_kernel(const RoutedDown a, co
         if (k0 + j < a.top) acc = fmaf(s_w[k0 + j], d[j], acc);
     }
     acc = warp_sum(acc);
-    if (lane == 0) out[row * a.ldo + n] = from_f<O>(acc);
+    if (lane == 0) out[row * a.ldo + n] = from_f<O>(a.add ? acc + to_f(out[row * a.ldo + n]) : acc);
   }
 }
 
@@ -315,8 +326,8 @@ static int launch_routed_down(const RoutedDown& a, const void* act, const void* 
 
 using namespace ve;
 
-#define VE_ROUTER int E, int top, int groups, int keep, int best2, int renorm, float factor
-#define VE_RMAKE Router{E, top, groups, keep, best2, renorm, factor}
+#define VE_ROUTER int E, int top, int groups, int keep, int best2, int renorm, float factor, int sigmoid
+#define VE_RMAKE Router{E, top, groups, keep, best2, renorm, factor, sigmoid}
 static bool router_ok(const Router& r) {
   return r.E > 0 && r.E <= kMaxExperts && r.top > 0 && r.top <= kMaxTop && r.groups > 0 && r.E % r.groups == 0 && r.keep > 0 && r.keep <= r.groups &&
          r.top <= r.keep * (r.E / r.groups);
@@ -337,24 +348,24 @@ int ve_route_rows(VE_ROUTER, const void* z, long ldz, void* ids, void* weights, 
 }
 
 // x [rows][K] fp32 when x32, else of the weights' type; f32: weights and output fp32 (else bf16). out [rows top][lda]; ids, weights
-// [rows][top] are written.
+// [rows][top] are written. wx: the weights multiply the inputs.
 int ve_routed_up(VE_ROUTER, const void* z, long ldz, const void* x, long ldx, int x32, const void* W, long ldw, void* out, long lda, void* ids, void* weights,
-                 int rows, int K, int ff, float alpha, float limit, float shift, int f32, cudaStream_t st) {
+                 int rows, int K, int ff, float alpha, float limit, float shift, int wx, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const Router r = VE_RMAKE;
   if (!router_ok(r) || K < 1 || ff < 1 || (ldw * (f32 ? 4 : 2)) % 16 || ((uintptr_t)W & 15) || ldw < K) return cudaErrorInvalidValue;
-  const RoutedUp a{(const float*)z, ldz, r, rows, 0, K, ff, ldx, ldw, lda, Glu{alpha, limit, shift}, (int*)ids, (float*)weights};
+  const RoutedUp a{(const float*)z, ldz, r, rows, 0, K, ff, ldx, ldw, lda, Glu{alpha, limit, shift}, (int*)ids, (float*)weights, wx};
   if (f32) return launch_routed_up<float, float>(a, x, W, out, st);
   if (x32) return launch_routed_up<float, __nv_bfloat16>(a, x, W, out, st);
   return launch_routed_up<__nv_bfloat16, __nv_bfloat16>(a, x, W, out, st);
 }
 
-// act [rows top][lda] of the weights' type; out [rows][ldo] fp32 when o32 or f32, else bf16.
+// act [rows top][lda] of the weights' type; out [rows][ldo] fp32 when o32 or f32, else bf16; add: out fp32 is added to. weights null: all one.
 int ve_routed_down(const void* act, long lda, const void* W, long ldw, const void* ids, const void* weights, int top, void* out, long ldo, int o32, int rows,
-                   int N, int ff, int f32, cudaStream_t st) {
+                   int N, int ff, int add, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (top < 1 || top > kMaxTop || N < 1 || ff < 1 || (ldw * (f32 ? 4 : 2)) % 16 || ((uintptr_t)W & 15) || ldw < ff) return cudaErrorInvalidValue;
-  const RoutedDown a{(const int*)ids, (const float*)weights, top, N, ff, lda, ldw, ldo};
+  if (top < 1 || top > kMaxTop || N < 1 || ff < 1 || (ldw * (f32 ? 4 : 2)) % 16 || ((uintptr_t)W & 15) || ldw < ff || (add && !o32 && !f32)) return cudaErrorInvalidValue;
+  const RoutedDown a{(const int*)ids, (const float*)weights, top, N, ff, lda, ldw, ldo, add};
   if (f32) return launch_routed_down<float, float>(a, act, W, out, rows, st);
   if (o32) return launch_routed_down<__nv_bfloat16, float>(a, act, W, out, rows, st);
   return launch_routed_down<__nv_bfloat16, __nv_bfloat16>(a, act, W, out, rows, st);

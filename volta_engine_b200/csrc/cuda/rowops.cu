@@ -6,8 +6,8 @@
 //   stream_norm  residual streams rewritten from the old ones and a sublayer's result (optional), then the layer norm (no shift) of
 //                their weighted sum
 //   group_rms    out = x / rms(x over groups of G columns) * w [* sigmoid(gate) or silu(gate)]; w repeats with its own length
-//   residual_norm  h += RMS norm of a sublayer's result (or of the weighted sum of a token's routed results), out = h or its RMS norm
-//   clamped_glu  out = gated unit of [gate | up] rows with both halves clamped
+//   residual_norm  h += a sublayer's result (or the weighted sum of a token's routed results) or its RMS norm, out = h or its RMS norm
+//   clamped_glu  out = gated unit of [gate | up] rows (optionally times a weight per row) with both halves clamped
 //   soft_cap     x = cap tanh(x / cap)
 //   polynorm     out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3, N = division by the row's root mean square
 //   scale_add    h += scale * part
@@ -277,11 +277,12 @@ __global__ void __launch_bounds__(256) stream_norm4_kernel(float* __restrict__ h
   }
 }
 
-// One sublayer result per row: rows of `part`, or (top > 0) sum_k rw[row][k] part[inv ? inv[row top + k] : row top + k].
+// One sublayer result per row: rows of `part`, or (top > 0) sum_k rw[row][k] part[inv ? inv[row top + k] : row top + k] (rw null: all one).
 struct ResultRows {
   const int* inv; const float* rw; int top;
 };
-// h [rows][H]. One CTA per row. wa null: no result; wo null: the residual itself; out null: only the residual.
+// h [rows][H]. One CTA per row. part null: no result; wa null: the result as it is, not normed; wo null: the residual itself; out null: only the
+// residual.
 template <typename T>
 __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ h, const T* __restrict__ part, long ldp, const ResultRows rr,
                                                             const float* __restrict__ wa, const float* __restrict__ wo, T* __restrict__ out, long ldo, int H,
@@ -296,7 +297,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ 
     float v = 0.f;
     for (int k = 0; k < rr.top; ++k) {
       const long r = row * rr.top + k;
-      v = fmaf(rr.rw[r], to_f(part[(rr.inv ? rr.inv[r] : r) * ldp + i]), v);
+      v = fmaf(rr.rw ? rr.rw[r] : 1.f, to_f(part[(rr.inv ? rr.inv[r] : r) * ldp + i]), v);
     }
     return v;
   };
@@ -311,8 +312,8 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(float* __restrict__ 
   }
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float v = hr[i];
-    if (wa) {
-      v = fmaf(result(i) * inv, wa[i], v);
+    if (part) {
+      v = wa ? fmaf(result(i) * inv, wa[i], v) : v + result(i);
       hr[i] = v;
     }
     if (!out) continue;
@@ -341,13 +342,13 @@ __global__ void __launch_bounds__(256) residual_norm4_kernel(float* __restrict__
     const int i = (j * 256 + threadIdx.x) * 4;
     x[j] = i < H ? load4(hr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     y[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (wa && !rr.top && i < H) y[j] = load4(part + row * ldp + i);
+    if (part && !rr.top && i < H) y[j] = load4(part + row * ldp + i);
   }
-  if (wa) {
+  if (part) {
     for (int k = 0; k < rr.top; ++k) {
       const long r = row * rr.top + k;
       const T* pr = part + (rr.inv ? rr.inv[r] : r) * ldp;
-      const float f = rr.rw[r];
+      const float f = rr.rw ? rr.rw[r] : 1.f;
 #pragma unroll
       for (int j = 0; j < NV; ++j) {
         const int i = (j * 256 + threadIdx.x) * 4;
@@ -357,15 +358,18 @@ __global__ void __launch_bounds__(256) residual_norm4_kernel(float* __restrict__
         }
       }
     }
+    float inv = 1.f;
+    if (wa) {
 #pragma unroll
-    for (int j = 0; j < NV; ++j) s += (y[j].x * y[j].x + y[j].y * y[j].y) + (y[j].z * y[j].z + y[j].w * y[j].w);
-    const float inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
-    s = 0.f;
+      for (int j = 0; j < NV; ++j) s += (y[j].x * y[j].x + y[j].y * y[j].y) + (y[j].z * y[j].z + y[j].w * y[j].w);
+      inv = 1.f / sqrtf(block_sum(s, red) / (float)H + eps);
+      s = 0.f;
+    }
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
       const int i = (j * 256 + threadIdx.x) * 4;
       if (i < H) {
-        const float4 w = load4(wa + i);
+        const float4 w = wa ? load4(wa + i) : make_float4(1.f, 1.f, 1.f, 1.f);
         x[j] = make_float4(fmaf(y[j].x * inv, w.x, x[j].x), fmaf(y[j].y * inv, w.y, x[j].y), fmaf(y[j].z * inv, w.z, x[j].z), fmaf(y[j].w * inv, w.w, x[j].w));
         store4(hr + i, x[j]);
       }
@@ -396,23 +400,30 @@ __global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ x, lo
   for (long i = blockIdx.x * 256l + threadIdx.x; i < n; i += gridDim.x * 256l) x[i] = soft_cap_of(x[i], cap);
 }
 
+// Factor of a row: w[index[row]] (w null: one).
+struct RowBy {
+  const float* w; const int* index;
+  VE_DEVINL float of(long row) const { return w ? w[index[row]] : 1.f; }
+};
+
 // z [rows][2 F]: gates, then ups (blk 0), or blocks of [4 gates | 4 ups].
 template <typename X, typename T>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, int blk, const Glu u) {
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const X* __restrict__ z, long ldz, T* __restrict__ out, long ldo, long total, int F, int blk, const Glu u, const RowBy by) {
   grid_dep_wait();
   grid_dep_launch();
   for (long q = blockIdx.x * 256l + threadIdx.x; q < total; q += gridDim.x * 256l) {
     const long row = q / F;
     const int i = (int)(q - row * F), g = blk ? (i >> 2) * 8 + (i & 3) : i, up = blk ? g + 4 : F + i;
-    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + g]), to_f(z[row * ldz + up]), u));
+    const float f = by.of(row);
+    out[row * ldo + i] = from_f<T>(clamped_glu_of(to_f(z[row * ldz + g]) * f, to_f(z[row * ldz + up]) * f, u));
   }
 }
-VE_DEVINL __nv_bfloat162 clamped_glu2(__nv_bfloat162 g, __nv_bfloat162 u, const Glu& c) {
+VE_DEVINL __nv_bfloat162 clamped_glu2(__nv_bfloat162 g, __nv_bfloat162 u, const Glu& c, float f) {
   const float2 a = __bfloat1622float2(g), b = __bfloat1622float2(u);
-  return __floats2bfloat162_rn(clamped_glu_of(a.x, b.x, c), clamped_glu_of(a.y, b.y, c));
+  return __floats2bfloat162_rn(clamped_glu_of(a.x * f, b.x * f, c), clamped_glu_of(a.y * f, b.y * f, c));
 }
 __global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* __restrict__ z, long ldz, __nv_bfloat16* __restrict__ out, long ldo, long total8,
-                                                           int F, int blk, const Glu u) {
+                                                           int F, int blk, const Glu u, const RowBy by) {
   grid_dep_wait();
   grid_dep_launch();
   const int f8 = F >> 3;
@@ -421,15 +432,16 @@ __global__ void __launch_bounds__(256) clamped_glu8_kernel(const __nv_bfloat16* 
     const int i = (int)(q - row * f8) * 8;
     const __nv_bfloat16* zr = z + row * ldz;
     const bf16x8 a = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i : i)), b = *reinterpret_cast<const bf16x8*>(zr + (blk ? 2 * i + 8 : F + i));
+    const float f = by.of(row);
     bf16x8 o;
     if (blk) {
-      o.v[0] = clamped_glu2(a.v[0], a.v[2], u);
-      o.v[1] = clamped_glu2(a.v[1], a.v[3], u);
-      o.v[2] = clamped_glu2(b.v[0], b.v[2], u);
-      o.v[3] = clamped_glu2(b.v[1], b.v[3], u);
+      o.v[0] = clamped_glu2(a.v[0], a.v[2], u, f);
+      o.v[1] = clamped_glu2(a.v[1], a.v[3], u, f);
+      o.v[2] = clamped_glu2(b.v[0], b.v[2], u, f);
+      o.v[3] = clamped_glu2(b.v[1], b.v[3], u, f);
     } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o.v[e] = clamped_glu2(a.v[e], b.v[e], u);
+      for (int e = 0; e < 4; ++e) o.v[e] = clamped_glu2(a.v[e], b.v[e], u, f);
     }
     *reinterpret_cast<bf16x8*>(out + row * ldo + i) = o;
   }
@@ -540,13 +552,14 @@ int ve_stream_norm(void* h, const void* part, long ldp, const void* mix, const v
   VE_CHECK_LAUNCH();
 }
 
-// h [rows][H] contiguous fp32 += RMS norm of the result * wa (wa null: no result); out = h, or its RMS norm * wo (null: not normed; out null: no
-// output). top > 0: a row's result is the sum of rw [rows][top] times rows inv [rows][top] (null: in order) of part.
+// h [rows][H] contiguous fp32 += RMS norm of the result * wa (wa null: the result as it is; part null: no result); out = h, or its RMS norm * wo
+// (null: not normed; out null: no output). top > 0: a row's result is the sum of rw [rows][top] (null: all one) times rows inv [rows][top]
+// (null: in order) of part.
 int ve_residual_norm(void* h, const void* part, long ldp, const void* inv, const void* rw, int top, const void* wa, const void* wo, void* out, long ldo, int rows,
                      int H, float eps, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (H < 1 || top < 0 || (wa && !part) || (top && !rw) || (!wa && !out)) return cudaErrorInvalidValue;
-  const ResultRows rr{(const int*)inv, (const float*)rw, wa ? top : 0};
+  if (H < 1 || top < 0 || (wa && !part) || (!part && !out)) return cudaErrorInvalidValue;
+  const ResultRows rr{(const int*)inv, (const float*)rw, part ? top : 0};
   const bool vec = !f32 && H % 4 == 0 && H <= 8192 && ldp % 4 == 0 && ldo % 4 == 0 && !(((uintptr_t)h | (uintptr_t)wa | (uintptr_t)wo) & 15) &&
                    !(((uintptr_t)part | (uintptr_t)out) & 7);
   if (f32) launch_pdl(residual_norm_kernel<float>, dim3(rows), dim3(256), 0, st, (float*)h, (const float*)part, ldp, rr, (const float*)wa, (const float*)wo,
@@ -571,20 +584,22 @@ int ve_soft_cap(void* x, long n, float cap, cudaStream_t st) {
   VE_CHECK_LAUNCH();
 }
 
-// z rows [gate F | up F] (blk 0) or blocks of [4 gate | 4 up] (F a multiple of 4); fp32 when x32, else of the activation type.
-int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, int blk, float alpha, float limit, float shift, int f32,
-                   cudaStream_t st) {
+// z rows [gate F | up F] (blk 0) or blocks of [4 gate | 4 up] (F a multiple of 4); fp32 when x32, else of the activation type. w (null:
+// none): row r is first multiplied with w[index[r]].
+int ve_clamped_glu(const void* z, long ldz, int x32, void* out, long ldo, int rows, int F, int blk, float alpha, float limit, float shift, const void* w,
+                   const void* index, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   const Glu u{alpha, limit, shift};
-  if (F < 1 || (blk && F % 4)) return cudaErrorInvalidValue;
+  const RowBy by{(const float*)w, (const int*)index};
+  if (F < 1 || (blk && F % 4) || (w && !index)) return cudaErrorInvalidValue;
   const bool vec = !f32 && !x32 && F % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && !((uintptr_t)z & 15) && !((uintptr_t)out & 15);
   const long total = (long)rows * F / (vec ? 8 : 1), blocks = (total + 255) / 256;
   const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
   if (vec) {
-    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, blk, u);
+    launch_pdl(clamped_glu8_kernel, grid, dim3(256), 0, st, (const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, ldo, total, F, blk, u, by);
     VE_CHECK_LAUNCH();
   }
-#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, blk, u)
+#define VE_CG(X, T) launch_pdl(clamped_glu_kernel<X, T>, grid, dim3(256), 0, st, (const X*)z, ldz, (T*)out, ldo, total, F, blk, u, by)
   if (f32) VE_CG(float, float);
   else if (x32) VE_CG(float, __nv_bfloat16);
   else VE_CG(__nv_bfloat16, __nv_bfloat16);

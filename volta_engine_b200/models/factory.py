@@ -22,7 +22,8 @@ DENSE_TYPES = {"llama", "mistral", "qwen2", "qwen3", "gemma2", "gemma3_text", "g
 MOE_TYPES = {"qwen3_moe", "glm4_moe", "mixtral", "moe"}
 MLA_TYPES = {"deepseek_v2", "deepseek_v3", "kimi_k2", "mla"}
 # designs that config.json names under "architecture": module and loader (config dict, tensor source, device, comm, dtype=)
-ARCHITECTURES = {"Fofosun": ("fofosun", "load_fofosun"), "Siditar": ("siditar", "load_siditar"), "Kutolix": ("kutolix", "load_kutolix")}
+ARCHITECTURES = {"Fofosun": ("fofosun", "load_fofosun"), "Siditar": ("siditar", "load_siditar"), "Kutolix": ("kutolix", "load_kutolix"),
+                 "Vugipel": ("vugipel", "load_vugipel")}
 
 
 def dense_config_from_hf(c: dict) -> DenseConfig:

@@ -78,5 +78,13 @@ class RoutedFF:
         return routed_many(self.choice, self.experts, z, x)
 
     def step(self, res, norm, write, b) -> None:
-        z = gemv_rows(self.router, b.n, out_f32=True, **res.read(norm))
-        res.later(routed_few(self.choice, self.experts, z, res.h, torch.float32), write)
+        pro, x = res.read(norm), res.h
+        if pro.get("b") is not None:                     # the experts read the normed row, which the router's linear stores
+            x = pro["x_out"] = torch.empty(x.shape, dtype=torch.bfloat16, device=x.device)
+        z = gemv_rows(self.router, b.n, out_f32=True, **pro)
+        if getattr(write, "deferred", False):
+            res.later(routed_few(self.choice, self.experts, z, x, torch.float32), write)
+        elif write is None:
+            routed_few(self.choice, self.experts, z, x, residual=res.h)
+        else:
+            raise NotImplementedError(f"routed results through {type(write).__name__}")

@@ -17,6 +17,7 @@ import copy
 import json
 from dataclasses import dataclass, field
 from pathlib import Path
+from typing import ClassVar
 
 import torch
 
@@ -31,6 +32,7 @@ DTYPES = {"bf16": torch.bfloat16, "bfloat16": torch.bfloat16, "fp32": torch.floa
 
 @dataclass
 class ListedConfig(DenseConfig):
+    mixers: ClassVar[dict] = MIXERS                 # the design's mixer types
     layers: list = field(default_factory=list)      # [{"type", "mixer": {sizes}, "mlp": {"kind", ...} | None}]
     loop: tuple = (0, 0, 1)                         # layers [start, stop) run this many times in a row
     v_width: int = 8                                # elements of a token's row in the value pool
@@ -41,7 +43,7 @@ class ListedConfig(DenseConfig):
         """The fields every design of this form has. ``feed_forwards``: the kinds the design has."""
         layers = [dict(L) for L in c["layers"]]
         for i, L in enumerate(layers):
-            if L["type"] not in MIXERS:
+            if L["type"] not in cls.mixers:
                 raise NotImplementedError(f"layer {i}: no mixer {L['type']!r} in this build")
             if L.get("mlp") is not None and L["mlp"].get("kind", "dense") not in feed_forwards:
                 raise NotImplementedError(f"layer {i}: no feed-forward {L['mlp']['kind']!r} in this build")
@@ -49,7 +51,7 @@ class ListedConfig(DenseConfig):
         loop = (int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else (0, 0, 1)
         if not 0 <= loop[0] <= loop[1] <= len(layers) or loop[2] < 1:
             raise ValueError(f"loop over layers {loop[0]} .. {loop[1]} of {len(layers)}, {loop[2]} times")
-        widths = [MIXERS[L["type"]].row_widths(L["mixer"]) for L in layers]
+        widths = [cls.mixers[L["type"]].row_widths(L["mixer"]) for L in layers]
         return cls(n_layers=len(layers), hidden=int(c["width"]), vocab=int(c["vocab"]), rms_eps=float(c["norm"]["eps"]), layers=layers, loop=loop,
                    n_q=1, n_kv=1, ffn=max([int((L["mlp"].get("expert") or L["mlp"])["ff"]) for L in layers if L.get("mlp") is not None] or [1]), quant="bf16",
                    head_dim=max([k for k, _ in widths] + [0]) or 64, v_width=max([v for _, v in widths] + [8]), **kw)

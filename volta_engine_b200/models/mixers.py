@@ -2,7 +2,7 @@
 reads normed rows and returns the rows of its output projection; ``step`` is the same on a few decode rows with the norm in
 front, the layer scale and the residual add inside the linears' launches (``finish(linear, **operands)`` runs the last one).
 
-``MIXERS`` maps the type names to classes; a class takes (mixer sizes, eps, tensor source, name prefix, device, dtype).
+``MIXERS`` maps type names to classes (a design may give its own names, ``ListedConfig.mixers``); a class takes (mixer sizes, eps, tensor source, name prefix, device, dtype).
 """
 from __future__ import annotations
 
@@ -14,17 +14,18 @@ from ..ops.gqa import GqaSpec, distance_bias, gqa_attend
 from ..ops.latent import LatentSpec, latent_rows
 from ..ops.linear import LinearBF16, LinearF32
 from ..ops.linear_attn import LinAttnSpec, LinAttnState, linattn_rows
+from ..ops.min_gru import MinGruState, min_gru_rows
 from ..ops.rotary import Rotation
 from ..ops.rowops import GroupRMS, gemv_rows
 
 
-def make_linear(src, names, device, dtype, dim: int = 0, join=None):
+def make_linear(src, names, device, dtype, dim: int = 0, join=None, bias=None):
     """One linear computing the stacked outputs of the tensors ``names`` (``dim`` 1: the sum of their outputs on stacked inputs;
-    ``join``: a function that makes one weight of them)."""
+    ``join``: a function that makes one weight of them; ``bias``: fp32, of its outputs)."""
     names = [names] if isinstance(names, str) else names
     parts = [src.tensor(n, device, dtype) for n in names]
     w = join(*parts) if join is not None else torch.cat(parts, dim) if len(parts) > 1 else parts[0]
-    return LinearF32(w) if dtype == torch.float32 else LinearBF16(w)
+    return LinearF32(w, bias) if dtype == torch.float32 else LinearBF16(w, bias)
 
 
 def apply_linear(lin, x, out_f32: bool = False):
@@ -67,21 +68,56 @@ class Mixer:
         return 0
 
 
+class MinGru(Mixer):
+    """A gated recurrence per channel whose gate and candidate read the current token alone: one fused input projection [gate | candidate |
+    output gate] with biases on the first two, the recurrence with the output gate, the output projection."""
+    recurrent = True
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
+        self.width = int(m["width"])
+        b = torch.cat([src.tensor(p + n, device, torch.float32).reshape(-1) for n in ("z.b", "x.b")])
+        self.in_proj = make_linear(src, [p + "z", p + "x", p + "g"], device, dtype, bias=torch.nn.functional.pad(b, (0, self.width)))
+        self.out = make_linear(src, p + "o", device, dtype)
+        if self.in_proj.out_features != 3 * self.width:
+            raise ValueError(f"{p}: projections of {self.in_proj.out_features} rows for three times {self.width} channels")
+        self.dtype = dtype
+        self.state: MinGruState | None = None
+
+    def bind(self, kv):
+        if self.state is None:
+            self.state = MinGruState(self.width, kv.max_slots, kv.page_table.device)
+        return self.state
+
+    def state_elements(self) -> int:
+        return self.width
+
+    def recur(self, proj, b, kv, journal):
+        return min_gru_rows(proj, b, self.bind(kv), self.dtype, self.out.weight.shape[1], *journal)
+
+    def rows(self, x, b, kv, journal=(None, None)):
+        return apply_linear(self.out, self.recur(apply_linear(self.in_proj, x, out_f32=True), b, kv, journal))
+
+    def step(self, pro, finish, b, kv, journal=(None, None)):
+        finish(self.out, x=self.recur(gemv_rows(self.in_proj, b.n, out_f32=True, **pro), b, kv, journal))
+
+
 class LinearRecurrence(Mixer):
-    """HGRN2, lightning attention and gated linear attention: one fused input projection [q | forget gate or k | v | gate | low-rank
+    """HGRN2, lightning attention, retention and gated linear attention: one fused input projection [q | forget gate or k | v | gate | low-rank
     decay], the decayed outer-product recurrence, an RMS norm of its output (per head, or over all heads; gated), the output
     projection. ``out_scale``: a factor on what enters the output projection."""
     recurrent = True
-    PARTS = {"hgrn2": ("q", "f", "v"), "lightning": ("q", "k", "v", "g"), "gated_linear_attention": ("q", "k", "v", "g", "a1")}
+    PARTS = {"hgrn2": ("q", "f", "v"), "lightning": ("q", "k", "v", "g"), "retention": ("q", "k", "v", "g"),
+             "gated_linear_attention": ("q", "k", "v", "g", "a1")}
 
     def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype, linears: bool = True, out_scale: float = 1.0):
         H, dk, dv = int(m["heads"]), int(m["dim"]), int(m["vdim"])
         f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
         self.parts = [p + n for n in self.PARTS[kind]]
         self.gated = "g" in self.PARTS[kind]
-        if kind == "lightning":
+        if kind in ("lightning", "retention"):
             decay = m["decay"] if isinstance(m["decay"], (list, tuple)) else [m["decay"]] * H
-            self.spec = LinAttnSpec(H, dk, dv, decay=torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device))
+            self.spec = LinAttnSpec(H, dk, dv, decay=torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device),
+                                    **({"plain": True, "q_scale": dk ** -0.5} if kind == "retention" else {}))
             if self.spec.decay.numel() != H:
                 raise ValueError(f"{p}: {self.spec.decay.numel()} decays for {H} heads")
         elif kind == "hgrn2":
@@ -92,7 +128,8 @@ class LinearRecurrence(Mixer):
         if linears:
             self.in_proj = make_linear(src, self.parts, device, dtype)
             self.out = make_linear(src, p + "o", device, dtype)
-        self.norm = GroupRMS(f32("norm") * out_scale, eps, 0 if kind == "lightning" else dv, silu=kind == "gated_linear_attention")
+        w = torch.ones(dv, device=device) if kind == "retention" else f32("norm")
+        self.norm = GroupRMS(w * out_scale, eps, 0 if kind == "lightning" else dv, silu=kind in ("retention", "gated_linear_attention"))
         self.dtype = dtype
         self.state: LinAttnState | None = None
 
@@ -146,6 +183,13 @@ class GroupedAttention(Mixer):
             self.out = make_linear(src, p + "o", device, dtype)
         self.dtype = dtype
 
+    def in_bias(self, src):
+        """Biases of the input projection's outputs, or None."""
+        return None
+
+    def out_bias(self, src):
+        return None
+
     def attend(self, proj, b, kv, out):
         return gqa_attend(self.spec, proj, b, kv, kv.k[self.cache_index], kv.v[self.cache_index], out)
 
@@ -183,9 +227,38 @@ class WindowedAttention(GroupedAttention):
         return apply_linear(self.out, self.attend(proj, b, kv, self._out(proj)))
 
 
+class RotatedValueAttention(GroupedAttention):
+    """Grouped-query softmax attention with rotary positions on queries and keys (behind their norm) and on values (taken back from the
+    result), a number per head on the scores, a soft cap, a sliding window that keeps the first tokens in sight, and biases on all
+    projections. ``out_scale`` as above."""
+
+    def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype, linears: bool = True, out_scale: float = 1.0):
+        f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
+        rot, vdim, window = m["rot"], int(m["vdim"]), window_of(m)
+        self.spec = GqaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), vdim, float(m["scale"]), eps, q_norm=f32("q.norm"), k_norm=f32("k.norm"),
+                            norm_first=True, head_mul=f32("temp"), softcap=float(m["softcap"]), out_scale=out_scale, window=window,
+                            keep_first=int(m["mask"].get("keep_first") or 0) if window else 0, rot=Rotation.from_config(rot, True).bind(device),
+                            v_rot=Rotation(vdim, float(rot["base"]), True).bind(device))
+        if self.spec.rot.dims > self.spec.dim:
+            raise ValueError(f"{p}: {self.spec.rot.dims} rotated columns of {self.spec.dim}")
+        self.p, self.out_scale, self.device = p, out_scale, device
+        self.parts = [p + n for n in self.PARTS]
+        if linears:
+            self.in_proj = make_linear(src, self.parts, device, dtype, bias=self.in_bias(src))
+            self.out = make_linear(src, p + "o", device, dtype, bias=self.out_bias(src))
+        self.dtype = dtype
+
+    def in_bias(self, src):
+        return torch.cat([src.tensor(self.p + n + ".b", self.device, torch.float32).reshape(-1) for n in self.PARTS])
+
+    def out_bias(self, src):
+        return (src.tensor(self.p + "o.b", self.device, torch.float32).reshape(-1) * self.out_scale).contiguous()
+
+
 class Parallel(Mixer):
-    """Grouped attention and gated linear attention side by side on the same rows: one input projection for both, and one output
-    projection over the two results put next to each other (each times its scale)."""
+    """Attention and a linear recurrence side by side on the same rows: one input projection for both, and one output projection over the
+    two results put next to each other (each times its scale)."""
+    LEFT, RIGHT = (GroupedAttention, "grouped_attention"), (LinearRecurrence, "gated_linear_attention")
     cached = recurrent = True
 
     @staticmethod
@@ -193,16 +266,19 @@ class Parallel(Mixer):
         return GroupedAttention.row_widths(m["left"])
 
     def __init__(self, kind: str, m: dict, eps: float, src, p: str, device, dtype):
-        self.left = GroupedAttention("grouped_attention", m["left"], eps, src, p + "left.", device, dtype, False, float(m["left_scale"]))
-        self.right = LinearRecurrence("gated_linear_attention", m["right"], eps, src, p + "right.", device, dtype, False, float(m["right_scale"]))
+        side = lambda which, name: which[0](which[1], m[name], eps, src, f"{p}{name}.", device, dtype, False, float(m[name + "_scale"]))
+        self.left, self.right = side(self.LEFT, "left"), side(self.RIGHT, "right")
         self.in_proj = make_linear(src, self.left.parts + self.right.parts, device, dtype)
-        self.out = make_linear(src, [p + "left.o", p + "right.o"], device, dtype, dim=1)
+        self.out = make_linear(src, [p + "left.o", p + "right.o"], device, dtype, dim=1, bias=self.left.out_bias(src))
+        b = self.left.in_bias(src)
+        if b is not None:
+            self.in_proj.bias = torch.nn.functional.pad(b, (0, self.in_proj.out_features - b.numel())).contiguous()
         self.k0 = self.left.spec.heads * self.left.spec.vdim         # columns of the left result
         self.k1 = self.right.spec.heads * self.right.spec.dv
         self.dtype = dtype
 
     def __copy__(self):
-        new = object.__new__(Parallel)
+        new = object.__new__(type(self))
         new.__dict__.update(self.__dict__)
         new.left, new.right = copy.copy(self.left), copy.copy(self.right)
         return new
@@ -234,6 +310,11 @@ class Parallel(Mixer):
         pr = proj[:, self.left.spec.cols:]
         o = self.right.recur(pr, b, kv, journal, True)
         finish(self.out, **self.right.norm.prologue(o, self.right.gate(pr), head=att))
+
+
+class RotatedRetention(Parallel):
+    """Attention with rotated values beside retention."""
+    LEFT, RIGHT = (RotatedValueAttention, "rotated_value_attention"), (LinearRecurrence, "retention")
 
 
 class LatentAttention(Mixer):
@@ -293,4 +374,5 @@ class LatentAttention(Mixer):
 
 
 MIXERS = {"hgrn2": LinearRecurrence, "lightning": LinearRecurrence, "latent_attention": LatentAttention,
-          "gated_linear_attention": LinearRecurrence, "grouped_attention": GroupedAttention, "parallel": Parallel, "attention": WindowedAttention}
+          "gated_linear_attention": LinearRecurrence, "grouped_attention": GroupedAttention, "parallel": Parallel, "attention": WindowedAttention,
+          "mingru": MinGru, "rotated_retention": RotatedRetention}

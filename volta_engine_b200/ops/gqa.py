@@ -1,6 +1,7 @@
 """Grouped-query softmax attention with its sizes and score terms as parameters (csrc/cuda/gqa.cu): rotary positions, RMS norm of
-queries and keys behind them (with or without a weight), query temperature by position, sliding window, bias by distance, sink, output
-gate, unlike query / key and value widths.
+queries and keys behind them or in front (with or without a weight), query temperature by position, factor per head, soft cap of the
+scores, sliding window (the first tokens in sight or not), bias by distance, sink, values rotated by their position (the result is turned
+back by the query's), output gate, unlike query / key and value widths.
 
 The paged cache's rows are as wide as the widest layer needs (``row_widths``); a layer sees a page as [kv heads, 64, width].
 
@@ -65,12 +66,19 @@ class GqaSpec:
     unit: bool = False                        # queries and keys are normed without a weight
     window: int = 0                           # a key is seen at distances below it (0: all in front)
     gated: bool = False                       # columns behind the values: the result is multiplied with their sigmoid
+    norm_first: bool = False                  # the norm of queries and keys stands in front of their rotation
+    head_mul: torch.Tensor | None = None      # fp32 [heads]: factor on a head's queries
+    softcap: float = 0.0                      # scores are softcap * tanh(score / softcap), in front of the bias (0: as they are)
+    keep_first: int = 0                       # the first tokens of a sequence that a window never leaves
+    v_rot: Rotation | None = None             # of the values over their whole width, pairs as in ``rot``
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads over {self.kv_heads} key / value heads")
         self.kw, self.vw = _up8(self.dim), _up8(self.vdim)
         self.group = self.heads // self.kv_heads
+        if self.v_rot is not None and (self.v_rot.dims != self.vdim or self.v_rot.mul != 1.0 or (self.rot is not None and self.rot.neighbours != self.v_rot.neighbours)):
+            raise ValueError("values are turned as a whole, in pairs laid out as those of the keys")
 
     @property
     def cols(self) -> int:
@@ -96,7 +104,7 @@ class GqaSpec:
 
     @property
     def tc_prefill(self) -> bool:
-        return self.kw <= 256 and self.vw <= 128 and self.group <= 128 and self.scale > 0
+        return self.kw <= 256 and self.vw <= 128 and self.group <= 128 and self.scale > 0 and (self.v_rot is None or self.v_rot.neighbours)
 
     def temperature(self, pos):
         return 1.0 + self.temp_coef * torch.log(((pos + 1) // self.temp_every + 1).float()) if self.temp_every > 0 else torch.ones(pos.shape)
@@ -115,10 +123,15 @@ def gqa_reference(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
     dt = kpool.dtype
     pf = proj.float()
     turn = (lambda x: spec.rot.turn(x, b.pos)) if spec.rot is not None else (lambda x: x)
-    q = _norm(turn(pf[:, : H * d].reshape(n, H, d)), spec.q_norm, spec.unit, spec.eps) * spec.temperature(b.pos)[:, None, None]
+    place = (lambda x, w: turn(_norm(x, w, spec.unit, spec.eps))) if spec.norm_first else (lambda x, w: _norm(turn(x), w, spec.unit, spec.eps))
+    q = place(pf[:, : H * d].reshape(n, H, d), spec.q_norm) * spec.temperature(b.pos)[:, None, None]
+    if spec.head_mul is not None:
+        q = q * spec.head_mul[:, None]
     q = q.to(dt).float()
-    k = _norm(turn(pf[:, H * d: (H + G) * d].reshape(n, G, d)), spec.k_norm, spec.unit, spec.eps)
+    k = place(pf[:, H * d: (H + G) * d].reshape(n, G, d), spec.k_norm)
     v = pf[:, (H + G) * d: spec.gate_col].reshape(n, G, dv)
+    if spec.v_rot is not None:
+        v = spec.v_rot.turn(v, b.pos)
     gate = torch.sigmoid(spec.gate(pf)) if spec.gated else None
     kp = kpool.reshape(kpool.shape[0], -1)[:, : G * PAGE * spec.kw].view(-1, G, PAGE, spec.kw)
     vp = vpool.reshape(vpool.shape[0], -1)[:, : G * PAGE * spec.vw].view(-1, G, PAGE, spec.vw)
@@ -133,16 +146,22 @@ def gqa_reference(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
             out[i] = 0
             continue
         a = max(0, p - spec.window + 1) if spec.window else 0          # first key it sees
-        pgs, o = cache.page_table[s, a // PAGE: p // PAGE + 1].long(), a // PAGE * PAGE
-        ks = kp[pgs].transpose(1, 2).reshape(-1, G, spec.kw)[a - o: p + 1 - o, :, :d].float()
-        vs = vp[pgs].transpose(1, 2).reshape(-1, G, spec.vw)[a - o: p + 1 - o, :, :dv].float()
+        seen = torch.cat([torch.arange(min(a, spec.keep_first)), torch.arange(a, p + 1)])
+        pgs = cache.page_table[s, : p // PAGE + 1].long()
+        ks = kp[pgs].transpose(1, 2).reshape(-1, G, spec.kw)[seen, :, :d].float()
+        vs = vp[pgs].transpose(1, 2).reshape(-1, G, spec.vw)[seen, :, :dv].float()
         sc = torch.einsum("gud,jgd->guj", q[i].reshape(G, spec.group, d), ks).reshape(H, -1) * spec.scale
+        if spec.softcap:
+            sc = spec.softcap * torch.tanh(sc / spec.softcap)
         if spec.bias is not None:
-            sc = sc + spec.bias[:, (p - torch.arange(a, p + 1)).clamp(max=spec.bias.shape[1] - 1)]
+            sc = sc + spec.bias[:, (p - seen).clamp(max=spec.bias.shape[1] - 1)]
         if spec.sink is not None:
             sc = torch.cat([sc, spec.sink[:, None]], 1)
-        pr = torch.softmax(sc, -1)[:, : p + 1 - a].reshape(G, spec.group, -1)
-        r = (torch.einsum("guj,jgv->guv", pr, vs) * spec.out_scale).reshape(-1)
+        pr = torch.softmax(sc, -1)[:, : len(seen)].reshape(G, spec.group, -1)
+        r = torch.einsum("guj,jgv->guv", pr, vs) * spec.out_scale
+        if spec.v_rot is not None:
+            r = spec.v_rot.turn(r[None], -b.pos[i: i + 1])
+        r = r.reshape(-1)
         out[i] = (r if gate is None else r * gate[i]).to(out.dtype)
     return out
 
@@ -157,7 +176,7 @@ def _ticket_words(dev):
     return t
 
 
-_D, _R, _S = "iiiiiill", "pppi", "fpipfipli"
+_D, _R, _S = "iiiiiill", "pppi", "fpipfipli" + "ifpii"
 
 
 def _dims(spec, kpool, vpool):
@@ -168,40 +187,45 @@ def _rows(pos, slot, cache):
     return (ptr(pos), ptr(slot), ptr(cache.page_table), cache.page_table.shape[1])
 
 
-def _score(spec, gate):
+def _score(spec, gate, back):
     return (float(spec.scale), ptr(spec.bias), spec.bias.shape[1] if spec.bias is not None else 0, ptr(spec.sink), float(spec.out_scale), spec.window,
-            ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.dtype == torch.float32))
+            ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.dtype == torch.float32), spec.keep_first, float(spec.softcap),
+            ptr(back), spec.v_rot.pairs if back is not None else 0, int(back is not None and spec.v_rot.neighbours))
 
 
 def gqa_store(spec: GqaSpec, proj, pos, slot, cache, kpool, vpool):
-    """Rotation, norms, temperature, cache rows -> queries [rows, heads, kw] of the cache's type."""
+    """Rotation, norms, temperature, cache rows -> (queries [rows, heads, kw] of the cache's type, fp32 [rows, pairs, 2] cosines and sines that
+    results are turned back by, or None)."""
     n, f32 = proj.shape[0], kpool.dtype == torch.float32
     q = torch.empty(n, spec.heads, spec.kw, dtype=kpool.dtype, device=proj.device)
-    rot = spec.rot
-    call("gqa_store", _D + _R + "pli" + "pifi" + "ippffi" + "pppii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), ptr(proj), proj.stride(0),
+    rot, vr = spec.rot, spec.v_rot
+    back = torch.empty(n, vr.pairs, 2, dtype=torch.float32, device=proj.device) if vr is not None else None
+    norm = int(spec.unit or spec.q_norm is not None or spec.k_norm is not None) * (2 if spec.norm_first else 1)
+    call("gqa_store", _D + _R + "pli" + "pifi" + "ippffi" + "ppip" + "pppii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), ptr(proj), proj.stride(0),
          int(proj.dtype == torch.float32), ptr(rot.half_turns) if rot is not None else 0, rot.pairs if rot is not None else 0, rot.mul if rot is not None else 1.0,
-         int(rot is not None and rot.neighbours), int(spec.unit or spec.q_norm is not None or spec.k_norm is not None), ptr(spec.q_norm), ptr(spec.k_norm), float(spec.eps), float(spec.temp_coef), int(spec.temp_every), ptr(q), ptr(kpool),
-         ptr(vpool), n, int(f32))
-    return q
+         int((rot or vr).neighbours) if rot is not None or vr is not None else 0, norm, ptr(spec.q_norm), ptr(spec.k_norm), float(spec.eps), float(spec.temp_coef),
+         int(spec.temp_every), ptr(spec.head_mul), ptr(vr.half_turns) if vr is not None else 0, vr.pairs if vr is not None else 0, ptr(back), ptr(q), ptr(kpool), ptr(vpool),
+         n, int(f32))
+    return q, back
 
 
-def _each_row(spec, q, gate, pos, slot, cache, kpool, vpool, out):
+def _each_row(spec, q, back, gate, pos, slot, cache, kpool, vpool, out):
     """Every row by itself: the split-key kernel, or the CUDA-core one."""
     n, dev, f32 = q.shape[0], q.device, kpool.dtype == torch.float32
     o32 = int(out.dtype == torch.float32)
     if f32 or not spec.tc_decode:
-        call("gqa_rows", _D + _R + _S + "ppp" + "pliii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate), ptr(q), ptr(kpool), ptr(vpool),
+        call("gqa_rows", _D + _R + _S + "ppp" + "pliii", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate, back), ptr(q), ptr(kpool), ptr(vpool),
              ptr(out), out.stride(0), o32, n, int(f32))
         return
     units = n * spec.kv_heads * ((spec.group + 15) // 16)
     nsplit = max(16, min(64, 148 // units)) if units <= MAX_TICKETS else 1          # a row takes as many of them as its position asks for,
     if spec.window:                                                                 # each at least two pages
-        nsplit = max(1, min(nsplit, ((spec.window + PAGE - 2) // PAGE + 2) // 2))
+        nsplit = max(1, min(nsplit, ((spec.window + PAGE - 2) // PAGE + 2 + (spec.keep_first + PAGE - 1) // PAGE) // 2))
     part = lse = None
     if nsplit > 1:
         part = torch.empty(n, spec.heads, nsplit, spec.vdim, dtype=torch.float32, device=dev)
         lse = torch.empty(n, spec.heads, nsplit, dtype=torch.float32, device=dev)
-    call("gqa_decode", _D + _R + _S + "pppl" + "pppi" + "pliip", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate), ptr(q), ptr(kpool), ptr(vpool),
+    call("gqa_decode", _D + _R + _S + "pppl" + "pppi" + "pliip", *_dims(spec, kpool, vpool), *_rows(pos, slot, cache), *_score(spec, gate, back), ptr(q), ptr(kpool), ptr(vpool),
          kpool.shape[0], ptr(part), ptr(lse), ptr(_ticket_words(dev)), nsplit, ptr(out), out.stride(0), o32, n, ptr(K.status_word(dev)))
 
 
@@ -210,21 +234,22 @@ def gqa_attend(spec: GqaSpec, proj, b, cache, kpool, vpool, out):
     view of any row pitch; fp32, or bf16 as the cache). ``kpool`` / ``vpool``: this layer's pages."""
     if not proj.is_cuda:
         return gqa_reference(spec, proj, b, cache, kpool, vpool, out)
-    return gqa_scores(spec, gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool), b, cache, kpool, vpool, out, spec.gate(proj))
+    q, back = gqa_store(spec, proj, b.pos, b.slot, cache, kpool, vpool)
+    return gqa_scores(spec, q, b, cache, kpool, vpool, out, spec.gate(proj), back)
 
 
-def gqa_scores(spec: GqaSpec, q, b, cache, kpool, vpool, out, gate=None):
-    """Attention of the queries of ``gqa_store`` over the cached rows. ``gate``: the gate's columns as projected."""
+def gqa_scores(spec: GqaSpec, q, b, cache, kpool, vpool, out, gate=None, back=None):
+    """Attention of the queries of ``gqa_store`` over the cached rows. ``gate``: the gate's columns as projected; ``back``: its second result."""
     n = q.shape[0]
     if b.row_path or kpool.dtype == torch.float32 or not spec.tc_prefill or out.dtype != torch.bfloat16:
-        _each_row(spec, q, gate, b.pos, b.slot, cache, kpool, vpool, out)
+        _each_row(spec, q, back, gate, b.pos, b.slot, cache, kpool, vpool, out)
         return out
     t = b.segments()
     r0 = t.short_rows
     if r0:
-        _each_row(spec, q[:r0], None if gate is None else gate[:r0], b.pos[:r0], b.slot[:r0], cache, kpool, vpool, out[:r0])
+        _each_row(spec, q[:r0], back, None if gate is None else gate[:r0], b.pos[:r0], b.slot[:r0], cache, kpool, vpool, out[:r0])
     if r0 < n:
         tf, tc = t.tiles(128 // spec.group)
-        call("gqa_prefill", _D + _R + _S + "pppl" + "ppi" + "plp", *_dims(spec, kpool, vpool), *_rows(b.pos, b.slot, cache), *_score(spec, gate), ptr(q), ptr(kpool),
+        call("gqa_prefill", _D + _R + _S + "pppl" + "ppi" + "plp", *_dims(spec, kpool, vpool), *_rows(b.pos, b.slot, cache), *_score(spec, gate, back), ptr(q), ptr(kpool),
              ptr(vpool), kpool.shape[0], ptr(tf), ptr(tc), tf.numel(), ptr(out), out.stride(0), ptr(K.status_word(q.device)))
     return out

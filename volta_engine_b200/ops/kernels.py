@@ -533,24 +533,24 @@ def bf16_wide(T: int, N: int) -> bool:
     return 1.75 * waves((N + 255) // 256 * tt) < waves((N + 127) // 128 * tt)
 
 
-def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False):
-    """out[t, n] = alpha * sum_k W[n,k] x[t,k] on tcgen05 (bf16 x bf16, fp32 accumulate)."""
+def gemm_bf16(W, x, out=None, residual=None, alpha=1.0, out_f32=False, bias=None):
+    """out[t, n] = alpha * sum_k W[n,k] x[t,k] (+ bias[n], fp32) on tcgen05 (bf16 x bf16, fp32 accumulate)."""
     N, K = W.shape
     T = x.shape[0]
     if out is None:
         out = torch.empty(T, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     f32 = out.dtype == torch.float32
-    call("gemm_bf16_wide" if bf16_wide(T, N) else "gemm_bf16", "plplplppliiifp", ptr(W), W.stride(0), ptr(x), x.stride(0), 0 if f32 else ptr(out),
+    call("gemm_bf16_wide" if bf16_wide(T, N) else "gemm_bf16", "plplplppliiifpp", ptr(W), W.stride(0), ptr(x), x.stride(0), 0 if f32 else ptr(out),
          out.stride(0), ptr(out) if f32 else 0, ptr(residual), residual.stride(0) if residual is not None else 0,
-         T, N, K, float(alpha), ptr(status_word(x.device)))
+         T, N, K, float(alpha), ptr(bias), ptr(status_word(x.device)))
     return out
 
 
-def gemm_f32(W, x):
-    """out[t, n] = sum_k W[n, k] x[t, k], true fp32."""
+def gemm_f32(W, x, bias=None):
+    """out[t, n] = sum_k W[n, k] x[t, k] (+ bias[n]), true fp32."""
     N, K = W.shape
     out = torch.empty(x.shape[0], N, dtype=torch.float32, device=x.device)
-    call("gemm_f32", "plplpliii", ptr(W), W.stride(0), ptr(x), x.stride(0), ptr(out), N, x.shape[0], N, K)
+    call("gemm_f32", "plplpliiip", ptr(W), W.stride(0), ptr(x), x.stride(0), ptr(out), N, x.shape[0], N, K, ptr(bias))
     return out
 
 

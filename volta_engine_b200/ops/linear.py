@@ -26,7 +26,8 @@ GEMV_KERNEL = os.environ.get("VOLTA_GEMV", "auto")
 
 
 class LinearBF16:
-    def __init__(self, weight: torch.Tensor):
+    def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None):
+        self.bias = bias                   # fp32 [N]
         self.out_features, self.in_features = weight.shape
         if self.in_features % 8:           # 16-byte rows for the loaders: zero columns behind the real ones
             weight = torch.nn.functional.pad(weight, (0, -self.in_features % 8))
@@ -37,17 +38,21 @@ class LinearBF16:
             x = torch.nn.functional.pad(x, (0, self.weight.shape[1] - x.shape[1]))
         if not x.is_cuda:
             y = x.float() @ self.weight.float().t()
+            if self.bias is not None:
+                y = y + self.bias
             if residual is not None:
                 y = y + residual.float()
             return y if out_f32 else y.to(x.dtype)
-        if x.shape[0] <= GEMV_MAX_ROWS and out_f32 and residual is None:
+        if x.shape[0] <= GEMV_MAX_ROWS and out_f32 and residual is None and self.bias is None:
             return K.bf16_gemv_f32(self.weight, x, out)
         if GEMM_BACKEND == "cublas":
             y = torch.matmul(x, self.weight.t())
+            if self.bias is not None:
+                y = y + self.bias.to(y.dtype)
             if residual is not None:
                 y = y + residual
             return y.float() if out_f32 else y
-        return K.gemm_bf16(self.weight, x, out=out, residual=residual, out_f32=out_f32)
+        return K.gemm_bf16(self.weight, x, out=out, residual=residual, out_f32=out_f32, bias=self.bias)
 
     def nbytes(self):
         return self.weight.numel() * self.weight.element_size()
@@ -56,14 +61,15 @@ class LinearBF16:
 class LinearF32:
     """fp32 weight and activations: the linears of a model's all-32-bit form."""
 
-    def __init__(self, weight: torch.Tensor):
-        self.weight = weight.float().contiguous()
+    def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None = None):
+        self.weight, self.bias = weight.float().contiguous(), bias
         self.out_features, self.in_features = weight.shape
 
     def forward(self, x, out_f32=True):
         if not x.is_cuda:
-            return x @ self.weight.t()
-        return K.gemm_f32(self.weight, x)
+            y = x @ self.weight.t()
+            return y if self.bias is None else y + self.bias
+        return K.gemm_f32(self.weight, x, self.bias)
 
     def nbytes(self):
         return self.weight.numel() * 4

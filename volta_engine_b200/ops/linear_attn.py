@@ -4,7 +4,8 @@
 
 over projection rows [ q (heads dk) | x (heads dk) | v (heads dv) | ... ] and one of
 
-  * ``decay`` given (lightning attention): d = decay[head], k = silu(x), v = silu(v), q = silu(q);
+  * ``decay`` given (lightning attention): d = decay[head], k = silu(x), v = silu(v), q = silu(q); with ``plain`` (retention) k = x and v as
+    projected, q times ``q_scale``;
   * ``lower`` / ``bias`` given (HGRN2): the forget gate f = lower + (1 - lower) sigmoid(x + bias) per channel is the decay and
     its complement 1 - f the key; v as projected, q = silu(q);
   * ``w2`` / ``bias`` given (gated linear attention): d = sigmoid(w2 a + bias)^(1 / tau) per channel from a low-rank part a of the
@@ -33,6 +34,7 @@ class LinAttnSpec:
     a_col: int = 0
     tau: float = 1.0
     q_scale: float = 1.0
+    plain: bool = False
 
     @property
     def mode(self) -> int:
@@ -77,7 +79,7 @@ def gates(pf, spec: LinAttnSpec):
         z = pf[:, spec.a_col: spec.a_col + spec.rank] @ spec.w2.t() + spec.bias
         return torch.exp(torch.nn.functional.logsigmoid(z) / spec.tau).reshape(n, spec.heads, spec.dk), x.reshape(n, spec.heads, spec.dk)
     if spec.mode == 0:
-        k = torch.nn.functional.silu(x).reshape(n, spec.heads, spec.dk)
+        k = (x if spec.plain else torch.nn.functional.silu(x)).reshape(n, spec.heads, spec.dk)
         return spec.decay.reshape(1, spec.heads, 1).expand_as(k), k
     z = x + spec.bias
     f = spec.lower + (1.0 - spec.lower) * torch.sigmoid(z)
@@ -89,10 +91,10 @@ def linattn_reference(proj, pos, slot, st: LinAttnState, spec: LinAttnSpec) -> t
     """CPU statement over the rows of a batch; updates ``st`` in place -> fp32 [rows, heads * dv]."""
     n, H, dk, dv = proj.shape[0], spec.heads, spec.dk, spec.dv
     pf = proj.float()
-    q = (pf[:, : H * dk] * spec.q_scale if spec.mode == 2 else torch.nn.functional.silu(pf[:, : H * dk])).reshape(n, H, dk)
+    q = (pf[:, : H * dk] * spec.q_scale if spec.mode == 2 or spec.plain else torch.nn.functional.silu(pf[:, : H * dk])).reshape(n, H, dk)
     d, k = gates(pf, spec)
     v = pf[:, 2 * H * dk: spec.cols].reshape(n, H, dv)
-    if spec.mode == 0:
+    if spec.mode == 0 and not spec.plain:
         v = torch.nn.functional.silu(v)
     o = torch.zeros(n, H, dv)
     for i in range(n):
@@ -110,9 +112,9 @@ def linattn_reference(proj, pos, slot, st: LinAttnState, spec: LinAttnSpec) -> t
 def _step(proj, pos, slot, st, spec, o, rows, segs=None):
     x32 = 1 if proj.dtype == torch.float32 else 0
     first, count, n = segs if segs is not None else (None, None, 0)
-    call("linattn_step", "plipp" + "ppi" + "pppp" + "pliiiii" + "piiff", ptr(proj), proj.stride(0), x32, ptr(pos), ptr(slot), ptr(first), ptr(count), n,
+    call("linattn_step", "plipp" + "ppi" + "pppp" + "pliiiii" + "piiffi", ptr(proj), proj.stride(0), x32, ptr(pos), ptr(slot), ptr(first), ptr(count), n,
          ptr(st.rec), ptr(spec.bias), ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), rows, spec.heads, spec.dk, spec.dv, spec.mode,
-         ptr(spec.w2), spec.rank, spec.a_col, 1.0 / spec.tau, float(spec.q_scale))
+         ptr(spec.w2), spec.rank, spec.a_col, 1.0 / spec.tau, float(spec.q_scale), int(spec.plain))
 
 
 def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJournal | None = None, rows=None,
@@ -150,7 +152,7 @@ def linattn_rows(proj, b, st: LinAttnState, spec: LinAttnSpec, journal: GDNJourn
             dec = torch.empty(n, spec.heads * spec.dk, dtype=torch.float32, device=proj.device)
             a = proj[:, spec.a_col:]
             call("linattn_decay", "plippp" + "iiif", ptr(a), a.stride(0), 1, ptr(spec.w2), ptr(spec.bias), ptr(dec), n, spec.heads * spec.dk, spec.rank, 1.0 / spec.tau)
-        call("linattn_chunk", "plpppppp" + "iii" + "ppp" + "pppp" + "liiii" + "pf", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
+        call("linattn_chunk", "plpppppp" + "iii" + "ppp" + "pppp" + "liiii" + "pfi", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
              ptr(t.chunk_count), ptr(t.seg_chunk0), t.chunks, t.seg_chunk0.numel() - 1, t.longest, ptr(st.rec), ptr(start), ptr(total), ptr(spec.bias),
-             ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), spec.heads, spec.dk, spec.dv, spec.mode, ptr(dec), float(spec.q_scale))
+             ptr(spec.lower), ptr(spec.decay), ptr(o), o.stride(0), spec.heads, spec.dk, spec.dv, spec.mode, ptr(dec), float(spec.q_scale), int(spec.plain))
     return o

@@ -18,9 +18,10 @@ FEW_ROWS = 16                             # rows that run route by route
 
 @dataclass
 class Router:
-    """Scores are the softmax over all experts, in fp32. With ``groups`` > ``keep`` the experts form equal groups of neighbours, of which
+    """Scores are the softmax over all experts, or (``sigmoid``) the sigmoid of every logit, in fp32. With ``groups`` > ``keep`` the experts form equal groups of neighbours, of which
     the ``keep`` best stay open; a group's score is its best member's (``best2``: the sum of its two best). The ``top`` best open experts
-    are taken, their scores are the weights (``renorm``: over their sum), times ``factor``. Ties go to the lower index."""
+    are taken, their scores are the weights (``renorm``: over their sum), times ``factor``. Ties go to the lower index. A weight multiplies
+    its expert's output, or (``weigh_input``) what the expert reads."""
     experts: int
     top: int
     groups: int = 1
@@ -28,6 +29,8 @@ class Router:
     best2: bool = False
     renorm: bool = False
     factor: float = 1.0
+    sigmoid: bool = False
+    weigh_input: bool = False
 
     def __post_init__(self):
         if self.experts > MAX_EXPERTS or self.top > MAX_TOP:
@@ -37,7 +40,7 @@ class Router:
 
     def choose(self, z):
         """CPU statement: logits [rows, experts] -> (experts int32 [rows, top], weights fp32 [rows, top])."""
-        s = torch.softmax(z.float(), -1)
+        s = torch.sigmoid(z.float()) if self.sigmoid else torch.softmax(z.float(), -1)
         rows = s.shape[0]
         open_ = s
         if self.keep < self.groups:
@@ -54,10 +57,10 @@ class Router:
 
     @property
     def args(self):
-        return self.experts, self.top, self.groups, self.keep, int(self.best2), int(self.renorm), float(self.factor)
+        return self.experts, self.top, self.groups, self.keep, int(self.best2), int(self.renorm), float(self.factor), int(self.sigmoid)
 
 
-_R = "iiiiiif"
+_R = "iiiiiifi"
 
 
 class ExpertWeights:
@@ -90,24 +93,28 @@ def routed_reference(router: Router, ex: ExpertWeights, z, x, out_dtype):
     for e in ids.unique().tolist():
         r, k = (ids == e).nonzero(as_tuple=True)
         gu = x[r] @ ex.gate_up[e, :, : ex.width].float().t()
+        f = w[r, k, None]
+        if router.weigh_input:
+            gu, f = gu * f, 1.0
         a = ex.unit.of(gu[:, : ex.ff], gu[:, ex.ff:]).to(dt).float()
-        y.index_add_(0, r, w[r, k, None] * (a @ ex.down[e, :, : ex.ff].float().t()))
+        y.index_add_(0, r, f * (a @ ex.down[e, :, : ex.ff].float().t()))
     return y.to(out_dtype)
 
 
-def routed_few(router: Router, ex: ExpertWeights, z, x, out_dtype):
-    """Rows one by one: two launches, the first routes too. ``x``: rows of the weights' type, or fp32 (rounded to it)."""
+def routed_few(router: Router, ex: ExpertWeights, z, x, out_dtype=None, residual=None):
+    """Rows one by one: two launches, the first routes too. ``x``: rows of the weights' type, or fp32 (rounded to it). ``residual``: fp32 rows
+    that the results are added to (nothing is returned)."""
     n, dev, dt = x.shape[0], x.device, ex.down.dtype
     f32 = int(dt == torch.float32)
     ids = torch.empty(n, router.top, dtype=torch.int32, device=dev)
     w = torch.empty(n, router.top, dtype=torch.float32, device=dev)
     a = torch.empty(n * router.top, ex.ff, dtype=dt, device=dev)
-    call("routed_up", _R + "plplipl" + "plpp" + "iiifffi", *router.args, ptr(z), z.stride(0), ptr(x), x.stride(0), int(x.dtype == torch.float32), ptr(ex.gate_up),
-         ex.gate_up.stride(1), ptr(a), a.stride(0), ptr(ids), ptr(w), n, ex.width, ex.ff, *ex.unit.constants, f32)
-    out = torch.empty(n, ex.width, dtype=out_dtype, device=dev)
-    call("routed_down", "plplppiplii" + "iii", ptr(a), a.stride(0), ptr(ex.down), ex.down.stride(1), ptr(ids), ptr(w), router.top, ptr(out), out.stride(0),
-         int(out_dtype == torch.float32), n, ex.width, ex.ff, f32)
-    return out
+    call("routed_up", _R + "plplipl" + "plpp" + "iiifffii", *router.args, ptr(z), z.stride(0), ptr(x), x.stride(0), int(x.dtype == torch.float32), ptr(ex.gate_up),
+         ex.gate_up.stride(1), ptr(a), a.stride(0), ptr(ids), ptr(w), n, ex.width, ex.ff, *ex.unit.constants, int(router.weigh_input), f32)
+    out = torch.empty(n, ex.width, dtype=out_dtype, device=dev) if residual is None else residual
+    call("routed_down", "plplppiplii" + "iiii", ptr(a), a.stride(0), ptr(ex.down), ex.down.stride(1), ptr(ids), 0 if router.weigh_input else ptr(w), router.top, ptr(out),
+         out.stride(0), int(out.dtype == torch.float32), n, ex.width, ex.ff, int(residual is not None), f32)
+    return out if residual is None else None
 
 
 def routed_many(router: Router, ex: ExpertWeights, z, x) -> RoutedRows:
@@ -132,7 +139,8 @@ def routed_many(router: Router, ex: ExpertWeights, z, x) -> RoutedRows:
         call("gemm_grouped_bf16", "plplpliiiiipip", ptr(W), W.stride(1), ptr(a), a.stride(0), ptr(out), out.stride(0), routes, ex.experts, cols, k, bn, ptr(tab),
              tiles, ptr(st))
         return out
-    a = ex.unit.rows(grouped(ex.gate_up, xs, 2 * ex.ff, ex.width), x.dtype)
+    by = (w.reshape(-1), order) if router.weigh_input else None
+    a = ex.unit.rows(grouped(ex.gate_up, xs, 2 * ex.ff, ex.width), x.dtype, by)
     if ex.ff % 8:
         a = torch.nn.functional.pad(a, (0, -ex.ff % 8))
-    return RoutedRows(grouped(ex.down, a, ex.width, ex.ff), inv, w)
+    return RoutedRows(grouped(ex.down, a, ex.width, ex.ff), inv, None if router.weigh_input else w)

@@ -135,13 +135,17 @@ class ClampedGlu:
         F, K = gate.shape
         return torch.stack([gate.reshape(F // 4, 4, K), up.reshape(F // 4, 4, K)], 1).reshape(2 * F, K)
 
-    def rows(self, z, out_dtype):
+    def rows(self, z, out_dtype, by=None):
+        """``by`` = (weights fp32, index int32 [rows]): row r of z is first multiplied with weights[index[r]]."""
         rows, F = z.shape[0], z.shape[1] // 2
         if not z.is_cuda:
+            if by is not None:
+                z = z.float() * by[0][by[1].long()][:, None]
             v = z.float().reshape(rows, F // 4, 2, 4).transpose(1, 2).reshape(rows, 2 * F) if self.blocks else z.float()
             return self.of(v[:, :F], v[:, F:]).to(out_dtype)
         out = torch.empty(rows, F, dtype=out_dtype, device=z.device)
-        call("clamped_glu", "plipliiifffi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, int(self.blocks), *self.constants, _f32(out))
+        w, index = by if by is not None else (None, None)
+        call("clamped_glu", "plipliiifffppi", ptr(z), z.stride(0), _f32(z), ptr(out), out.stride(0), rows, F, int(self.blocks), *self.constants, ptr(w), ptr(index), _f32(out))
         return out
 
     def epilogue(self):
@@ -194,11 +198,12 @@ class RoutedRows:
     """Results of a routed feed-forward that are not summed yet: a row's result is sum_k w[row, k] d[inv[row, k]]."""
     d: torch.Tensor           # [routes, H]
     inv: torch.Tensor         # int32 [rows, top]
-    w: torch.Tensor           # fp32 [rows, top]
+    w: torch.Tensor | None = None         # fp32 [rows, top] (None: all one)
 
     def tensor(self):
-        rows, top = self.w.shape
-        return torch.einsum("rk,rkh->rh", self.w, self.d[self.inv.long().reshape(-1)].reshape(rows, top, -1).float()).to(self.d.dtype)
+        rows, top = self.inv.shape
+        d = self.d[self.inv.long().reshape(-1)].reshape(rows, top, -1).float()
+        return (d.sum(1) if self.w is None else torch.einsum("rk,rkh->rh", self.w, d)).to(self.d.dtype)
 
 
 @dataclass
@@ -216,24 +221,33 @@ class NormedWrite:
 
 @dataclass
 class ResidualNorm:
-    """What is read of an fp32 residual whose sublayers norm their results: the residual itself (``w`` None) or its RMS norm."""
+    """What is read of an fp32 residual: the residual itself (``w`` None) or its RMS norm. A sublayer's result enters it behind a norm of its
+    own (``write``: NormedWrite) or as it is (None)."""
     w: torch.Tensor | None
     eps: float
     takes_routed = True
+
+    @staticmethod
+    def add(h, part, write: NormedWrite | None = None):
+        """CPU statement: a result enters the residual."""
+        if write is not None:
+            write.add(h, part)
+        else:
+            h += (part.tensor() if isinstance(part, RoutedRows) else part).float()
 
     def rows(self, h, out_dtype, part=None, write: NormedWrite | None = None):
         """The result in front enters the residual (in place, optional), then what is read of it."""
         rows, H = h.shape
         if not h.is_cuda:
             if part is not None:
-                write.add(h, part)
+                self.add(h, part, write)
             v = h if self.w is None else h / torch.sqrt(h.pow(2).mean(-1, keepdim=True) + self.eps) * self.w
             return v.to(out_dtype)
-        assert part is None or write.eps == self.eps
+        assert part is None or write is None or write.eps == self.eps
         out = torch.empty(rows, H, dtype=out_dtype, device=h.device)
-        d, inv, w, top = (part.d, part.inv, part.w, part.w.shape[1]) if isinstance(part, RoutedRows) else (part, None, None, 0)
+        d, inv, w, top = (part.d, part.inv, part.w, part.inv.shape[1]) if isinstance(part, RoutedRows) else (part, None, None, 0)
         call("residual_norm", "pplppippplii" + "fi", ptr(h), ptr(d), d.stride(0) if d is not None else 0, ptr(inv), ptr(w), top,
-             ptr(write.w) if part is not None else 0, ptr(self.w), ptr(out), out.stride(0), rows, H, float(self.eps), _f32(out))
+             ptr(write.w) if part is not None and write is not None else 0, ptr(self.w), ptr(out), out.stride(0), rows, H, float(self.eps), _f32(out))
         return out
 
     def prologue(self, h, part=None, write: NormedWrite | None = None):
@@ -289,8 +303,8 @@ def fused_fits(lin, rows: int) -> bool:
 
 
 def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wlen=0, gate=None, coef=None, eps=0.0, head=None, silu=False,
-              glu=None, unit=None, part=None, h_out=None, cap=0.0, out_f32=False, residual=None):
-    """A bf16 linear on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
+              glu=None, unit=None, part=None, h_out=None, x_out=None, cap=0.0, out_f32=False, residual=None):
+    """A bf16 linear (with its bias, if it has one) on ``M`` <= 16 rows. ``pro`` and its operands: the ``prologue`` dictionaries above (0: ``x`` is bf16).
     ``glu`` = (alpha, limit, shift): the clamped gated unit of its outputs, which come in blocks, in bf16. ``cap``: soft cap of fp32 outputs.
     ``residual`` = (h fp32, scale | None): h += scale * y in place, (streams, StreamWrite): the streams rewritten in place; otherwise
     the product is returned."""
@@ -308,9 +322,9 @@ def gemv_rows(lin, M: int, *, x, pro=0, kx=0, w=None, b=None, alpha=0.0, G=0, wl
     streams, mix = 0, None
     if isinstance(scale, StreamWrite):
         streams, mix, scale = h.shape[1], scale.mix, scale.out
-    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiifffip" + "fplp", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
+    call("gemv_rows", "pliiiii" + "plppfiiplpf" + "pplplp" + "pliiifffip" + "fplppp", ptr(W), W.stride(0), N, K, M, pro, kx or k0 + x.shape[1], ptr(x), x.stride(0), ptr(w), ptr(b),
          float(alpha), G, wlen, ptr(gate), gate.stride(0) if gate is not None else 0, ptr(coef), float(eps),
          ptr(out) if out_f32 else 0, ptr(out) if out is not None and not out_f32 else 0, out.stride(0) if out is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(scale),
          ptr(head), head.stride(0) if head is not None else 0, k0, int(silu), int(glu is not None), *(glu or unit or (0.0, 0.0, 0.0)), streams, ptr(mix),
-         float(cap), ptr(part), part.stride(0) if part is not None else 0, ptr(h_out))
+         float(cap), ptr(part), part.stride(0) if part is not None else 0, ptr(h_out), ptr(x_out), ptr(getattr(lin, "bias", None)))
     return out

@@ -113,7 +113,7 @@ def run_kernels(width: int, dev) -> dict:
         pairs = _kept(n, ctx)
         proj = torch.randn(n, mx.in_proj.out_features, device=dev).to(ty)
         out = torch.empty(n, D, dtype=bf, device=dev)
-        q = gqa_store(spec, proj, b.pos, b.slot, kv, kv.k[0], kv.v[0])
+        q, _ = gqa_store(spec, proj, b.pos, b.slot, kv, kv.k[0], kv.v[0])
         kb.add(f"attention {kind}", "kutolix (gate, sink)", lambda: gqa_scores(spec, q, b, kv, kv.k[0], kv.v[0], out, spec.gate(proj)),
                keys * G * 512 + n * D * (4 + size), 4.0 * pairs * D)
         qkv = torch.randn(n, (H + 2 * G) * 128, device=dev).to(bf)

@@ -99,7 +99,7 @@ def run_kernels(width: int, dev) -> dict:
         kvb = ctx * G * 256 * 2
         out = torch.empty(n, D, dtype=bf if n > 1 else torch.float32, device=dev)
         spec = mx.left.spec
-        q = gqa_store(spec, proj, b.pos, b.slot, kv, kv.k[0], kv.v[0])
+        q, _ = gqa_store(spec, proj, b.pos, b.slot, kv, kv.k[0], kv.v[0])
         kb.add(f"attention {kind}", "siditar", lambda: gqa_scores(spec, q, b, kv, kv.k[0], kv.v[0], out), kvb + n * D * 4, flops)
         qkv = torch.randn(n, (H + 2 * G) * 128, device=dev).to(bf)
         kp, vp = kvd.layer(0)
