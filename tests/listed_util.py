@@ -1,9 +1,12 @@
-"""What the tests of decoders with listed layers share: engines, portions, schedules of several requests, the scheduler."""
+"""What the tests of decoders with listed layers share: engines, portions, schedules of several requests, rows through one operator, the
+scheduler."""
+import dataclasses
 import json
 
 import pytest
 import torch
 
+from volta_engine_b200.runtime.batch import BatchRows
 from volta_engine_b200.runtime.engine import Engine
 from volta_engine_b200.runtime.generator import Generator
 from volta_engine_b200.runtime.kv_cache import PagedKVCache
@@ -77,6 +80,38 @@ def schedule(lengths, seed):
         if step:
             steps.append((step, ended))
     return steps
+
+
+# ------------------------------------------------------------------------------------------ one operator
+class Rows:
+    """A paged cache (its rows wider than this layer's, filled with an earlier request's rows) and batches through an operator."""
+
+    def __init__(self, dtype, device, kw, vw, extra=0, pages=24):
+        self.dtype, self.device = dtype, device
+        self.kv = PagedKVCache(2, 1, kw + extra, pages, 3, 1024, torch.device(device), dtype=dtype, v_head_dim=vw + extra)
+        self.kv.k.fill_(3.0)
+        self.kv.v.fill_(-3.0)
+
+    def batch(self, parts):
+        """parts: [(slot, first position, rows)] one batch, shortest first."""
+        pos, slots = [], []
+        for s, p0, x in parts:
+            self.kv.reserve(s, p0 + x.shape[0])
+            pos += range(p0, p0 + x.shape[0])
+            slots += [s] * x.shape[0]
+        b = BatchRows.make(pos, pos, slots, self.device)
+        return self.run(b, torch.cat([p[2] for p in parts]))
+
+    def walk(self, slot, x, cuts):
+        at, got = 0, []
+        for c in cuts:
+            got.append(self.batch([(slot, at, x[at:at + c])]))
+            at += c
+        return torch.cat(got)
+
+
+def vars_of(spec):
+    return {f.name: getattr(spec, f.name) for f in dataclasses.fields(spec)}
 
 
 # ------------------------------------------------------------------------------------------ scheduler

@@ -135,12 +135,15 @@ def test_wide_gemm_at_the_edges_of_its_tiles(T, N, K):
     W[:, :K], x[:, :K] = rnd(N, K, seed=1).to(torch.bfloat16), rnd(T, K, seed=2).to(torch.bfloat16)
     res = rnd(T, N, seed=3).to(torch.bfloat16)
     e = x.double() @ W.double().t()
-    Wd, xd, rd = W.cuda(), x.cuda(), res.cuda()
-    for f32 in (True, False):
+    bias = rnd(N, seed=4)
+    Wd, xd, rd, bd = W.cuda(), x.cuda(), res.cuda(), bias.cuda()
+    for f32, biased in ((True, False), (False, False), (True, True), (False, True)):
         out = torch.full((T + 1, N), 9.0, dtype=torch.float32 if f32 else torch.bfloat16, device="cuda")
-        call("gemm_bf16_wide", "plplplppliiifp", ptr(Wd), Kp, ptr(xd), Kp, 0 if f32 else ptr(out), N, ptr(out) if f32 else 0, 0 if f32 else ptr(rd), N, T, N, Kp,
-             1.0, ptr(status_word(Wd.device)))
+        call("gemm_bf16_wide", "plplplppliiifpp", ptr(Wd), Kp, ptr(xd), Kp, 0 if f32 else ptr(out), N, ptr(out) if f32 else 0, 0 if f32 else ptr(rd), N, T, N, Kp,
+             1.0, ptr(bd) if biased else 0, ptr(status_word(Wd.device)))
         want = e if f32 else e + res.double()
+        if biased:
+            want = want + bias.double()
         assert (out[:T].double().cpu() - want).abs().max() < (1e-5 if f32 else 6e-3) * want.abs().max()
         assert bool((out[T] == 9.0).all())
 

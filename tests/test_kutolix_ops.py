@@ -8,15 +8,13 @@ import pytest
 import torch
 
 import kutolix_plain as plain
-from listed_util import DEVICES, one_thread  # noqa: F401
+from listed_util import DEVICES, Rows, one_thread, vars_of  # noqa: F401
 from volta_engine_b200.ops.gqa import GqaSpec, gqa_attend, gqa_store
 from volta_engine_b200.ops.latent import LatentSpec, latent_rows
 from volta_engine_b200.ops.linear import LinearBF16, LinearF32
 from volta_engine_b200.ops.rotary import Rotation
 from volta_engine_b200.ops.routed import ExpertWeights, Router, route, routed_few, routed_many, routed_reference
 from volta_engine_b200.ops.rowops import ClampedGlu, NormedWrite, ResidualNorm, RoutedRows, embed_rows, gemv_rows, soft_cap_
-from volta_engine_b200.runtime.batch import BatchRows
-from volta_engine_b200.runtime.kv_cache import PagedKVCache
 
 TYPES = [torch.float32, torch.bfloat16]
 TOL = {torch.float32: 3e-5, torch.bfloat16: 0.03}
@@ -92,33 +90,6 @@ def att_case(H, G, d, dv, window, dims=None, base=500.0, scale=None, sink=0.0, s
     return spec, {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "scale": spec.scale, "mask": {"size": window}, "rot": {"dims": dims, "base": base}}, W
 
 
-class Rows:
-    """A paged cache (its rows wider than this layer's, filled with an earlier request's rows) and batches through an operator."""
-
-    def __init__(self, dtype, device, kw, vw, extra=0, pages=24):
-        self.dtype, self.device = dtype, device
-        self.kv = PagedKVCache(2, 1, kw + extra, pages, 3, 1024, torch.device(device), dtype=dtype, v_head_dim=vw + extra)
-        self.kv.k.fill_(3.0)
-        self.kv.v.fill_(-3.0)
-
-    def batch(self, parts):
-        """parts: [(slot, first position, rows)] one batch, shortest first."""
-        pos, slots = [], []
-        for s, p0, x in parts:
-            self.kv.reserve(s, p0 + x.shape[0])
-            pos += range(p0, p0 + x.shape[0])
-            slots += [s] * x.shape[0]
-        b = BatchRows.make(pos, pos, slots, self.device)
-        return self.run(b, torch.cat([p[2] for p in parts]))
-
-    def walk(self, slot, x, cuts):
-        at, got = 0, []
-        for c in cuts:
-            got.append(self.batch([(slot, at, x[at:at + c])]))
-            at += c
-        return torch.cat(got)
-
-
 class AttnRows(Rows):
     def __init__(self, spec, dtype, device, extra=0, x32=False):
         super().__init__(dtype, device, *spec.row_widths, extra)
@@ -134,11 +105,6 @@ class AttnRows(Rows):
         gqa_attend(self.spec, x, b, self.kv, self.kv.k[1], self.kv.v[1], y[:, :w])
         assert bool((y[:, w:] == 5.0).all())
         return y[:, :w].float().cpu()
-
-
-def vars_of(spec):
-    import dataclasses
-    return {f.name: getattr(spec, f.name) for f in dataclasses.fields(spec)}
 
 
 ATT = [(4, 2, 24, 40, 37, 16), (3, 3, 21, 13, 19, 10), (8, 2, 128, 128, 64, 128), (18, 1, 16, 8, 65, 2), (2, 1, 64, 136, 100, 64), (1, 1, 264, 24, 50, 100), (5, 5, 8, 64, 1, 8),

@@ -28,15 +28,14 @@ def centred_norm(x, w, eps):
     return over_rms(x, eps) * (1.0 + w)
 
 
-def turn_pairs(v, p, base, dims):
-    """Neighbouring entries (2 i, 2 i + 1) of the first ``dims`` of v [..., width] turned by p base^(-2 i / dims)."""
+def turn_pairs(v, positions, base, dims):
+    """Row t of v [rows, heads, width]: neighbouring entries (2 i, 2 i + 1) of the first ``dims`` turned by positions[t] base^(-2 i / dims)."""
+    a = torch.tensor([[p * base ** (-2.0 * i / dims) for i in range(dims // 2)] for p in positions], dtype=F64)[:, None]
+    c, s = torch.cos(a).to(v.dtype), torch.sin(a).to(v.dtype)
     out = v.clone()
-    for i in range(dims // 2):
-        a = torch.tensor(p * base ** (-2.0 * i / dims), dtype=F64)
-        c, s = torch.cos(a).to(v.dtype), torch.sin(a).to(v.dtype)
-        x, y = v[..., 2 * i], v[..., 2 * i + 1]
-        out[..., 2 * i] = x * c - y * s
-        out[..., 2 * i + 1] = y * c + x * s
+    x, y = v[..., 0:dims:2], v[..., 1:dims:2]
+    out[..., 0:dims:2] = x * c - y * s
+    out[..., 1:dims:2] = y * c + x * s
     return out
 
 
@@ -77,9 +76,8 @@ def rotated_value_attention(W, p, m, h, eps):
     q = over_rms(proj("q", H, d), eps) * W[p + "q.norm"]
     k = over_rms(proj("k", G, d), eps) * W[p + "k.norm"]
     v = proj("v", G, dv)
-    q = torch.stack([turn_pairs(q[t], t, rot["base"], rot["dims"]) for t in range(T)])
-    k = torch.stack([turn_pairs(k[t], t, rot["base"], rot["dims"]) for t in range(T)])
-    v = torch.stack([turn_pairs(v[t], t, rot["base"], dv) for t in range(T)])
+    q, k = (turn_pairs(x, range(T), rot["base"], rot["dims"]) for x in (q, k))
+    v = turn_pairs(v, range(T), rot["base"], dv)
     out = torch.zeros(T, H, dv, dtype=h.dtype)
     for t in range(T):
         j = visible(t, m["mask"])
@@ -88,7 +86,7 @@ def rotated_value_attention(W, p, m, h, eps):
             s = soft_cap(k[j, g] @ q[t, n] * m["scale"] * W[p + "temp"][n], m["softcap"])
             e = torch.exp(s - s.max())
             out[t, n] = (e @ v[j, g]) / e.sum()
-        out[t] = turn_pairs(out[t], -t, rot["base"], dv)
+    out = turn_pairs(out, [-t for t in range(T)], rot["base"], dv)
     return out.reshape(T, H * dv) @ W[p + "o"].T + W[p + "o.b"]
 
 

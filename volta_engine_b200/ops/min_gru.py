@@ -36,7 +36,7 @@ class MinGruState:
 def min_gru_reference(proj, pos, slot, st: MinGruState) -> torch.Tensor:
     """CPU statement over the rows of a batch; updates ``st`` in place -> fp32 [rows, width]."""
     W = st.rec.shape[1]
-    z, u, g = proj.float().split(W, 1)
+    z, u, g = proj[:, : 3 * W].float().split(W, 1)
     take, keep = torch.sigmoid(z), torch.sigmoid(-z)
     c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
     S = torch.zeros(proj.shape[0], W)

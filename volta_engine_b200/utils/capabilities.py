@@ -30,6 +30,7 @@ TABLE = {
     "latent_rope_store": ("LatentAttention", P), "latent_absorb": ("LatentAttention", P), "latent_attn": ("LatentAttention", P),
     "latent_expand": ("LatentAttention", P), "latent_gather": ("LatentAttention", P), "latent_prefill": ("LatentAttention", P), "latent_prefill_tc": ("LatentAttention", P),
     "latent_decode": ("LatentAttention", P), "linattn_step": ("LinearAttention", P), "linattn_chunk": ("LinearAttention", P), "linattn_decay": ("LinearAttention", P),
+    "mingru_step": ("MinGru", P), "mingru_chunk": ("MinGru", P),
     "gqa_store": ("GroupedAttention", P), "gqa_rows": ("GroupedAttention", P), "gqa_decode": ("GroupedAttention", P), "gqa_prefill": ("GroupedAttention", P),
     "embed_rows": ("RowOps (fp32 residual)", P), "dyt_rows": ("RowOps (fp32 residual)", P), "group_rms": ("RowOps (fp32 residual)", P),
     "stream_norm": ("RowOps (fp32 residual)", P), "clamped_glu": ("RowOps (fp32 residual)", P),
