@@ -15,6 +15,7 @@ from volta_engine_b200.ops.linear import LinearBF16, LinearF32
 from volta_engine_b200.ops.rotary import Rotation
 from volta_engine_b200.ops.routed import ExpertWeights, Router, route, routed_few, routed_many, routed_reference
 from volta_engine_b200.ops.rowops import ClampedGlu, NormedWrite, ResidualNorm, RoutedRows, embed_rows, gemv_rows, soft_cap_
+from volta_engine_b200.runtime.kv_cache import PagedKVCache
 
 TYPES = [torch.float32, torch.bfloat16]
 TOL = {torch.float32: 3e-5, torch.bfloat16: 0.03}

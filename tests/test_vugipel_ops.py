@@ -430,4 +430,4 @@ def test_routed_results_without_weights_are_summed_into_the_residual(rows, width
     hd = h.clone().to(device)
     got = ResidualNorm((1.0 + w).to(device), 1e-5).rows(hd, torch.bfloat16, RoutedRows(d.to(device), inv.to(device)))
     close(got, plain.centred_norm(x, w.double(), 1e-5), torch.bfloat16, bf16=2 ** -6)
-    close(hd, x, torch.float32, f32=5e-6 if device == "cuda" else 2 ** -8)
+    close(hd, x, torch.float32, f32=5e-6 if device == "cuda" else 2 ** -7)
