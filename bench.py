@@ -95,10 +95,10 @@ def main():
     ap.add_argument("--comm", default=os.environ.get("VOLTA_COMM", "symm"))
     ap.add_argument("--kv-format", default="bf16", help="bf16 (the configuration of record) | fp8 | k8v4 | nvfp4 (quantised caches, A/B)")
     ap.add_argument("--config", default="dense27b", choices=["dense27b", "moe80b", "moe80b_exl3", "mla_mtp", "dsv3_gguf", "flash_next", "qwen3_5", "glm5_next", "fofosun",
-                                                               "siditar", "kutolix"],
+                                                               "siditar", "kutolix", "vugipel"],
                     help="dense27b: the configuration of record (default); the others are the reference's further headline "
-                         "models (volta_engine_b200/tools/bench_configs.py); fofosun, siditar, kutolix: that design beside "
-                         "the closest assembly at equal size (volta_engine_b200/tools/bench_fofosun.py, bench_siditar.py, bench_kutolix.py)")
+                         "models (volta_engine_b200/tools/bench_configs.py); fofosun, siditar, kutolix, vugipel: that design beside "
+                         "the closest assembly at equal size (volta_engine_b200/tools/bench_fofosun.py, bench_siditar.py, bench_kutolix.py, bench_vugipel.py)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
@@ -111,6 +111,9 @@ def main():
     if args.config == "kutolix":
         from volta_engine_b200.tools import bench_kutolix
         return bench_kutolix.run(args, ClockSampler)
+    if args.config == "vugipel":
+        from volta_engine_b200.tools import bench_vugipel
+        return bench_vugipel.run(args, ClockSampler)
     if args.config != "dense27b":
         from volta_engine_b200.tools import bench_configs
         return bench_configs.run(args, ClockSampler)
