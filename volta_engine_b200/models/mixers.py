@@ -236,7 +236,7 @@ class RotatedValueAttention(GroupedAttention):
         f32 = lambda name: src.tensor(p + name, device, torch.float32).reshape(-1).contiguous()
         rot, vdim, window = m["rot"], int(m["vdim"]), window_of(m)
         self.spec = GqaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), vdim, float(m["scale"]), eps, q_norm=f32("q.norm"), k_norm=f32("k.norm"),
-                            norm_first=True, head_mul=f32("temp"), softcap=float(m["softcap"]), out_scale=out_scale, window=window,
+                            norm_first=True, head_mul=f32("temp"), softcap=float(m.get("softcap") or 0.0), out_scale=out_scale, window=window,
                             keep_first=int(m["mask"].get("keep_first") or 0) if window else 0, rot=Rotation.from_config(rot, True).bind(device),
                             v_rot=Rotation(vdim, float(rot["base"]), True).bind(device))
         if self.spec.rot.dims > self.spec.dim:

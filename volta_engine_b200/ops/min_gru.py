@@ -13,8 +13,6 @@ import torch
 from .._lib import call, ptr
 from .gdn import GDNJournal
 
-PARTS = 4                 # of a chunk, walked side by side (csrc/cuda/mingru.cu)
-
 
 class MinGruState:
     """rec [slots, width] fp32 of one layer."""
@@ -81,8 +79,8 @@ def min_gru_rows(proj, b, st: MinGruState, dtype, cols: int = 0, journal: GDNJou
         _step(proj, pos, slot, st, y, n, (t.first, t.count, t.n_short))
     if t.chunks:
         new = lambda *s: torch.empty(*s, dtype=torch.float32, device=proj.device)
-        total, part, start = new(t.chunks, W, 2), new(t.chunks, PARTS, W, 2), new(t.seg_chunk0.numel() - 1, W)
-        call("mingru_chunk", "plpp" + "ppppi" + "pppp" + "pliii", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
-             ptr(t.chunk_count), ptr(t.seg_chunk0), t.chunks, ptr(st.rec), ptr(total), ptr(part), ptr(start), ptr(y), y.stride(0), W, y.shape[1],
+        total, start = new(t.chunks, 2, W), new(t.seg_chunk0.numel() - 1, W)
+        call("mingru_chunk", "plpp" + "ppppi" + "ppp" + "pliii", ptr(proj), proj.stride(0), ptr(pos), ptr(slot), ptr(t.chunk_seg), ptr(t.chunk_first),
+             ptr(t.chunk_count), ptr(t.seg_chunk0), t.chunks, ptr(st.rec), ptr(total), ptr(start), ptr(y), y.stride(0), W, y.shape[1],
              int(dtype == torch.float32))
     return y
