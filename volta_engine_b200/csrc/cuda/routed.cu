@@ -34,10 +34,12 @@ VE_DEVINL int warp_argmax(float v, int i, float* best = nullptr) {
   return i;
 }
 
-// One warp, one row. sc: E floats of scratch in shared memory, with groups > 1 `groups` more behind them. A closed expert's score is
-// -1, a taken one's -2, a taken group's -1: scores are never negative.
+// One warp, one row. sc: E floats of scratch in shared memory, with groups > 1 `groups` more behind them: what experts and groups are ranked by
+// (the softmax, or the logit: sigmoids near one cannot be told apart). A closed or taken expert's and a taken group's rank is -infinity.
 VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* sc, int* ids, float* w) {
   const int lane = threadIdx.x & 31;
+  const float NONE = __int_as_float(0xff800000);
+  auto score = [&](float v) { return r.sigmoid ? sigmoid_of(v) : v; };
   float m = -FLT_MAX;
   for (int e = lane; e < r.E; e += 32) {
     float l = z[e];
@@ -45,9 +47,7 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
     sc[e] = l;
     m = fmaxf(m, l);
   }
-  if (r.sigmoid) {
-    for (int e = lane; e < r.E; e += 32) sc[e] = sigmoid_of(sc[e]);
-  } else {
+  if (!r.sigmoid) {
     m = warp_max(m);
     float s = 0.f;
     for (int e = lane; e < r.E; e += 32) {
@@ -63,7 +63,7 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
     float* gs = sc + r.E;
     const int per = r.E / r.groups;
     for (int g = lane; g < r.groups; g += 32) {
-      float b1 = 0.f, b2 = 0.f;
+      float b1 = NONE, b2 = NONE;
       for (int e = g * per; e < (g + 1) * per; ++e) {
         const float v = sc[e];
         if (v > b1) {
@@ -71,11 +71,11 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
           b1 = v;
         } else if (v > b2) b2 = v;
       }
-      gs[g] = r.best2 ? b1 + b2 : b1;
+      gs[g] = r.best2 ? score(b1) + (per > 1 ? score(b2) : 0.f) : b1;
     }
     __syncwarp();
     for (int k = 0; k < r.keep; ++k) {
-      float v = -3.f;
+      float v = NONE;
       int i = 0x7fffffff;
       for (int g = lane; g < r.groups; g += 32)
         if (gs[g] > v) {
@@ -83,16 +83,16 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
           i = g;
         }
       i = warp_argmax(v, i);
-      if (lane == 0) gs[i] = -1.f;
+      if (lane == 0) gs[i] = NONE;
       __syncwarp();
     }
     for (int e = lane; e < r.E; e += 32)
-      if (gs[e / per] >= 0.f) sc[e] = -1.f;
+      if (gs[e / per] != NONE) sc[e] = NONE;
     __syncwarp();
   }
   float sum = 0.f;
   for (int k = 0; k < r.top; ++k) {
-    float v = -3.f;
+    float v = NONE;
     int i = 0x7fffffff;
     for (int e = lane; e < r.E; e += 32)
       if (sc[e] > v) {
@@ -100,11 +100,12 @@ VE_DEVINL void route_warp(const float* __restrict__ z, const Router& r, float* s
         i = e;
       }
     i = warp_argmax(v, i, &v);
+    v = score(v);
     sum += v;
     if (lane == 0) {
       ids[k] = i;
       w[k] = v;
-      sc[i] = -2.f;
+      sc[i] = NONE;
     }
     __syncwarp();
   }

@@ -42,13 +42,13 @@ class Router:
         """CPU statement: logits [rows, experts] -> (experts int32 [rows, top], weights fp32 [rows, top])."""
         s = torch.sigmoid(z.float()) if self.sigmoid else torch.softmax(z.float(), -1)
         rows = s.shape[0]
-        open_ = s
+        rank = open_ = z.float() if self.sigmoid else s                  # (sigmoids near one cannot be told apart)
         if self.keep < self.groups:
-            g = s.reshape(rows, self.groups, -1)
-            gs = g.topk(min(2, g.shape[2]), -1).values.sum(-1) if self.best2 else g.amax(-1)
+            g = rank.reshape(rows, self.groups, -1)
+            gs = s.reshape(g.shape).topk(min(2, g.shape[2]), -1).values.sum(-1) if self.best2 else g.amax(-1)
             best = torch.sort(gs, dim=-1, descending=True, stable=True).indices[:, : self.keep]
             kept = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, best, True)
-            open_ = torch.where(kept[:, :, None], g, torch.full_like(g, -1.0)).reshape(rows, -1)
+            open_ = torch.where(kept[:, :, None], g, torch.full_like(g, -torch.inf)).reshape(rows, -1)
         ids = torch.sort(open_, dim=-1, descending=True, stable=True).indices[:, : self.top]
         w = s.gather(1, ids)
         if self.renorm:
