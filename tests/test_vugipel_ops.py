@@ -1,6 +1,6 @@
 """Every mechanism of the Vugipel decoder alone against the plain statement: attention with rotated values (one key per row that stands out:
 just inside and just outside the window, among the first tokens and behind them, at page borders), soft caps, head factors, retention, the
-gated recurrence per channel, sigmoid routers and experts weighed at their input, linears with biases, norms with weights around zero."""
+gated recurrence per channel, sigmoid routers and experts weighed at their input, linears with biases, norms with offset weights."""
 import pytest
 import torch
 
@@ -300,7 +300,7 @@ def test_rows_of_no_slot_and_rows_of_one_slot_in_a_step():
 
 # ------------------------------------------------------------------------------------------ routers and experts
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("experts,top", [(12, 1), (7, 2), (40, 8), (1, 1), (6, 6), (300, 20), (1024, 32)])
+@pytest.mark.parametrize("experts,top", [(13, 1), (7, 2), (40, 8), (1, 1), (6, 6), (300, 20), (1024, 32)])
 def test_sigmoid_routers(experts, top, device):
     """Experts and weights of every row, best first; every weight is the sigmoid of its own logit, whatever the others are."""
     z = rnd(37, experts, seed=experts, scale=1.5)
@@ -325,7 +325,7 @@ def test_a_row_of_nan_logits_still_gives_experts():
     assert all(len(set(r)) == 4 and 0 <= min(r) and max(r) < 24 for r in ids.tolist())
 
 
-EXP = [(18, 4, 104, 40), (7, 2, 75, 19), (64, 8, 256, 88), (12, 1, 136, 264), (3, 3, 512, 8), (1, 1, 64, 64), (5, 4, 33, 130), (9, 8, 24, 6272)]
+EXP = [(18, 4, 104, 40), (7, 2, 75, 19), (64, 8, 256, 88), (13, 1, 120, 264), (3, 3, 512, 8), (1, 1, 64, 64), (5, 4, 33, 130), (9, 8, 24, 6272)]
 
 
 @pytest.mark.parametrize("device", DEVICES)

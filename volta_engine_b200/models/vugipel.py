@@ -1,6 +1,6 @@
 """Vugipel: a decoder whose configuration lists its layers one by one. Every layer mixes tokens by a gated recurrence per channel (minGRU) or
 by windowed attention with rotated values beside retention, and has a mixture of gated SiLU experts (sigmoid router, weights on the
-experts' inputs) or no feed-forward. RMS norms whose weights are stored around zero stand in front of the sublayers, whose results are
+experts' inputs) or no feed-forward. RMS norms whose weights are stored as offsets from one stand in front of the sublayers, whose results are
 added to an fp32 residual.
 
 The decoder is the one of :mod:`.listed`, mixers and feed-forwards those of :mod:`.mixers` and :mod:`.feed_forward`, norms and
